@@ -31,7 +31,7 @@ extern "C" {
 #endif
 
 /* TensorSharp.DType (TensorSharp/DType.cs:6-13) */
-enum { TSB200_F32 = 0, TSB200_F16 = 1, TSB200_F64 = 2, TSB200_I32 = 3, TSB200_U8 = 4 };
+enum { TSB200_F32 = 0, TSB200_F16 = 1, TSB200_F64 = 2, TSB200_I32 = 3, TSB200_U8 = 4, TSB200_BF16 = 5 /* layered engines only */ };
 
 /* A strided view over device memory: the (sizes, strides, storage, offset) of TensorSharp.Tensor with the
  * offset already applied to `data`.  Outermost dimension first; strides in elements. */
@@ -171,7 +171,9 @@ TSB200_API int TSB200_PhiloxUniform(int device, float* u, int n, uint64_t seed, 
  * always fp32. */
 enum { TSB200_ACT_NONE = -1, TSB200_ACT_RELU = 0, TSB200_ACT_SILU = 1, TSB200_ACT_LEAKYRELU = 2,
        TSB200_ACT_GLU_NOACT = 3 /* the reference's "SwiGLU": (xW1+b1)*(xW3+b3), PositionwiseFeedForward.cs:82-89 */,
-       TSB200_ACT_SWIGLU = 4 /* silu(xW1+b1)*(xW3+b3): extension */, TSB200_ACT_GELU = 5 /* erf GELU: extension */ };
+       TSB200_ACT_SWIGLU = 4 /* silu(xW1+b1)*(xW3+b3): extension */, TSB200_ACT_GELU = 5 /* erf GELU: extension */,
+       TSB200_ACT_SIGMOID = 6 /* layered engines: gates */,
+       TSB200_ACT_CLAMP_GLU = 7 /* layered engines: a sigmoid(s a) (g + t) with a, g clamped */ };
 
 /* y[M,N] = act(bias + x[M,K] W[K,N]) (+ residual); W row-major [in,out] as the reference stores it
  * (Seq2SeqSharp/Layers/FeedForwardLayer.cs:43).  x, y in `dtype`; residual and y_f32 optional:
@@ -330,6 +332,37 @@ TSB200_API int TSB200_DebugSetGemvTrace(void* device_buffer);
 #endif
 
 TSB200_API int TSB200_GptCreate(const TSB200GptConfig* cfg, void** gpt);
+/* Layered models: every layer has its own description, so that sizes, order and sharing may differ from layer to layer.  The
+ * handle is an ordinary engine: prefill, decode, slots, snapshots, beams and sampling work as for TSB200_GptCreate.  (The reference
+ * has no counterpart: its GPTDecoder repeats one layer, Networks/GPTDecoder.cs:104-133.)  dtype TSB200_F32 or TSB200_BF16; the
+ * residual stream, norms, scores, softmax and angles are fp32 in both.  One GPU.
+ *   x = embed[id] * embed_scale
+ *   x <- x + gate1 * attention(h1 + conv(h1)) + gate2 * experts(h2),   h1 / h2: RMS norm in norm_groups equal parts, weights norm1 /
+ *        norm2; gate = sigmoid(h G + b); conv: causal, per channel, conv_taps taps (the newest is the position itself)
+ *   logits = norm(x) embed^T * logit_scale
+ * Weights (TSB200_GptSetWeight; matrices [out, in] row-major, F32 or BF16, tables I32): embed [V, d], final_norm [1, d] and per layer i
+ *   layer.<i>.{norm1, norm2 [1, d], conv1 [d, taps], gate1.w, gate2.w [d, d], gate1.b, gate2.b [1, d]}
+ *   layer.<i>.attn.{q [H (dim + rot), d], dkv [rank + rot, d], dkv_norm [1, rank], uk [H dim, rank], uv [H vdim, rank], o [d, H vdim]}
+ *   layer.<i>.experts.{table [V, top] I32, <e>.gate, <e>.up [ff, d], <e>.down [d, ff]}
+ * Layers with kv_from >= 0 have no dkv / dkv_norm; layers without experts have no norm2 / gate2 / experts. */
+typedef struct TSB200LayerDesc {
+  int32_t mixer;              /* 0: latent attention */
+  int32_t heads, dim, rot_dim, vdim, kv_rank;   /* per head: unrotated and rotated query/key size, value size; size of the latent */
+  int32_t rot_dims;           /* leading dimensions of the rotated part that turn (pairs i, i + rot_dims / 2) */
+  int32_t kv_from;            /* -1: own latent and cache; else the layer whose cached latents and rotated keys are attended to */
+  float scale;                /* of the scores */
+  double rot_base;
+  int32_t experts, top;       /* experts 0: no feed-forward; else `top` experts per token id by table, each with weight 1 / top */
+  int32_t ff;
+  float glu_limit, glu_slope, glu_shift;   /* expert: a = min(gate, limit), u = clamp(up, limit), a sigmoid(slope a) (u + shift) */
+} TSB200LayerDesc;
+typedef struct TSB200LayeredConfig {
+  int32_t L, d, V, dtype;
+  int32_t norm_groups, conv_taps;
+  float eps, embed_scale, logit_scale;
+  int32_t max_batch, max_tokens, device;
+} TSB200LayeredConfig;
+TSB200_API int TSB200_GptCreateLayered(const TSB200LayeredConfig* cfg, const TSB200LayerDesc* layers, void** gpt);
 TSB200_API int TSB200_GptDestroy(void* gpt);
 /* name = the reference's weight key (IModel.AddWeights/GetWeights, Seq2SeqSharp/Tools/WeightTensor.cs:571-604),
  * e.g. "GPTDecoder.SelfAttn_3.QKV", "GPTDecoder.PosFFN_3.feedForwardLayer1.m_Whd", "TgtEmbeddings",
@@ -415,6 +448,10 @@ TSB200_API int TSB200_GptSlotReset(void* gpt, int slot);   /* empties the slot; 
 TSB200_API int TSB200_GptSetPerSequenceState(void* gpt, int on);
 TSB200_API int TSB200_GptSlotExtend(void* gpt, int slot, const int32_t* ids, int S, const TSB200DecodingOptions* opt,
                                     int32_t* out_id);
+/* S given tokens for one sequence on top of what its slot holds (nothing after TSB200_GptSlotReset), WITHOUT sampling: logits
+ * [n_want, V] (F32, host) at the places want[] (0 .. S - 1, host) of the portion; n_want may be 0.  Scoring a text, or feeding a
+ * prompt in portions.  No next id is pending afterwards: continue with this call, TSB200_GptSlotExtend or TSB200_GptStepHost. */
+TSB200_API int TSB200_GptSlotLogits(void* gpt, int slot, const int32_t* ids, int S, const int32_t* want, int n_want, float* logits);
 /* device-timed duration (ms, CUDA events on the engine's stream) of the last GptDecode / GptPrefill call and
  * the number of kernel launches it issued (graph replays count their nodes) */
 TSB200_API int TSB200_GptLastTiming(void* gpt, float* ms, int64_t* launches);

@@ -14,7 +14,7 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.environ.get("TSB200_LIB") or os.path.join(_HERE, "libtsb200.so")
 HEADER_PATH = os.path.join(_HERE, "..", "include", "tsb200.h")
 
-F32, F16, F64, I32, U8 = 0, 1, 2, 3, 4
+F32, F16, F64, I32, U8, BF16 = 0, 1, 2, 3, 4, 5
 ACT_NONE, ACT_RELU, ACT_SILU, ACT_LEAKYRELU, ACT_GLU_NOACT, ACT_SWIGLU, ACT_GELU = -1, 0, 1, 2, 3, 4, 5
 
 
@@ -38,6 +38,18 @@ class GptConfig(C.Structure):
                [("eps", C.c_float), ("rope_base", C.c_float)] + \
                [(n, C.c_int32) for n in ("ape_decode_pos0", "max_batch", "max_tokens", "device", "tp_rank", "tp_size", "n_experts",
                                          "experts_per_token", "cross_attn", "max_src_tokens")]
+
+
+class LayerDescC(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "rot_dim", "vdim", "kv_rank", "rot_dims", "kv_from")] + \
+               [("scale", C.c_float), ("rot_base", C.c_double)] + [(n, C.c_int32) for n in ("experts", "top", "ff")] + \
+               [(n, C.c_float) for n in ("glu_limit", "glu_slope", "glu_shift")]
+
+
+class LayeredConfigC(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("L", "d", "V", "dtype", "norm_groups", "conv_taps")] + \
+               [(n, C.c_float) for n in ("eps", "embed_scale", "logit_scale")] + \
+               [(n, C.c_int32) for n in ("max_batch", "max_tokens", "device")]
 
 
 class DecodingOptionsC(C.Structure):
@@ -121,6 +133,7 @@ def lib():
         "TSB200_PrefillAttention": (i32, [i32, i32, vp, vp, i64, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp]),
         "TSB200_SoftmaxArgmax": (i32, [i32, vp, vp, vp, i32, i32, f32, vp, i32, vp]),
         "TSB200_GptCreate": (i32, [C.POINTER(GptConfig), C.POINTER(vp)]),
+        "TSB200_GptCreateLayered": (i32, [C.POINTER(LayeredConfigC), C.POINTER(LayerDescC), C.POINTER(vp)]),
         "TSB200_GptDestroy": (i32, [vp]),
         "TSB200_GptSetWeight": (i32, [vp, C.c_char_p, vp, i32, i64, i64, i32]),
         "TSB200_GptGetWeightPtr": (i32, [vp, C.c_char_p, C.POINTER(vp), C.POINTER(i64), C.POINTER(i64)]),
@@ -152,6 +165,7 @@ def lib():
         "TSB200_GptSlotReset": (i32, [vp, i32]),
         "TSB200_GptSetPerSequenceState": (i32, [vp, i32]),
         "TSB200_GptSlotExtend": (i32, [vp, i32, vp, i32, C.POINTER(DecodingOptionsC), vp]),
+        "TSB200_GptSlotLogits": (i32, [vp, i32, vp, i32, vp, i32, vp]),
         "TSB200_GptExtend": (i32, [vp, vp, i32, i32, C.POINTER(DecodingOptionsC), vp]),
         "TSB200_GptCacheSnapshot": (i32, [vp, C.POINTER(vp)]),
         "TSB200_GptCacheSnapshotInfo": (i32, [vp, C.POINTER(i32), C.POINTER(i32), C.POINTER(i64), vp]),

@@ -1,5 +1,6 @@
 // Shared host/device helpers for libtsb200: error convention, device/stream bookkeeping, dtype utilities.
 #pragma once
+#include <cuda_bf16.h>
 #include <cuda_fp16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -90,7 +91,8 @@ inline cudaError_t launch_k(void (*kernel)(KArgs...), dim3 grid, dim3 block, siz
 inline size_t dtype_size(int dt) {
   switch (dt) {
     case TSB200_F32: return 4;
-    case TSB200_F16: return 2;
+    case TSB200_F16:
+    case TSB200_BF16: return 2;
     case TSB200_F64: return 8;
     case TSB200_I32: return 4;
     case TSB200_U8: return 1;
@@ -98,12 +100,51 @@ inline size_t dtype_size(int dt) {
   return 0;
 }
 
+inline bool is_16bit(int dt) { return dt == TSB200_F16 || dt == TSB200_BF16; }
+
 template <typename T> __device__ __forceinline__ float to_f(T v);
 template <> __device__ __forceinline__ float to_f<float>(float v) { return v; }
 template <> __device__ __forceinline__ float to_f<__half>(__half v) { return __half2float(v); }
 template <typename T> __device__ __forceinline__ T from_f(float v);
 template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
 template <> __device__ __forceinline__ __half from_f<__half>(float v) { return __float2half_rn(v); }
+template <> __device__ __forceinline__ float to_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+// The two 16-bit model types side by side: a pair of values in one register, and what the tensor-core instructions need to know.
+template <typename H> struct Pair16;
+template <> struct Pair16<__half> {
+  static constexpr uint32_t kUmmaFormat = 0;   // A / B format field of the tcgen05 instruction descriptor
+  static constexpr bool kBf16 = false;
+  static __device__ __forceinline__ float2 get(uint32_t r) { return __half22float2(*reinterpret_cast<const __half2*>(&r)); }
+  static __device__ __forceinline__ uint32_t put(float a, float b) {
+    const __half2 h = __floats2half2_rn(a, b);
+    return *reinterpret_cast<const uint32_t*>(&h);
+  }
+};
+template <> struct Pair16<__nv_bfloat16> {
+  static constexpr uint32_t kUmmaFormat = 1;
+  static constexpr bool kBf16 = true;
+  static __device__ __forceinline__ float2 get(uint32_t r) { return make_float2(__uint_as_float(r << 16), __uint_as_float(r & 0xffff0000u)); }
+  static __device__ __forceinline__ uint32_t put(float a, float b) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const uint32_t*>(&h);
+  }
+};
+// D[16x8] += A[16x16] B[16x8] on the warp-level tensor cores, fp32 accumulators
+template <typename H>
+__device__ __forceinline__ void mma_16816(float* d, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  if constexpr (Pair16<H>::kBf16)
+    asm volatile(
+        "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+        : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+        : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+  else
+    asm volatile(
+        "mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+        : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+        : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

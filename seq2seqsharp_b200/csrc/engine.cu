@@ -12,9 +12,12 @@
 //  * a decode step is one CUDA graph: the cache length and the step counter live in device memory so the same
 //    graph is replayed for every token, sampled ids are fed back on the device, and the host reads ids only
 //    when asked (every step only if it must test the reference's stop rule, GPT.cs:300-303).
+#include <algorithm>
 #include <cmath>
+#include <cstdio>
 #include <cstdlib>
 #include <cstring>
+#include <set>
 #include <string>
 #include <vector>
 
@@ -70,6 +73,10 @@ __global__ void gather_last_kernel(float* xl, const float* x, int B, int S, int 
     last = last < 0 ? 0 : (last >= S ? S - 1 : last);
     for (int i = threadIdx.x; i < d; i += blockDim.x) xl[(int64_t)b * d + i] = x[((int64_t)b * S + last) * d + i];
   }
+}
+
+__global__ void gather_rows_kernel(float* out, const float* x, const int* rows, int d) {
+  for (int i = threadIdx.x; i < d; i += blockDim.x) out[(int64_t)blockIdx.x * d + i] = x[(int64_t)rows[blockIdx.x] * d + i];
 }
 
 // state: the device step state (kernels.cuh).  The per-sequence pointers (ids, history, out) address sequence b0 + b of
@@ -156,8 +163,21 @@ struct GraphKey {
   }
 };
 
+struct Layered;
+
 struct Gpt {
   TSB200GptConfig c;
+  Layered* ly = nullptr;       // models whose layers are described one by one (engine_layers.cuh); null: GPTDecoder's uniform layers
+  int64_t x_bytes = 0;         // layered: size of the residual buffer
+  // rows whose logits are asked for instead of the last of each sequence (TSB200_GptSlotLogits): device list, count, destination
+  const int* want_rows = nullptr;
+  int n_want = 0;
+  float* want_logits = nullptr;
+  float* want_x = nullptr;     // [n_want, d] gathered rows and their normed form (uniform layers)
+  void* want_h = nullptr;
+  int* want_list = nullptr;
+  float* want_out = nullptr;
+  int64_t want_cap = 0;        // rows the two buffers, the list and the logits have room for
   DeviceState* st = nullptr;
   cudaStream_t s = nullptr;
   int es = 4;  // element size of the model dtype
@@ -194,7 +214,8 @@ struct Gpt {
   int cross_T = 0;                // longest encoder output of the current call (0: none set)
   int* beam_ids = nullptr;
   float* beam_p = nullptr;
-  void** beam_layers = nullptr;   // [2 * L]: K cache, V cache of layer 0, 1, ...
+  struct SeqPiece* beam_pieces = nullptr;   // one entry per (cache part, head)
+  int n_beam_pieces = 0;
   int* beam_pairs = nullptr;      // [2 * max_batch]
   int* moe_picks = nullptr;      // [rows, experts_per_token] experts chosen by the router, ascending per token
   float* moe_scores = nullptr;   // their router probabilities
@@ -325,22 +346,31 @@ constexpr size_t kGuardBytes = 256;
 constexpr int kGuardByte = 0xC5;
 constexpr int kMaxBeam = 32;
 
-// Copies whole sequences inside the engine: for every pair (src, dst) the first T cache rows of every (layer, K or V, KV
-// head), the token history and the pending id.  grid = (pairs, 2 * L * Hkv); sources and destinations are disjoint.
-__global__ void __launch_bounds__(256) seq_copy_kernel(void* const* layers, const int* pairs, int Hkv, int64_t seq_bytes, int64_t head_pitch,
-                                                       int64_t head_bytes, int* hist, int* hist_len, int* ids_cur, int hist_stride) {
+// One contiguous piece of a sequence's cache: bytes per cached token, or a fixed state (row_bytes 0, state_bytes).
+struct SeqPiece {
+  unsigned char* base;
+  long long seq_bytes, row_bytes, state_bytes;
+};
+// Copies whole sequences inside the engine: for every pair (src, dst) and every piece the rows of the first T tokens (or the state),
+// the token history and the pending id.  grid = (pairs, pieces); sources and destinations are disjoint.
+__global__ void __launch_bounds__(256) seq_copy_kernel(const SeqPiece* pieces, const int* pairs, int T, int Tmax, int* hist, int* hist_len, int* ids_cur,
+                                                       int hist_stride) {
   const int src = pairs[2 * blockIdx.x], dst = pairs[2 * blockIdx.x + 1];
-  TSB_DEV_CHECK(engine, src >= 0 && dst >= 0 && src != dst && head_bytes <= head_pitch, 0x104, return)   // bad pair or rows beyond the cache
-  const int lw = blockIdx.y / Hkv, kvh = blockIdx.y % Hkv;
-  unsigned char* base = reinterpret_cast<unsigned char*>(layers[lw]);
-  const uint4* from = reinterpret_cast<const uint4*>(base + (size_t)src * seq_bytes + (size_t)kvh * head_pitch);
-  uint4* to = reinterpret_cast<uint4*>(base + (size_t)dst * seq_bytes + (size_t)kvh * head_pitch);
-  for (int64_t i = threadIdx.x; i < head_bytes / 16; i += blockDim.x) to[i] = from[i];
+  TSB_DEV_CHECK(engine, src >= 0 && dst >= 0 && src != dst && T <= Tmax, 0x104, return)   // bad pair or rows beyond the cache
+  const SeqPiece p = pieces[blockIdx.y];
+  const long long n = p.row_bytes ? p.row_bytes * T : p.state_bytes;
+  const unsigned char* from = p.base + src * p.seq_bytes;
+  unsigned char* to = p.base + dst * p.seq_bytes;
+  if (((p.seq_bytes | n | (long long)(uintptr_t)p.base) & 15) == 0) {
+    for (long long i = threadIdx.x; i < n / 16; i += blockDim.x) reinterpret_cast<uint4*>(to)[i] = reinterpret_cast<const uint4*>(from)[i];
+  } else {
+    for (long long i = threadIdx.x; i < n; i += blockDim.x) to[i] = from[i];
+  }
   if (blockIdx.y == 0) {
-    const int n = hist_len[src];
-    for (int i = threadIdx.x; i < n && i < hist_stride; i += blockDim.x) hist[(size_t)dst * hist_stride + i] = hist[(size_t)src * hist_stride + i];
+    const int n_h = hist_len[src];
+    for (int i = threadIdx.x; i < n_h && i < hist_stride; i += blockDim.x) hist[(size_t)dst * hist_stride + i] = hist[(size_t)src * hist_stride + i];
     if (threadIdx.x == 0) {
-      hist_len[dst] = n;
+      hist_len[dst] = n_h;
       ids_cur[dst] = ids_cur[src];
     }
   }
@@ -372,7 +402,8 @@ static int dev_free(Gpt* g, void* user) {
 }
 
 static int fill_const(Gpt* g, void* p, int64_t n, float v) {
-  if (g->c.dtype == TSB200_F32) fill_const_kernel<float><<<(int)((n + 255) / 256), 256, 0, g->s>>>((float*)p, n, v);
+  if (g->c.dtype == TSB200_BF16) fill_const_kernel<__nv_bfloat16><<<(int)((n + 255) / 256), 256, 0, g->s>>>((__nv_bfloat16*)p, n, v);
+  else if (g->c.dtype == TSB200_F32) fill_const_kernel<float><<<(int)((n + 255) / 256), 256, 0, g->s>>>((float*)p, n, v);
   else fill_const_kernel<__half><<<(int)((n + 255) / 256), 256, 0, g->s>>>((__half*)p, n, v);
   count_launch(g->c.device);
   return check_launch("fill_const");
@@ -572,6 +603,7 @@ static std::vector<std::string> weight_names(const Gpt* g, bool biases, bool nor
 }
 
 static int ensure_act(Gpt* g, int64_t rows) {
+  if (g->ly) return 1;   // a layered engine sizes its scratch per forward pass
   if (rows <= g->act_rows) return 1;
   const TSB200GptConfig& c = g->c;
   TSB_CUDA(cudaStreamSynchronize(g->s));
@@ -611,6 +643,68 @@ static Epilogue make_ep(const void* bias, const float* residual, void* y, float*
   Epilogue e{};
   e.bias = bias; e.residual = residual; e.y = y32 ? nullptr : y; e.y32 = y32; e.act = act; e.glu = glu;
   return e;
+}
+
+}  // namespace tsb
+
+#include "engine_layers.cuh"
+
+namespace tsb {
+
+// What a sequence owns in the engine, piece by piece: rows per cached token ([max_batch][heads][max_tokens][row_bytes]) or a state of
+// fixed size ([max_batch][state_bytes]).  Slots, snapshots and sequence copies work on this list, whatever the model is made of.
+struct CachePart {
+  void** base;
+  int heads;
+  size_t row_bytes;     // 0: a state
+  size_t state_bytes;
+  size_t seq_bytes(const Gpt* g) const { return row_bytes ? (size_t)heads * g->c.max_tokens * row_bytes : state_bytes; }
+  size_t used_bytes(int T) const { return row_bytes ? (size_t)heads * T * row_bytes : state_bytes; }   // of a sequence of T tokens
+};
+static std::vector<CachePart> cache_parts(Gpt* g) {
+  std::vector<CachePart> v;
+  if (g->ly) {
+    for (auto& L : g->ly->L) {
+      if (L.cache) v.push_back({&L.cache, 1, (size_t)L.sh.row * g->es, 0});
+      v.push_back({&L.ring, 1, 0, (size_t)g->ly->c.conv_taps * g->ly->c.d * g->es});
+    }
+    return v;
+  }
+  for (LayerW& L : g->L) {
+    v.push_back({&L.cK, g->c.Hkv, (size_t)g->c.hd * g->es, 0});
+    v.push_back({&L.cV, g->c.Hkv, (size_t)g->c.hd * g->es, 0});
+  }
+  return v;
+}
+// n_seq sequences from `slot` on <-> a compact buffer ([part][sequence][used bytes])
+static int copy_parts(Gpt* g, unsigned char* compact, int slot, int n_seq, int T, bool save) {
+  for (const CachePart& p : cache_parts(g)) {
+    unsigned char* at = (unsigned char*)*p.base + (size_t)slot * p.seq_bytes(g);
+    if (p.row_bytes) {
+      const size_t row = (size_t)T * p.row_bytes, pitch = (size_t)g->c.max_tokens * p.row_bytes, rows = (size_t)n_seq * p.heads;
+      if (save) TSB_CUDA(cudaMemcpy2DAsync(compact, row, at, pitch, row, rows, cudaMemcpyDeviceToDevice, g->s));
+      else TSB_CUDA(cudaMemcpy2DAsync(at, pitch, compact, row, row, rows, cudaMemcpyDeviceToDevice, g->s));
+    } else {
+      const size_t bytes = (size_t)n_seq * p.state_bytes;
+      TSB_CUDA(cudaMemcpyAsync(save ? compact : at, save ? at : compact, bytes, cudaMemcpyDeviceToDevice, g->s));
+    }
+    compact += (size_t)n_seq * p.used_bytes(T);
+  }
+  return 1;
+}
+static size_t parts_bytes(Gpt* g, int T) {   // of one sequence of T tokens
+  size_t n = 0;
+  for (const CachePart& p : cache_parts(g)) n += p.used_bytes(T);
+  return n;
+}
+static std::vector<size_t> parts_layout(Gpt* g) {   // two engines with the same layout can exchange snapshots
+  std::vector<size_t> v;
+  for (const CachePart& p : cache_parts(g)) {
+    v.push_back((size_t)p.heads);
+    v.push_back(p.row_bytes);
+    v.push_back(p.state_bytes);
+  }
+  return v;
 }
 
 // One linear layer of the engine on packed weights.  With `ng` the input is the fp32 residual stream and the layer's
@@ -689,6 +783,8 @@ static int row_parallel_linear(Gpt* g, int rows, const void* in, const void* Wp,
 // then the LM head behind the final norm.
 static int ensure_stack(Gpt* g, int B) {
   const TSB200GptConfig& c = g->c;
+  g->own_B = 0;
+  if (g->ly) return 1;                        // layered models run one launch per operation
   g->stack_max_B = (c.dtype == TSB200_F16) ? 8 : 4;  // fp16: tensor-core consumers take up to 8 rows
   const int cap = g->stack_cap >= 0 ? g->stack_cap : (c.dtype == TSB200_F16 ? 0 : 2);
   if (g->tp == 1 && cap < g->stack_max_B) g->stack_max_B = cap;
@@ -805,6 +901,10 @@ static int ensure_stack(Gpt* g, int B) {
 // One forward pass over `rows = B*S` new tokens whose ids are in g->ids_in; leaves logits [B,V] in g->logits.
 // With use_state the cache length is read from g->state[0] by the kernels (graph replay), else from T0.
 static int enqueue_forward(Gpt* g, int B, int S, int T0, bool use_state, int splits) {
+  if (g->ly) {
+    if (!use_state) TSB_TRY(ensure_layered(g, B, S, T0 + S));
+    return enqueue_layered(g, B, S, T0, use_state, use_state ? splits : T0 + S);
+  }
   NvtxRange nvtx_(S == 1 ? "tsb200.forward.step" : "tsb200.forward.prompt");
   PdlScope pdl_scope(g->pdl && S == 1);
   const TSB200GptConfig& c = g->c;
@@ -905,6 +1005,13 @@ static int enqueue_forward(Gpt* g, int B, int S, int T0, bool use_state, int spl
     TSB_TRY(row_parallel_linear(g, rows, g->ffn, L.w2, c.F, L.b2));
   }
   const float* xlast = g->x;
+  if (g->want_rows) {
+    if (g->n_want == 0) return 1;
+    gather_rows_kernel<<<g->n_want, 256, 0, g->s>>>(g->want_x, g->x, g->want_rows, d);
+    count_launch(dev);
+    TSB_TRY(check_launch("gather_rows"));
+    return engine_linear(g, g->n_want, nullptr, g->want_x, g->nf_g, g->nf_b, g->want_h, g->head_w, d, c.V, make_ep(g->head_b, nullptr, nullptr, g->want_logits, TSB200_ACT_NONE, 0));
+  }
   if (S > 1) {
     gather_last_kernel<<<B, 256, 0, g->s>>>(g->xl, g->x, B, S, d, g->gather_lens);
     count_launch(dev);
@@ -959,6 +1066,8 @@ static int check_err_flag(Gpt* g, const int* pre = nullptr) {
     int c = chk_take_engine();
     if (!c) c = chk_take_attention();
     if (!c) c = chk_take_moe();
+    if (!c) c = chk_take_blocks();
+    if (!c) c = chk_take_latent();
     if (!c) c = chk_take_sampling();
     TSB_CHECK(c == 0, "checked build: device-side check 0x%x failed (an index or a capacity was out of range; the access was skipped)", c);
   }
@@ -1064,7 +1173,11 @@ static int ensure_graph(Gpt* g, const TSB200DecodingOptions* opt, int n_steps) {
   while (Tp < g->T + n_steps) Tp <<= 1;
   TSB_TRY(ensure_stack(g, B));
   GraphKey key;
-  key.B = B; key.strategy = opt->strategy; key.splits = attn_pick_splits(g->st, c.dtype, B, c.H, c.Hkv, c.hd, Tp);
+  if (g->ly) {
+    if (Tp > c.max_tokens) Tp = c.max_tokens;
+    TSB_TRY(ensure_layered(g, B, 1, Tp));
+  }
+  key.B = B; key.strategy = opt->strategy; key.splits = g->ly ? Tp : attn_pick_splits(g->st, c.dtype, B, c.H, c.Hkv, c.hd, Tp);
   key.n_blocked = opt->n_blocked; key.blocked_hash = hash_blocked(opt->blocked, opt->n_blocked);
   key.topP = opt->topP; key.temperature = opt->temperature; key.penalty = opt->repeatPenalty;
   key.seed = opt->seed; key.seq_base = opt->seq_base;
@@ -1271,6 +1384,125 @@ int TSB200_GptCreate(const TSB200GptConfig* cfg, void** out) {
   return 1;
 }
 
+int TSB200_GptCreateLayered(const TSB200LayeredConfig* cfg, const TSB200LayerDesc* layers, void** out) {
+  TSB_CHECK(cfg && layers && out, "gpt_create_layered: null argument");
+  *out = nullptr;
+  const TSB200LayeredConfig& c = *cfg;
+  TSB_CHECK(c.L > 0 && c.d > 0 && c.V > 0, "gpt_create_layered: bad dimensions");
+  TSB_CHECK(c.dtype == TSB200_F32 || c.dtype == TSB200_BF16, "gpt_create_layered: dtype must be F32 or BF16");
+  TSB_CHECK(c.norm_groups > 0 && c.d % c.norm_groups == 0, "gpt_create_layered: a width of %d is not cut into %d norm groups", c.d, c.norm_groups);
+  TSB_CHECK(c.conv_taps >= 1 && c.conv_taps <= 64, "gpt_create_layered: %d convolution taps are not supported", c.conv_taps);
+  TSB_CHECK(c.max_batch > 0 && c.max_batch <= 1024 && c.max_tokens > 0, "gpt_create_layered: bad cache capacity");
+  for (int i = 0; i < c.L; ++i) {
+    const TSB200LayerDesc& l = layers[i];
+    TSB_CHECK(l.mixer == 0, "gpt_create_layered: layer %d has an unknown mixer %d", i, l.mixer);
+    TSB_CHECK(l.heads > 0 && l.dim > 0 && l.rot_dim > 0 && l.vdim > 0 && l.kv_rank > 0 && l.kv_rank <= 1024 && l.dim <= 768,
+              "gpt_create_layered: layer %d has unsupported attention sizes (latent up to 1024, unrotated head size up to 768)", i);
+    TSB_CHECK(l.rot_dims > 0 && l.rot_dims <= l.rot_dim && l.rot_dims % 2 == 0 && l.rot_base > 0.0, "gpt_create_layered: layer %d has a bad rotation", i);
+    if (l.kv_from >= 0) {
+      TSB_CHECK(l.kv_from < i && layers[l.kv_from].kv_from < 0, "gpt_create_layered: layer %d reads the cache of layer %d, which is not an earlier layer with its own", i, l.kv_from);
+      const TSB200LayerDesc& o = layers[l.kv_from];
+      TSB_CHECK(o.kv_rank == l.kv_rank && o.rot_dim == l.rot_dim && o.rot_dims == l.rot_dims && o.rot_base == l.rot_base,
+                "gpt_create_layered: layer %d and layer %d, whose cache it reads, differ in the latent or the rotation", i, l.kv_from);
+    }
+    TSB_CHECK(l.experts >= 0 && l.experts <= 4096 && (l.experts == 0 || (l.top >= 1 && l.top <= l.experts && l.ff > 0)),
+              "gpt_create_layered: layer %d has %d experts with %d per token", i, l.experts, l.top);
+  }
+  DeviceState* st;
+  TSB_TRY(use_device(c.device, &st));
+  Gpt* g = new Gpt();
+  std::memset(&g->c, 0, sizeof(g->c));
+  g->c.L = c.L; g->c.d = c.d; g->c.V = c.V; g->c.H = g->c.Hkv = g->c.hd = g->c.F = 1;
+  g->c.norm_type = 1; g->c.act = TSB200_ACT_SILU; g->c.attn_type = 1; g->c.dtype = c.dtype; g->c.eps = c.eps;
+  g->c.max_batch = c.max_batch; g->c.max_tokens = c.max_tokens; g->c.device = c.device; g->c.tp_size = 1;
+  g->c.n_experts = g->c.experts_per_token = 1;
+  g->st = st;
+  g->s = st->stream;
+  g->es = (int)dtype_size(c.dtype);
+  {
+    const char* e = getenv("TSB200_PDL");
+    g->pdl = !(e && e[0] == '0');
+  }
+  Layered* ly = new Layered();
+  g->ly = ly;
+  ly->c = c;
+  ly->L.resize((size_t)c.L);
+  const int64_t d = c.d, V = c.V, es = g->es, MB = c.max_batch;
+  const int dt = c.dtype, NT = packed_tile_cols(dt);
+  auto fail = [&]() { TSB200_GptDestroy(g); return 0; };
+#define G_ALLOC(p, bytes) if (!dev_alloc(g, (void**)&(p), (bytes))) return fail()
+  G_ALLOC(g->E, V * d * es);
+  G_ALLOC(g->nf_g, d * es);
+  G_ALLOC(g->head_w, packed_bytes(dt, (int)d, (int)V));
+  for (int i = 0; i < c.L; ++i) {
+    LayeredLayer& L = ly->L[i];
+    L.d = layers[i];
+    L.sh = LatentShape{L.d.heads, L.d.dim, L.d.rot_dim, L.d.vdim, L.d.kv_rank, L.d.rot_dims, latent_row_elems(L.d.kv_rank, L.d.rot_dim), L.d.scale};
+    L.Nq = L.sh.H * (L.sh.dim + L.sh.rot);
+    L.Nkv = L.d.kv_from < 0 ? L.sh.rank + L.sh.rot : 0;
+    const bool ff = L.d.experts > 0;
+    const int dct = (int)((d + NT - 1) / NT);
+    L.ct_gate2 = dct;
+    L.ct_qkv = ff ? 2 * dct : dct;
+    G_ALLOC(L.norm1, d * es); G_ALLOC(L.conv_w, d * c.conv_taps * es); G_ALLOC(L.g1b, d * es);
+    G_ALLOC(L.fused, packed_bytes(dt, (int)d, L.ct_qkv * NT + L.Nq + L.Nkv));
+    G_ALLOC(L.uk, (int64_t)L.sh.H * L.sh.dim * L.sh.rank * es); G_ALLOC(L.uv, (int64_t)L.sh.H * L.sh.vdim * L.sh.rank * es);
+    G_ALLOC(L.ukv, packed_bytes(dt, L.sh.row, L.sh.H * (L.sh.dim + L.sh.vdim)));
+    G_ALLOC(L.wo, packed_bytes(dt, L.sh.H * L.sh.vdim, (int)d));
+    if (L.Nkv) {
+      G_ALLOC(L.kv_norm, (int64_t)L.sh.rank * es);
+      G_ALLOC(L.cache, MB * c.max_tokens * L.sh.row * es);
+    }
+    G_ALLOC(L.ring, MB * c.conv_taps * d * es);
+    if (ff) {
+      G_ALLOC(L.norm2, d * es); G_ALLOC(L.g2b, d * es);
+      L.up_bytes = packed_bytes(dt, (int)d, 2 * L.d.ff);
+      L.down_bytes = packed_bytes(dt, L.d.ff, (int)d);
+      G_ALLOC(L.up, L.up_bytes * L.d.experts); G_ALLOC(L.down, L.down_bytes * L.d.experts);
+      G_ALLOC(L.table, V * L.d.top * 4);
+      L.route_index = ly->n_route++;
+      ly->max_experts = std::max(ly->max_experts, L.d.experts);
+    }
+    for (int j = 0; j < i && !L.tab; ++j)
+      if (layers[j].rot_dims == L.d.rot_dims && layers[j].rot_base == L.d.rot_base) L.tab = ly->L[j].tab;
+    if (!L.tab) {
+      float2* tab = nullptr;
+      G_ALLOC(tab, (int64_t)c.max_tokens * (L.d.rot_dims / 2) * sizeof(float2));
+      if (!launch_angle_table(c.device, st, tab, c.max_tokens, L.d.rot_dims, L.d.rot_base, g->s)) return fail();
+      L.tab = tab;
+    }
+  }
+  for (auto& w : layered_weights(ly)) ly->missing.insert(w.first);
+  G_ALLOC(g->hl, MB * d * es);
+  G_ALLOC(g->logits, MB * V * 4);
+  G_ALLOC(g->probs, MB * V * 4);
+  G_ALLOC(g->u, MB * 4);
+  G_ALLOC(g->ids_cur, MB * 4);
+  G_ALLOC(g->ids_new, MB * 4);
+  G_ALLOC(g->hist, MB * c.max_tokens * 4);
+  G_ALLOC(g->hist_len, MB * 4);
+  G_ALLOC(g->state, (int64_t)(kStateLens + 2 * MB) * 4 + 64);
+  mirror_uniform(g);
+  G_ALLOC(g->out_dev, MB * (c.max_tokens + 1) * 4);
+  G_ALLOC(g->blocked, 1024);
+  g->blocked_cap = 256;
+  G_ALLOC(g->err_flag, 64);
+  g->topp_ws_bytes = TSB200_TopPWorkspaceBytes((int)MB, c.V);
+  G_ALLOC(g->topp_ws, g->topp_ws_bytes);
+#undef G_ALLOC
+  if (!init_linear_attrs(c.device) || !init_topp_attrs(c.device) || !init_tc_attrs(c.device)) return fail();
+  if (cudaEventCreate(&g->ev0) != cudaSuccess || cudaEventCreate(&g->ev1) != cudaSuccess) {
+    set_last_error("gpt_create_layered: cudaEventCreate failed");
+    return fail();
+  }
+  if (cudaStreamSynchronize(g->s) != cudaSuccess) {
+    set_last_error("gpt_create_layered: initialisation failed: %s", cudaGetErrorString(cudaGetLastError()));
+    return fail();
+  }
+  *out = g;
+  return 1;
+}
+
 int TSB200_GptDestroy(void* h) {
   if (!h) return 1;
   Gpt* g = (Gpt*)h;
@@ -1288,6 +1520,7 @@ int TSB200_GptDestroy(void* h) {
   owner_destroy(g->own);
   for (auto& a : g->allocs)
     if (a.base) cudaFree(a.base);
+  delete g->ly;
   delete g;
   return 1;
 }
@@ -1296,6 +1529,10 @@ int TSB200_GptSetWeight(void* h, const char* name, const void* data, int dtype, 
   NvtxRange nvtx_("tsb200.gpt.set_weight");
   Gpt* g = (Gpt*)h;
   TSB_CHECK(g && name && data, "gpt_set_weight: null argument");
+  if (g->ly) {
+    TSB_TRY(use_device(g->c.device, nullptr));
+    return layered_set_weight(g, name, data, dtype, rows, cols, on_device);
+  }
   TSB_CHECK(dtype == TSB200_F32 || dtype == TSB200_F16, "gpt_set_weight: data must be F32 or F16");
   TSB_TRY(use_device(g->c.device, nullptr));
   Dest dst;
@@ -1336,6 +1573,7 @@ int TSB200_GptSetWeight(void* h, const char* name, const void* data, int dtype, 
 int TSB200_GptGetWeightPtr(void* h, const char* name, void** ptr, int64_t* rows, int64_t* cols) {
   Gpt* g = (Gpt*)h;
   TSB_CHECK(g && name && ptr, "gpt_get_weight_ptr: null argument");
+  TSB_CHECK(!g->ly, "gpt_get_weight_ptr: not available for layered engines");
   Dest dst;
   TSB_TRY(resolve(g, name, &dst));
   TSB_CHECK(!dst.packed && dst.col_stride == 1 && dst.row_stride == dst.cols, "gpt_get_weight_ptr: '%s' is stored in the engine's packed layout", name);
@@ -1349,6 +1587,7 @@ int TSB200_GptFillSynthetic(void* h, uint64_t seed, float std, float bias_std) {
   Gpt* g = (Gpt*)h;
   TSB_CHECK(g, "gpt_fill_synthetic: null engine");
   TSB_TRY(use_device(g->c.device, nullptr));
+  if (g->ly) return layered_fill_synthetic(g, seed, std, bias_std);
   std::vector<std::string> names = weight_names(g, bias_std > 0.0f, false, true);
   if (g->PE) names.push_back("PosEmbedding");
   int64_t max_elems = 0;
@@ -1723,9 +1962,10 @@ int TSB200_GptCacheLengths(void* h, int* lens, int n) {
 // A parked KV cache: rows [0, T) of every layer's K and V for B sequences, compacted, plus what a later call needs
 // to continue the text (token history, the pending id, the sampling step counter).
 struct GptSnapshot {
-  int device = 0, B = 0, T = 0, L = 0, Hkv = 0, hd = 0, es = 0;
+  int device = 0, B = 0, T = 0;
+  std::vector<size_t> layout;  // of the engine it was taken from (parts_layout)
   uint32_t step = 0;
-  void* kv = nullptr;          // [L][2][B * Hkv][T * hd] elements
+  void* kv = nullptr;          // [cache part][sequence][bytes in use]
   size_t bytes = 0;
   std::vector<int> hist;       // [B][T + 1]: the cached tokens and the pending one
   std::vector<int> pending;    // [B]
@@ -1742,26 +1982,16 @@ int TSB200_GptCacheSnapshot(void* h, void** snap_out) {
   TSB_CHECK(g->T > 0 && g->B > 0, "gpt_cache_snapshot: nothing is cached");
   TSB_CHECK(!g->ragged, "gpt_cache_snapshot: the sequences have different lengths; park them one by one (TSB200_GptSlotSnapshot)");
   GptSnapshot* sn = new GptSnapshot();
-  sn->device = c.device; sn->B = g->B; sn->T = g->T; sn->L = c.L; sn->Hkv = c.Hkv; sn->hd = c.hd; sn->es = g->es;
+  sn->device = c.device; sn->B = g->B; sn->T = g->T; sn->layout = parts_layout(g);
   sn->step = g->step;
-  const size_t row = (size_t)sn->T * c.hd * g->es, pitch = (size_t)c.max_tokens * c.hd * g->es;
-  const size_t rows = (size_t)sn->B * c.Hkv;
-  sn->bytes = (size_t)c.L * 2 * rows * row;
+  sn->bytes = (size_t)sn->B * parts_bytes(g, sn->T);
   auto fail = [&]() { if (sn->kv) cudaFree(sn->kv); delete sn; return 0; };
   if (cudaMalloc(&sn->kv, sn->bytes) != cudaSuccess) {
     cudaGetLastError();
     set_last_error("OOM: gpt_cache_snapshot could not allocate %zu bytes", sn->bytes);
     return fail();
   }
-  for (int k = 0; k < c.L; ++k)
-    for (int w = 0; w < 2; ++w) {
-      unsigned char* dst = (unsigned char*)sn->kv + ((size_t)k * 2 + w) * rows * row;
-      const void* src = w == 0 ? g->L[k].cK : g->L[k].cV;
-      if (cudaMemcpy2DAsync(dst, row, src, pitch, row, rows, cudaMemcpyDeviceToDevice, g->s) != cudaSuccess) {
-        set_last_error("gpt_cache_snapshot: cache copy failed");
-        return fail();
-      }
-    }
+  if (!copy_parts(g, (unsigned char*)sn->kv, 0, sn->B, sn->T, true)) return fail();
   sn->hist.assign((size_t)sn->B * (sn->T + 1), 0);
   sn->pending.assign(sn->B, 0);
   // a cache decoded to capacity has no history slot for the pending id (it stays in `pending`)
@@ -1803,22 +2033,16 @@ int TSB200_GptCacheRestore(void* h, void* snap, int B_new) {
   TSB_CHECK(g && sn, "gpt_cache_restore: null argument");
   const TSB200GptConfig& c = g->c;
   TSB_TRY(use_device(c.device, nullptr));
-  TSB_CHECK(sn->device == c.device && sn->L == c.L && sn->Hkv == c.Hkv && sn->hd == c.hd && sn->es == g->es,
-            "gpt_cache_restore: the snapshot was taken from a different model or device");
+  TSB_CHECK(sn->device == c.device && sn->layout == parts_layout(g), "gpt_cache_restore: the snapshot was taken from a different model or device");
   if (B_new <= 0) B_new = sn->B;
   TSB_CHECK(B_new == sn->B || sn->B == 1, "gpt_cache_restore: a snapshot of %d sequences cannot serve %d", sn->B, B_new);
   TSB_CHECK(B_new <= c.max_batch, "gpt_cache_restore: batch %d exceeds capacity %d", B_new, c.max_batch);
   TSB_CHECK(sn->T < c.max_tokens, "OOM: snapshot of %d tokens exceeds the KV-cache capacity %d", sn->T, c.max_tokens);
-  const size_t row = (size_t)sn->T * c.hd * g->es, pitch = (size_t)c.max_tokens * c.hd * g->es;
-  const size_t rows = (size_t)sn->B * c.Hkv;
-  const int copies = (B_new == sn->B) ? 1 : B_new;  // one sequence parked, many served: the rows go to every slot
-  for (int k = 0; k < c.L; ++k)
-    for (int w = 0; w < 2; ++w) {
-      const unsigned char* src = (const unsigned char*)sn->kv + ((size_t)k * 2 + w) * rows * row;
-      unsigned char* dst = (unsigned char*)(w == 0 ? g->L[k].cK : g->L[k].cV);
-      for (int r = 0; r < copies; ++r)
-        TSB_CUDA(cudaMemcpy2DAsync(dst + (size_t)r * c.Hkv * pitch, pitch, src, row, row, rows, cudaMemcpyDeviceToDevice, g->s));
-    }
+  if (B_new == sn->B) {
+    TSB_TRY(copy_parts(g, (unsigned char*)sn->kv, 0, B_new, sn->T, false));
+  } else {   // one sequence parked, many served: it goes to every slot
+    for (int r = 0; r < B_new; ++r) TSB_TRY(copy_parts(g, (unsigned char*)sn->kv, r, 1, sn->T, false));
+  }
   std::vector<int> lens(B_new, sn->T + 1), pend(B_new);
   for (int b = 0; b < B_new; ++b) {
     const int sb = (B_new == sn->B) ? b : 0;
@@ -1847,26 +2071,16 @@ int TSB200_GptSlotSnapshot(void* h, int slot, void** snap_out) {
   TSB_TRY(use_device(c.device, nullptr));
   TSB_CHECK(slot >= 0 && slot < g->B && g->Ts[slot] > 0, "gpt_slot_snapshot: sequence %d holds nothing", slot);
   GptSnapshot* sn = new GptSnapshot();
-  sn->device = c.device; sn->B = 1; sn->T = g->Ts[slot]; sn->L = c.L; sn->Hkv = c.Hkv; sn->hd = c.hd; sn->es = g->es;
+  sn->device = c.device; sn->B = 1; sn->T = g->Ts[slot]; sn->layout = parts_layout(g);
   sn->step = (uint32_t)g->steps_v[slot];
-  const size_t row = (size_t)sn->T * c.hd * g->es, pitch = (size_t)c.max_tokens * c.hd * g->es;
-  const size_t rows = (size_t)c.Hkv;
-  sn->bytes = (size_t)c.L * 2 * rows * row;
+  sn->bytes = parts_bytes(g, sn->T);
   auto fail = [&]() { if (sn->kv) cudaFree(sn->kv); delete sn; return 0; };
   if (cudaMalloc(&sn->kv, sn->bytes) != cudaSuccess) {
     cudaGetLastError();
     set_last_error("OOM: gpt_slot_snapshot could not allocate %zu bytes", sn->bytes);
     return fail();
   }
-  for (int k = 0; k < c.L; ++k)
-    for (int w = 0; w < 2; ++w) {
-      unsigned char* dst = (unsigned char*)sn->kv + ((size_t)k * 2 + w) * rows * row;
-      const unsigned char* src = (const unsigned char*)(w == 0 ? g->L[k].cK : g->L[k].cV) + (size_t)slot * c.Hkv * pitch;
-      if (cudaMemcpy2DAsync(dst, row, src, pitch, row, rows, cudaMemcpyDeviceToDevice, g->s) != cudaSuccess) {
-        set_last_error("gpt_slot_snapshot: cache copy failed");
-        return fail();
-      }
-    }
+  if (!copy_parts(g, (unsigned char*)sn->kv, slot, 1, sn->T, true)) return fail();
   sn->hist.assign((size_t)sn->T + 1, 0);
   sn->pending.assign(1, 0);
   const size_t hist_w = (size_t)(sn->T + 1 <= c.max_tokens ? sn->T + 1 : c.max_tokens) * 4;
@@ -1925,19 +2139,11 @@ int TSB200_GptSlotRestore(void* h, void* snap, int slot) {
   TSB_CHECK(g && sn, "gpt_slot_restore: null argument");
   const TSB200GptConfig& c = g->c;
   TSB_TRY(use_device(c.device, nullptr));
-  TSB_CHECK(sn->device == c.device && sn->L == c.L && sn->Hkv == c.Hkv && sn->hd == c.hd && sn->es == g->es,
-            "gpt_slot_restore: the snapshot was taken from a different model or device");
+  TSB_CHECK(sn->device == c.device && sn->layout == parts_layout(g), "gpt_slot_restore: the snapshot was taken from a different model or device");
   TSB_CHECK(sn->B == 1, "gpt_slot_restore: the snapshot holds %d sequences; a slot takes one", sn->B);
   TSB_CHECK(sn->T < c.max_tokens, "OOM: snapshot of %d tokens exceeds the KV-cache capacity %d", sn->T, c.max_tokens);
   TSB_TRY(slot_claim(g, slot, "gpt_slot_restore"));
-  const size_t row = (size_t)sn->T * c.hd * g->es, pitch = (size_t)c.max_tokens * c.hd * g->es;
-  const size_t rows = (size_t)c.Hkv;
-  for (int k = 0; k < c.L; ++k)
-    for (int w = 0; w < 2; ++w) {
-      const unsigned char* src = (const unsigned char*)sn->kv + ((size_t)k * 2 + w) * rows * row;
-      unsigned char* dst = (unsigned char*)(w == 0 ? g->L[k].cK : g->L[k].cV) + (size_t)slot * c.Hkv * pitch;
-      TSB_CUDA(cudaMemcpy2DAsync(dst, pitch, src, row, row, rows, cudaMemcpyDeviceToDevice, g->s));
-    }
+  TSB_TRY(copy_parts(g, (unsigned char*)sn->kv, slot, 1, sn->T, false));
   const int len = sn->T + 1;
   TSB_CUDA(cudaMemcpyAsync(g->hist + (size_t)slot * c.max_tokens, sn->hist.data(), (size_t)len * 4, cudaMemcpyHostToDevice, g->s));
   TSB_CUDA(cudaMemcpyAsync(g->hist_len + slot, &len, 4, cudaMemcpyHostToDevice, g->s));
@@ -1950,30 +2156,43 @@ int TSB200_GptSlotRestore(void* h, void* snap, int slot) {
   return 1;
 }
 
-// S prompt tokens for ONE sequence on top of what it has cached (nothing after TSB200_GptSlotReset), then its next id.
-// The run addresses the sequence's rows of every per-sequence buffer; the other sequences are not touched.
-int TSB200_GptSlotExtend(void* h, int slot, const int32_t* ids, int S, const TSB200DecodingOptions* opt, int32_t* out_id) {
-  NvtxRange nvtx_("tsb200.gpt.slot_extend");
-  Gpt* g = (Gpt*)h;
-  TSB_CHECK(g && ids && opt, "gpt_slot_extend: null argument");
+// S prompt tokens for ONE sequence on top of what it has cached (nothing after TSB200_GptSlotReset), then its next id (opt given) or
+// the logits at the places want[0, n_want) of the portion (opt null).  The run addresses the sequence's rows of every per-sequence
+// buffer; the other sequences are not touched.
+static int slot_run(Gpt* g, int slot, const int32_t* ids, int S, const TSB200DecodingOptions* opt, int32_t* out_id, const int32_t* want, int n_want,
+                    float* logits, const char* who) {
   const TSB200GptConfig& c = g->c;
   TSB_TRY(use_device(c.device, nullptr));
-  TSB_TRY(slot_claim(g, slot, "gpt_slot_extend"));
+  TSB_TRY(slot_claim(g, slot, who));
   const int T0 = g->Ts[slot];
-  TSB_CHECK(S > 0 && T0 + S < c.max_tokens, "OOM: prompt of %d tokens exceeds the KV-cache capacity %d", T0 + S, c.max_tokens);
-  for (int i = 0; i < S; ++i) TSB_CHECK(ids[i] >= 0 && ids[i] < c.V, "gpt_slot_extend: token id %d out of range", ids[i]);
+  TSB_CHECK(S > 0 && (opt ? T0 + S < c.max_tokens : T0 + S <= c.max_tokens), "OOM: prompt of %d tokens exceeds the KV-cache capacity %d", T0 + S, c.max_tokens);
+  for (int i = 0; i < S; ++i) TSB_CHECK(ids[i] >= 0 && ids[i] < c.V, "%s: token id %d out of range", who, ids[i]);
   TSB_TRY(ensure_act(g, (int64_t)S));
+  if (!opt) {
+    for (int i = 0; i < n_want; ++i) TSB_CHECK(want[i] >= 0 && want[i] < S, "%s: place %d is outside the portion of %d tokens", who, want[i], S);
+    if (n_want > g->want_cap || !g->want_cap) {
+      const int64_t cap = n_want > 16 ? n_want : 16;
+      const int64_t es = g->es;
+      void* p[4] = {(void*)g->want_list, g->want_out, g->want_x, g->want_h};
+      for (void* q : p)
+        if (q) TSB_TRY(dev_free(g, q));
+      g->want_list = nullptr; g->want_out = nullptr; g->want_x = nullptr; g->want_h = nullptr; g->want_cap = 0;
+      TSB_TRY(dev_alloc(g, (void**)&g->want_list, cap * 4));
+      TSB_TRY(dev_alloc(g, (void**)&g->want_out, cap * c.V * 4));
+      TSB_TRY(dev_alloc(g, (void**)&g->want_x, cap * c.d * 4));
+      TSB_TRY(dev_alloc(g, (void**)&g->want_h, cap * c.d * es));
+      g->want_cap = cap;
+    }
+  }
   void* ids_dev = nullptr;
   TSB_CUDA(cudaMalloc(&ids_dev, (size_t)S * 4));
   // the view of one sequence: every per-sequence pointer moves to the sequence's rows
   struct View {
-    Gpt* g; int slot; std::vector<std::pair<void*, void*>> kv; int *hist, *hist_len, *ids_cur; uint32_t step;
-    View(Gpt* g_, int slot_) : g(g_), slot(slot_), hist(g_->hist), hist_len(g_->hist_len), ids_cur(g_->ids_cur), step(g_->step) {
-      const size_t pitch = (size_t)g->c.max_tokens * g->c.hd * g->es * g->c.Hkv;
-      for (LayerW& L : g->L) {
-        kv.push_back({L.cK, L.cV});
-        L.cK = (char*)L.cK + (size_t)slot * pitch;
-        L.cV = (char*)L.cV + (size_t)slot * pitch;
+    Gpt* g; std::vector<std::pair<void**, void*>> kv; int *hist, *hist_len, *ids_cur; uint32_t step;
+    View(Gpt* g_, int slot) : g(g_), hist(g_->hist), hist_len(g_->hist_len), ids_cur(g_->ids_cur), step(g_->step) {
+      for (const CachePart& p : cache_parts(g)) {
+        kv.push_back({p.base, *p.base});
+        *p.base = (char*)*p.base + (size_t)slot * p.seq_bytes(g);
       }
       g->hist += (size_t)slot * g->c.max_tokens;
       g->hist_len += slot;
@@ -1982,46 +2201,66 @@ int TSB200_GptSlotExtend(void* h, int slot, const int32_t* ids, int S, const TSB
       g->step = (uint32_t)g->steps_v[slot];
     }
     ~View() {
-      for (size_t k = 0; k < kv.size(); ++k) { g->L[k].cK = kv[k].first; g->L[k].cV = kv[k].second; }
+      for (auto& k : kv) *k.first = k.second;
       g->hist = hist; g->hist_len = hist_len; g->ids_cur = ids_cur; g->seq0 = 0; g->step = step;
       g->ids_in = nullptr;
+      g->want_rows = nullptr; g->n_want = 0; g->want_logits = nullptr;
     }
   };
   int ok = 1;
   {
     // the device state is set for the whole batch first (the commit kernel counts the sequence's step there)
-    if (!upload_blocked(g, opt) || !set_state(g, 0)) { cudaFree(ids_dev); return 0; }
+    if ((opt && !upload_blocked(g, opt)) || !set_state(g, 0)) { cudaFree(ids_dev); return 0; }
     View view(g, slot);
     g->ids_in = (int*)ids_dev;
-    TSB200DecodingOptions o2 = *opt;
-    o2.seq_base += (uint64_t)slot;
     const int len = T0 + S;
     do {
       if (cudaMemcpyAsync(ids_dev, ids, (size_t)S * 4, cudaMemcpyHostToDevice, g->s) != cudaSuccess ||
           cudaMemcpyAsync(g->hist + T0, ids_dev, (size_t)S * 4, cudaMemcpyDeviceToDevice, g->s) != cudaSuccess ||
           cudaMemcpyAsync(g->hist_len, &len, 4, cudaMemcpyHostToDevice, g->s) != cudaSuccess ||
-          cudaStreamSynchronize(g->s) != cudaSuccess) { ok = 0; set_last_error("gpt_slot_extend: upload failed"); break; }
+          (n_want > 0 && cudaMemcpyAsync(g->want_list, want, (size_t)n_want * 4, cudaMemcpyHostToDevice, g->s) != cudaSuccess) ||
+          cudaStreamSynchronize(g->s) != cudaSuccess) { ok = 0; set_last_error("%s: upload failed", who); break; }
+      if (!opt) { g->want_rows = g->want_list; g->n_want = n_want; g->want_logits = g->want_out; }
       const long long l0 = g->st->launches;
       cudaEventRecord(g->ev0, g->s);
       if (!(ok = enqueue_forward(g, 1, S, T0, false, 1))) break;
-      if (!(ok = enqueue_sample(g, 1, &o2, false, false))) break;
-      // the sequence's logits also go to its own row of the logits buffer
-      if (slot != 0) cudaMemcpyAsync(g->logits + (size_t)slot * c.V, g->logits, (size_t)c.V * 4, cudaMemcpyDeviceToDevice, g->s);
+      if (opt) {
+        TSB200DecodingOptions o2 = *opt;
+        o2.seq_base += (uint64_t)slot;
+        if (!(ok = enqueue_sample(g, 1, &o2, false, false))) break;
+        // the sequence's logits also go to its own row of the logits buffer
+        if (slot != 0) cudaMemcpyAsync(g->logits + (size_t)slot * c.V, g->logits, (size_t)c.V * 4, cudaMemcpyDeviceToDevice, g->s);
+      }
       cudaEventRecord(g->ev1, g->s);
-      if (cudaStreamSynchronize(g->s) != cudaSuccess) { ok = 0; set_last_error("gpt_slot_extend: %s", cudaGetErrorString(cudaGetLastError())); break; }
+      if (cudaStreamSynchronize(g->s) != cudaSuccess) { ok = 0; set_last_error("%s: %s", who, cudaGetErrorString(cudaGetLastError())); break; }
       cudaEventElapsedTime(&g->last_ms, g->ev0, g->ev1);
       if (!(ok = check_err_flag(g))) break;
       g->last_launches = g->st->launches - l0;
-      if (out_id && cudaMemcpy(out_id, g->out_dev, 4, cudaMemcpyDeviceToHost) != cudaSuccess) { ok = 0; set_last_error("gpt_slot_extend: id download failed"); break; }
+      if (opt && out_id && cudaMemcpy(out_id, g->out_dev, 4, cudaMemcpyDeviceToHost) != cudaSuccess) { ok = 0; set_last_error("%s: id download failed", who); break; }
+      if (n_want > 0 && cudaMemcpy(logits, g->want_out, (size_t)n_want * c.V * 4, cudaMemcpyDeviceToHost) != cudaSuccess) { ok = 0; set_last_error("%s: logits download failed", who); break; }
     } while (0);
   }
   cudaFree(ids_dev);
   if (!ok) return 0;
   g->Ts[slot] = T0 + S;
-  g->steps_v[slot] += 1;
+  if (opt) g->steps_v[slot] += 1;
   refresh_ragged(g);
   g->probs_valid = false;
   return 1;
+}
+
+int TSB200_GptSlotExtend(void* h, int slot, const int32_t* ids, int S, const TSB200DecodingOptions* opt, int32_t* out_id) {
+  NvtxRange nvtx_("tsb200.gpt.slot_extend");
+  Gpt* g = (Gpt*)h;
+  TSB_CHECK(g && ids && opt, "gpt_slot_extend: null argument");
+  return slot_run(g, slot, ids, S, opt, out_id, nullptr, 0, nullptr, "gpt_slot_extend");
+}
+
+int TSB200_GptSlotLogits(void* h, int slot, const int32_t* ids, int S, const int32_t* want, int n_want, float* logits) {
+  NvtxRange nvtx_("tsb200.gpt.slot_logits");
+  Gpt* g = (Gpt*)h;
+  TSB_CHECK(g && ids && n_want >= 0 && (n_want == 0 || (want && logits)), "gpt_slot_logits: null argument");
+  return slot_run(g, slot, ids, S, nullptr, nullptr, want, n_want, logits, "gpt_slot_logits");
 }
 
 int TSB200_GptLastTiming(void* h, float* ms, int64_t* launches) {
@@ -2043,6 +2282,10 @@ int TSB200_GptStepBytes(void* h, int B, int T, int64_t* bytes) {
   Gpt* g = (Gpt*)h;
   TSB_CHECK(g && bytes, "gpt_step_bytes: null argument");
   const TSB200GptConfig& c = g->c;
+  if (g->ly) {
+    *bytes = layered_step_bytes(g, B, T);
+    return 1;
+  }
   const int64_t d = c.d, F = c.F, V = c.V, Hd = (int64_t)c.H * c.hd, KVd = (int64_t)c.Hkv * c.hd, s = g->es;
   const int64_t p_attn = d * (Hd + 2 * KVd) + Hd * d;
   const int64_t p_ffn = (g->glu ? 3 : 2) * d * F;
@@ -2244,15 +2487,15 @@ int TSB200_GptBeamCopy(void* h, const int32_t* src, const int32_t* dst, int n) {
     for (int j = 0; j < n; ++j) TSB_CHECK(dst[j] != src[i], "gpt_beam_copy: sequence %d is both a source and a destination", src[i]);
     for (int j = 0; j < i; ++j) TSB_CHECK(dst[j] != dst[i], "gpt_beam_copy: destination %d named twice", dst[i]);
   }
-  if (!g->beam_layers) {
-    TSB_TRY(dev_alloc(g, (void**)&g->beam_layers, (int64_t)2 * c.L * sizeof(void*)));
+  if (!g->beam_pieces) {
+    std::vector<SeqPiece> pc;
+    for (const CachePart& p : cache_parts(g))
+      for (int h = 0; h < p.heads; ++h)
+        pc.push_back({(unsigned char*)*p.base + (size_t)h * c.max_tokens * p.row_bytes, (long long)p.seq_bytes(g), (long long)p.row_bytes, (long long)p.state_bytes});
+    TSB_TRY(dev_alloc(g, (void**)&g->beam_pieces, (int64_t)pc.size() * sizeof(SeqPiece)));
     TSB_TRY(dev_alloc(g, (void**)&g->beam_pairs, (int64_t)2 * c.max_batch * 4));
-    std::vector<void*> lp((size_t)2 * c.L);
-    for (int k = 0; k < c.L; ++k) {
-      lp[2 * k] = g->L[k].cK;
-      lp[2 * k + 1] = g->L[k].cV;
-    }
-    TSB_CUDA(cudaMemcpy(g->beam_layers, lp.data(), lp.size() * sizeof(void*), cudaMemcpyHostToDevice));
+    TSB_CUDA(cudaMemcpy(g->beam_pieces, pc.data(), pc.size() * sizeof(SeqPiece), cudaMemcpyHostToDevice));
+    g->n_beam_pieces = (int)pc.size();
   }
   std::vector<int> pairs((size_t)2 * n);
   int Tmax = 0;
@@ -2265,11 +2508,8 @@ int TSB200_GptBeamCopy(void* h, const int32_t* src, const int32_t* dst, int n) {
     Tmax = g->Ts[src[i]] > Tmax ? g->Ts[src[i]] : Tmax;
   }
   TSB_CUDA(cudaMemcpyAsync(g->beam_pairs, pairs.data(), pairs.size() * 4, cudaMemcpyHostToDevice, g->s));
-  const int64_t head_pitch = (int64_t)c.max_tokens * c.hd * g->es;
-  const int64_t head_bytes = (((int64_t)Tmax * c.hd * g->es) + 15) / 16 * 16;   // rows of 16-byte multiples (hd * es is one)
   if (Tmax > 0)
-    seq_copy_kernel<<<dim3(n, 2 * c.L * c.Hkv), 256, 0, g->s>>>(g->beam_layers, g->beam_pairs, c.Hkv, head_pitch * c.Hkv, head_pitch, head_bytes,
-                                                                  g->hist, g->hist_len, g->ids_cur, c.max_tokens);
+    seq_copy_kernel<<<dim3(n, g->n_beam_pieces), 256, 0, g->s>>>(g->beam_pieces, g->beam_pairs, Tmax, c.max_tokens, g->hist, g->hist_len, g->ids_cur, c.max_tokens);
   count_launch(c.device);
   TSB_TRY(check_launch("seq_copy"));
   TSB_CUDA(cudaStreamSynchronize(g->s));   // `pairs` is pageable
@@ -2311,7 +2551,8 @@ int TSB200_GptProfileDecode(void* h, int n_steps, const TSB200DecodingOptions* o
   TSB_TRY(set_state(g, 0));
   int Tp = 256;
   while (Tp < g->T + n_steps) Tp <<= 1;
-  const int splits = attn_pick_splits(g->st, c.dtype, g->B, c.H, c.Hkv, c.hd, Tp);
+  if (g->ly) TSB_TRY(ensure_layered(g, g->B, 1, Tp));
+  const int splits = g->ly ? Tp : attn_pick_splits(g->st, c.dtype, g->B, c.H, c.Hkv, c.hd, Tp);
   TSB_TRY(ensure_stack(g, g->B));
   g->prof = true;
   g->prof_n = 0;

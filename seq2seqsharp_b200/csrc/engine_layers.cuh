@@ -1,0 +1,523 @@
+// Layered engines: models whose layers are described one by one (TSB200LayerDesc) instead of by one shape for all.  Part of
+// engine.cu: the same Gpt object, cache manager, slots, snapshots, captured decode step and sampling serve both kinds; this
+// file holds what differs - weights, cache rows, scratch and the forward pass.
+//
+// A layer (residual stream x in fp32):
+//   block norm   h1, h2 = two weights on one group-wise RMS norm of x (the previous layer's expert outputs join x here);
+//                hc = h1 + short convolution of h1
+//   one linear   gate1 = sigmoid(h1 G1 + b1), gate2 = sigmoid(h2 G2 + b2), q | dkv = hc W: three sections of one packed matrix,
+//                one launch up to 16 rows
+//   append       latent norm, rotation, cache row (or only the query's rotation when the layer reads another layer's cache)
+//   attention    latent attention over the cache rows (ops_latent.cu)
+//   out          x += gate1 * (attn W_o)
+//   experts      two grouped products over rows sorted by expert; their outputs wait for the next block norm
+#pragma once
+
+namespace tsb {
+
+struct LayeredLayer {
+  TSB200LayerDesc d;
+  LatentShape sh;
+  int Nq = 0, Nkv = 0;            // columns of q and dkv (0: the layer reads another layer's cache)
+  int ct_gate2 = 0, ct_qkv = 0;   // first column tile of the sections of `fused`
+  const float2* tab = nullptr;
+  void *norm1 = nullptr, *norm2 = nullptr, *conv_w = nullptr, *g1b = nullptr, *g2b = nullptr;
+  void *fused = nullptr, *kv_norm = nullptr, *uk = nullptr, *uv = nullptr, *ukv = nullptr, *wo = nullptr;
+  void *up = nullptr, *down = nullptr;   // [experts] packed matrices, columns of `up` are interleaved (gate, up) pairs
+  int64_t up_bytes = 0, down_bytes = 0;
+  int* table = nullptr;
+  void* cache = nullptr;          // [max_batch][max_tokens][row]; null: kv_from's
+  void* ring = nullptr;           // [max_batch][taps][d]
+  RouteLayer route{};             // host copy of the routing scratch
+  int route_index = -1;
+};
+
+struct Layered {
+  TSB200LayeredConfig c;
+  std::vector<LayeredLayer> L;
+  std::set<std::string> missing;  // weights not given yet
+  int n_route = 0, max_experts = 0;
+  // scratch, grown on demand (ensure_layered)
+  struct Buf { void* p = nullptr; int64_t bytes = 0; };
+  Buf hcat, gate1, gate2, qkv, attn, hs, hidden, y, q_lat, part, kv, ints, routes, ws;
+  int64_t route_rows = 0;
+  int route_block = 0;
+};
+
+template <typename TD, typename TS>
+__global__ void convert_kernel(TD* dst, const TS* src, int64_t n) {
+  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) dst[i] = from_f<TD>(to_f<TS>(src[i]));
+}
+static int convert_into(Gpt* g, void* dst, const void* src, int src_dtype, int64_t n) {
+  const int gsz = (int)((n + 255) / 256 < 4096 ? (n + 255) / 256 : 4096);
+  if (g->c.dtype == TSB200_BF16 && src_dtype == TSB200_BF16) convert_kernel<<<gsz, 256, 0, g->s>>>((__nv_bfloat16*)dst, (const __nv_bfloat16*)src, n);
+  else if (g->c.dtype == TSB200_BF16 && src_dtype == TSB200_F32) convert_kernel<<<gsz, 256, 0, g->s>>>((__nv_bfloat16*)dst, (const float*)src, n);
+  else if (g->c.dtype == TSB200_F32 && src_dtype == TSB200_BF16) convert_kernel<<<gsz, 256, 0, g->s>>>((float*)dst, (const __nv_bfloat16*)src, n);
+  else if (g->c.dtype == TSB200_F32 && src_dtype == TSB200_F32) convert_kernel<<<gsz, 256, 0, g->s>>>((float*)dst, (const float*)src, n);
+  else TSB_FAIL("layered engine: weights are F32 or BF16 tensors");
+  count_launch(g->c.device);
+  return check_launch("convert");
+}
+
+// Every weight of the model by name with its shape ([out, in] for matrices); "table" tensors are int32.
+static std::vector<std::pair<std::string, std::pair<int64_t, int64_t>>> layered_weights(const Layered* ly) {
+  std::vector<std::pair<std::string, std::pair<int64_t, int64_t>>> v;
+  const int64_t d = ly->c.d, V = ly->c.V;
+  auto add = [&](const std::string& n, int64_t r, int64_t c) { v.push_back({n, {r, c}}); };
+  add("embed", V, d);
+  add("final_norm", 1, d);
+  for (size_t i = 0; i < ly->L.size(); ++i) {
+    const LayeredLayer& L = ly->L[i];
+    const std::string p = "layer." + std::to_string(i) + ".";
+    add(p + "norm1", 1, d);
+    add(p + "conv1", d, ly->c.conv_taps);
+    add(p + "gate1.w", d, d);
+    add(p + "gate1.b", 1, d);
+    add(p + "attn.q", L.Nq, d);
+    if (L.Nkv) {
+      add(p + "attn.dkv", L.Nkv, d);
+      add(p + "attn.dkv_norm", 1, L.sh.rank);
+    }
+    add(p + "attn.uk", (int64_t)L.sh.H * L.sh.dim, L.sh.rank);
+    add(p + "attn.uv", (int64_t)L.sh.H * L.sh.vdim, L.sh.rank);
+    add(p + "attn.o", d, (int64_t)L.sh.H * L.sh.vdim);
+    if (L.d.experts > 0) {
+      add(p + "norm2", 1, d);
+      add(p + "gate2.w", d, d);
+      add(p + "gate2.b", 1, d);
+      add(p + "experts.table", V, L.d.top);
+      for (int e = 0; e < L.d.experts; ++e) {
+        const std::string q = p + "experts." + std::to_string(e) + ".";
+        add(q + "gate", L.d.ff, d);
+        add(q + "up", L.d.ff, d);
+        add(q + "down", d, L.d.ff);
+      }
+    }
+  }
+  return v;
+}
+
+// One weight from device memory (src) into its place(s).
+static int layered_put(Gpt* g, const std::string& name, const void* src, int dt, int64_t rows, int64_t cols) {
+  Layered* ly = g->ly;
+  const int dev = g->c.device, T = g->c.dtype, d = ly->c.d;
+  const int64_t n = rows * cols;
+  auto pack = [&](void* dst, int N, int K, int Kp, int c0, int cs) {   // [N, K] (out x in) -> columns c0 + j cs of a packed [Kp, ..] matrix
+    return launch_pack(dev, g->st, T, dst, dt, src, K, N, K, Kp, c0, cs, g->s, true);
+  };
+  if (name == "embed") {
+    TSB_TRY(convert_into(g, g->E, src, dt, n));
+    return pack(g->head_w, ly->c.V, d, d, 0, 1);
+  }
+  if (name == "final_norm") return convert_into(g, g->nf_g, src, dt, n);
+  int i = -1, used = 0;
+  TSB_CHECK(std::sscanf(name.c_str(), "layer.%d.%n", &i, &used) == 1 && used > 0 && i >= 0 && i < (int)ly->L.size(), "unknown weight name '%s'", name.c_str());
+  LayeredLayer& L = ly->L[i];
+  const std::string f = name.substr(used);
+  const int NT = packed_tile_cols(T);
+  if (f == "norm1") return convert_into(g, L.norm1, src, dt, n);
+  if (f == "norm2") return convert_into(g, L.norm2, src, dt, n);
+  if (f == "conv1") return convert_into(g, L.conv_w, src, dt, n);
+  if (f == "gate1.w") return pack(L.fused, d, d, d, 0, 1);
+  if (f == "gate1.b") return convert_into(g, L.g1b, src, dt, n);
+  if (f == "gate2.w") return pack(L.fused, d, d, d, L.ct_gate2 * NT, 1);
+  if (f == "gate2.b") return convert_into(g, L.g2b, src, dt, n);
+  if (f == "attn.q") return pack(L.fused, L.Nq, d, d, L.ct_qkv * NT, 1);
+  if (f == "attn.dkv") return pack(L.fused, L.Nkv, d, d, L.ct_qkv * NT + L.Nq, 1);
+  if (f == "attn.dkv_norm") return convert_into(g, L.kv_norm, src, dt, n);
+  if (f == "attn.uk") {
+    TSB_TRY(convert_into(g, L.uk, src, dt, n));
+    return pack(L.ukv, L.sh.H * L.sh.dim, L.sh.rank, L.sh.row, 0, 1);
+  }
+  if (f == "attn.uv") {
+    TSB_TRY(convert_into(g, L.uv, src, dt, n));
+    return pack(L.ukv, L.sh.H * L.sh.vdim, L.sh.rank, L.sh.row, L.sh.H * L.sh.dim, 1);
+  }
+  if (f == "attn.o") return pack(L.wo, d, L.sh.H * L.sh.vdim, L.sh.H * L.sh.vdim, 0, 1);
+  if (f == "experts.table") {
+    TSB_CUDA(cudaMemcpyAsync(L.table, src, (size_t)n * 4, cudaMemcpyDeviceToDevice, g->s));
+    return 1;
+  }
+  int e = -1, at = 0;
+  TSB_CHECK(std::sscanf(f.c_str(), "experts.%d.%n", &e, &at) == 1 && at > 0 && e >= 0 && e < L.d.experts, "unknown weight name '%s'", name.c_str());
+  const std::string w = f.substr(at);
+  if (w == "gate") return pack((char*)L.up + e * L.up_bytes, L.d.ff, d, d, 0, 2);
+  if (w == "up") return pack((char*)L.up + e * L.up_bytes, L.d.ff, d, d, 1, 2);
+  if (w == "down") return pack((char*)L.down + e * L.down_bytes, d, L.d.ff, L.d.ff, 0, 1);
+  TSB_FAIL("unknown weight name '%s'", name.c_str());
+}
+
+static int layered_check_table(const LayeredLayer& L, const int32_t* t, int64_t rows) {
+  for (int64_t r = 0; r < rows; ++r)
+    for (int j = 0; j < L.d.top; ++j)
+      TSB_CHECK(t[r * L.d.top + j] >= 0 && t[r * L.d.top + j] < L.d.experts, "expert table: entry %d of token %lld names expert %d of %d", j, (long long)r,
+                t[r * L.d.top + j], L.d.experts);
+  return 1;
+}
+
+static int layered_set_weight(Gpt* g, const char* name, const void* data, int dtype, int64_t rows, int64_t cols, int on_device) {
+  Layered* ly = g->ly;
+  int64_t er = 0, ec = 0;
+  for (auto& w : layered_weights(ly))
+    if (w.first == name) {
+      er = w.second.first;
+      ec = w.second.second;
+      break;
+    }
+  TSB_CHECK(er > 0, "unknown weight name '%s'", name);
+  TSB_CHECK(rows == er && cols == ec, "gpt_set_weight: '%s' expects [%lld, %lld], got [%lld, %lld]", name, (long long)er, (long long)ec, (long long)rows,
+            (long long)cols);
+  const bool table = ends_with(name, "experts.table");
+  TSB_CHECK(table ? dtype == TSB200_I32 : (dtype == TSB200_F32 || dtype == TSB200_BF16), "gpt_set_weight: '%s' has an unsupported element type", name);
+  const int64_t bytes = rows * cols * (int64_t)dtype_size(dtype);
+  if (table) {
+    std::vector<int32_t> host;
+    const int32_t* t = (const int32_t*)data;
+    if (on_device) {
+      host.resize((size_t)(rows * cols));
+      TSB_CUDA(cudaMemcpy(host.data(), data, (size_t)bytes, cudaMemcpyDeviceToHost));
+      t = host.data();
+    }
+    int i = -1;
+    std::sscanf(name, "layer.%d.", &i);
+    TSB_TRY(layered_check_table(ly->L[i], t, rows));
+  }
+  const void* src = data;
+  void* tmp = nullptr;
+  if (!on_device) {
+    cudaError_t e = cudaMalloc(&tmp, (size_t)bytes);
+    if (e != cudaSuccess) {
+      cudaGetLastError();
+      TSB_FAIL("OOM: staging buffer of %lld bytes: %s", (long long)bytes, cudaGetErrorString(e));
+    }
+    if (cudaMemcpyAsync(tmp, data, (size_t)bytes, cudaMemcpyHostToDevice, g->s) != cudaSuccess) {
+      cudaFree(tmp);
+      TSB_FAIL("gpt_set_weight: host to device copy failed: %s", cudaGetErrorString(cudaGetLastError()));
+    }
+    src = tmp;
+  }
+  int ok = layered_put(g, name, src, dtype, rows, cols);
+  if (cudaStreamSynchronize(g->s) != cudaSuccess && ok) {
+    set_last_error("gpt_set_weight: %s", cudaGetErrorString(cudaGetLastError()));
+    ok = 0;
+  }
+  if (tmp) cudaFree(tmp);
+  if (ok) ly->missing.erase(name);
+  return ok;
+}
+
+// matrices N(0, std), biases N(0, bias_std), norm gains 1, tables by a hash of (token, choice)
+static int layered_fill_synthetic(Gpt* g, uint64_t seed, float std, float bias_std) {
+  Layered* ly = g->ly;
+  int64_t most = 1;
+  const auto all = layered_weights(ly);
+  for (auto& w : all) most = std::max(most, w.second.first * w.second.second);
+  void* tmp = nullptr;
+  if (cudaMalloc(&tmp, (size_t)most * 4) != cudaSuccess) {
+    cudaGetLastError();
+    TSB_FAIL("OOM: synthetic staging buffer of %lld bytes", (long long)most * 4);
+  }
+  int ok = 1;
+  std::vector<int32_t> host;
+  for (auto& w : all) {
+    const std::string& n = w.first;
+    const int64_t r = w.second.first, c = w.second.second;
+    int dt = TSB200_F32;
+    if (ends_with(n, "experts.table")) {
+      int i = -1;
+      std::sscanf(n.c_str(), "layer.%d.", &i);
+      const uint64_t E = (uint64_t)ly->L[i].d.experts;
+      host.resize((size_t)(r * c));
+      for (int64_t t = 0; t < r; ++t) {
+        uint64_t h = (seed + 0x9E3779B97F4A7C15ull * (uint64_t)(t + 1) + (uint64_t)i * 0xBF58476D1CE4E5B9ull);
+        h = (h ^ (h >> 30)) * 0xBF58476D1CE4E5B9ull;
+        h = (h ^ (h >> 27)) * 0x94D049BB133111EBull;
+        for (int64_t j = 0; j < c; ++j) host[(size_t)(t * c + j)] = (int32_t)(((h >> 8) + (uint64_t)j) % E);   // neighbours: the entries of a row differ
+      }
+      dt = TSB200_I32;
+      ok = cudaMemcpyAsync(tmp, host.data(), host.size() * 4, cudaMemcpyHostToDevice, g->s) == cudaSuccess;
+      if (!ok) set_last_error("gpt_fill_synthetic: table upload failed");
+    } else if (n == "final_norm" || ends_with(n, "norm1") || ends_with(n, "norm2") || ends_with(n, "dkv_norm")) {
+      fill_const_kernel<float><<<(int)((r * c + 255) / 256), 256, 0, g->s>>>((float*)tmp, r * c, 1.0f);
+    } else {
+      const bool bias = ends_with(n, ".b");
+      if (bias && bias_std <= 0.0f) ok = cudaMemsetAsync(tmp, 0, (size_t)(r * c) * 4, g->s) == cudaSuccess;
+      else ok = launch_synthetic(g->c.device, g->st, tmp, TSB200_F32, r * c, seed, fnv1a64(n.c_str()), bias ? bias_std : std, g->s);
+    }
+    ok = ok && layered_put(g, n, tmp, dt, r, c);
+    if (!ok) break;
+    ly->missing.erase(n);
+    if (dt == TSB200_I32) cudaStreamSynchronize(g->s);   // `host` is reused
+  }
+  if (cudaStreamSynchronize(g->s) != cudaSuccess && ok) {
+    set_last_error("gpt_fill_synthetic: %s", cudaGetErrorString(cudaGetLastError()));
+    ok = 0;
+  }
+  cudaFree(tmp);
+  if (g->gexec) { cudaGraphExecDestroy(g->gexec); g->gexec = nullptr; }
+  return ok;
+}
+
+static int layered_block_rows(const Layered* ly, int rows) {
+  if (rows > 64) return 128;
+  int64_t picks = 0, experts = 1;
+  for (auto& L : ly->L)
+    if (L.d.experts > 0 && (int64_t)rows * L.d.top * experts > picks * L.d.experts) {
+      picks = (int64_t)rows * L.d.top;
+      experts = L.d.experts;
+    }
+  return picks > 4 * experts ? 16 : 8;
+}
+static int layered_max_blocks(int64_t picks, int experts, int block_rows) { return (int)(std::min<int64_t>(picks, experts) + picks / block_rows); }
+
+static int grow(Gpt* g, Layered::Buf& b, int64_t bytes, bool zero = false) {
+  if (bytes <= b.bytes) return 1;
+  if (b.p) TSB_TRY(dev_free(g, b.p));
+  b.p = nullptr;
+  b.bytes = 0;
+  TSB_TRY(dev_alloc(g, &b.p, bytes, zero));
+  b.bytes = bytes;
+  // the captured decode step holds the old buffer as a kernel argument
+  if (g->gexec) { cudaGraphExecDestroy(g->gexec); g->gexec = nullptr; }
+  return 1;
+}
+
+// Scratch of a forward pass over B sequences of S new positions on up to T cached ones (T: after the pass).
+static int ensure_layered(Gpt* g, int B, int S, int T) {
+  Layered* ly = g->ly;
+  const int64_t rows = (int64_t)B * S, d = ly->c.d, es = g->es;
+  const int dt = g->c.dtype;
+  const int br = layered_block_rows(ly, (int)rows);
+  bool big = rows * d * 4 > g->x_bytes;
+  int64_t nq = 0, na = 0, npk = 0, nhid = 0, nlat = 0, npart = 0, nkv = 0, nints = 0;
+  int64_t ws = kWsCounterBytes + 1024;
+  auto lin = [&](int64_t K, int64_t N) {
+    for (int64_t m : {(int64_t)1, std::min<int64_t>(rows, 64)}) {
+      ws = std::max(ws, linear_workspace_bytes((int)m, (int)K, (int)N));
+      if (is_16bit(dt)) ws = std::max(ws, gemm_stream_mma_workspace_bytes((int)m, (int)K, (int)N, g->st->sm_count));
+    }
+  };
+  lin(d, ly->c.V);
+  for (auto& L : ly->L) {
+    nq = std::max(nq, rows * (L.Nq + L.Nkv));
+    na = std::max(na, rows * L.sh.H * L.sh.vdim);
+    if (!latent_expanded(dt, L.sh, L.Nq + L.Nkv, S)) {
+      nlat = std::max(nlat, rows * L.sh.H * L.sh.row);
+      npart = std::max(npart, rows * L.sh.H * latent_pick_splits(g->st, L.sh, B, S, T) * (L.sh.rank + 2));
+    } else {
+      nkv = std::max(nkv, (int64_t)B * T * L.sh.H * (L.sh.dim + L.sh.vdim));
+      for (int64_t m : {(int64_t)16, (int64_t)64})
+        ws = std::max(ws, gemm_stream_mma_workspace_bytes((int)m, L.sh.row, L.sh.H * (L.sh.dim + L.sh.vdim), g->st->sm_count));
+    }
+    if (is_16bit(dt)) ws = std::max(ws, gemm_stream_sections_workspace_bytes((int)std::min<int64_t>(rows, 16), (int)d, (int)(2 * d + L.Nq + L.Nkv), g->st->sm_count));
+    lin(d, d);
+    lin(d, L.Nq + L.Nkv);
+    lin(L.sh.H * L.sh.vdim, d);
+    if (L.d.experts > 0) {
+      const int64_t p = rows * L.d.top;
+      npk = std::max(npk, p);
+      nhid = std::max(nhid, p * L.d.ff);
+      const int mb = layered_max_blocks(p, L.d.experts, br);
+      nints += 2 * p + 4 * (int64_t)mb + 16;
+      if (is_16bit(dt) && br <= 16) {
+        ws = std::max(ws, gemm_stream_grouped_workspace_bytes(br, 2 * L.d.ff, mb, g->st->sm_count));
+        ws = std::max(ws, gemm_stream_grouped_workspace_bytes(br, (int)d, mb, g->st->sm_count));
+      }
+    }
+  }
+  if (is_16bit(dt)) ws = std::max<int64_t>(ws, 64LL << 20);   // split-K partials of the tensor-core GEMM
+  if (big) {
+    TSB_CUDA(cudaStreamSynchronize(g->s));
+    if (g->x) TSB_TRY(dev_free(g, g->x));
+    g->x = nullptr;
+    g->x_bytes = 0;
+    TSB_TRY(dev_alloc(g, (void**)&g->x, rows * d * 4, false));
+    g->x_bytes = rows * d * 4;
+    if (g->gexec) { cudaGraphExecDestroy(g->gexec); g->gexec = nullptr; }
+  }
+  TSB_TRY(grow(g, ly->hcat, 3 * rows * d * es));
+  TSB_TRY(grow(g, ly->gate1, rows * d * es));
+  TSB_TRY(grow(g, ly->gate2, rows * d * es));
+  TSB_TRY(grow(g, ly->qkv, nq * es));
+  TSB_TRY(grow(g, ly->attn, na * es));
+  TSB_TRY(grow(g, ly->hs, npk * d * es));
+  TSB_TRY(grow(g, ly->hidden, nhid * es));
+  TSB_TRY(grow(g, ly->y, npk * d * es));
+  TSB_TRY(grow(g, ly->q_lat, nlat * es));
+  TSB_TRY(grow(g, ly->part, npart * 4));
+  TSB_TRY(grow(g, ly->kv, nkv * es));
+  TSB_TRY(grow(g, ly->ws, ws, true));
+  if (ly->n_route > 0 && (ly->route_rows != rows || ly->route_block != br)) {
+    // routing scratch of every expert layer, laid out for this many rows; the captured step holds pointers into it
+    TSB_TRY(grow(g, ly->ints, nints * 4 + 64));
+    TSB_TRY(grow(g, ly->routes, (int64_t)ly->n_route * sizeof(RouteLayer)));
+    if (g->gexec) { cudaGraphExecDestroy(g->gexec); g->gexec = nullptr; }
+    std::vector<RouteLayer> host((size_t)ly->n_route);
+    int* at = (int*)ly->ints.p;
+    for (auto& L : ly->L) {
+      if (L.d.experts <= 0) continue;
+      const int64_t p = rows * L.d.top;
+      RouteLayer& r = L.route;
+      r.table = L.table;
+      r.top = L.d.top;
+      r.experts = L.d.experts;
+      r.blocks = (RowBlock*)at;   // 16-byte aligned: every piece is a multiple of four ints
+      at += 4 * (int64_t)layered_max_blocks(p, L.d.experts, br);
+      r.n_blocks = at;
+      at += 4;
+      r.pos = at;
+      at += (p + 3) / 4 * 4;
+      r.matrix_of = at;
+      at += (p + 3) / 4 * 4;
+      host[(size_t)L.route_index] = r;
+    }
+    TSB_CUDA(cudaMemcpyAsync(ly->routes.p, host.data(), host.size() * sizeof(RouteLayer), cudaMemcpyHostToDevice, g->s));
+    TSB_CUDA(cudaStreamSynchronize(g->s));   // `host` is pageable
+    ly->route_rows = rows;
+    ly->route_block = br;
+  }
+  return 1;
+}
+
+// Forward pass over B * S new tokens (ids in g->ids_in, or g->ids_cur in a captured step); logits of each sequence's last position
+// to g->logits, or of the rows g->want_rows (device, g->n_want of them) to g->want_logits.  T_plan: the longest cache the splits of
+// the attention are chosen for.
+static int enqueue_layered(Gpt* g, int B, int S, int T0, bool use_state, int T_plan) {
+  NvtxRange nvtx_(S == 1 ? "tsb200.forward.step" : "tsb200.forward.prompt");
+  PdlScope pdl_scope(g->pdl && S == 1);
+  Layered* ly = g->ly;
+  const int dev = g->c.device, dt = g->c.dtype, d = ly->c.d, rows = B * S;
+  const int64_t es = g->es;
+  const int* dT = use_state ? g->state : nullptr;
+  TSB_CHECK(ly->missing.empty(), "layered engine: %d weights have not been given, the first is '%s'", (int)ly->missing.size(), ly->missing.begin()->c_str());
+  const int* ids = (S == 1 && use_state) ? g->ids_cur : g->ids_in;
+  const bool pdl = g->pdl;
+  void *ws = ly->ws.p;
+  const int64_t wsb = ly->ws.bytes;
+  g->lin_syms_used = true;
+  {
+    prof_begin(g, KC_EMBED);
+    const int gsz = rows < g->st->sm_count * 8 ? rows : g->st->sm_count * 8;
+    if (dt == TSB200_F32)
+      TSB_CUDA(launch_k(embed_kernel<float>, dim3(gsz), dim3(256), 0, g->s, g->x, (const float*)g->E, (const float*)nullptr, ids, rows, S, d, g->c.V, ly->c.embed_scale, 0, 0, T0, dT));
+    else
+      TSB_CUDA(launch_k(embed_kernel<__nv_bfloat16>, dim3(gsz), dim3(256), 0, g->s, g->x, (const __nv_bfloat16*)g->E, (const __nv_bfloat16*)nullptr, ids, rows, S, d, g->c.V, ly->c.embed_scale, 0, 0, T0, dT));
+    count_launch(dev);
+    TSB_TRY(check_launch("embed"));
+    TSB_TRY(launch_table_route(dev, (const RouteLayer*)ly->routes.p, ly->n_route, ly->max_experts, ids, rows, g->c.V, ly->route_block, g->s));
+    prof_end(g, KC_EMBED);
+  }
+  char* h1 = (char*)ly->hcat.p;
+  char *h2 = h1 + (int64_t)rows * d * es, *hc = h2 + (int64_t)rows * d * es;
+  const LayeredLayer* prev = nullptr;   // the layer whose expert outputs wait in ly->y
+  auto pending = [&](BlockNormArgs& a) {
+    if (!prev) return;
+    a.y = ly->y.p;
+    a.y_pos = prev->route.pos;
+    a.top = prev->d.top;
+    a.y_gate = ly->gate2.p;
+  };
+  for (auto& L : ly->L) {
+    const LayeredLayer& src = L.Nkv ? L : ly->L[L.d.kv_from];
+    const int KB = (d + 31) / 32, Nqkv = L.Nq + L.Nkv;
+    const bool ff = L.d.experts > 0;
+    BlockNormArgs a{};
+    a.x = g->x; a.d = d; a.groups = ly->c.norm_groups; a.eps = ly->c.eps;
+    a.w1 = L.norm1; a.h1 = h1; a.out_scale = 1.0f;
+    if (ff) {
+      a.w2 = L.norm2; a.h2 = h2; a.h2_sorted = ly->hs.p; a.next_pos = L.route.pos; a.next_top = L.d.top;
+    }
+    pending(a);
+    a.write_x = 1;
+    if (S == 1) {
+      a.conv_w = L.conv_w; a.conv_ring = L.ring; a.hc = hc; a.taps = ly->c.conv_taps; a.T0 = T0; a.state = dT;
+    }
+    PROF(KC_NORM, launch_block_norm(dev, dt, a, rows, g->s));
+    if (S > 1) PROF(KC_NORM, launch_short_conv(dev, g->st, dt, hc, h1, L.conv_w, L.ring, B, S, d, ly->c.conv_taps, T0, dT, g->gather_lens, g->s));
+    // gates and projections
+    {
+      Epilogue e1 = make_ep(L.g1b, nullptr, ly->gate1.p, nullptr, TSB200_ACT_SIGMOID, 0);
+      Epilogue e2 = make_ep(L.g2b, nullptr, ly->gate2.p, nullptr, TSB200_ACT_SIGMOID, 0);
+      Epilogue e3 = make_ep(nullptr, nullptr, ly->qkv.p, nullptr, TSB200_ACT_NONE, 0);
+      int r = 2;
+      if (rows <= 16 && ff) {
+        const LinearSection sec[3] = {{d, e1}, {d, e2}, {Nqkv, e3}};
+        prof_begin(g, KC_LINEAR);
+        r = launch_gemm_stream_sections(dev, g->st, dt, h1, L.fused, rows, d, sec, 3, pdl, ws, wsb, g->s);
+        if (r == 0) return 0;
+        if (r == 1) prof_end(g, KC_LINEAR);
+      }
+      if (r == 2) {
+        PROF(KC_LINEAR, launch_linear(dev, g->st, dt, h1, L.fused, rows, d, d, e1, ws, wsb, g->s, true));
+        if (ff) PROF(KC_LINEAR, launch_linear(dev, g->st, dt, h2, (char*)L.fused + (int64_t)L.ct_gate2 * KB * 16384, rows, d, d, e2, ws, wsb, g->s, true));
+        PROF(KC_LINEAR, launch_linear(dev, g->st, dt, hc, (char*)L.fused + (int64_t)L.ct_qkv * KB * 16384, rows, d, Nqkv, e3, ws, wsb, g->s, true));
+      }
+    }
+    const int64_t seq_stride = (int64_t)g->c.max_tokens * src.sh.row;
+    PROF(KC_ROPE_APPEND, launch_latent_append(dev, dt, L.sh, ly->qkv.p, Nqkv, L.Nkv ? L.Nq : -1, L.kv_norm, ly->c.eps, src.cache, seq_stride, B, S, T0, dT,
+                                              g->c.max_tokens, L.tab, g->s));
+    LatentArgs at{};
+    at.shape = L.sh; at.q = ly->qkv.p; at.q_stride = Nqkv; at.cache = src.cache; at.seq_stride = seq_stride;
+    at.B = B; at.S = S; at.T0 = T0; at.Tmax = g->c.max_tokens; at.state = dT;
+    at.splits = latent_pick_splits(g->st, L.sh, B, S, T_plan);
+    at.uk = L.uk; at.uv = L.uv; at.ukv_packed = L.ukv; at.q_lat = ly->q_lat.p; at.part = (float*)ly->part.p; at.part_elems = ly->part.bytes / 4;
+    at.kv = ly->kv.p; at.kv_elems = ly->kv.bytes / es; at.out = ly->attn.p; at.lin_ws = ws; at.lin_ws_bytes = wsb;
+    PROF(KC_ATTENTION, launch_latent_attention(dev, g->st, dt, at, g->s));
+    {
+      Epilogue e = make_ep(nullptr, g->x, nullptr, g->x, TSB200_ACT_NONE, 0);
+      e.gate = ly->gate1.p;
+      PROF(KC_LINEAR, launch_linear(dev, g->st, dt, ly->attn.p, L.wo, rows, L.sh.H * L.sh.vdim, d, e, ws, wsb, g->s, true));
+    }
+    prev = nullptr;
+    if (ff) {
+      const int picks = rows * L.d.top;
+      RowGroups gr{};
+      gr.table = L.route.blocks; gr.n_blocks = L.route.n_blocks;
+      gr.max_blocks = layered_max_blocks(picks, L.d.experts, ly->route_block);
+      auto grouped = [&](const void* x, const void* W, int64_t matrix_bytes, int K, int N, const Epilogue& e) -> int {
+        gr.matrix_bytes = matrix_bytes;
+        int r = 2;
+        if (ly->route_block <= 16) r = launch_gemm_stream_grouped(dev, g->st, dt, x, W, picks, ly->route_block, K, N, e, gr, pdl, ws, wsb, g->s);
+        if (r == 2) r = launch_gemm_tc_grouped(dev, g->st, dt, x, W, picks, K, N, e, gr, g->s);
+        if (r == 2) r = launch_pick_linear(dev, dt, x, W, L.route.matrix_of, matrix_bytes, picks, K, N, e, g->s);
+        return r;
+      };
+      Epilogue eu = make_ep(nullptr, nullptr, ly->hidden.p, nullptr, TSB200_ACT_CLAMP_GLU, 1);
+      eu.glu_limit = L.d.glu_limit; eu.glu_slope = L.d.glu_slope; eu.glu_shift = L.d.glu_shift;
+      PROF(KC_LINEAR, grouped(ly->hs.p, L.up, L.up_bytes, d, 2 * L.d.ff, eu));
+      PROF(KC_LINEAR, grouped(ly->hidden.p, L.down, L.down_bytes, L.d.ff, d, make_ep(nullptr, nullptr, ly->y.p, nullptr, TSB200_ACT_NONE, 0)));
+      prev = &L;
+    }
+  }
+  // final norm on the rows whose logits are asked for, head
+  const int n_out = g->want_rows ? g->n_want : B;
+  if (n_out == 0) return 1;
+  void* hl = g->want_rows ? g->want_h : g->hl;
+  BlockNormArgs a{};
+  a.x = g->x; a.d = d; a.groups = ly->c.norm_groups; a.eps = ly->c.eps; a.w1 = g->nf_g; a.h1 = hl; a.out_scale = ly->c.logit_scale;
+  pending(a);
+  a.rows_of = g->want_rows;
+  if (!g->want_rows && S > 1) { a.last_of_S = S; a.lens = g->gather_lens; }
+  PROF(KC_NORM, launch_block_norm(dev, dt, a, n_out, g->s));
+  PROF(KC_LINEAR, launch_linear(dev, g->st, dt, hl, g->head_w, n_out, d, g->c.V, make_ep(nullptr, nullptr, nullptr, g->want_rows ? g->want_logits : g->logits, TSB200_ACT_NONE, 0),
+                                ws, wsb, g->s, true));
+  return 1;
+}
+
+// bytes a decode step of B sequences at cache length T has to move: weights once (experts: as many as B tokens can name), the
+// cache rows every layer reads and writes, convolution states, logits
+static int64_t layered_step_bytes(const Gpt* g, int B, int T) {
+  const Layered* ly = g->ly;
+  const int64_t d = ly->c.d, es = g->es;
+  int64_t n = d * ly->c.V + d;
+  int64_t total = 0;
+  for (auto& L : ly->L) {
+    const int64_t ex = std::min<int64_t>(L.d.experts, (int64_t)B * std::max(L.d.top, 0));
+    n += (L.d.experts > 0 ? 2 : 1) * d * d + d * (L.Nq + L.Nkv) + (int64_t)L.sh.H * (L.sh.dim + L.sh.vdim) * L.sh.rank + (int64_t)L.sh.H * L.sh.vdim * d +
+         3 * ex * d * L.d.ff + 4 * d + d * ly->c.conv_taps;
+    total += (int64_t)B * T * (L.sh.rank + L.sh.rot) * es + (L.Nkv ? (int64_t)B * L.Nkv * es : 0) + (int64_t)B * ly->c.conv_taps * d * es;
+  }
+  return total + n * es + (int64_t)B * d * es + (int64_t)B * ly->c.V * 4;
+}
+
+}  // namespace tsb

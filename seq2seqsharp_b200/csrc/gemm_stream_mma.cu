@@ -1,4 +1,4 @@
-// Linear layer for decode batches of 5..64 rows on packed fp16 weights: y[M,N] = epilogue(x[M,K] * W[K,N]).
+// Linear layer for decode batches of 5..64 rows on packed fp16 or bf16 weights: y[M,N] = epilogue(x[M,K] * W[K,N]).
 //
 // At these row counts the product is still bound by streaming the weights once (HBM), but there are too many rows
 // for FMA pipes and too few output tiles for a tile-per-CTA tensor-core GEMM (its split-K variants spend most of their
@@ -30,6 +30,15 @@ constexpr int kGsStageBytes = kTileBytes + kGsXBytes;
 // Raised by a kernel whose bounded wait ran out; read and cleared by gs_take_error().
 __device__ int g_gs_error;
 
+// what a launch computes: one linear / several linears of equal K on stacked row blocks / the blocks of a row-grouped product
+constexpr int kGsPlain = 0, kGsSections = 1, kGsGrouped = 2;
+constexpr int kGsMaxSections = 4;
+struct GsSection {
+  int ct_end;   // first column tile after the section
+  int N;
+  Epilogue ep;
+};
+
 struct GsArgs {
   const unsigned char* Wp;
   int M, K, N, KB, CT;
@@ -37,8 +46,8 @@ struct GsArgs {
   int prefetch;             // 1: the first ring-full of weight tiles is requested before the wait on the previous kernel
   // KQ > 0 instantiations: the rows come from the fp32 residual stream and are normed here (no activation tiles by TMA)
   const float* xres;        // [M][K]
-  const __half* gamma;
-  const __half* beta;       // may be null
+  const void* gamma;
+  const void* beta;         // may be null
   int norm_type;            // 0 LayerNorm, 1 RMSNorm
   float eps;
   int rope_on;              // 1: the epilogue rotates q / k and appends k / v to the cache (see RopeFuse)
@@ -47,6 +56,9 @@ struct GsArgs {
   unsigned int* counters;   // [CT], zero on entry, self-resetting
   int* error_flag;
   Epilogue ep;
+  int n_sec;                // kGsSections
+  GsSection sec[kGsMaxSections];
+  RowGroups groups;         // kGsGrouped: CT counts the column tiles of ONE matrix
 };
 
 __device__ __forceinline__ void gs_tma_load_2d(void* dst, const CUtensorMap* map, int c0, int c1, uint64_t* bar) {
@@ -65,33 +77,19 @@ __device__ __forceinline__ void gs_ldmatrix_x4(uint32_t addr, uint32_t& r0, uint
                : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3)
                : "r"(addr));
 }
-__device__ __forceinline__ void gs_mma_16816(float* d, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
 __device__ __forceinline__ unsigned gs_atom_add_acq_rel(unsigned* p, unsigned v) {
   unsigned old;
   asm volatile("atom.acq_rel.gpu.global.add.u32 %0, [%1], %2;" : "=r"(old) : "l"(p), "r"(v) : "memory");
   return old;
 }
 __device__ __forceinline__ void gs_consumers_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
-__device__ __forceinline__ float gs_act(float v, int act) {
-  switch (act) {
-    case TSB200_ACT_RELU: return v < 0.0f ? 0.0f : v;
-    case TSB200_ACT_SILU: return v / (1.0f + expf(-v));
-    case TSB200_ACT_LEAKYRELU: return v < 0.0f ? 0.01f * v : v;
-    case TSB200_ACT_GELU: return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
-    default: return v;
-  }
-}
-
 // KQ == 0: activation rows arrive as TMA tiles beside every weight tile.  KQ > 0 (NB == 1, K == KQ * 1024, M * KQ <= 16): the
 // rows are read from the fp32 residual stream, normed by the consumer warps (LayerNorm / RMSNorm, the arithmetic of
 // norm_kernel) and kept in shared memory as fp16 for the whole kernel - the norm launch in front of the linear disappears and
 // a stage is the weight tile alone.
-template <int NB, int KQ = 0>  // row blocks of 8: M <= 8 * NB
+// MODE kGsSections: column tile ct belongs to section i (the first with ct < ct_end), which reads activation rows i * M ..;
+// MODE kGsGrouped: "column tiles" run over (row block, column tile of its matrix) pairs; how many there are is read from the device.
+template <typename H, int NB, int KQ = 0, int MODE = kGsPlain>  // row blocks of 8: M <= 8 * NB
 __global__ void __launch_bounds__(kStreamThreads, 1) gemm_stream_mma_kernel(const __grid_constant__ CUtensorMap mapX, GsArgs a) {
   constexpr int NT = 256;
   constexpr bool NORM = KQ > 0;
@@ -107,9 +105,7 @@ __global__ void __launch_bounds__(kStreamThreads, 1) gemm_stream_mma_kernel(cons
   __shared__ float s_red[8][16];
 
   const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
-  const int M = a.M, N = a.N, KB = a.KB;
-  const long long U = (long long)KB * a.CT, G = gridDim.x;  // the host launches at most U CTAs: no range is empty
-  const int u_begin = (int)(U * blockIdx.x / G), u_end = (int)(U * (blockIdx.x + 1) / G);
+  const int KB = a.KB;
 
   if (tid == 0) {
     for (int i = 0; i < S; ++i) {
@@ -123,16 +119,45 @@ __global__ void __launch_bounds__(kStreamThreads, 1) gemm_stream_mma_kernel(cons
   __syncthreads();
   grid_dep_launch();
 
+  long long U = (long long)KB * a.CT, G = gridDim.x;  // the host launches at most U CTAs: no range is empty
+  int max_contrib = a.max_contrib;
+  if constexpr (MODE == kGsGrouped) {
+    grid_dep_wait();   // the row blocks come from an earlier kernel
+    U *= min(*a.groups.n_blocks, a.groups.max_blocks);
+    if (G > U) G = U;
+    if (blockIdx.x >= G) return;
+    max_contrib = (int)(KB / (U / G)) + 2;
+  }
+  const int u_begin = (int)(U * blockIdx.x / G), u_end = (int)(U * (blockIdx.x + 1) / G);
+  const int MS = MODE == kGsGrouped ? NB * 8 : a.M;   // rows of a scratch slot
+  // where the weight tiles and the activation rows of "column tile" vct are
+  auto tile_src = [&](int vct) {
+    if constexpr (MODE == kGsGrouped)
+      return a.Wp + (size_t)a.groups.table[vct / a.CT].matrix * a.groups.matrix_bytes + (size_t)(vct % a.CT) * KB * kTileBytes;
+    else
+      return a.Wp + (size_t)vct * KB * kTileBytes;
+  };
+  auto tile_row = [&](int vct) {
+    if constexpr (MODE == kGsGrouped) return a.groups.table[vct / a.CT].row0;
+    if constexpr (MODE == kGsSections) {
+      int i = 0;
+      while (i < a.n_sec - 1 && vct >= a.sec[i].ct_end) ++i;
+      return i * a.M;
+    }
+    return 0;
+  };
+
   if (w == kConsumerWarps) {
     if (lane == 0) {
-      const unsigned char* src = a.Wp + (size_t)u_begin * kTileBytes;
-      int s = 0, kb = u_begin % KB;
+      int s = 0, kb = u_begin % KB, vct = u_begin / KB;
+      const unsigned char* src = tile_src(vct) + (size_t)kb * kTileBytes;
+      int xrow = tile_row(vct);
       unsigned round = 0;
       long long issued = 0;
       // The weights do not depend on the previous kernel: the first ring-full of tiles is requested before the wait on it,
       // so the stream starts while that kernel's last CTAs still reduce and store (and while a norm kernel in between runs).
       constexpr unsigned TX = NORM ? kTileBytes : kTileBytes + NB * 8 * 64;
-      const int n_pre = (a.prefetch || NORM) ? min(S, u_end - u_begin) : 0;
+      const int n_pre = MODE != kGsGrouped && (a.prefetch || NORM) ? min(S, u_end - u_begin) : 0;
       for (int i = 0; i < n_pre; ++i) {
         mbar_expect_tx(&full[i], TX);
         bulk_g2s(smem + (size_t)i * STAGE, src + (size_t)i * kTileBytes, kTileBytes, &full[i]);
@@ -149,10 +174,17 @@ __global__ void __launch_bounds__(kStreamThreads, 1) gemm_stream_mma_kernel(cons
           mbar_expect_tx(&full[s], TX);
           bulk_g2s(dst, src, kTileBytes, &full[s]);
         }
-        if (!NORM) gs_tma_load_2d(dst + kTileBytes, &mapX, kb * kKT, 0, &full[s]);  // x = kb * 32 halves: a 64-byte multiple
+        if (!NORM) gs_tma_load_2d(dst + kTileBytes, &mapX, kb * kKT, xrow, &full[s]);  // x = kb * 32 halves: a 64-byte multiple
         src += kTileBytes;
         ++issued;
-        if (++kb == KB) kb = 0;
+        if (++kb == KB) {
+          kb = 0;
+          ++vct;
+          if (MODE != kGsPlain && u + 1 < u_end) {
+            src = tile_src(vct);
+            xrow = tile_row(vct);
+          }
+        }
         if (++s == S) {
           s = 0;
           ++round;
@@ -240,26 +272,26 @@ __global__ void __launch_bounds__(kStreamThreads, 1) gemm_stream_mma_kernel(cons
 #pragma unroll
     for (int j = 0; j < KQ; ++j) {
       const int c4 = tid + 256 * j;   // float4 index inside a row
-      const __half2 g01 = reinterpret_cast<const __half2*>(a.gamma)[2 * c4], g23 = reinterpret_cast<const __half2*>(a.gamma)[2 * c4 + 1];
-      __half2 b01 = __floats2half2_rn(0.0f, 0.0f), b23 = b01;
+      const uint32_t g01p = reinterpret_cast<const uint32_t*>(a.gamma)[2 * c4], g23p = reinterpret_cast<const uint32_t*>(a.gamma)[2 * c4 + 1];
+      const float2 g01 = Pair16<H>::get(g01p), g23 = Pair16<H>::get(g23p);
+      float2 b01 = make_float2(0.0f, 0.0f), b23 = b01;
       if (a.beta) {
-        b01 = reinterpret_cast<const __half2*>(a.beta)[2 * c4];
-        b23 = reinterpret_cast<const __half2*>(a.beta)[2 * c4 + 1];
+        b01 = Pair16<H>::get(reinterpret_cast<const uint32_t*>(a.beta)[2 * c4]);
+        b23 = Pair16<H>::get(reinterpret_cast<const uint32_t*>(a.beta)[2 * c4 + 1]);
       }
 #pragma unroll
       for (int r = 0; r < 8; ++r) {
         uint2 out = make_uint2(0u, 0u);   // rows beyond M are zero rows of the 8-row operand
         if (r < R && r < M_) {
           const int rr = r < R ? r : 0;
-          float t0 = __low2float(g01) * ((v[rr][j].x - shift[rr]) / inv[rr]), t1 = __high2float(g01) * ((v[rr][j].y - shift[rr]) / inv[rr]);
-          float t2 = __low2float(g23) * ((v[rr][j].z - shift[rr]) / inv[rr]), t3 = __high2float(g23) * ((v[rr][j].w - shift[rr]) / inv[rr]);
+          float t0 = g01.x * ((v[rr][j].x - shift[rr]) / inv[rr]), t1 = g01.y * ((v[rr][j].y - shift[rr]) / inv[rr]);
+          float t2 = g23.x * ((v[rr][j].z - shift[rr]) / inv[rr]), t3 = g23.y * ((v[rr][j].w - shift[rr]) / inv[rr]);
           if (a.beta) {
-            t0 += __low2float(b01); t1 += __high2float(b01);
-            t2 += __low2float(b23); t3 += __high2float(b23);
+            t0 += b01.x; t1 += b01.y;
+            t2 += b23.x; t3 += b23.y;
           }
-          const __half2 h01 = __floats2half2_rn(t0, t1), h23 = __floats2half2_rn(t2, t3);
-          out.x = *reinterpret_cast<const uint32_t*>(&h01);
-          out.y = *reinterpret_cast<const uint32_t*>(&h23);
+          out.x = Pair16<H>::put(t0, t1);
+          out.y = Pair16<H>::put(t2, t3);
         }
         *reinterpret_cast<uint2*>(xs + (size_t)r * XROW + (size_t)c4 * 8) = out;
       }
@@ -281,9 +313,6 @@ __global__ void __launch_bounds__(kStreamThreads, 1) gemm_stream_mma_kernel(cons
 #pragma unroll
       for (int e = 0; e < 4; ++e) d[cb][nb][e] = 0.0f;
 
-  const int max_contrib = a.max_contrib;
-  const Epilogue ep = a.ep;
-  const __half* bias = reinterpret_cast<const __half*>(ep.bias);
   int s = 0;
   unsigned round = 0;
   bool dead = false;
@@ -317,7 +346,7 @@ __global__ void __launch_bounds__(kStreamThreads, 1) gemm_stream_mma_kernel(cons
         uint32_t a0, a1, a2, a3;
         gs_ldmatrix_x4_trans(wbase + k * 128 + ((unit ^ (k & 7)) << 4), a0, a1, a2, a3);
 #pragma unroll
-        for (int nb = 0; nb < NB; ++nb) gs_mma_16816(d[cb][nb], a0, a1, a2, a3, bf[nb][2 * kk], bf[nb][2 * kk + 1]);
+        for (int nb = 0; nb < NB; ++nb) mma_16816<H>(d[cb][nb], a0, a1, a2, a3, bf[nb][2 * kk], bf[nb][2 * kk + 1]);
       }
     }
     __syncwarp();
@@ -339,7 +368,13 @@ __global__ void __launch_bounds__(kStreamThreads, 1) gemm_stream_mma_kernel(cons
     const int c_last = (int)(((ct_last_u + 1) * G + U - 1) / U - 1);
     const int n_contrib = c_last - c_first + 1;
     const int slot = blockIdx.x - c_first;
-    float* mine = a.partials + (((size_t)cur_ct * max_contrib + slot) * M) * NT;
+    int M = a.M, row_base = 0;
+    if constexpr (MODE == kGsGrouped) {
+      const RowBlock rb = a.groups.table[cur_ct / a.CT];
+      M = rb.rows;
+      row_base = rb.row0;
+    }
+    float* mine = a.partials + (((size_t)cur_ct * max_contrib + slot) * MS) * NT;
 #pragma unroll
     for (int cb = 0; cb < 2; ++cb) {
       const int col = chunk * 64 + hf * 32 + cb * 16 + g8;
@@ -361,14 +396,21 @@ __global__ void __launch_bounds__(kStreamThreads, 1) gemm_stream_mma_kernel(cons
     }
     gs_consumers_sync();
     if (*(volatile int*)&s_last) {
-      const float* all = a.partials + ((size_t)cur_ct * max_contrib * M) * NT;
+      const float* all = a.partials + ((size_t)cur_ct * max_contrib * MS) * NT;
+      int si = 0;
+      if constexpr (MODE == kGsSections)
+        while (si < a.n_sec - 1 && cur_ct >= a.sec[si].ct_end) ++si;
+      const Epilogue& ep = MODE == kGsSections ? a.sec[si].ep : a.ep;
+      const int N = MODE == kGsSections ? a.sec[si].N : a.N;
+      const int lct = MODE == kGsSections ? (si ? cur_ct - a.sec[si - 1].ct_end : cur_ct) : (MODE == kGsGrouped ? cur_ct % a.CT : cur_ct);
+      const H* bias = reinterpret_cast<const H*>(ep.bias);
       const int No = ep.glu ? N / 2 : N;
       // work items: (row, group of 4 columns); per item up to eight slots are read at once and added in slot order
       for (int idx = tid; idx < M * 64; idx += 256) {
         {
           float4 sum = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
           const float4* src = reinterpret_cast<const float4*>(all) + idx;
-          const size_t slot_stride = (size_t)M * NT / 4;
+          const size_t slot_stride = (size_t)MS * NT / 4;
           for (int j0 = 0; j0 < n_contrib; j0 += 8) {
             float4 t[8];
 #pragma unroll
@@ -380,7 +422,7 @@ __global__ void __launch_bounds__(kStreamThreads, 1) gemm_stream_mma_kernel(cons
                 sum.x += t[q].x; sum.y += t[q].y; sum.z += t[q].z; sum.w += t[q].w;
               }
           }
-          const int row = idx >> 6, c = cur_ct * NT + (idx & 63) * 4;
+          const int row = row_base + (idx >> 6), c = lct * NT + (idx & 63) * 4;
           const float v[4] = {sum.x, sum.y, sum.z, sum.w};
           if (a.rope_on) {
             // four columns = two rotation pairs of one head (hd and the section boundaries are multiples of four)
@@ -392,21 +434,20 @@ __global__ void __launch_bounds__(kStreamThreads, 1) gemm_stream_mma_kernel(cons
               const int head = cc / rf.hd, e0 = cc % rf.hd;
               float t[4];
 #pragma unroll
-              for (int e = 0; e < 4; ++e) t[e] = __half2float(__float2half_rn(v[e] + (bias ? __half2float(bias[c + e]) : 0.0f)));
+              for (int e = 0; e < 4; ++e) t[e] = to_f<H>(from_f<H>(v[e] + (bias ? to_f<H>(bias[c + e]) : 0.0f)));
               if (rf.use_rope && sec < 2 && pos < rf.Tmax) {
                 const float2 cs0 = rf.tab[(int64_t)pos * (rf.hd / 2) + e0 / 2], cs1 = rf.tab[(int64_t)pos * (rf.hd / 2) + e0 / 2 + 1];
                 const float a0 = t[0], b0 = t[1], a1 = t[2], b1 = t[3];
                 t[0] = a0 * cs0.x - b0 * cs0.y; t[1] = b0 * cs0.x + a0 * cs0.y;
                 t[2] = a1 * cs1.x - b1 * cs1.y; t[3] = b1 * cs1.x + a1 * cs1.y;
               }
-              const __half2 h01 = __floats2half2_rn(t[0], t[1]), h23 = __floats2half2_rn(t[2], t[3]);
               uint2 out;
-              out.x = *reinterpret_cast<const uint32_t*>(&h01);
-              out.y = *reinterpret_cast<const uint32_t*>(&h23);
+              out.x = Pair16<H>::put(t[0], t[1]);
+              out.y = Pair16<H>::put(t[2], t[3]);
               if (sec == 0) {
-                *reinterpret_cast<uint2*>(reinterpret_cast<__half*>(ep.y) + (size_t)row * N + c) = out;
+                *reinterpret_cast<uint2*>(reinterpret_cast<H*>(ep.y) + (size_t)row * N + c) = out;
               } else if (pos < rf.Tmax) {   // capacity is checked on the host; never write past the cache
-                __half* dst = reinterpret_cast<__half*>(sec == 1 ? rf.cK : rf.cV) + (((int64_t)row * (rf.KVd / rf.hd) + head) * rf.Tmax + pos) * rf.hd + e0;
+                H* dst = reinterpret_cast<H*>(sec == 1 ? rf.cK : rf.cV) + (((int64_t)row * (rf.KVd / rf.hd) + head) * rf.Tmax + pos) * rf.hd + e0;
                 *reinterpret_cast<uint2*>(dst) = out;
               }
             }
@@ -414,25 +455,15 @@ __global__ void __launch_bounds__(kStreamThreads, 1) gemm_stream_mma_kernel(cons
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
               if (c + e < N) {
-                float x = gs_act(v[e] + (bias ? __half2float(bias[c + e]) : 0.0f), ep.act);
-                const size_t o = (size_t)row * N + c + e;
-                if (ep.residual) x += ep.residual[o];
-                if (ep.y32) ep.y32[o] = x;
-                else reinterpret_cast<__half*>(ep.y)[o] = __float2half_rn(x);
+                ep_store<H>(ep, (size_t)row * N + c + e, ep_act(v[e] + (bias ? to_f<H>(bias[c + e]) : 0.0f), ep.act));
               }
             }
           } else {
 #pragma unroll
             for (int e = 0; e < 4; e += 2) {
               if (c + e + 1 < N) {
-                float av = v[e] + (bias ? __half2float(bias[c + e]) : 0.0f);
-                const float gv = v[e + 1] + (bias ? __half2float(bias[c + e + 1]) : 0.0f);
-                if (ep.act == TSB200_ACT_SWIGLU) av = av / (1.0f + expf(-av));
-                float x = av * gv;
-                const size_t o = (size_t)row * No + ((c + e) >> 1);
-                if (ep.residual) x += ep.residual[o];
-                if (ep.y32) ep.y32[o] = x;
-                else reinterpret_cast<__half*>(ep.y)[o] = __float2half_rn(x);
+                const float av = v[e] + (bias ? to_f<H>(bias[c + e]) : 0.0f), gv = v[e + 1] + (bias ? to_f<H>(bias[c + e + 1]) : 0.0f);
+                ep_store<H>(ep, (size_t)row * No + ((c + e) >> 1), ep_glu(av, gv, ep));
               }
             }
           }
@@ -469,7 +500,7 @@ struct GcArgs {
   Epilogue ep;
 };
 
-template <int NB>
+template <typename H, int NB>
 __global__ void __launch_bounds__(kGcThreads, 3) gemm_chunk_mma_kernel(const __grid_constant__ CUtensorMap mapX, GcArgs a) {
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
@@ -576,7 +607,7 @@ __global__ void __launch_bounds__(kGcThreads, 3) gemm_chunk_mma_kernel(const __g
           uint32_t a0, a1, a2, a3;
           gs_ldmatrix_x4_trans(wbase + h2 * 4096 + k * 128 + ((unit ^ (k & 7)) << 4), a0, a1, a2, a3);
 #pragma unroll
-          for (int nb = 0; nb < NB; ++nb) gs_mma_16816(d[nb], a0, a1, a2, a3, bf[nb][2 * kk], bf[nb][2 * kk + 1]);
+          for (int nb = 0; nb < NB; ++nb) mma_16816<H>(d[nb], a0, a1, a2, a3, bf[nb][2 * kk], bf[nb][2 * kk + 1]);
         }
       }
       __syncwarp();
@@ -620,7 +651,7 @@ __global__ void __launch_bounds__(kGcThreads, 3) gemm_chunk_mma_kernel(const __g
     }
     if (finish) {
       const Epilogue ep = a.ep;
-      const __half* bias = reinterpret_cast<const __half*>(ep.bias);
+      const H* bias = reinterpret_cast<const H*>(ep.bias);
       const int No = ep.glu ? N / 2 : N;
       for (int idx = tid; idx < M * 16; idx += 128) {
         const int row = idx >> 4, c = ct * 256 + j * 64 + (idx & 15) * 4;
@@ -630,25 +661,15 @@ __global__ void __launch_bounds__(kGcThreads, 3) gemm_chunk_mma_kernel(const __g
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             if (c + e < N) {
-              float x = gs_act(v[e] + (bias ? __half2float(bias[c + e]) : 0.0f), ep.act);
-              const size_t o = (size_t)row * N + c + e;
-              if (ep.residual) x += ep.residual[o];
-              if (ep.y32) ep.y32[o] = x;
-              else reinterpret_cast<__half*>(ep.y)[o] = __float2half_rn(x);
+              ep_store<H>(ep, (size_t)row * N + c + e, ep_act(v[e] + (bias ? to_f<H>(bias[c + e]) : 0.0f), ep.act));
             }
           }
         } else {
 #pragma unroll
           for (int e = 0; e < 4; e += 2) {
             if (c + e + 1 < N) {
-              float av = v[e] + (bias ? __half2float(bias[c + e]) : 0.0f);
-              const float gv = v[e + 1] + (bias ? __half2float(bias[c + e + 1]) : 0.0f);
-              if (ep.act == TSB200_ACT_SWIGLU) av = av / (1.0f + expf(-av));
-              float x = av * gv;
-              const size_t o = (size_t)row * No + ((c + e) >> 1);
-              if (ep.residual) x += ep.residual[o];
-              if (ep.y32) ep.y32[o] = x;
-              else reinterpret_cast<__half*>(ep.y)[o] = __float2half_rn(x);
+              const float av = v[e] + (bias ? to_f<H>(bias[c + e]) : 0.0f), gv = v[e + 1] + (bias ? to_f<H>(bias[c + e + 1]) : 0.0f);
+              ep_store<H>(ep, (size_t)row * No + ((c + e) >> 1), ep_glu(av, gv, ep));
             }
           }
         }
@@ -680,11 +701,15 @@ static GsEncodeTiledFn gs_get_encode() {
   return fn;
 }
 
-template <int NB, int KQ = 0>
+static CUtensorMapDataType gs_map_type(int dtype) {
+  return dtype == TSB200_BF16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
+}
+
+template <typename H, int NB, int KQ = 0, int MODE = kGsPlain>
 static int gs_launch(int device, const CUtensorMap& mapX, const GsArgs& a, int grid, size_t smem, bool pdl, cudaStream_t s) {
   static bool attr_done[kMaxDevices] = {};
   if (!attr_done[device]) {
-    TSB_CUDA(cudaFuncSetAttribute(gemm_stream_mma_kernel<NB, KQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024));
+    TSB_CUDA(cudaFuncSetAttribute(gemm_stream_mma_kernel<H, NB, KQ, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024));
     attr_done[device] = true;
   }
   cudaLaunchConfig_t cfg{};
@@ -697,7 +722,7 @@ static int gs_launch(int device, const CUtensorMap& mapX, const GsArgs& a, int g
   at[0].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = at;
   cfg.numAttrs = (pdl && pdl_enabled()) ? 1 : 0;
-  TSB_CUDA(cudaLaunchKernelEx(&cfg, gemm_stream_mma_kernel<NB, KQ>, mapX, a));
+  TSB_CUDA(cudaLaunchKernelEx(&cfg, gemm_stream_mma_kernel<H, NB, KQ, MODE>, mapX, a));
   count_launch(device);
   return 1;
 }
@@ -736,12 +761,12 @@ static int gs_prefetch_enabled() {
   return on;
 }
 
-template <int NB>
+template <typename H, int NB>
 static int gc_launch(int device, const CUtensorMap& mapX, const GcArgs& a, int grid, bool pdl, cudaStream_t s) {
   static bool attr_done[kMaxDevices] = {};
   const size_t smem = kGcStages * kGcStageBytes + 1024 + 128;
   if (!attr_done[device]) {
-    TSB_CUDA(cudaFuncSetAttribute(gemm_chunk_mma_kernel<NB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    TSB_CUDA(cudaFuncSetAttribute(gemm_chunk_mma_kernel<H, NB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     attr_done[device] = true;
   }
   cudaLaunchConfig_t cfg{};
@@ -754,13 +779,13 @@ static int gc_launch(int device, const CUtensorMap& mapX, const GcArgs& a, int g
   at[0].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = at;
   cfg.numAttrs = (pdl && pdl_enabled()) ? 1 : 0;
-  TSB_CUDA(cudaLaunchKernelEx(&cfg, gemm_chunk_mma_kernel<NB>, mapX, a));
+  TSB_CUDA(cudaLaunchKernelEx(&cfg, gemm_chunk_mma_kernel<H, NB>, mapX, a));
   count_launch(device);
   return 1;
 }
 
 // Column-chunk variant (17..64 rows).  1 ok, 0 error, 2 not handled.
-static int launch_gemm_chunk_mma(int device, DeviceState* st, const void* x, const void* Wp, int M, int K, int N, const Epilogue& ep,
+static int launch_gemm_chunk_mma(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int M, int K, int N, const Epilogue& ep,
                                  int* error_flag, bool pdl, void* ws, int64_t ws_bytes, cudaStream_t s) {
   GsEncodeTiledFn enc = gs_get_encode();
   if (!enc) return 2;
@@ -793,18 +818,18 @@ static int launch_gemm_chunk_mma(int device, DeviceState* st, const void* x, con
     const cuuint64_t strides[1] = {(cuuint64_t)K * 2};
     const cuuint32_t box[2] = {64, (cuuint32_t)(NB * 8)};
     const cuuint32_t el[2] = {1, 1};
-    const CUresult r = enc(&mapX, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(x), dims, strides, box, el,
+    const CUresult r = enc(&mapX, gs_map_type(dtype), 2, const_cast<void*>(x), dims, strides, box, el,
                            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
                            CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     TSB_CHECK(r == CUDA_SUCCESS, "gemm_chunk: cuTensorMapEncodeTiled failed with %d", (int)r);
   }
   const int grid = boxes * ks;
-  if (NB == 4) return gc_launch<4>(device, mapX, a, grid, pdl, s);
-  return gc_launch<8>(device, mapX, a, grid, pdl, s);
+  if (dtype == TSB200_BF16) return NB == 4 ? gc_launch<__nv_bfloat16, 4>(device, mapX, a, grid, pdl, s) : gc_launch<__nv_bfloat16, 8>(device, mapX, a, grid, pdl, s);
+  return NB == 4 ? gc_launch<__half, 4>(device, mapX, a, grid, pdl, s) : gc_launch<__half, 8>(device, mapX, a, grid, pdl, s);
 }
 
 // 1 ok, 0 error, 2 shape not handled (caller falls back).
-int launch_gemm_stream_mma(int device, DeviceState* st, const void* x, const void* Wp, int M, int K, int N, const Epilogue& ep,
+int launch_gemm_stream_mma(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int M, int K, int N, const Epilogue& ep,
                            int* error_flag, bool pdl, void* ws, int64_t ws_bytes, cudaStream_t s) {
   {
     static int enabled = -1;
@@ -822,7 +847,7 @@ int launch_gemm_stream_mma(int device, DeviceState* st, const void* x, const voi
       chunk = (e && e[0] == '0') ? 0 : 1;
     }
     if (chunk) {
-      const int r = launch_gemm_chunk_mma(device, st, x, Wp, M, K, N, ep, error_flag, pdl, ws, ws_bytes, s);
+      const int r = launch_gemm_chunk_mma(device, st, dtype, x, Wp, M, K, N, ep, error_flag, pdl, ws, ws_bytes, s);
       if (r != 2) return r;
     }
   }
@@ -855,18 +880,111 @@ int launch_gemm_stream_mma(int device, DeviceState* st, const void* x, const voi
     const cuuint64_t strides[1] = {(cuuint64_t)K * 2};
     const cuuint32_t box[2] = {32, (cuuint32_t)(NB * 8)};
     const cuuint32_t el[2] = {1, 1};
-    const CUresult r = enc(&mapX, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(x), dims, strides, box, el,
+    const CUresult r = enc(&mapX, gs_map_type(dtype), 2, const_cast<void*>(x), dims, strides, box, el,
                            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_64B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
                            CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     TSB_CHECK(r == CUDA_SUCCESS, "gemm_stream: cuTensorMapEncodeTiled failed with %d", (int)r);
   }
   const size_t smem = fixed + (size_t)stages * kGsStageBytes;
-  switch (NB) {
-    case 1: return gs_launch<1>(device, mapX, a, (int)g, smem, pdl, s);
-    case 2: return gs_launch<2>(device, mapX, a, (int)g, smem, pdl, s);
-    case 4: return gs_launch<4>(device, mapX, a, (int)g, smem, pdl, s);
-    default: return gs_launch<8>(device, mapX, a, (int)g, smem, pdl, s);
+  if (dtype == TSB200_BF16) {
+    if (NB > 2) return 2;   // the column-chunk variant serves more rows of this type
+    return NB == 1 ? gs_launch<__nv_bfloat16, 1>(device, mapX, a, (int)g, smem, pdl, s) : gs_launch<__nv_bfloat16, 2>(device, mapX, a, (int)g, smem, pdl, s);
   }
+  switch (NB) {
+    case 1: return gs_launch<__half, 1>(device, mapX, a, (int)g, smem, pdl, s);
+    case 2: return gs_launch<__half, 2>(device, mapX, a, (int)g, smem, pdl, s);
+    case 4: return gs_launch<__half, 4>(device, mapX, a, (int)g, smem, pdl, s);
+    default: return gs_launch<__half, 8>(device, mapX, a, (int)g, smem, pdl, s);
+  }
+}
+
+// activation tiles [NB * 8 rows][32 k] of a row-major [rows, K] matrix
+static int gs_map_x(CUtensorMap* map, int dtype, const void* x, int rows, int K, int NB) {
+  GsEncodeTiledFn enc = gs_get_encode();
+  if (!enc) return 2;
+  const cuuint64_t dims[2] = {(cuuint64_t)K, (cuuint64_t)rows};
+  const cuuint64_t strides[1] = {(cuuint64_t)K * 2};
+  const cuuint32_t box[2] = {32, (cuuint32_t)(NB * 8)};
+  const cuuint32_t el[2] = {1, 1};
+  const CUresult r = enc(map, gs_map_type(dtype), 2, const_cast<void*>(x), dims, strides, box, el, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                         CU_TENSOR_MAP_SWIZZLE_64B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  TSB_CHECK(r == CUDA_SUCCESS, "gemm_stream: cuTensorMapEncodeTiled failed with %d", (int)r);
+  return 1;
+}
+static size_t gs_ring(GsArgs* a) {   // stages and shared memory of a launch without the norm prologue
+  const size_t fixed = 32 * sizeof(uint64_t) + 1024 + 128;
+  int stages = (int)((225 * 1024 - fixed) / kGsStageBytes);
+  if (stages > 16) stages = 16;
+  a->stages = stages;
+  return fixed + (size_t)stages * kGsStageBytes;
+}
+
+int64_t gemm_stream_sections_workspace_bytes(int M, int K, int total_N, int sm_count) {
+  return gemm_stream_mma_workspace_bytes(M, K, total_N + 256 * kGsMaxSections, sm_count);
+}
+
+int launch_gemm_stream_sections(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int M, int K, const LinearSection* sec,
+                                int n_sec, bool pdl, void* ws, int64_t ws_bytes, cudaStream_t s) {
+  if (dtype != TSB200_BF16 || M < 1 || M > 16 || n_sec < 1 || n_sec > kGsMaxSections || K % 8 != 0 || ((uintptr_t)x % 16) != 0 ||
+      ((uintptr_t)Wp % 16) != 0)
+    return 2;
+  const int NB = M <= 8 ? 1 : 2;
+  GsArgs a{};
+  a.Wp = reinterpret_cast<const unsigned char*>(Wp);
+  a.M = M; a.K = K;
+  a.KB = (K + kKT - 1) / kKT;
+  a.n_sec = n_sec;
+  for (int i = 0; i < n_sec; ++i) {
+    a.CT += (sec[i].N + 255) / 256;
+    a.sec[i].ct_end = a.CT;
+    a.sec[i].N = sec[i].N;
+    a.sec[i].ep = sec[i].ep;
+  }
+  const long long U = (long long)a.KB * a.CT;
+  long long g = st->sm_count;
+  if (g > U) g = U;
+  a.max_contrib = (int)(a.KB / (U / g)) + 2;
+  a.prefetch = gs_prefetch_enabled();
+  const int64_t need = kWsCounterBytes + (int64_t)a.CT * a.max_contrib * M * 256 * 4;
+  if (!ws || ws_bytes < need || (int64_t)a.CT * 4 > kWsCounterBytes - 256) return 2;
+  a.counters = reinterpret_cast<unsigned int*>(ws);
+  a.partials = reinterpret_cast<float*>(reinterpret_cast<char*>(ws) + kWsCounterBytes);
+  CUtensorMap mapX;
+  const int r = gs_map_x(&mapX, dtype, x, n_sec * M, K, NB);
+  if (r != 1) return r;
+  const size_t smem = gs_ring(&a);
+  return NB == 1 ? gs_launch<__nv_bfloat16, 1, 0, kGsSections>(device, mapX, a, (int)g, smem, pdl, s)
+                 : gs_launch<__nv_bfloat16, 2, 0, kGsSections>(device, mapX, a, (int)g, smem, pdl, s);
+}
+
+// slots: every (block, column tile) has KB / per + 2 of them, per = units per CTA >= 1, and units / per <= 2 CTAs
+int64_t gemm_stream_grouped_workspace_bytes(int block_rows, int N, int max_blocks, int sm_count) {
+  const int64_t vct = (int64_t)((N + 255) / 256) * max_blocks;
+  return kWsCounterBytes + (2 * (int64_t)sm_count + 3 * vct) * block_rows * 256 * 4 + 256;
+}
+
+int launch_gemm_stream_grouped(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int rows, int block_rows, int K, int N,
+                               const Epilogue& ep, const RowGroups& groups, bool pdl, void* ws, int64_t ws_bytes, cudaStream_t s) {
+  if (dtype != TSB200_BF16 || (block_rows != 8 && block_rows != 16) || K % 8 != 0 || ((uintptr_t)x % 16) != 0 || ((uintptr_t)Wp % 16) != 0) return 2;
+  GsArgs a{};
+  a.Wp = reinterpret_cast<const unsigned char*>(Wp);
+  a.M = rows; a.K = K; a.N = N;
+  a.KB = (K + kKT - 1) / kKT;
+  a.CT = (N + 255) / 256;
+  a.groups = groups;
+  a.ep = ep;
+  if (!ws || ws_bytes < gemm_stream_grouped_workspace_bytes(block_rows, N, groups.max_blocks, st->sm_count) ||
+      (int64_t)a.CT * groups.max_blocks * 4 > kWsCounterBytes - 256 || (int64_t)a.CT * groups.max_blocks * a.KB > 0x7fffffffLL)
+    return 2;
+  a.counters = reinterpret_cast<unsigned int*>(ws);
+  a.partials = reinterpret_cast<float*>(reinterpret_cast<char*>(ws) + kWsCounterBytes);
+  const int NB = block_rows / 8;
+  CUtensorMap mapX;
+  const int r = gs_map_x(&mapX, dtype, x, rows, K, NB);
+  if (r != 1) return r;
+  const size_t smem = gs_ring(&a);
+  return NB == 1 ? gs_launch<__nv_bfloat16, 1, 0, kGsGrouped>(device, mapX, a, st->sm_count, smem, pdl, s)
+                 : gs_launch<__nv_bfloat16, 2, 0, kGsGrouped>(device, mapX, a, st->sm_count, smem, pdl, s);
 }
 
 // y = epilogue(norm(x32[M,K]) * W[K,N]) in one launch, for up to 8 rows of a fp16 model whose width is 1024, 2048 or 4096
@@ -903,8 +1021,8 @@ int launch_gemm_stream_mma_norm(int device, DeviceState* st, const float* x32, c
   a.stages = stages;
   a.prefetch = 1;
   a.xres = x32;
-  a.gamma = reinterpret_cast<const __half*>(gamma);
-  a.beta = reinterpret_cast<const __half*>(beta);
+  a.gamma = gamma;
+  a.beta = beta;
   a.norm_type = norm_type;
   a.eps = eps;
   if (rope) {
@@ -925,9 +1043,9 @@ int launch_gemm_stream_mma_norm(int device, DeviceState* st, const float* x32, c
   CUtensorMap none{};   // unused by these instantiations
   const size_t smem = fixed + (size_t)stages * kTileBytes;
   switch (KQ) {
-    case 1: return gs_launch<1, 1>(device, none, a, (int)g, smem, pdl, s);
-    case 2: return gs_launch<1, 2>(device, none, a, (int)g, smem, pdl, s);
-    default: return gs_launch<1, 4>(device, none, a, (int)g, smem, pdl, s);
+    case 1: return gs_launch<__half, 1, 1>(device, none, a, (int)g, smem, pdl, s);
+    case 2: return gs_launch<__half, 1, 2>(device, none, a, (int)g, smem, pdl, s);
+    default: return gs_launch<__half, 1, 4>(device, none, a, (int)g, smem, pdl, s);
   }
 }
 

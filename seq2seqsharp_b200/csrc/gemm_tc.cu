@@ -1,4 +1,5 @@
-// Tensor-core GEMM for prefill and large-batch decode: y[M,N] = epilogue(x[M,K] * W[K,N]), fp16 in, fp32 accumulate.
+// Tensor-core GEMM for prefill and large-batch decode: y[M,N] = epilogue(x[M,K] * W[K,N]), fp16 or bf16 in,
+// fp32 accumulate.
 //
 // sm_100a design (5th-generation tensor cores):
 //  * operands are staged in shared memory by TMA tensor copies (cp.async.bulk.tensor, 128-byte swizzle, completion
@@ -117,27 +118,15 @@ struct TcArgs {
 };
 
 // Fused epilogue for 32 consecutive columns of one row: bias first, activation, gate product on interleaved
-// (a_j, g_j) column pairs, fp32 residual, store in fp16 or fp32.
+// (a_j, g_j) column pairs, gate, fp32 residual, store in the model type or fp32.
+template <typename H>
 __device__ __forceinline__ void tc_finish(const TcArgs& a, int row, int col0, const float* v) {
-  const __half* bias = reinterpret_cast<const __half*>(a.ep.bias);
+  const H* bias = reinterpret_cast<const H*>(a.ep.bias);
   if (!a.ep.glu) {
 #pragma unroll
     for (int j = 0; j < 32; ++j) {
       const int col = col0 + j;
-      if (col < a.N) {
-        float x = v[j] + (bias ? __half2float(bias[col]) : 0.0f);
-        switch (a.ep.act) {
-          case TSB200_ACT_RELU: x = x < 0.0f ? 0.0f : x; break;
-          case TSB200_ACT_SILU: x = x / (1.0f + expf(-x)); break;
-          case TSB200_ACT_LEAKYRELU: x = x < 0.0f ? 0.01f * x : x; break;
-          case TSB200_ACT_GELU: x = 0.5f * x * (1.0f + erff(x * 0.70710678118654752f)); break;
-          default: break;
-        }
-        const size_t o = (size_t)row * a.N + col;
-        if (a.ep.residual) x += a.ep.residual[o];
-        if (a.ep.y32) a.ep.y32[o] = x;
-        else reinterpret_cast<__half*>(a.ep.y)[o] = __float2half_rn(x);
-      }
+      if (col < a.N) ep_store<H>(a.ep, (size_t)row * a.N + col, ep_act(v[j] + (bias ? to_f<H>(bias[col]) : 0.0f), a.ep.act));
     }
   } else {
     const int No = a.N / 2;
@@ -145,14 +134,8 @@ __device__ __forceinline__ void tc_finish(const TcArgs& a, int row, int col0, co
     for (int j = 0; j < 32; j += 2) {
       const int col = col0 + j;
       if (col + 1 < a.N) {
-        float av = v[j] + (bias ? __half2float(bias[col]) : 0.0f);
-        const float gv = v[j + 1] + (bias ? __half2float(bias[col + 1]) : 0.0f);
-        if (a.ep.act == TSB200_ACT_SWIGLU) av = av / (1.0f + expf(-av));
-        float x = av * gv;
-        const size_t o = (size_t)row * No + (col >> 1);
-        if (a.ep.residual) x += a.ep.residual[o];
-        if (a.ep.y32) a.ep.y32[o] = x;
-        else reinterpret_cast<__half*>(a.ep.y)[o] = __float2half_rn(x);
+        const float av = v[j] + (bias ? to_f<H>(bias[col]) : 0.0f), gv = v[j + 1] + (bias ? to_f<H>(bias[col + 1]) : 0.0f);
+        ep_store<H>(a.ep, (size_t)row * No + (col >> 1), ep_glu(av, gv, a.ep));
       }
     }
   }
@@ -161,26 +144,18 @@ __device__ __forceinline__ void tc_finish(const TcArgs& a, int row, int col0, co
 // The same epilogue for a full chunk of 32 columns when every pointer is 16-byte aligned and N is a multiple of 32
 // (TcArgs::vec_ok): 16-byte loads of bias and residual, 16-byte stores, i.e. whole 32-byte sectors instead of one
 // 2-byte store per element (scalar stores made the epilogue longer than the mainloop of a 128 x 256 x 4096 tile).
-__device__ __forceinline__ float tc_act(float x, int act) {
-  switch (act) {
-    case TSB200_ACT_RELU: return x < 0.0f ? 0.0f : x;
-    case TSB200_ACT_SILU: return x / (1.0f + expf(-x));
-    case TSB200_ACT_LEAKYRELU: return x < 0.0f ? 0.01f * x : x;
-    case TSB200_ACT_GELU: return 0.5f * x * (1.0f + erff(x * 0.70710678118654752f));
-    default: return x;
-  }
-}
+template <typename H>
 __device__ __forceinline__ void tc_finish_fast(const TcArgs& a, int row, int col0, const float* v) {
   float b[32];
   if (a.ep.bias) {
-    const uint4* bp = reinterpret_cast<const uint4*>(reinterpret_cast<const __half*>(a.ep.bias) + col0);
+    const uint4* bp = reinterpret_cast<const uint4*>(reinterpret_cast<const H*>(a.ep.bias) + col0);
 #pragma unroll
     for (int q = 0; q < 4; ++q) {
       const uint4 t = bp[q];
-      const __half2* h = reinterpret_cast<const __half2*>(&t);
+      const uint32_t h[4] = {t.x, t.y, t.z, t.w};
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const float2 f = __half22float2(h[i]);
+        const float2 f = Pair16<H>::get(h[i]);
         b[q * 8 + 2 * i] = f.x;
         b[q * 8 + 2 * i + 1] = f.y;
       }
@@ -194,19 +169,30 @@ __device__ __forceinline__ void tc_finish_fast(const TcArgs& a, int row, int col
   size_t o;
   if (!a.ep.glu) {
 #pragma unroll
-    for (int j = 0; j < 32; ++j) x[j] = tc_act(v[j] + b[j], a.ep.act);
+    for (int j = 0; j < 32; ++j) x[j] = ep_act(v[j] + b[j], a.ep.act);
     n_out = 32;
     o = (size_t)row * a.N + col0;
   } else {
 #pragma unroll
-    for (int j = 0; j < 16; ++j) {
-      float av = v[2 * j] + b[2 * j];
-      const float gv = v[2 * j + 1] + b[2 * j + 1];
-      if (a.ep.act == TSB200_ACT_SWIGLU) av = av / (1.0f + expf(-av));
-      x[j] = av * gv;
-    }
+    for (int j = 0; j < 16; ++j) x[j] = ep_glu(v[2 * j] + b[2 * j], v[2 * j + 1] + b[2 * j + 1], a.ep);
     n_out = 16;
     o = (size_t)row * (a.N / 2) + (col0 >> 1);
+  }
+  if (a.ep.gate) {
+    const uint4* gp = reinterpret_cast<const uint4*>(reinterpret_cast<const H*>(a.ep.gate) + o);
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      if (q * 8 < n_out) {
+        const uint4 t = gp[q];
+        const uint32_t h[4] = {t.x, t.y, t.z, t.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float2 f = Pair16<H>::get(h[i]);
+          x[q * 8 + 2 * i] *= f.x;
+          x[q * 8 + 2 * i + 1] *= f.y;
+        }
+      }
+    }
   }
   if (a.ep.residual) {
     const float4* rp = reinterpret_cast<const float4*>(a.ep.residual + o);
@@ -224,20 +210,22 @@ __device__ __forceinline__ void tc_finish_fast(const TcArgs& a, int row, int col
     for (int q = 0; q < 8; ++q)
       if (q * 4 < n_out) yp[q] = make_float4(x[q * 4], x[q * 4 + 1], x[q * 4 + 2], x[q * 4 + 3]);
   } else {
-    uint4* yp = reinterpret_cast<uint4*>(reinterpret_cast<__half*>(a.ep.y) + o);
+    uint4* yp = reinterpret_cast<uint4*>(reinterpret_cast<H*>(a.ep.y) + o);
 #pragma unroll
     for (int q = 0; q < 4; ++q) {
       if (q * 8 < n_out) {
         uint4 t;
-        __half2* h = reinterpret_cast<__half2*>(&t);
-#pragma unroll
-        for (int i = 0; i < 4; ++i) h[i] = __floats2half2_rn(x[q * 8 + 2 * i], x[q * 8 + 2 * i + 1]);
+        t.x = Pair16<H>::put(x[q * 8], x[q * 8 + 1]);
+        t.y = Pair16<H>::put(x[q * 8 + 2], x[q * 8 + 3]);
+        t.z = Pair16<H>::put(x[q * 8 + 4], x[q * 8 + 5]);
+        t.w = Pair16<H>::put(x[q * 8 + 6], x[q * 8 + 7]);
         yp[q] = t;
       }
     }
   }
 }
 
+template <typename H>
 __global__ void __launch_bounds__(kTcThreads, 2) gemm_tc_kernel(const __grid_constant__ CUtensorMap mapA, TcArgs a) {
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   // carve: [stages][A 16K][B 16K] (1024-byte aligned for the 128B swizzle atoms), then barriers
@@ -295,8 +283,8 @@ __global__ void __launch_bounds__(kTcThreads, 2) gemm_tc_kernel(const __grid_con
     }
   } else if (w == 1 && lane == 0) {
     // ---------------- MMA issuer
-    // instruction descriptor: D fp32, A/B fp16, A K-major, B MN-major, N = 128, M = 128
-    const uint32_t idesc = (1u << 4) | (0u << 7) | (0u << 10) | (0u << 15) | (1u << 16) | ((uint32_t)(kBN >> 3) << 17) |
+    // instruction descriptor: D fp32, A/B fp16 or bf16, A K-major, B MN-major, N = 128, M = 128
+    const uint32_t idesc = (1u << 4) | (Pair16<H>::kUmmaFormat << 7) | (Pair16<H>::kUmmaFormat << 10) | (0u << 15) | (1u << 16) | ((uint32_t)(kBN >> 3) << 17) |
                            ((uint32_t)(kBM >> 4) << 24);
     for (int it = 0; it < k_iters; ++it) {
       const int s = it % kTcStages, r = it / kTcStages;
@@ -339,8 +327,8 @@ __global__ void __launch_bounds__(kTcThreads, 2) gemm_tc_kernel(const __grid_con
         float f[32];
 #pragma unroll
         for (int j = 0; j < 32; ++j) f[j] = __uint_as_float(v[j]);
-        if (a.vec_ok && n0 + c + 32 <= a.N) tc_finish_fast(a, row, n0 + c, f);
-        else tc_finish(a, row, n0 + c, f);
+        if (a.vec_ok && n0 + c + 32 <= a.N) tc_finish_fast<H>(a, row, n0 + c, f);
+        else tc_finish<H>(a, row, n0 + c, f);
       } else {
         // raw partial sums of this K slice; the last CTA of the tile adds the slices in a fixed order
         float4* dst = reinterpret_cast<float4*>(a.partials + ((size_t)blockIdx.z * a.M + row) * Npad + n0 + c);
@@ -392,8 +380,8 @@ __global__ void __launch_bounds__(kTcThreads, 2) gemm_tc_kernel(const __grid_con
               f[4 * j] += t.x; f[4 * j + 1] += t.y; f[4 * j + 2] += t.z; f[4 * j + 3] += t.w;
             }
           }
-          if (a.vec_ok && n0 + c + 32 <= a.N) tc_finish_fast(a, row, n0 + c, f);
-          else tc_finish(a, row, n0 + c, f);
+          if (a.vec_ok && n0 + c + 32 <= a.N) tc_finish_fast<H>(a, row, n0 + c, f);
+          else tc_finish<H>(a, row, n0 + c, f);
         }
       }
     }
@@ -438,8 +426,12 @@ __device__ __forceinline__ TcTile tc_tile_of(int t, int m_tiles, int n_tiles) {
   return o;
 }
 
+// GROUPED: the row tiles are the blocks of `g` (rows sorted by the matrix they meet): tile m covers rows [row0, row0 + rows) and
+// multiplies them with the packed matrix `matrix`; m_tiles is read from the device.
+template <typename H, bool GROUPED>
 __global__ void __launch_bounds__(kTcThreads, 1) gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap mapA, TcArgs a,
-                                                                           int m_tiles, int n_tiles) {
+                                                                           int m_tiles, int n_tiles, RowGroups g) {
+  if constexpr (GROUPED) m_tiles = min(*g.n_blocks, g.max_blocks);
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   unsigned char* sA = smem;
@@ -483,6 +475,12 @@ __global__ void __launch_bounds__(kTcThreads, 1) gemm_tc_persistent_kernel(const
       const TcTile tl = tc_tile_of(t, m_tiles, n_tiles);
       const int it_begin = 0, it_end = k_total;
       const unsigned char* wsrc = a.Wp + ((size_t)tl.n_tile * a.KB) * 16384;
+      int row0 = tl.m_tile * kBM;
+      if constexpr (GROUPED) {
+        const RowBlock rb = g.table[tl.m_tile];
+        row0 = rb.row0;
+        wsrc += (size_t)rb.matrix * g.matrix_bytes;
+      }
       for (int it = it_begin; it < it_end; ++it, ++it_g) {
         const int s = it_g % kP_Stages, r = it_g / kP_Stages;
         if (it_g >= kP_Stages && !tc_mbar_wait(&empty[s], (unsigned)((r - 1) & 1))) {
@@ -492,15 +490,15 @@ __global__ void __launch_bounds__(kTcThreads, 1) gemm_tc_persistent_kernel(const
         const int kb0 = it * 2;
         const bool two = kb0 + 1 < a.KB;
         tc_mbar_expect_tx(&full[s], kP_ABytes + (two ? 32768 : 16384));
-        tma_load_2d(sA + s * kP_ABytes, &mapA, it * kBK, tl.m_tile * kBM, &full[s]);
+        tma_load_2d(sA + s * kP_ABytes, &mapA, it * kBK, row0, &full[s]);
         tc_bulk_g2s(sB + s * kP_BBytes, wsrc + (size_t)kb0 * 16384, 16384, &full[s]);
         if (two) tc_bulk_g2s(sB + s * kP_BBytes + 16384, wsrc + (size_t)(kb0 + 1) * 16384, 16384, &full[s]);
       }
     }
   } else if (w == 1 && lane == 0) {
     // ---------------- MMA issuer
-    // instruction descriptor: D fp32, A/B fp16, A K-major, B MN-major, N = 256, M = 128
-    const uint32_t idesc = (1u << 4) | (1u << 16) | ((uint32_t)(kP_BN >> 3) << 17) | ((uint32_t)(kBM >> 4) << 24);
+    // instruction descriptor: D fp32, A/B fp16 or bf16, A K-major, B MN-major, N = 256, M = 128
+    const uint32_t idesc = (1u << 4) | (Pair16<H>::kUmmaFormat << 7) | (Pair16<H>::kUmmaFormat << 10) | (1u << 16) | ((uint32_t)(kP_BN >> 3) << 17) | ((uint32_t)(kBM >> 4) << 24);
     int it_g = 0, n_done = 0;
     for (int t = blockIdx.x; t < n_total && !s_err; t += gridDim.x, ++n_done) {
       const int buf = n_done & 1;
@@ -547,9 +545,14 @@ __global__ void __launch_bounds__(kTcThreads, 1) gemm_tc_persistent_kernel(const
         break;
       }
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const int row = tl.m_tile * kBM + q * 32 + lane;
+      int row = tl.m_tile * kBM + q * 32 + lane;
       const int n0 = tl.n_tile * kP_BN;
-      const bool live = row < a.M;
+      bool live = row < a.M;
+      if constexpr (GROUPED) {
+        const RowBlock rb = g.table[tl.m_tile];
+        row = rb.row0 + q * 32 + lane;
+        live = q * 32 + lane < rb.rows && row < a.M;
+      }
 #pragma unroll 1
       for (int c = 0; c < kP_BN; c += 32) {
         uint32_t v[32];
@@ -558,8 +561,8 @@ __global__ void __launch_bounds__(kTcThreads, 1) gemm_tc_persistent_kernel(const
         float f[32];
 #pragma unroll
         for (int j = 0; j < 32; ++j) f[j] = __uint_as_float(v[j]);
-        if (a.vec_ok && n0 + c + 32 <= a.N) tc_finish_fast(a, row, n0 + c, f);
-        else tc_finish(a, row, n0 + c, f);
+        if (a.vec_ok && n0 + c + 32 <= a.N) tc_finish_fast<H>(a, row, n0 + c, f);
+        else tc_finish<H>(a, row, n0 + c, f);
       }
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       __syncwarp();
@@ -603,10 +606,13 @@ static EncodeTiledFn get_encode() {
 int init_tc_attrs(int device) {
   static bool done[kMaxDevices] = {};
   if (done[device]) return 1;
-  TSB_CUDA(cudaFuncSetAttribute(gemm_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                kTcStages * (kABytes + kBBytes) + 1024 + 256));
-  TSB_CUDA(cudaFuncSetAttribute(gemm_tc_persistent_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                kP_Stages * (kP_ABytes + kP_BBytes) + 1024 + 256));
+  const int one = kTcStages * (kABytes + kBBytes) + 1024 + 256, pers = kP_Stages * (kP_ABytes + kP_BBytes) + 1024 + 256;
+  const auto dyn = cudaFuncAttributeMaxDynamicSharedMemorySize;
+  TSB_CUDA(cudaFuncSetAttribute(gemm_tc_kernel<__half>, dyn, one));
+  TSB_CUDA(cudaFuncSetAttribute(gemm_tc_kernel<__nv_bfloat16>, dyn, one));
+  TSB_CUDA(cudaFuncSetAttribute(gemm_tc_persistent_kernel<__half, false>, dyn, pers));
+  TSB_CUDA(cudaFuncSetAttribute(gemm_tc_persistent_kernel<__nv_bfloat16, false>, dyn, pers));
+  TSB_CUDA(cudaFuncSetAttribute(gemm_tc_persistent_kernel<__nv_bfloat16, true>, dyn, pers));
   done[device] = true;
   return 1;
 }
@@ -634,7 +640,42 @@ int64_t gemm_tc_workspace_bytes(int M, int N, int sm_count) {
   return 4096 + kWsCounterBytes + ks * M * (int64_t)((N + kBN - 1) / kBN) * kBN * 4;
 }
 
-int launch_gemm_tc(int device, DeviceState* st, const void* x, const void* Wp, int M, int K, int N, const Epilogue& ep,
+static int tc_map_rows(CUtensorMap* map, int dtype, const void* x, int M, int K) {
+  EncodeTiledFn enc = get_encode();
+  if (!enc) return 2;
+  const cuuint64_t dims[2] = {(cuuint64_t)K, (cuuint64_t)M};
+  const cuuint64_t strides[1] = {(cuuint64_t)K * 2};
+  const cuuint32_t box[2] = {(cuuint32_t)kBK, (cuuint32_t)kBM};
+  const cuuint32_t el[2] = {1, 1};
+  const CUresult r = enc(map, dtype == TSB200_BF16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(x),
+                         dims, strides, box, el, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
+                         CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  TSB_CHECK(r == CUDA_SUCCESS, "gemm_tc: cuTensorMapEncodeTiled(A) failed with %d", (int)r);
+  return 1;
+}
+static int tc_vec_ok(int N, const Epilogue& ep) {
+  const uintptr_t al = (uintptr_t)ep.bias | (uintptr_t)ep.residual | (uintptr_t)ep.y | (uintptr_t)ep.y32 | (uintptr_t)ep.gate;
+  return (N % 32 == 0) && (al % 16 == 0) ? 1 : 0;
+}
+
+int launch_gemm_tc_grouped(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int rows, int K, int N, const Epilogue& ep,
+                           const RowGroups& groups, cudaStream_t s) {
+  if (dtype != TSB200_BF16 || K % 8 != 0 || ((uintptr_t)x % 16) != 0 || ((uintptr_t)Wp % 16) != 0) return 2;
+  TSB_TRY(init_tc_attrs(device));
+  CUtensorMap mapA;
+  const int r = tc_map_rows(&mapA, dtype, x, rows, K);
+  if (r != 1) return r;
+  TcArgs a{};
+  a.M = rows; a.N = N; a.K = K; a.KB = (K + 31) / 32; a.ep = ep; a.ksplit = 1;
+  a.Wp = reinterpret_cast<const unsigned char*>(Wp);
+  a.vec_ok = tc_vec_ok(N, ep);
+  const size_t smem_p = kP_Stages * (kP_ABytes + kP_BBytes) + 1024 + 256;
+  gemm_tc_persistent_kernel<__nv_bfloat16, true><<<st->sm_count, kTcThreads, smem_p, s>>>(mapA, a, 0, (N + kP_BN - 1) / kP_BN, groups);
+  count_launch(device);
+  return check_launch("gemm_tc_grouped");
+}
+
+int launch_gemm_tc(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int M, int K, int N, const Epilogue& ep,
                    int* error_flag, void* ws, int64_t ws_bytes, cudaStream_t s) {
   {
     static int enabled = -1;
@@ -645,28 +686,17 @@ int launch_gemm_tc(int device, DeviceState* st, const void* x, const void* Wp, i
     if (!enabled) return 2;
   }
   if (K % 8 != 0 || ((uintptr_t)x % 16) != 0 || ((uintptr_t)Wp % 16) != 0) return 2;
-  EncodeTiledFn enc = get_encode();
-  if (!enc) return 2;
   TSB_TRY(init_tc_attrs(device));
   const int KB = (K + 31) / 32;
   CUtensorMap mapA;
   {
-    const cuuint64_t dims[2] = {(cuuint64_t)K, (cuuint64_t)M};
-    const cuuint64_t strides[1] = {(cuuint64_t)K * 2};
-    const cuuint32_t box[2] = {(cuuint32_t)kBK, (cuuint32_t)kBM};
-    const cuuint32_t el[2] = {1, 1};
-    const CUresult r = enc(&mapA, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(x), dims, strides, box, el,
-                           CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
-                           CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-    TSB_CHECK(r == CUDA_SUCCESS, "gemm_tc: cuTensorMapEncodeTiled(A) failed with %d", (int)r);
+    const int r = tc_map_rows(&mapA, dtype, x, M, K);
+    if (r != 1) return r;
   }
   TcArgs a{};
   a.M = M; a.N = N; a.K = K; a.KB = KB; a.error_flag = error_flag; a.ep = ep;
   a.Wp = reinterpret_cast<const unsigned char*>(Wp);
-  {
-    const uintptr_t al = (uintptr_t)ep.bias | (uintptr_t)ep.residual | (uintptr_t)ep.y | (uintptr_t)ep.y32;
-    a.vec_ok = (N % 32 == 0) && (al % 16 == 0) ? 1 : 0;
-  }
+  a.vec_ok = tc_vec_ok(N, ep);
   {
     // large M: persistent 128 x 256 tiles with a double-buffered accumulator
     static int pers = -1;
@@ -680,7 +710,8 @@ int launch_gemm_tc(int device, DeviceState* st, const void* x, const void* Wp, i
       a.ksplit = 1;
       int g = st->sm_count;
       const size_t smem_p = kP_Stages * (kP_ABytes + kP_BBytes) + 1024 + 256;
-      gemm_tc_persistent_kernel<<<g, kTcThreads, smem_p, s>>>(mapA, a, m_tiles, n_tiles);
+      if (dtype == TSB200_BF16) gemm_tc_persistent_kernel<__nv_bfloat16, false><<<g, kTcThreads, smem_p, s>>>(mapA, a, m_tiles, n_tiles, RowGroups{});
+      else gemm_tc_persistent_kernel<__half, false><<<g, kTcThreads, smem_p, s>>>(mapA, a, m_tiles, n_tiles, RowGroups{});
       count_launch(device);
       return check_launch("gemm_tc_persistent");
     }
@@ -715,7 +746,8 @@ int launch_gemm_tc(int device, DeviceState* st, const void* x, const void* Wp, i
     }
   }
   const size_t smem = kTcStages * (kABytes + kBBytes) + 1024 + 256;
-  gemm_tc_kernel<<<grid, kTcThreads, smem, s>>>(mapA, a);
+  if (dtype == TSB200_BF16) gemm_tc_kernel<__nv_bfloat16><<<grid, kTcThreads, smem, s>>>(mapA, a);
+  else gemm_tc_kernel<__half><<<grid, kTcThreads, smem, s>>>(mapA, a);
   count_launch(device);
   return check_launch("gemm_tc");
 }

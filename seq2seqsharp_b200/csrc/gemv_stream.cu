@@ -358,17 +358,19 @@ __global__ void __launch_bounds__(kStreamThreads, 1) gemv_stream_kernel(StreamAr
 // ---- packing: row-major logical columns [c0 + j*cs] of a [K, Np] matrix into the tiled layout -----------------------
 template <typename TD, typename TS>
 __global__ void pack_tiles_kernel(TD* __restrict__ dst, const TS* __restrict__ src, int rows, int cols, int src_ld, int KB,
-                                  int NT, int c0, int cs) {
+                                  int NT, int c0, int cs, int transposed, int k0) {
   const long long n = (long long)rows * cols;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
-    const int k = (int)(i / cols), j = (int)(i % cols);
-    const int c = c0 + j * cs;
+    // consecutive threads read consecutive source elements in either orientation
+    const int ks = transposed ? (int)(i % rows) : (int)(i / cols), j = transposed ? (int)(i / rows) : (int)(i % cols);
+    const int c = c0 + j * cs, k = k0 + ks;
     const long long tile = (long long)(c / NT) * KB + (k / kKT);
-    dst[tile * (kKT * NT) + packed_tile_off<TD>(k % kKT, c % NT)] = from_f<TD>(to_f<TS>(src[(long long)k * src_ld + j]));
+    const TS v = transposed ? src[(long long)j * src_ld + ks] : src[(long long)ks * src_ld + j];
+    dst[tile * (kKT * NT) + packed_tile_off<TD>(k % kKT, c % NT)] = from_f<TD>(to_f<TS>(v));
   }
 }
 
-int packed_tile_cols(int dtype) { return dtype == TSB200_F16 ? 256 : 128; }
+int packed_tile_cols(int dtype) { return is_16bit(dtype) ? 256 : 128; }
 int64_t packed_bytes(int dtype, int K, int N) {
   const int NT = packed_tile_cols(dtype);
   const int64_t KB = (K + kKT - 1) / kKT, CT = (N + NT - 1) / NT;
@@ -376,18 +378,21 @@ int64_t packed_bytes(int dtype, int K, int N) {
 }
 
 int launch_pack(int device, DeviceState* st, int dst_dtype, void* dst, int src_dtype, const void* src, int rows, int cols,
-                int src_ld, int K, int c0, int cs, cudaStream_t s) {
+                int src_ld, int K, int c0, int cs, cudaStream_t s, bool transposed, int k0) {
   const int NT = packed_tile_cols(dst_dtype);
   const int KB = (K + kKT - 1) / kKT;
   const long long n = (long long)rows * cols;
   if (n == 0) return 1;
   long long g = (n + 255) / 256;
   if (g > (long long)st->sm_count * 16) g = (long long)st->sm_count * 16;
-#define TSB_PACK(TD, TS) pack_tiles_kernel<TD, TS><<<(int)g, 256, 0, s>>>((TD*)dst, (const TS*)src, rows, cols, src_ld, KB, NT, c0, cs)
+#define TSB_PACK(TD, TS) pack_tiles_kernel<TD, TS><<<(int)g, 256, 0, s>>>((TD*)dst, (const TS*)src, rows, cols, src_ld, KB, NT, c0, cs, transposed ? 1 : 0, k0)
   if (dst_dtype == TSB200_F16 && src_dtype == TSB200_F16) TSB_PACK(__half, __half);
   else if (dst_dtype == TSB200_F16 && src_dtype == TSB200_F32) TSB_PACK(__half, float);
   else if (dst_dtype == TSB200_F32 && src_dtype == TSB200_F32) TSB_PACK(float, float);
   else if (dst_dtype == TSB200_F32 && src_dtype == TSB200_F16) TSB_PACK(float, __half);
+  else if (dst_dtype == TSB200_BF16 && src_dtype == TSB200_BF16) TSB_PACK(__nv_bfloat16, __nv_bfloat16);
+  else if (dst_dtype == TSB200_BF16 && src_dtype == TSB200_F32) TSB_PACK(__nv_bfloat16, float);
+  else if (dst_dtype == TSB200_F32 && src_dtype == TSB200_BF16) TSB_PACK(float, __nv_bfloat16);
   else TSB_FAIL("pack: unsupported dtypes");
 #undef TSB_PACK
   count_launch(device);

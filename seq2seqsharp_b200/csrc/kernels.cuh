@@ -11,7 +11,40 @@ struct Epilogue {
   float* y32;             // [M, N_out] fp32
   int act;                // TSB200_ACT_*
   int glu;                // 1: columns are interleaved (a_j, g_j) pairs, out_j = act(a_j) * g_j, N_out = N/2
+  const void* gate;       // [M, N_out] in T, may be null: the result is multiplied by it before the residual is added
+  // TSB200_ACT_CLAMP_GLU: a' = min(a, limit), g' = clamp(g, -limit, limit), out = a' sigmoid(slope a') (g' + shift)
+  float glu_limit, glu_slope, glu_shift;
 };
+#ifdef __CUDACC__
+// activation and gate of the linear kernels' epilogues
+__device__ __forceinline__ float ep_act(float v, int act) {
+  switch (act) {
+    case TSB200_ACT_RELU: return v < 0.0f ? 0.0f : v;
+    case TSB200_ACT_SILU:
+    case TSB200_ACT_SWIGLU: return v / (1.0f + expf(-v));
+    case TSB200_ACT_LEAKYRELU: return v < 0.0f ? 0.01f * v : v;
+    case TSB200_ACT_GELU: return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
+    case TSB200_ACT_SIGMOID: return 1.0f / (1.0f + expf(-v));
+    default: return v;  // NONE, GLU_NOACT
+  }
+}
+__device__ __forceinline__ float ep_glu(float a, float g, const Epilogue& ep) {
+  if (ep.act == TSB200_ACT_CLAMP_GLU) {
+    a = fminf(a, ep.glu_limit);
+    g = fminf(fmaxf(g, -ep.glu_limit), ep.glu_limit);
+    return a / (1.0f + expf(-ep.glu_slope * a)) * (g + ep.glu_shift);
+  }
+  return ep_act(a, ep.act) * g;
+}
+// one finished value (activation applied) at element o of the output
+template <typename T>
+__device__ __forceinline__ void ep_store(const Epilogue& ep, size_t o, float v) {
+  if (ep.gate) v *= to_f<T>(reinterpret_cast<const T*>(ep.gate)[o]);
+  if (ep.residual) v += ep.residual[o];
+  if (ep.y32) ep.y32[o] = v;
+  else reinterpret_cast<T*>(ep.y)[o] = from_f<T>(v);
+}
+#endif
 
 int launch_norm_residual(int device, DeviceState* st, int dtype, void* h, float* x, const void* delta, const void* gamma,
                          const void* beta, int norm_type, float eps, int M, int d, cudaStream_t s);
@@ -101,6 +134,8 @@ int chk_take_engine();
 int chk_take_attention();
 int chk_take_moe();
 int chk_take_sampling();
+int chk_take_blocks();
+int chk_take_latent();
 
 constexpr int kStackMaxRanks = 8;
 constexpr int kStackXchSites = 4;     // exchange buffers: {out-projection, FFN down} x layer parity
@@ -165,8 +200,9 @@ __host__ __device__ __forceinline__ int packed_tile_off(int k, int c) {
   return k * 128 + c;
 }
 int packed_tile_cols(int dtype);
+// transposed: the source holds [cols, rows] (out x in) instead of [rows, cols]; k0: first row (of K) the block goes to
 int launch_pack(int device, DeviceState* st, int dst_dtype, void* dst, int src_dtype, const void* src, int rows, int cols,
-                int src_ld, int K, int c0, int cs, cudaStream_t s);
+                int src_ld, int K, int c0, int cs, cudaStream_t s, bool transposed = false, int k0 = 0);
 // NCCL binding (comm.cu)
 int comm_all_reduce_f32(void* comm, float* buf, int64_t count, cudaStream_t s);
 int comm_nranks(void* comm);
@@ -177,8 +213,34 @@ int comm_peer_take_error();
 int comm_rank(void* comm);
 int init_stream_attrs(int device);
 // tcgen05/TMEM GEMM on packed fp16 weights (gemm_tc.cu): 1 ok, 0 error, 2 shape not handled
-int launch_gemm_tc(int device, DeviceState* st, const void* x, const void* Wp, int M, int K, int N, const Epilogue& ep,
+int launch_gemm_tc(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int M, int K, int N, const Epilogue& ep,
                    int* error_flag, void* ws, int64_t ws_bytes, cudaStream_t s);
+// Grouped products: the rows of x are sorted by the matrix they meet; `table` (device) lists blocks of rows of one matrix,
+// *n_blocks (device) says how many there are.  Matrix e starts at Wp + e * matrix_bytes.
+struct RowBlock {
+  int matrix, row0, rows, pad;
+};
+struct RowGroups {
+  const RowBlock* table;
+  const int* n_blocks;
+  int max_blocks;          // host bound of *n_blocks
+  int64_t matrix_bytes;
+};
+// blocks of up to 128 rows (tcgen05) / up to 8 or 16 rows (streamed weights, mma.sync).  1 ok, 0 error, 2 shape not handled
+int launch_gemm_tc_grouped(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int rows, int K, int N, const Epilogue& ep,
+                           const RowGroups& groups, cudaStream_t s);
+int launch_gemm_stream_grouped(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int rows, int block_rows, int K, int N,
+                               const Epilogue& ep, const RowGroups& groups, bool pdl, void* ws, int64_t ws_bytes, cudaStream_t s);
+int64_t gemm_stream_grouped_workspace_bytes(int block_rows, int N, int max_blocks, int sm_count);
+// Several linears of equal K in one launch: section i multiplies rows [i * M, (i + 1) * M) of x (stacked [sections * M, K])
+// with columns of its own in Wp (each section starts on a column tile).  At most 16 rows.
+struct LinearSection {
+  int N;
+  Epilogue ep;
+};
+int launch_gemm_stream_sections(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int M, int K, const LinearSection* sec,
+                                int n_sec, bool pdl, void* ws, int64_t ws_bytes, cudaStream_t s);
+int64_t gemm_stream_sections_workspace_bytes(int M, int K, int total_N, int sm_count);
 int64_t gemm_tc_workspace_bytes(int M, int N, int sm_count);
 // stream-K mma.sync GEMM for decode batches of up to 64 rows on packed fp16 weights (gemm_stream_mma.cu)
 // mixture-of-experts feed-forward (ops_moe.cu): x32 += sum over the token's experts of score * W2_e act(W1_e h)
@@ -206,10 +268,91 @@ struct RopeFuse {
 int launch_gemm_stream_mma_norm(int device, DeviceState* st, const float* x32, const void* gamma, const void* beta, int norm_type, float eps,
                                 const void* Wp, int M, int K, int N, const Epilogue& ep, int* error_flag, bool pdl, void* ws, int64_t ws_bytes,
                                 cudaStream_t s, const RopeFuse* rope = nullptr);
-int launch_gemm_stream_mma(int device, DeviceState* st, const void* x, const void* Wp, int M, int K, int N, const Epilogue& ep,
+int launch_gemm_stream_mma(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int M, int K, int N, const Epilogue& ep,
                            int* error_flag, bool pdl, void* ws, int64_t ws_bytes, cudaStream_t s);
 int64_t gemm_stream_mma_workspace_bytes(int M, int K, int N, int sm_count);
 int gs_take_error();
+// ---- blocks of layered engines (ops_blocks.cu) ---------------------------------------------------------------------------
+struct BlockNormArgs {
+  float* x;               // [rows, d] residual stream
+  int d, groups;
+  float eps;
+  const void* w1;         // first norm weight -> h1 (times out_scale)
+  void* h1;
+  float out_scale;
+  const void* w2;         // second norm weight -> h2, both of the same row (may be null)
+  void* h2;
+  void* h2_sorted;        // copies of h2 at rows next_pos[row * next_top + j] (next_top = 0: none)
+  const int* next_pos;
+  int next_top;
+  // pending expert outputs of the previous layer: x += y_gate * mean_j y[y_pos[row * top + j]]; y == null: nothing pending
+  const void* y;
+  const int* y_pos;
+  int top;
+  const void* y_gate;     // may be null (1)
+  int write_x;            // store the sum back into x
+  // which row of x an output row is: rows_of[r], or the last of each sequence's last_of_S rows (lens: their own lengths), or r
+  const int* rows_of;
+  int last_of_S;
+  const int* lens;
+  // one new position per sequence: hc = h1 + causal convolution of h1, state ring [sequences][taps][d]; null: none
+  const void* conv_w;     // [d, taps]
+  void* conv_ring;
+  void* hc;
+  int taps, T0;
+  const int* state;
+};
+int launch_block_norm(int device, int dtype, const BlockNormArgs& a, int out_rows, cudaStream_t s);
+int launch_short_conv(int device, DeviceState* st, int dtype, void* out, const void* h, const void* w, void* ring, int B, int S, int d, int taps,
+                      int T0, const int* state, const int* lens, cudaStream_t s);
+struct RouteLayer {       // one expert layer of table_route_kernel
+  const int* table;       // [vocab, top]
+  int top, experts;
+  int* pos;               // [rows * top] sorted row of every pick
+  int* matrix_of;         // [rows * top] expert of every sorted row
+  RowBlock* blocks;
+  int* n_blocks;
+};
+int launch_table_route(int device, const RouteLayer* layers_dev, int n_layers, int max_experts, const int* ids, int rows, int V, int block_rows,
+                       cudaStream_t s);
+int launch_pick_linear(int device, int dtype, const void* x, const void* Wp, const int* matrix_of, int64_t matrix_bytes, int rows, int K, int N,
+                       const Epilogue& ep, cudaStream_t s);
+// ---- latent attention (ops_latent.cu) -------------------------------------------------------------------------------------
+struct LatentShape {
+  int H, dim, rot, vdim, rank;   // heads, unrotated / rotated query-key size, value size, latent size
+  int rot_dims;                  // how many of the `rot` dimensions turn
+  int row;                       // elements of a cache row: [latent | rotated key part | zeros]
+  float scale;
+};
+inline int latent_row_elems(int rank, int rot) { return (rank + rot + 15) / 16 * 16; }
+// full-precision cos / sin table [Tmax, dims / 2] of base^(-2 i / dims) * position
+int launch_angle_table(int device, DeviceState* st, float2* tab, int Tmax, int dims, double base, cudaStream_t s);
+// per row of q | dkv: the query's rotated parts turned in place, and (dkv_col >= 0) latent norm + rotation + cache append
+int launch_latent_append(int device, int dtype, const LatentShape& a, void* qkv, int row_stride, int dkv_col, const void* norm_w, float eps, void* cache,
+                         int64_t seq_stride, int B, int S, int T0, const int* state, int Tmax, const float2* tab, cudaStream_t s);
+struct LatentArgs {
+  LatentShape shape;
+  const void* q;                 // rows of q | dkv, turned
+  int q_stride;
+  const void* cache;             // [sequences][Tmax][row]
+  int64_t seq_stride;
+  int B, S, T0, Tmax;
+  const int* state;
+  int splits;
+  const void *uk, *uv;           // [H * dim, rank], [H * vdim, rank] row-major in the model type
+  const void* ukv_packed;        // packed [row, H * (dim + vdim)]: latent -> keys | values (zero rows beyond the latent)
+  void* q_lat;                   // scratch [B * S, H, row]
+  float* part;                   // scratch [B * S * H][splits][rank + 2]
+  int64_t part_elems;
+  void* kv;                      // scratch [B][T0 + S][H * (dim + vdim)], expanded form only
+  int64_t kv_elems;
+  void* out;                     // [B * S, H * vdim]
+  void* lin_ws;
+  int64_t lin_ws_bytes;
+};
+int latent_pick_splits(DeviceState* st, const LatentShape& a, int B, int S, int T);
+bool latent_expanded(int dtype, const LatentShape& a, int q_stride, int S);
+int launch_latent_attention(int device, DeviceState* st, int dtype, const LatentArgs& a, cudaStream_t s);
 int init_tc_attrs(int device);
 int tc_take_error();
 int64_t linear_workspace_bytes(int M, int K, int N);

@@ -1,0 +1,372 @@
+// Building blocks of layered engines (engine_layers.cuh) around their linears and attention:
+//   block_norm_kernel    pending expert outputs -> residual, RMS norm in groups with one or two weights from one pass over the
+//                        row, the second result optionally also in the row order of a grouped product, and for one new
+//                        position per sequence the short causal convolution with its state;
+//   short_conv_kernel    the same convolution for many new positions; short_conv_state_kernel then leaves the sequence's last
+//                        inputs in its ring (a kernel of its own: the ring is read by the first positions of a portion);
+//   table_route_kernel   experts chosen by token id: for every layer the picks of all rows sorted by expert, cut into blocks of
+//                        rows of one expert (the unit of the grouped products), all layers in one launch at the start of a step;
+//   pick_linear_kernel   one row times its own expert's matrix on CUDA cores: fp32 models and shapes the grouped
+//                        tensor-core products do not take.
+// Convolution state: a ring of `taps` rows per sequence, position p at row p % taps.  With one row more than the convolution looks
+// back, a step that is run again at the same position (a sequence that stands still while others go on) finds the ring as it was.
+#include "kernels.cuh"
+
+namespace tsb {
+
+TSB_CHECKED_WORD(blocks)
+#ifndef TSB200_CHECKED
+int chk_take_blocks() { return 0; }
+#endif
+
+template <typename T, int V> struct VecIO;   // V consecutive elements
+template <typename T> struct VecIO<T, 1> {
+  static __device__ __forceinline__ void load(const T* p, float* f) { f[0] = to_f<T>(p[0]); }
+  static __device__ __forceinline__ void store(T* p, const float* f) { p[0] = from_f<T>(f[0]); }
+};
+template <> struct VecIO<float, 4> {
+  static __device__ __forceinline__ void load(const float* p, float* f) {
+    const float4 t = *reinterpret_cast<const float4*>(p);
+    f[0] = t.x; f[1] = t.y; f[2] = t.z; f[3] = t.w;
+  }
+  static __device__ __forceinline__ void store(float* p, const float* f) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+};
+template <> struct VecIO<__nv_bfloat16, 4> {
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float* f) {
+    const uint2 t = *reinterpret_cast<const uint2*>(p);
+    const float2 a = Pair16<__nv_bfloat16>::get(t.x), b = Pair16<__nv_bfloat16>::get(t.y);
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float* f) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(Pair16<__nv_bfloat16>::put(f[0], f[1]), Pair16<__nv_bfloat16>::put(f[2], f[3]));
+  }
+};
+
+constexpr int kBlockNormThreads = 256;
+
+// shared memory: the row in fp32 [d], partial sums [max(groups, 8)]
+template <typename T, int V>
+__global__ void __launch_bounds__(kBlockNormThreads) block_norm_kernel(BlockNormArgs a) {
+  extern __shared__ float s_row[];
+  float* s_part = s_row + a.d;
+  pdl_trigger();
+  pdl_wait();
+  const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
+  const int d = a.d, gsz = d / a.groups;
+  const int out_row = blockIdx.x;
+  int row = out_row;
+  if (a.rows_of) row = a.rows_of[out_row];
+  else if (a.last_of_S > 0) {
+    const int n = a.lens ? a.lens[out_row] : a.last_of_S;
+    row = out_row * a.last_of_S + min(max(n, 1), a.last_of_S) - 1;
+  }
+  float* xr = a.x + (int64_t)row * d;
+  const float inv_top = a.top > 0 ? 1.0f / (float)a.top : 0.0f;
+  for (int i = tid * V; i < d; i += kBlockNormThreads * V) {
+    float v[V];
+    VecIO<float, V>::load(xr + i, v);
+    if (a.y) {   // the previous layer's experts: their mean, gated, joins the residual here
+      float sum[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) sum[e] = 0.0f;
+      for (int j = 0; j < a.top; ++j) {
+        float t[V];
+        VecIO<T, V>::load(reinterpret_cast<const T*>(a.y) + (int64_t)a.y_pos[(int64_t)row * a.top + j] * d + i, t);
+#pragma unroll
+        for (int e = 0; e < V; ++e) sum[e] += t[e];
+      }
+      float g[V];
+      if (a.y_gate) VecIO<T, V>::load(reinterpret_cast<const T*>(a.y_gate) + (int64_t)row * d + i, g);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] += sum[e] * inv_top * (a.y_gate ? g[e] : 1.0f);
+      if (a.write_x) VecIO<float, V>::store(xr + i, v);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) s_row[i + e] = v[e];
+  }
+  __syncthreads();
+  // sums of squares: several warps per group when there are few groups, several groups per warp otherwise
+  const int wpg = a.groups >= 8 ? 1 : 8 / a.groups;
+  if (a.groups >= 8) {
+    for (int g = w; g < a.groups; g += 8) {
+      float s = 0.0f;
+      for (int i = lane; i < gsz; i += 32) s += s_row[g * gsz + i] * s_row[g * gsz + i];
+      s = warp_sum(s);
+      if (lane == 0) s_part[g] = s;
+    }
+  } else {
+    const int g = w / wpg, part = w % wpg;
+    float s = 0.0f;
+    if (g < a.groups)
+      for (int i = part * 32 + lane; i < gsz; i += wpg * 32) s += s_row[g * gsz + i] * s_row[g * gsz + i];
+    s = warp_sum(s);
+    if (lane == 0) s_part[w] = s;
+  }
+  __syncthreads();
+  auto inv_rms = [&](int g) {
+    float s = 0.0f;
+    for (int q = 0; q < wpg; ++q) s += s_part[g * wpg + q];
+    return 1.0f / sqrtf(s / (float)gsz + a.eps);
+  };
+  int b = 0, pos = 0;
+  if (a.conv_ring) {
+    b = out_row;
+    pos = state_len(a.state, b, a.T0);
+  }
+  int cur_g = -1;
+  float inv = 0.0f;
+  for (int i = tid * V; i < d; i += kBlockNormThreads * V) {
+    float n[V], h[V], wt[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      const int g = (i + e) / gsz;
+      if (g != cur_g) {
+        cur_g = g;
+        inv = inv_rms(g);
+      }
+      n[e] = s_row[i + e] * inv;
+    }
+    VecIO<T, V>::load(reinterpret_cast<const T*>(a.w1) + i, wt);
+#pragma unroll
+    for (int e = 0; e < V; ++e) h[e] = n[e] * wt[e] * a.out_scale;
+    VecIO<T, V>::store(reinterpret_cast<T*>(a.h1) + (int64_t)out_row * d + i, h);
+    if (a.w2) {
+      float h2[V];
+      VecIO<T, V>::load(reinterpret_cast<const T*>(a.w2) + i, wt);
+#pragma unroll
+      for (int e = 0; e < V; ++e) h2[e] = n[e] * wt[e];
+      VecIO<T, V>::store(reinterpret_cast<T*>(a.h2) + (int64_t)out_row * d + i, h2);
+      for (int j = 0; j < a.next_top; ++j)
+        VecIO<T, V>::store(reinterpret_cast<T*>(a.h2_sorted) + (int64_t)a.next_pos[(int64_t)row * a.next_top + j] * d + i, h2);
+    }
+    if (a.conv_ring) {
+      T* ring = reinterpret_cast<T*>(a.conv_ring) + (int64_t)b * a.taps * d;
+      float out[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        const float hr = to_f<T>(from_f<T>(h[e]));   // the value the state keeps
+        float acc = hr;
+        const T* cw = reinterpret_cast<const T*>(a.conv_w) + (int64_t)(i + e) * a.taps;
+        for (int j = 0; j < a.taps; ++j) {
+          const int p = pos - a.taps + 1 + j;
+          if (p < 0) continue;
+          acc += to_f<T>(cw[j]) * (p == pos ? hr : to_f<T>(ring[(int64_t)(p % a.taps) * d + i + e]));
+        }
+        out[e] = acc;
+      }
+      VecIO<T, V>::store(ring + (int64_t)(pos % a.taps) * d + i, h);
+      VecIO<T, V>::store(reinterpret_cast<T*>(a.hc) + (int64_t)out_row * d + i, out);
+    }
+  }
+}
+
+// out[b, s] = h[b, s] + sum_j w[:, j] h[b, s - taps + 1 + j]; positions before the portion come from the ring, none before 0
+template <typename T>
+__global__ void __launch_bounds__(256) short_conv_kernel(T* out, const T* h, const T* wgt, const T* ring, int B, int S, int d, int taps, int T0_arg,
+                                                         const int* state) {
+  const int64_t n = (int64_t)B * S * d;
+  for (int64_t q = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; q < n; q += (int64_t)gridDim.x * blockDim.x) {
+    const int i = (int)(q % d);
+    const int64_t row = q / d;
+    const int b = (int)(row / S), s = (int)(row % S);
+    const int T0 = state_len(state, b, T0_arg);
+    float acc = to_f<T>(h[q]);
+    for (int j = 0; j < taps; ++j) {
+      const int back = taps - 1 - j, p = T0 + s - back;
+      if (p < 0) continue;
+      const float v = s >= back ? to_f<T>(h[q - (int64_t)back * d]) : to_f<T>(ring[((int64_t)b * taps + p % taps) * d + i]);
+      acc += to_f<T>(wgt[(int64_t)i * taps + j]) * v;
+    }
+    out[q] = from_f<T>(acc);
+  }
+}
+template <typename T>
+__global__ void __launch_bounds__(256) short_conv_state_kernel(T* ring, const T* h, int S, int d, int taps, int T0_arg, const int* state, const int* lens) {
+  const int b = blockIdx.y;
+  const int T0 = state_len(state, b, T0_arg);
+  const int n = lens ? min(max(lens[b], 1), S) : S;
+  const int keep = min(n, taps);
+  for (int q = blockIdx.x * blockDim.x + threadIdx.x; q < keep * d; q += gridDim.x * blockDim.x) {
+    const int s = n - keep + q / d, i = q % d;
+    ring[((int64_t)b * taps + (T0 + s) % taps) * d + i] = h[((int64_t)b * S + s) * d + i];
+  }
+}
+
+// ---- routing by token id ---------------------------------------------------------------------------------------------------
+constexpr int kRouteThreads = 512;
+
+// exclusive prefix sum of s_v[0, n) in place, total returned to every thread; s_tmp: 32 ints
+__device__ __forceinline__ int block_exclusive_scan(int* s_v, int n, int* s_tmp) {
+  const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, nw = kRouteThreads / 32;
+  int carry = 0;
+  for (int base = 0; base < n; base += kRouteThreads) {
+    const int i = base + tid;
+    const int v = i < n ? s_v[i] : 0;
+    int x = v;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int y = __shfl_up_sync(0xffffffffu, x, o);
+      if (lane >= o) x += y;
+    }
+    if (lane == 31) s_tmp[w] = x;
+    __syncthreads();
+    int off = carry, tot = 0;
+    for (int q = 0; q < nw; ++q) {
+      if (q < w) off += s_tmp[q];
+      tot += s_tmp[q];
+    }
+    if (i < n) s_v[i] = off + x - v;
+    carry += tot;
+    __syncthreads();
+  }
+  return carry;
+}
+
+// one CTA per expert layer; dynamic shared memory: 3 * max_experts ints
+__global__ void __launch_bounds__(kRouteThreads) table_route_kernel(const RouteLayer* layers, const int* ids, int rows, int V, int block_rows) {
+  extern __shared__ int s_int[];
+  __shared__ int s_tmp[32];
+  pdl_trigger();
+  pdl_wait();
+  const RouteLayer L = layers[blockIdx.x];
+  const int E = L.experts, top = L.top, n = rows * top, tid = threadIdx.x;
+  int* cnt = s_int;             // picks per expert
+  int* first = s_int + E;       // first sorted row of an expert
+  int* blk = s_int + 2 * E;     // first block of an expert
+  for (int e = tid; e < E; e += kRouteThreads) cnt[e] = 0;
+  __syncthreads();
+  auto expert_of = [&](int p) {
+    int id = ids[p / top];
+    TSB_DEV_CHECK(blocks, id >= 0 && id < V, 0x501, (void)0)   // token id outside the vocabulary (routed as id 0)
+    if (id < 0 || id >= V) id = 0;
+    int e = L.table[(int64_t)id * top + p % top];
+    TSB_DEV_CHECK(blocks, e >= 0 && e < E, 0x502, (void)0)     // the table names an expert that does not exist (checked when it is loaded)
+    return min(max(e, 0), E - 1);
+  };
+  for (int p = tid; p < n; p += kRouteThreads) atomicAdd(&cnt[expert_of(p)], 1);
+  __syncthreads();
+  for (int e = tid; e < E; e += kRouteThreads) {
+    first[e] = cnt[e];
+    blk[e] = (cnt[e] + block_rows - 1) / block_rows;
+  }
+  __syncthreads();
+  block_exclusive_scan(first, E, s_tmp);
+  const int n_blocks = block_exclusive_scan(blk, E, s_tmp);
+  for (int e = tid; e < E; e += kRouteThreads) {
+    for (int q = 0; q * block_rows < cnt[e]; ++q) {
+      RowBlock rb;
+      rb.matrix = e;
+      rb.row0 = first[e] + q * block_rows;
+      rb.rows = min(block_rows, cnt[e] - q * block_rows);
+      rb.pad = 0;
+      L.blocks[blk[e] + q] = rb;
+    }
+  }
+  if (tid == 0) *L.n_blocks = n_blocks;
+  __syncthreads();
+  // the order inside an expert is of no consequence: every row is computed by itself
+  for (int p = tid; p < n; p += kRouteThreads) {
+    const int e = expert_of(p);
+    const int at = atomicAdd(&first[e], 1);
+    L.pos[p] = at;
+    L.matrix_of[at] = e;
+  }
+}
+
+// y[r] = epilogue(x[r] W_{matrix_of[r]}) for packed matrices, two columns per thread
+template <typename T>
+__global__ void __launch_bounds__(128) pick_linear_kernel(const T* x, const T* Wp, const int* matrix_of, int64_t matrix_elems, int K, int N, Epilogue ep) {
+  extern __shared__ float s_x[];
+  constexpr int NT = sizeof(T) == 2 ? 256 : 128;
+  pdl_trigger();
+  pdl_wait();
+  const int r = blockIdx.x, KB = (K + 31) / 32;
+  for (int i = threadIdx.x; i < K; i += 128) s_x[i] = to_f<T>(x[(int64_t)r * K + i]);
+  __syncthreads();
+  const int c = (blockIdx.y * 128 + threadIdx.x) * 2;
+  if (c >= N) return;
+  const T* W = Wp + (int64_t)matrix_of[r] * matrix_elems + (int64_t)(c / NT) * KB * (32 * NT);
+  const int cc = c % NT;
+  float a0 = 0.0f, a1 = 0.0f;
+#pragma unroll 4
+  for (int k = 0; k < K; ++k) {
+    const T* wp = W + (int64_t)(k >> 5) * (32 * NT) + packed_tile_off<T>(k & 31, cc);   // c is even: its neighbour is the next element
+    a0 = fmaf(s_x[k], to_f<T>(wp[0]), a0);
+    a1 = fmaf(s_x[k], to_f<T>(wp[1]), a1);
+  }
+  const T* bias = reinterpret_cast<const T*>(ep.bias);
+  const float b0 = bias ? to_f<T>(bias[c]) : 0.0f, b1 = bias && c + 1 < N ? to_f<T>(bias[c + 1]) : 0.0f;
+  if (ep.glu) {
+    if (c + 1 < N) ep_store<T>(ep, (size_t)r * (N / 2) + (c >> 1), ep_glu(a0 + b0, a1 + b1, ep));
+  } else {
+    ep_store<T>(ep, (size_t)r * N + c, ep_act(a0 + b0, ep.act));
+    if (c + 1 < N) ep_store<T>(ep, (size_t)r * N + c + 1, ep_act(a1 + b1, ep.act));
+  }
+}
+
+// ---- host side -------------------------------------------------------------------------------------------------------------
+int launch_block_norm(int device, int dtype, const BlockNormArgs& a, int out_rows, cudaStream_t s) {
+  if (out_rows == 0) return 1;
+  TSB_CHECK(a.groups >= 1 && a.d % a.groups == 0, "block_norm: a width of %d is not cut into %d groups", a.d, a.groups);
+  const size_t smem = ((size_t)a.d + (a.groups > 8 ? a.groups : 8)) * sizeof(float);
+  TSB_CHECK(smem <= 200 * 1024, "block_norm: rows of %d elements are not supported", a.d);
+  static bool done[kMaxDevices] = {};
+  if (!done[device]) {
+    TSB_CUDA(cudaFuncSetAttribute(block_norm_kernel<float, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    TSB_CUDA(cudaFuncSetAttribute(block_norm_kernel<float, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    TSB_CUDA(cudaFuncSetAttribute(block_norm_kernel<__nv_bfloat16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    TSB_CUDA(cudaFuncSetAttribute(block_norm_kernel<__nv_bfloat16, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    done[device] = true;
+  }
+  const bool v4 = a.d % 4 == 0;
+  if (dtype == TSB200_F32)
+    TSB_CUDA(launch_k(v4 ? block_norm_kernel<float, 4> : block_norm_kernel<float, 1>, dim3(out_rows), dim3(kBlockNormThreads), smem, s, a));
+  else
+    TSB_CUDA(launch_k(v4 ? block_norm_kernel<__nv_bfloat16, 4> : block_norm_kernel<__nv_bfloat16, 1>, dim3(out_rows), dim3(kBlockNormThreads), smem, s, a));
+  count_launch(device);
+  return check_launch("block_norm");
+}
+
+int launch_short_conv(int device, DeviceState* st, int dtype, void* out, const void* h, const void* w, void* ring, int B, int S, int d, int taps,
+                      int T0, const int* state, const int* lens, cudaStream_t s) {
+  int64_t g = ((int64_t)B * S * d + 255) / 256;
+  if (g > (int64_t)st->sm_count * 32) g = (int64_t)st->sm_count * 32;
+  const dim3 g2((unsigned)((taps * d + 255) / 256), B);
+  if (dtype == TSB200_F32) {
+    short_conv_kernel<float><<<(int)g, 256, 0, s>>>((float*)out, (const float*)h, (const float*)w, (const float*)ring, B, S, d, taps, T0, state);
+    short_conv_state_kernel<float><<<g2, 256, 0, s>>>((float*)ring, (const float*)h, S, d, taps, T0, state, lens);
+  } else {
+    typedef __nv_bfloat16 H;
+    short_conv_kernel<H><<<(int)g, 256, 0, s>>>((H*)out, (const H*)h, (const H*)w, (const H*)ring, B, S, d, taps, T0, state);
+    short_conv_state_kernel<H><<<g2, 256, 0, s>>>((H*)ring, (const H*)h, S, d, taps, T0, state, lens);
+  }
+  count_launch(device, 2);
+  return check_launch("short_conv");
+}
+
+int launch_table_route(int device, const RouteLayer* layers_dev, int n_layers, int max_experts, const int* ids, int rows, int V, int block_rows,
+                       cudaStream_t s) {
+  if (n_layers == 0 || rows == 0) return 1;
+  const size_t smem = (size_t)3 * max_experts * sizeof(int);
+  TSB_CHECK(smem <= 48 * 1024, "table_route: %d experts are not supported (at most 4096)", max_experts);
+  TSB_CUDA(launch_k(table_route_kernel, dim3(n_layers), dim3(kRouteThreads), smem, s, layers_dev, ids, rows, V, block_rows));
+  count_launch(device);
+  return check_launch("table_route");
+}
+
+int launch_pick_linear(int device, int dtype, const void* x, const void* Wp, const int* matrix_of, int64_t matrix_bytes, int rows, int K, int N,
+                       const Epilogue& ep, cudaStream_t s) {
+  if (rows == 0) return 1;
+  const size_t smem = (size_t)K * sizeof(float);
+  TSB_CHECK(smem <= 48 * 1024, "pick_linear: rows of %d inputs are not supported", K);
+  const dim3 grid(rows, (N + 255) / 256);
+  if (dtype == TSB200_F32)
+    TSB_CUDA(launch_k(pick_linear_kernel<float>, grid, dim3(128), smem, s, (const float*)x, (const float*)Wp, matrix_of, matrix_bytes / 4, K, N, ep));
+  else
+    TSB_CUDA(launch_k(pick_linear_kernel<__nv_bfloat16>, grid, dim3(128), smem, s, (const __nv_bfloat16*)x, (const __nv_bfloat16*)Wp, matrix_of,
+                      matrix_bytes / 2, K, N, ep));
+  count_launch(device);
+  return check_launch("pick_linear");
+}
+
+}  // namespace tsb

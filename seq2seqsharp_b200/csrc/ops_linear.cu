@@ -13,24 +13,6 @@
 namespace tsb {
 
 
-__device__ __forceinline__ float apply_act(int act, float v) {
-  switch (act) {
-    case TSB200_ACT_RELU: return v < 0.0f ? 0.0f : v;
-    case TSB200_ACT_SILU:
-    case TSB200_ACT_SWIGLU: return v / (1.0f + expf(-v));
-    case TSB200_ACT_LEAKYRELU: return v < 0.0f ? 0.01f * v : v;
-    case TSB200_ACT_GELU: return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
-    default: return v;  // NONE, GLU_NOACT
-  }
-}
-
-template <typename T>
-__device__ __forceinline__ void store_out(const Epilogue& ep, int64_t idx, float v) {
-  if (ep.residual) v += ep.residual[idx];
-  if (ep.y32) ep.y32[idx] = v;
-  else reinterpret_cast<T*>(ep.y)[idx] = from_f<T>(v);
-}
-
 template <typename T> struct WVec;
 template <> struct WVec<__half> {
   static constexpr int N = 8;
@@ -42,6 +24,21 @@ template <> struct WVec<__half> {
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const float2 t = __half22float2(h[i]);
+      f[2 * i] = t.x;
+      f[2 * i + 1] = t.y;
+    }
+  }
+};
+template <> struct WVec<__nv_bfloat16> {
+  static constexpr int N = 8;
+  uint4 raw;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { raw = __ldg(reinterpret_cast<const uint4*>(p)); }
+  __device__ __forceinline__ void zero() { raw = make_uint4(0, 0, 0, 0); }
+  __device__ __forceinline__ void get(float* f) const {
+    const uint32_t r[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 t = Pair16<__nv_bfloat16>::get(r[i]);
       f[2 * i] = t.x;
       f[2 * i + 1] = t.y;
     }
@@ -155,8 +152,7 @@ __global__ void __launch_bounds__(kGemvThreads) gemv_kernel(const T* __restrict_
       const int m = i / NT, c = ct * NT + (i % NT);
       if (c < N) {
         float v = red[i] + (bias ? to_f<T>(bias[c]) : 0.0f);
-        v = apply_act(ep.act, v);
-        store_out<T>(ep, (int64_t)m * N + c, v);
+        ep_store<T>(ep, (size_t)m * N + c, ep_act(v, ep.act));
       }
     }
   } else {
@@ -167,7 +163,7 @@ __global__ void __launch_bounds__(kGemvThreads) gemv_kernel(const T* __restrict_
       if (c + 1 < N) {
         const float a = red[m * NT + 2 * j] + (bias ? to_f<T>(bias[c]) : 0.0f);
         const float g = red[m * NT + 2 * j + 1] + (bias ? to_f<T>(bias[c + 1]) : 0.0f);
-        store_out<T>(ep, (int64_t)m * No + (c >> 1), apply_act(ep.act, a) * g);
+        ep_store<T>(ep, (size_t)m * No + (c >> 1), ep_glu(a, g, ep));
       }
     }
   }
@@ -252,7 +248,7 @@ __global__ void __launch_bounds__(256) gemm_generic_kernel(GemmArgs g, Epilogue 
           const int n = n0 + tx * 4 + j;
           if (n < g.N) {
             float v = acc[i][j] + (bias ? to_f<T>(bias[n]) : 0.0f);
-            store_out<T>(ep, (int64_t)m * g.N + n, apply_act(ep.act, v));
+            ep_store<T>(ep, (size_t)m * g.N + n, ep_act(v, ep.act));
           }
         }
       } else {
@@ -262,7 +258,7 @@ __global__ void __launch_bounds__(256) gemm_generic_kernel(GemmArgs g, Epilogue 
           if (n + 1 < g.N) {
             const float a = acc[i][j] + (bias ? to_f<T>(bias[n]) : 0.0f);
             const float gg = acc[i][j + 1] + (bias ? to_f<T>(bias[n + 1]) : 0.0f);
-            store_out<T>(ep, (int64_t)m * (g.N / 2) + (n >> 1), apply_act(ep.act, a) * gg);
+            ep_store<T>(ep, (size_t)m * (g.N / 2) + (n >> 1), ep_glu(a, gg, ep));
           }
         }
       }
@@ -313,7 +309,7 @@ static int gemv_attr(int) {
 int init_linear_attrs(int device) {
   static bool done[kMaxDevices] = {};
   if (done[device]) return 1;
-#define TSB_ATTR(M) TSB_TRY((gemv_attr<float, M>(device))); TSB_TRY((gemv_attr<__half, M>(device)))
+#define TSB_ATTR(M) TSB_TRY((gemv_attr<float, M>(device))); TSB_TRY((gemv_attr<__half, M>(device))); TSB_TRY((gemv_attr<__nv_bfloat16, M>(device)))
   TSB_ATTR(1); TSB_ATTR(2); TSB_ATTR(3); TSB_ATTR(4); TSB_ATTR(5); TSB_ATTR(6); TSB_ATTR(7); TSB_ATTR(8);
 #undef TSB_ATTR
   done[device] = true;
@@ -356,21 +352,21 @@ static int launch_generic(int device, const GemmArgs& g, const Epilogue* ep, cud
 int launch_linear(int device, DeviceState* st, int dtype, const void* x, const void* W, int M, int K, int N,
                   const Epilogue& ep, void* ws, int64_t ws_bytes, cudaStream_t s, bool packed) {
   if (M == 0) return 1;
-  const int vec = dtype == TSB200_F16 ? 8 : 4;
+  const int vec = is_16bit(dtype) ? 8 : 4;
   const int packedKB = packed ? (K + 31) / 32 : 0;
   if (packed && dtype == TSB200_F16 && M > 16 && M <= 64) {
     // 17..64 rows: the weights stream once through tcgen05 with the activation rows as the N dimension
     const int r = launch_gemm_stream_tc(device, st, x, W, M, K, N, ep, nullptr, true, ws, ws_bytes, s);
     if (r != 2) return r;
   }
-  if (packed && dtype == TSB200_F16 && M >= 1 && M <= 64) {
+  if (packed && is_16bit(dtype) && M >= 1 && M <= 64) {
     // decode batches: weights streamed once through a ring, mma.sync consumers (measured: for 33..64 rows and wide
     // outputs the split-K tcgen05 kernel below is faster, its partial sums being a smaller share of the traffic)
-    const int r = launch_gemm_stream_mma(device, st, x, W, M, K, N, ep, nullptr, true, ws, ws_bytes, s);
+    const int r = launch_gemm_stream_mma(device, st, dtype, x, W, M, K, N, ep, nullptr, true, ws, ws_bytes, s);
     if (r != 2) return r;
   }
-  if (packed && dtype == TSB200_F16 && M > 16) {
-    const int r = launch_gemm_tc(device, st, x, W, M, K, N, ep, nullptr, ws, ws_bytes, s);
+  if (packed && is_16bit(dtype) && M > 16) {
+    const int r = launch_gemm_tc(device, st, dtype, x, W, M, K, N, ep, nullptr, ws, ws_bytes, s);
     if (r != 2) return r;
   }
   const bool gemv_ok = (packed || N % vec == 0) && (((uintptr_t)W % 16) == 0) && M <= 16;
@@ -381,7 +377,8 @@ int launch_linear(int device, DeviceState* st, int dtype, const void* x, const v
       const int No = ep.glu ? N / 2 : N;
       if (e2.residual) e2.residual += (int64_t)m0 * No;
       if (e2.y32) e2.y32 += (int64_t)m0 * No;
-      if (e2.y) e2.y = (char*)e2.y + (int64_t)m0 * No * (dtype == TSB200_F16 ? 2 : 4);
+      if (e2.y) e2.y = (char*)e2.y + (int64_t)m0 * No * (is_16bit(dtype) ? 2 : 4);
+      if (e2.gate) e2.gate = (const char*)e2.gate + (int64_t)m0 * No * (is_16bit(dtype) ? 2 : 4);
 #define TSB_GEMV(T, MM) launch_gemv_m<T, MM>(device, st, (const T*)x + (int64_t)m0 * K, (const T*)W, K, N, e2, ws, ws_bytes, s, packedKB)
 #define TSB_GEMV_SW(T)                                  \
   switch (mb) {                                         \
@@ -394,7 +391,7 @@ int launch_linear(int device, DeviceState* st, int dtype, const void* x, const v
     case 7: TSB_TRY(TSB_GEMV(T, 7)); break;             \
     default: TSB_TRY(TSB_GEMV(T, 8)); break;            \
   }
-      if (dtype == TSB200_F16) { TSB_GEMV_SW(__half) } else { TSB_GEMV_SW(float) }
+      if (dtype == TSB200_F16) { TSB_GEMV_SW(__half) } else if (dtype == TSB200_BF16) { TSB_GEMV_SW(__nv_bfloat16) } else { TSB_GEMV_SW(float) }
 #undef TSB_GEMV_SW
 #undef TSB_GEMV
     }
@@ -408,6 +405,7 @@ int launch_linear(int device, DeviceState* st, int dtype, const void* x, const v
   g.b_packedKB = packedKB;
   g.b_NT = 32 * vec;
   if (dtype == TSB200_F16) return launch_generic<__half>(device, g, &ep, s);
+  if (dtype == TSB200_BF16) return launch_generic<__nv_bfloat16>(device, g, &ep, s);
   return launch_generic<float>(device, g, &ep, s);
 }
 

@@ -230,7 +230,7 @@ class GPT:
         self.tp_rank, self.tp_size = tp_rank, tp_size
         self._h = C.c_void_p()
         N.call("TSB200_GptCreate", C.byref(c), C.byref(self._h))
-        self._keep = None
+        self._keep, self._B = None, 0
 
     def InitComm(self, group=None, peer=True):
         """Creates the NCCL communicator of the tensor-parallel group: rank 0 makes the id, torch.distributed (any
@@ -400,6 +400,16 @@ class GPT:
                out.ctypes.data_as(C.c_void_p))
         self._B = max(self._B, slot + 1)
         return int(out[0])
+
+    def SlotLogits(self, slot: int, tokens, want=()) -> np.ndarray:
+        """Runs `tokens` on top of what the slot holds without sampling; logits [len(want), V] at the places `want` of the portion."""
+        ids = np.ascontiguousarray(np.asarray(tokens, dtype=np.int32).reshape(-1))
+        w = np.ascontiguousarray(np.asarray(list(want), dtype=np.int32))
+        out = np.empty((w.size, self.cfg.V), dtype=np.float32)
+        N.call("TSB200_GptSlotLogits", self._h, int(slot), ids.ctypes.data_as(C.c_void_p), int(ids.size), w.ctypes.data_as(C.c_void_p), int(w.size),
+               out.ctypes.data_as(C.c_void_p))
+        self._B = max(self._B, slot + 1)
+        return out
 
     def Decode(self, n_steps: int, opts: DecodingOptions, stop_on_eos: bool = False):
         out = np.zeros((self._B, n_steps), dtype=np.int32)
