@@ -15,6 +15,8 @@ Workloads (synthetic seeded weights and prompts of the named shapes; no dataset 
     c4_b4   the same 1B-class model, B=4, 16384-token prompts, greedy (long-context KV-cache stress)
     c1      tiny fp32 model, B=1, prompt 32, greedy
 
+`--design pepilix` measures prefill and decode of a layered design at a few sizes beside the closest uniform model instead (one GPU).
+
 With N > 1 the 7B-class workloads (c5_*) run ONE model tensor-parallel over the N GPUs (strong scaling: `value` is the
 tokens/s of the one sharded model); the other workloads run N batch-sharded replicas (weak scaling).  `--parallelism`
 overrides.  After the timed region the benchmarked engine is checked against an independent engine (one GPU, one launch
@@ -639,6 +641,120 @@ def run_b200(args):
                  (line["parity_check"]["max_rel_logit_err"], line["parity_check"]["tolerance"]))
 
 
+# ---- layered designs beside the closest uniform model ---------------------------------------------------------------------------
+# sizes that resemble the layers of real models; every entry: layers, width, heads, unrotated / rotated / value head size, latent,
+# experts, experts per token, expert width.  The closest existing model of equal size: GPTDecoder with grouped-query attention, RoPE,
+# RMSNorm and a dense gated feed-forward as wide as the experts a token uses, fp16.
+DESIGN_SIZES = {
+    "1k": dict(L=12, d=1024, H=16, dim=64, rot=32, vdim=64, rank=256, E=16, top=2, ff=1024),
+    "2k": dict(L=12, d=2048, H=16, dim=128, rot=64, vdim=128, rank=512, E=32, top=4, ff=1408),
+    "4k": dict(L=6, d=4096, H=32, dim=128, rot=64, vdim=128, rank=512, E=16, top=2, ff=4096),
+}
+DESIGN_V = 32000
+
+
+def design_models(z, local, max_batch, max_tokens):
+    """(layered model, closest uniform model), random weights."""
+    from seq2seqsharp_b200.gpt import (ActivateFuncEnums as A, GPT, GPTConfig, MultiHeadAttentionTypeEnums as MA, NormEnums as Nm,
+                                       PositionEmbeddingEnums as PE)
+    from seq2seqsharp_b200.layered import BlockLayer, LatentAttention, LayeredConfig, LayeredGPT, TableExperts
+    from seq2seqsharp_b200.pepilix import EXPERT_SHIFT, EXPERT_SLOPE
+    ex = TableExperts(experts=z["E"], top=z["top"], ff=z["ff"], limit=7.0, slope=EXPERT_SLOPE, shift=EXPERT_SHIFT)
+    at = dict(heads=z["H"], dim=z["dim"], rot_dim=z["rot"], vdim=z["vdim"], kv_rank=z["rank"], rot_base=1e6, scale=(z["dim"] + z["rot"]) ** -0.5)
+    lay = LayeredConfig(d=z["d"], V=DESIGN_V, norm_groups=8, conv_taps=4, embed_scale=z["d"] ** 0.5,
+                        layers=[BlockLayer(LatentAttention(**at), ex) for _ in range(z["L"])])
+    uni = GPTConfig(L=z["L"], d=z["d"], H=z["H"], Hkv=max(1, z["H"] // 4), hd=z["vdim"], F=z["top"] * z["ff"], V=DESIGN_V, norm=Nm.RMSNorm, act=A.SwiGLU_SiLU,
+                    pe=PE.RoPE, attn=MA.GQA, dtype="float16")
+    return (lambda: LayeredGPT(lay, device_id=local, max_batch=max_batch, max_tokens=max_tokens),
+            lambda: GPT(uni, device_id=local, max_batch=max_batch, max_tokens=max_tokens), lay, uni)
+
+
+def design_costs(z, which, B, S, T):
+    """Algorithmic (bytes of a decode step at context T with B sequences, flops of a prefill of B x S) per kernel class."""
+    L, d, H, V = z["L"], z["d"], z["H"], DESIGN_V
+    if which == "layered":
+        proj = 2 * d * d + d * (H * (z["dim"] + z["rot"]) + z["rank"] + z["rot"]) + H * z["vdim"] * d
+        lat = H * (z["dim"] + z["vdim"]) * z["rank"]
+        seen = z["E"] * (1.0 - (1.0 - z["top"] / z["E"]) ** B)       # experts that B tokens use, on average
+        by = {"linear": 2.0 * (L * proj + d * V), "experts": 2.0 * L * 3 * d * z["ff"] * seen,
+              "attention": 2.0 * L * (lat + B * T * (z["rank"] + z["rot"]))}
+        fl = {"linear": 2.0 * B * S * L * proj + 2.0 * B * d * V, "experts": 2.0 * B * S * L * 3 * d * z["ff"] * z["top"],
+              "attention": L * (2.0 * B * S * lat + 2.0 * B * H * (z["dim"] + z["rot"] + z["vdim"]) * S * S / 2.0)}
+    else:
+        hd, kv = z["vdim"], max(1, H // 4)
+        proj = d * (H + 2 * kv) * hd + H * hd * d + 3 * d * z["top"] * z["ff"]
+        by = {"linear": 2.0 * (L * proj + d * V), "attention": 2.0 * L * B * T * 2 * kv * hd}
+        fl = {"linear": 2.0 * B * S * L * proj + 2.0 * B * d * V, "attention": L * 4.0 * B * H * hd * S * S / 2.0}
+    return by, fl
+
+
+def run_design(args):
+    import torch
+
+    from seq2seqsharp_b200 import _native
+    from seq2seqsharp_b200.configs import SEED
+    from seq2seqsharp_b200.synthetic import prompt_ids
+    local = 0
+    torch.cuda.set_device(local)
+    if not _native.lib().TSB200_IsAvailable(local):
+        raise RuntimeError("bench: device %d is not an sm_100 GPU; this backend has no CPU fallback" % local)
+    hbm, _ = peaks()
+    burst, sustained, which_peak = tensor_peaks()
+    K, W = args.steps, max(args.warmup, 3)
+    out = {"design": args.design, "unit": "tokens/s", "data": "synthetic", "steps": K, "warmup": W, "peaks": which_peak, "sizes": {}}
+    sampler = ClockSampler(local)
+    sampler.start()
+    for name in args.design_sizes.split(","):
+        z = DESIGN_SIZES[name]
+        res = {}
+        for which in ("layered", "uniform"):
+            r = {}
+            for B, S in ((1, 1024), (8, 1024), (64, 512)):
+                max_tokens = S + W + K + 24
+                lay, uni, _, _ = design_models(z, local, B, max_tokens)
+                g = (lay if which == "layered" else uni)()
+                g.FillSynthetic(SEED, 0.02, 0.0)
+                opts = make_options("greedy", 1.0, max_tokens, SEED, 0)
+                ids = prompt_ids(SEED, B, S, DESIGN_V)
+                g.Prefill(ids, opts)
+                g.Decode(W, opts)
+                g.Decode(K, opts)
+                ms, _ = g.LastTiming()
+                T = S + W + K // 2
+                prof = g.ProfileDecode(8, opts)
+                by, _ = design_costs(z, which, B, S, T)
+                r["decode_B%d_T%d" % (B, T)] = {
+                    "tokens_per_s": B * K / (ms / 1e3), "ms_per_step": ms / K, "launches_per_step": sum(v[1] for v in prof.values()) // 8,
+                    "classes": {k: {"ms": v[0] / 8, **({"gbs": by[k] / 1e6 / (v[0] / 8), "frac_of_hbm_peak": by[k] / 1e6 / (v[0] / 8) / hbm} if k in by else {})}
+                                for k, v in prof.items() if v[1]}}
+                g.close()
+            for B, S in ((1, 2048), (4, 2048)):
+                lay, uni, _, _ = design_models(z, local, B, S + 8)
+                g = (lay if which == "layered" else uni)()
+                g.FillSynthetic(SEED, 0.02, 0.0)
+                opts = make_options("greedy", 1.0, S + 8, SEED, 0)
+                ids = prompt_ids(SEED, B, S, DESIGN_V)
+                times = []
+                for _ in range(W + 5):
+                    g.Reset()
+                    g.Prefill(ids, opts)
+                    times.append(g.LastTiming()[0])
+                ms = statistics.median(times[W:])
+                g.Reset()
+                prof = g.ProfilePrefill(ids, opts)
+                _, fl = design_costs(z, which, B, S, 0)
+                r["prefill_B%d_S%d" % (B, S)] = {
+                    "tokens_per_s": B * S / (ms / 1e3), "ms": ms, "tflops": sum(fl.values()) / 1e9 / ms, "frac_of_tensor_peak": sum(fl.values()) / 1e9 / ms / burst,
+                    "classes": {k: {"ms": v[0], **({"tflops": fl[k] / 1e9 / v[0], "frac_of_tensor_peak": fl[k] / 1e9 / v[0] / burst} if k in fl else {})}
+                                for k, v in prof.items() if v[1]}}
+                g.close()
+            res[which] = r
+        out["sizes"][name] = {"shape": z, **res}
+    clocks = sampler.stop()
+    out["clocks"] = {"sm_mhz": clocks["sm_mhz"], "sm_max_mhz": clocks["sm_max_mhz"], "reasons": clocks["reasons"]}
+    print(json.dumps(out))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -646,6 +762,9 @@ def main():
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--workload", default="c5_b1", choices=sorted(WORKLOADS))
+    ap.add_argument("--design", default="", choices=["", "pepilix"],
+                    help="instead of a workload: prefill and decode throughput of a layered design at a few sizes beside the closest uniform model")
+    ap.add_argument("--design-sizes", default="1k,2k,4k")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-parity-check", action="store_true")
     ap.add_argument("--no-secondary", action="store_true")
@@ -656,7 +775,9 @@ def main():
     args = ap.parse_args()
     # stdout carries the ONE JSON line: whatever NCCL has to say (its version banner, INFO lines) goes to stderr
     os.environ.setdefault("NCCL_DEBUG_FILE", "/dev/stderr")
-    if args.impl == "reference":
+    if args.design:
+        run_design(args)
+    elif args.impl == "reference":
         run_reference(args)
     else:
         run_b200(args)

@@ -488,9 +488,13 @@ TSB200_API int TSB200_GptGetStepTimes(void* gpt, float* ms, int n, int* n_out);
 /* Runs n_steps decode steps un-captured with CUDA events around every launch group and returns, per kernel class
  * (0 embed, 1 norm, 2 linear (GEMV/GEMM), 3 rope+append, 4 attention, 5 sampling, 6 commit), the summed device
  * time in ms and the number of launches.  Consecutive launches of one class are timed as one run (events only at its two
- * ends), so that they chain as they do in the captured step.  n_classes >= 8. */
+ * ends), so that they chain as they do in the captured step.  Classes also: 7 all-reduce, 8 persistent step kernel, 9 experts.
+ * n_classes >= 10. */
 TSB200_API int TSB200_GptProfileDecode(void* gpt, int n_steps, const TSB200DecodingOptions* opt, float* class_ms,
                                        int64_t* class_groups, int n_classes);
+/* the same for one prefill (ids [B, S] on an empty cache, as TSB200_GptPrefill) */
+TSB200_API int TSB200_GptProfilePrefill(void* gpt, const int32_t* ids, int B, int S, const TSB200DecodingOptions* opt, float* class_ms,
+                                        int64_t* class_groups, int n_classes);
 /* the engine's stream (cudaStream_t) */
 TSB200_API int TSB200_GptStream(void* gpt, void** stream);
 /* algorithmic bytes of one decode step at cache length T for B sequences (weights once + KV read/write +

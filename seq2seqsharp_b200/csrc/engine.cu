@@ -294,7 +294,7 @@ struct Gpt {
   int own_B = 0;                     // batch the owner kernel serves for the current program (0: not in use)
 };
 
-enum KernelClass { KC_EMBED = 0, KC_NORM = 1, KC_LINEAR = 2, KC_ROPE_APPEND = 3, KC_ATTENTION = 4, KC_SAMPLE = 5, KC_COMMIT = 6, KC_ALLREDUCE = 7, KC_STACK = 8, KC_COUNT = 9 };
+enum KernelClass { KC_EMBED = 0, KC_NORM = 1, KC_LINEAR = 2, KC_ROPE_APPEND = 3, KC_ATTENTION = 4, KC_SAMPLE = 5, KC_COMMIT = 6, KC_ALLREDUCE = 7, KC_STACK = 8, KC_EXPERTS = 9, KC_COUNT = 10 };
 
 // Profiling pass (TSB200_GptProfileDecode): CUDA events around RUNS of consecutive launches of one class.  Inside a run no
 // event is recorded between the launches, so they chain exactly as they do in the captured step (an event between two
@@ -997,7 +997,7 @@ static int enqueue_forward(Gpt* g, int B, int S, int T0, bool use_state, int spl
     if (L.moe) {
       // MoEFeedForward.Process: the layer's own LayerNorm (whatever the model's norm type), router, experts, residual add
       PROF(KC_NORM, launch_norm_residual(dev, g->st, dt, g->h, g->x, nullptr, L.moe_g, L.moe_b, 0, c.eps, rows, d, g->s));
-      PROF(KC_LINEAR, launch_moe_ffn(dev, g->st, dt, g->x, g->h, L.router_w, L.router_b, L.moe_w1, L.moe_w2, g->ffn, g->moe_picks, g->moe_scores,
+      PROF(KC_EXPERTS, launch_moe_ffn(dev, g->st, dt, g->x, g->h, L.router_w, L.router_b, L.moe_w1, L.moe_w2, g->ffn, g->moe_picks, g->moe_scores,
                                      rows, d, c.n_experts, c.experts_per_token, act, g->s));
       continue;
     }
@@ -2536,6 +2536,35 @@ int TSB200_GptSetWaitLimit(void* h, int polls) {
   return 1;
 }
 
+static int prof_sum(Gpt* g, float* class_ms, int64_t* class_groups) {
+  for (size_t i = 0; i < g->prof_n; ++i) {
+    float ms = 0.0f;
+    TSB_CUDA(cudaEventElapsedTime(&ms, g->prof_ev[2 * i], g->prof_ev[2 * i + 1]));
+    class_ms[g->prof_cls[i]] += ms;
+    class_groups[g->prof_cls[i]] += g->prof_cnt[i];   // launches, however many of them shared a run
+  }
+  return 1;
+}
+
+int TSB200_GptProfilePrefill(void* h, const int32_t* ids, int B, int S, const TSB200DecodingOptions* opt, float* class_ms, int64_t* class_groups,
+                             int n_classes) {
+  NvtxRange nvtx_("tsb200.gpt.profile_prefill");
+  Gpt* g = (Gpt*)h;
+  TSB_CHECK(g && ids && opt && class_ms && class_groups, "gpt_profile_prefill: null argument");
+  TSB_TRY(use_device(g->c.device, nullptr));
+  TSB_CHECK(n_classes >= KC_COUNT, "gpt_profile_prefill: need room for %d classes", (int)KC_COUNT);
+  for (int i = 0; i < n_classes; ++i) { class_ms[i] = 0.0f; class_groups[i] = 0; }
+  g->prof = true;
+  g->prof_n = 0;
+  const int ok = run_prompt(g, ids, B, S, opt, nullptr, false);
+  prof_flush(g);
+  g->prof = false;
+  g->prof_open = false;
+  TSB_CUDA(cudaStreamSynchronize(g->s));
+  if (!ok) return 0;
+  return prof_sum(g, class_ms, class_groups);
+}
+
 int TSB200_GptProfileDecode(void* h, int n_steps, const TSB200DecodingOptions* opt, float* class_ms, int64_t* class_groups,
                             int n_classes) {
   NvtxRange nvtx_("tsb200.gpt.profile_decode");
@@ -2565,12 +2594,7 @@ int TSB200_GptProfileDecode(void* h, int n_steps, const TSB200DecodingOptions* o
   if (!ok) return 0;
   TSB_CUDA(e);
   TSB_TRY(check_err_flag(g));
-  for (size_t i = 0; i < g->prof_n; ++i) {
-    float ms = 0.0f;
-    TSB_CUDA(cudaEventElapsedTime(&ms, g->prof_ev[2 * i], g->prof_ev[2 * i + 1]));
-    class_ms[g->prof_cls[i]] += ms;
-    class_groups[g->prof_cls[i]] += g->prof_cnt[i];   // launches, however many of them shared a run
-  }
+  TSB_TRY(prof_sum(g, class_ms, class_groups));
   g->T += n_steps;
   g->step += (uint32_t)n_steps;
   g->probs_valid = (opt->strategy == 1);

@@ -6,9 +6,9 @@
 //   block norm   h1, h2 = two weights on one group-wise RMS norm of x (the previous layer's expert outputs join x here);
 //                hc = h1 + short convolution of h1
 //   one linear   gate1 = sigmoid(h1 G1 + b1), gate2 = sigmoid(h2 G2 + b2), q | dkv = hc W: three sections of one packed matrix,
-//                one launch up to 16 rows
-//   append       latent norm, rotation, cache row (or only the query's rotation when the layer reads another layer's cache)
-//   attention    latent attention over the cache rows (ops_latent.cu)
+//                one launch up to 64 rows
+//   attention    latent norm, rotation, cache row (or only the query's rotation when the layer reads another layer's cache), latent
+//                attention over the cache rows (ops_latent.cu)
 //   out          x += gate1 * (attn W_o)
 //   experts      two grouped products over rows sorted by expert; their outputs wait for the next block norm
 #pragma once
@@ -39,7 +39,7 @@ struct Layered {
   int n_route = 0, max_experts = 0;
   // scratch, grown on demand (ensure_layered)
   struct Buf { void* p = nullptr; int64_t bytes = 0; };
-  Buf hcat, gate1, gate2, qkv, attn, hs, hidden, y, q_lat, part, kv, ints, routes, ws;
+  Buf hcat, gate1, gate2, qkv, attn, hs, hidden, y, q_lat, part, kv, compact, ints, routes, ws;
   int64_t route_rows = 0;
   int route_block = 0;
 };
@@ -289,7 +289,7 @@ static int ensure_layered(Gpt* g, int B, int S, int T) {
   const int dt = g->c.dtype;
   const int br = layered_block_rows(ly, (int)rows);
   bool big = rows * d * 4 > g->x_bytes;
-  int64_t nq = 0, na = 0, npk = 0, nhid = 0, nlat = 0, npart = 0, nkv = 0, nints = 0;
+  int64_t nq = 0, na = 0, npk = 0, nhid = 0, nlat = 0, npart = 0, nkv = 0, ncomp = 0, nints = 0;
   int64_t ws = kWsCounterBytes + 1024;
   auto lin = [&](int64_t K, int64_t N) {
     for (int64_t m : {(int64_t)1, std::min<int64_t>(rows, 64)}) {
@@ -306,10 +306,11 @@ static int ensure_layered(Gpt* g, int B, int S, int T) {
       npart = std::max(npart, rows * L.sh.H * latent_pick_splits(g->st, L.sh, B, S, T) * (L.sh.rank + 2));
     } else {
       nkv = std::max(nkv, (int64_t)B * T * L.sh.H * (L.sh.dim + L.sh.vdim));
+      if (B > 1) ncomp = std::max(ncomp, (int64_t)B * T * L.sh.row);
       for (int64_t m : {(int64_t)16, (int64_t)64})
         ws = std::max(ws, gemm_stream_mma_workspace_bytes((int)m, L.sh.row, L.sh.H * (L.sh.dim + L.sh.vdim), g->st->sm_count));
     }
-    if (is_16bit(dt)) ws = std::max(ws, gemm_stream_sections_workspace_bytes((int)std::min<int64_t>(rows, 16), (int)d, (int)(2 * d + L.Nq + L.Nkv), g->st->sm_count));
+    if (is_16bit(dt)) ws = std::max(ws, gemm_stream_sections_workspace_bytes((int)std::min<int64_t>(rows, 64), (int)d, (int)(2 * d + L.Nq + L.Nkv), g->st->sm_count));
     lin(d, d);
     lin(d, L.Nq + L.Nkv);
     lin(L.sh.H * L.sh.vdim, d);
@@ -346,6 +347,7 @@ static int ensure_layered(Gpt* g, int B, int S, int T) {
   TSB_TRY(grow(g, ly->q_lat, nlat * es));
   TSB_TRY(grow(g, ly->part, npart * 4));
   TSB_TRY(grow(g, ly->kv, nkv * es));
+  TSB_TRY(grow(g, ly->compact, ncomp * es));
   TSB_TRY(grow(g, ly->ws, ws, true));
   if (ly->n_route > 0 && (ly->route_rows != rows || ly->route_block != br)) {
     // routing scratch of every expert layer, laid out for this many rows; the captured step holds pointers into it
@@ -440,7 +442,7 @@ static int enqueue_layered(Gpt* g, int B, int S, int T0, bool use_state, int T_p
       Epilogue e2 = make_ep(L.g2b, nullptr, ly->gate2.p, nullptr, TSB200_ACT_SIGMOID, 0);
       Epilogue e3 = make_ep(nullptr, nullptr, ly->qkv.p, nullptr, TSB200_ACT_NONE, 0);
       int r = 2;
-      if (rows <= 16 && ff) {
+      if (rows <= 64 && ff) {
         const LinearSection sec[3] = {{d, e1}, {d, e2}, {Nqkv, e3}};
         prof_begin(g, KC_LINEAR);
         r = launch_gemm_stream_sections(dev, g->st, dt, h1, L.fused, rows, d, sec, 3, pdl, ws, wsb, g->s);
@@ -454,14 +456,13 @@ static int enqueue_layered(Gpt* g, int B, int S, int T0, bool use_state, int T_p
       }
     }
     const int64_t seq_stride = (int64_t)g->c.max_tokens * src.sh.row;
-    PROF(KC_ROPE_APPEND, launch_latent_append(dev, dt, L.sh, ly->qkv.p, Nqkv, L.Nkv ? L.Nq : -1, L.kv_norm, ly->c.eps, src.cache, seq_stride, B, S, T0, dT,
-                                              g->c.max_tokens, L.tab, g->s));
     LatentArgs at{};
-    at.shape = L.sh; at.q = ly->qkv.p; at.q_stride = Nqkv; at.cache = src.cache; at.seq_stride = seq_stride;
+    at.shape = L.sh; at.q = ly->qkv.p; at.q_stride = Nqkv; at.dkv_col = L.Nkv ? L.Nq : -1; at.norm_w = L.kv_norm; at.eps = ly->c.eps; at.tab = L.tab;
+    at.cache = src.cache; at.seq_stride = seq_stride;
     at.B = B; at.S = S; at.T0 = T0; at.Tmax = g->c.max_tokens; at.state = dT;
     at.splits = latent_pick_splits(g->st, L.sh, B, S, T_plan);
     at.uk = L.uk; at.uv = L.uv; at.ukv_packed = L.ukv; at.q_lat = ly->q_lat.p; at.part = (float*)ly->part.p; at.part_elems = ly->part.bytes / 4;
-    at.kv = ly->kv.p; at.kv_elems = ly->kv.bytes / es; at.out = ly->attn.p; at.lin_ws = ws; at.lin_ws_bytes = wsb;
+    at.kv = ly->kv.p; at.kv_elems = ly->kv.bytes / es; at.compact = ly->compact.p; at.compact_elems = ly->compact.bytes / es; at.out = ly->attn.p; at.lin_ws = ws; at.lin_ws_bytes = wsb;
     PROF(KC_ATTENTION, launch_latent_attention(dev, g->st, dt, at, g->s));
     {
       Epilogue e = make_ep(nullptr, g->x, nullptr, g->x, TSB200_ACT_NONE, 0);
@@ -484,8 +485,8 @@ static int enqueue_layered(Gpt* g, int B, int S, int T0, bool use_state, int T_p
       };
       Epilogue eu = make_ep(nullptr, nullptr, ly->hidden.p, nullptr, TSB200_ACT_CLAMP_GLU, 1);
       eu.glu_limit = L.d.glu_limit; eu.glu_slope = L.d.glu_slope; eu.glu_shift = L.d.glu_shift;
-      PROF(KC_LINEAR, grouped(ly->hs.p, L.up, L.up_bytes, d, 2 * L.d.ff, eu));
-      PROF(KC_LINEAR, grouped(ly->hidden.p, L.down, L.down_bytes, L.d.ff, d, make_ep(nullptr, nullptr, ly->y.p, nullptr, TSB200_ACT_NONE, 0)));
+      PROF(KC_EXPERTS, grouped(ly->hs.p, L.up, L.up_bytes, d, 2 * L.d.ff, eu));
+      PROF(KC_EXPERTS, grouped(ly->hidden.p, L.down, L.down_bytes, L.d.ff, d, make_ep(nullptr, nullptr, ly->y.p, nullptr, TSB200_ACT_NONE, 0)));
       prev = &L;
     }
   }

@@ -498,9 +498,11 @@ struct GcArgs {
   unsigned int* counters;    // [boxes], zero on entry, self-resetting
   int* error_flag;
   Epilogue ep;
+  int n_sec;                 // kGsSections
+  GsSection sec[kGsMaxSections];
 };
 
-template <typename H, int NB>
+template <typename H, int NB, int MODE>
 __global__ void __launch_bounds__(kGcThreads, 3) gemm_chunk_mma_kernel(const __grid_constant__ CUtensorMap mapX, GcArgs a) {
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
@@ -510,9 +512,13 @@ __global__ void __launch_bounds__(kGcThreads, 3) gemm_chunk_mma_kernel(const __g
   __shared__ int s_err, s_last;
 
   const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
-  const int M = a.M, N = a.N, KB = a.KB;
+  const int M = a.M, KB = a.KB;
   const int box = blockIdx.x / a.ksplit, ks = blockIdx.x % a.ksplit;   // the K ranges of a box run side by side
   const int ct = box >> 2, j = box & 3;
+  int si = 0;
+  if constexpr (MODE == kGsSections)
+    while (si < a.n_sec - 1 && ct >= a.sec[si].ct_end) ++si;
+  const int xrow = si * M;
   const int k2_total = (KB + 1) / 2;
   const int k2_beg = ks * a.k2_per, k2_end = min(k2_total, k2_beg + a.k2_per);
   const int n_st = max(k2_end - k2_beg, 0);
@@ -554,7 +560,7 @@ __global__ void __launch_bounds__(kGcThreads, 3) gemm_chunk_mma_kernel(const __g
           break;
         }
         if (i >= n_pre) put_w(i);
-        gs_tma_load_2d(smem + (size_t)s * kGcStageBytes + 8192, &mapX, (k2_beg + i) * 2 * kKT, 0, &full[s]);  // x = kb0 * 32 halves: a 64-byte multiple
+        gs_tma_load_2d(smem + (size_t)s * kGcStageBytes + 8192, &mapX, (k2_beg + i) * 2 * kKT, xrow, &full[s]);  // x = kb0 * 32 halves: a 64-byte multiple
         done = i + 1;
       }
       if (*(volatile int*)&s_err) {
@@ -650,11 +656,13 @@ __global__ void __launch_bounds__(kGcThreads, 3) gemm_chunk_mma_kernel(const __g
       }
     }
     if (finish) {
-      const Epilogue ep = a.ep;
+      const Epilogue& ep = MODE == kGsSections ? a.sec[si].ep : a.ep;
+      const int N = MODE == kGsSections ? a.sec[si].N : a.N;
+      const int lct = MODE == kGsSections && si ? ct - a.sec[si - 1].ct_end : ct;
       const H* bias = reinterpret_cast<const H*>(ep.bias);
       const int No = ep.glu ? N / 2 : N;
       for (int idx = tid; idx < M * 16; idx += 128) {
-        const int row = idx >> 4, c = ct * 256 + j * 64 + (idx & 15) * 4;
+        const int row = idx >> 4, c = lct * 256 + j * 64 + (idx & 15) * 4;
         const float4 t = reinterpret_cast<const float4*>(red)[idx];
         const float v[4] = {t.x, t.y, t.z, t.w};
         if (!ep.glu) {
@@ -761,12 +769,12 @@ static int gs_prefetch_enabled() {
   return on;
 }
 
-template <typename H, int NB>
+template <typename H, int NB, int MODE = kGsPlain>
 static int gc_launch(int device, const CUtensorMap& mapX, const GcArgs& a, int grid, bool pdl, cudaStream_t s) {
   static bool attr_done[kMaxDevices] = {};
   const size_t smem = kGcStages * kGcStageBytes + 1024 + 128;
   if (!attr_done[device]) {
-    TSB_CUDA(cudaFuncSetAttribute(gemm_chunk_mma_kernel<H, NB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    TSB_CUDA(cudaFuncSetAttribute(gemm_chunk_mma_kernel<H, NB, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     attr_done[device] = true;
   }
   cudaLaunchConfig_t cfg{};
@@ -779,16 +787,45 @@ static int gc_launch(int device, const CUtensorMap& mapX, const GcArgs& a, int g
   at[0].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = at;
   cfg.numAttrs = (pdl && pdl_enabled()) ? 1 : 0;
-  TSB_CUDA(cudaLaunchKernelEx(&cfg, gemm_chunk_mma_kernel<H, NB>, mapX, a));
+  TSB_CUDA(cudaLaunchKernelEx(&cfg, gemm_chunk_mma_kernel<H, NB, MODE>, mapX, a));
   count_launch(device);
+  return 1;
+}
+
+static int gc_map_x(CUtensorMap* map, int dtype, const void* x, int rows, int K, int NB) {
+  GsEncodeTiledFn enc = gs_get_encode();
+  if (!enc) return 2;
+  const cuuint64_t dims[2] = {(cuuint64_t)K, (cuuint64_t)rows};
+  const cuuint64_t strides[1] = {(cuuint64_t)K * 2};
+  const cuuint32_t box[2] = {64, (cuuint32_t)(NB * 8)};
+  const cuuint32_t el[2] = {1, 1};
+  const CUresult r = enc(map, gs_map_type(dtype), 2, const_cast<void*>(x), dims, strides, box, el, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                         CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  TSB_CHECK(r == CUDA_SUCCESS, "gemm_chunk: cuTensorMapEncodeTiled failed with %d", (int)r);
+  return 1;
+}
+// K ranges per box and scratch; 1 ok, 2 the scratch does not suffice
+static int gc_plan(GcArgs* a, DeviceState* st, int boxes, void* ws, int64_t ws_bytes) {
+  const int k2_total = (a->KB + 1) / 2;
+  // about two CTAs per SM in flight (three fit); a K range is at least 8 stages long
+  int ks = (2 * st->sm_count + boxes - 1) / boxes;
+  if (ks > k2_total / 8) ks = k2_total / 8;
+  if (ks < 1) ks = 1;
+  if (ks > 8) ks = 8;
+  a->k2_per = (k2_total + ks - 1) / ks;
+  ks = (k2_total + a->k2_per - 1) / a->k2_per;     // no empty range
+  a->ksplit = ks;
+  a->prefetch = gs_prefetch_enabled();
+  const int64_t need = kWsCounterBytes + (int64_t)boxes * ks * a->M * 64 * 4;
+  if (ks > 1 && (!ws || ws_bytes < need || (int64_t)boxes * 4 > kWsCounterBytes - 256)) return 2;
+  a->counters = reinterpret_cast<unsigned int*>(ws);
+  a->partials = ws ? reinterpret_cast<float*>(reinterpret_cast<char*>(ws) + kWsCounterBytes) : nullptr;
   return 1;
 }
 
 // Column-chunk variant (17..64 rows).  1 ok, 0 error, 2 not handled.
 static int launch_gemm_chunk_mma(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int M, int K, int N, const Epilogue& ep,
                                  int* error_flag, bool pdl, void* ws, int64_t ws_bytes, cudaStream_t s) {
-  GsEncodeTiledFn enc = gs_get_encode();
-  if (!enc) return 2;
   const int NB = M <= 32 ? 4 : 8;
   GcArgs a{};
   a.Wp = reinterpret_cast<const unsigned char*>(Wp);
@@ -796,34 +833,13 @@ static int launch_gemm_chunk_mma(int device, DeviceState* st, int dtype, const v
   a.KB = (K + kKT - 1) / kKT;
   a.CT = (N + 255) / 256;
   const int boxes = (N + 63) / 64;                 // boxes that hold real columns (the last column tile may have fewer than 4)
-  const int k2_total = (a.KB + 1) / 2;
-  // about two CTAs per SM in flight (three fit); a K range is at least 8 stages long
-  int ks = (2 * st->sm_count + boxes - 1) / boxes;
-  if (ks > k2_total / 8) ks = k2_total / 8;
-  if (ks < 1) ks = 1;
-  if (ks > 8) ks = 8;
-  a.k2_per = (k2_total + ks - 1) / ks;
-  ks = (k2_total + a.k2_per - 1) / a.k2_per;       // no empty range
-  a.ksplit = ks;
-  a.prefetch = gs_prefetch_enabled();
-  const int64_t need = kWsCounterBytes + (int64_t)boxes * ks * M * 64 * 4;
-  if (ks > 1 && (!ws || ws_bytes < need || (int64_t)boxes * 4 > kWsCounterBytes - 256)) return 2;
-  a.counters = reinterpret_cast<unsigned int*>(ws);
-  a.partials = ws ? reinterpret_cast<float*>(reinterpret_cast<char*>(ws) + kWsCounterBytes) : nullptr;
+  if (gc_plan(&a, st, boxes, ws, ws_bytes) != 1) return 2;
   a.error_flag = error_flag;
   a.ep = ep;
   CUtensorMap mapX;
-  {
-    const cuuint64_t dims[2] = {(cuuint64_t)K, (cuuint64_t)M};
-    const cuuint64_t strides[1] = {(cuuint64_t)K * 2};
-    const cuuint32_t box[2] = {64, (cuuint32_t)(NB * 8)};
-    const cuuint32_t el[2] = {1, 1};
-    const CUresult r = enc(&mapX, gs_map_type(dtype), 2, const_cast<void*>(x), dims, strides, box, el,
-                           CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
-                           CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-    TSB_CHECK(r == CUDA_SUCCESS, "gemm_chunk: cuTensorMapEncodeTiled failed with %d", (int)r);
-  }
-  const int grid = boxes * ks;
+  const int r = gc_map_x(&mapX, dtype, x, M, K, NB);
+  if (r != 1) return r;
+  const int grid = boxes * a.ksplit;
   if (dtype == TSB200_BF16) return NB == 4 ? gc_launch<__nv_bfloat16, 4>(device, mapX, a, grid, pdl, s) : gc_launch<__nv_bfloat16, 8>(device, mapX, a, grid, pdl, s);
   return NB == 4 ? gc_launch<__half, 4>(device, mapX, a, grid, pdl, s) : gc_launch<__half, 8>(device, mapX, a, grid, pdl, s);
 }
@@ -925,9 +941,30 @@ int64_t gemm_stream_sections_workspace_bytes(int M, int K, int total_N, int sm_c
 
 int launch_gemm_stream_sections(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int M, int K, const LinearSection* sec,
                                 int n_sec, bool pdl, void* ws, int64_t ws_bytes, cudaStream_t s) {
-  if (dtype != TSB200_BF16 || M < 1 || M > 16 || n_sec < 1 || n_sec > kGsMaxSections || K % 8 != 0 || ((uintptr_t)x % 16) != 0 ||
+  if (dtype != TSB200_BF16 || M < 1 || M > 64 || n_sec < 1 || n_sec > kGsMaxSections || K % 8 != 0 || ((uintptr_t)x % 16) != 0 ||
       ((uintptr_t)Wp % 16) != 0)
     return 2;
+  if (M > 16) {   // the column-chunk kernel; every section starts on a column tile, so its boxes are whole tiles but for the last section's
+    GcArgs c{};
+    c.Wp = reinterpret_cast<const unsigned char*>(Wp);
+    c.M = M; c.K = K;
+    c.KB = (K + kKT - 1) / kKT;
+    c.n_sec = n_sec;
+    for (int i = 0; i < n_sec; ++i) {
+      c.CT += (sec[i].N + 255) / 256;
+      c.sec[i].ct_end = c.CT;
+      c.sec[i].N = sec[i].N;
+      c.sec[i].ep = sec[i].ep;
+    }
+    const int last = (sec[n_sec - 1].N + 255) / 256, boxes = (c.CT - last) * 4 + (sec[n_sec - 1].N + 63) / 64;
+    if (gc_plan(&c, st, boxes, ws, ws_bytes) != 1) return 2;
+    const int nb = M <= 32 ? 4 : 8;
+    CUtensorMap map;
+    const int r = gc_map_x(&map, dtype, x, n_sec * M, K, nb);
+    if (r != 1) return r;
+    return nb == 4 ? gc_launch<__nv_bfloat16, 4, kGsSections>(device, map, c, boxes * c.ksplit, pdl, s)
+                   : gc_launch<__nv_bfloat16, 8, kGsSections>(device, map, c, boxes * c.ksplit, pdl, s);
+  }
   const int NB = M <= 8 ? 1 : 2;
   GsArgs a{};
   a.Wp = reinterpret_cast<const unsigned char*>(Wp);

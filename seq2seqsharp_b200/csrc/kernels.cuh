@@ -233,7 +233,7 @@ int launch_gemm_stream_grouped(int device, DeviceState* st, int dtype, const voi
                                const Epilogue& ep, const RowGroups& groups, bool pdl, void* ws, int64_t ws_bytes, cudaStream_t s);
 int64_t gemm_stream_grouped_workspace_bytes(int block_rows, int N, int max_blocks, int sm_count);
 // Several linears of equal K in one launch: section i multiplies rows [i * M, (i + 1) * M) of x (stacked [sections * M, K])
-// with columns of its own in Wp (each section starts on a column tile).  At most 16 rows.
+// with columns of its own in Wp (each section starts on a column tile).  At most 64 rows.
 struct LinearSection {
   int N;
   Epilogue ep;
@@ -327,14 +327,15 @@ struct LatentShape {
 inline int latent_row_elems(int rank, int rot) { return (rank + rot + 15) / 16 * 16; }
 // full-precision cos / sin table [Tmax, dims / 2] of base^(-2 i / dims) * position
 int launch_angle_table(int device, DeviceState* st, float2* tab, int Tmax, int dims, double base, cudaStream_t s);
-// per row of q | dkv: the query's rotated parts turned in place, and (dkv_col >= 0) latent norm + rotation + cache append
-int launch_latent_append(int device, int dtype, const LatentShape& a, void* qkv, int row_stride, int dkv_col, const void* norm_w, float eps, void* cache,
-                         int64_t seq_stride, int B, int S, int T0, const int* state, int Tmax, const float2* tab, cudaStream_t s);
 struct LatentArgs {
   LatentShape shape;
-  const void* q;                 // rows of q | dkv, turned
+  void* q;                       // rows of q | dkv as projected (the expanded form turns the queries in place)
   int q_stride;
-  const void* cache;             // [sequences][Tmax][row]
+  int dkv_col;                   // column of dkv in a row: latent norm, rotation and cache append; < 0: the layer reads another layer's cache
+  const void* norm_w;
+  float eps;
+  const float2* tab;             // launch_angle_table
+  void* cache;                   // [sequences][Tmax][row]
   int64_t seq_stride;
   int B, S, T0, Tmax;
   const int* state;
@@ -346,6 +347,8 @@ struct LatentArgs {
   int64_t part_elems;
   void* kv;                      // scratch [B][T0 + S][H * (dim + vdim)], expanded form only
   int64_t kv_elems;
+  void* compact;                 // scratch [B][T0 + S][row], expanded form of several sequences
+  int64_t compact_elems;
   void* out;                     // [B * S, H * vdim]
   void* lin_ws;
   int64_t lin_ws_bytes;

@@ -160,6 +160,144 @@ __global__ void __launch_bounds__(kBlockNormThreads) block_norm_kernel(BlockNorm
   }
 }
 
+// The same for the usual widths, the row in registers: thread t holds elements (t + u * threads) * 4 .. + 3.  Weights are requested
+// before the wait on the previous kernel, everything that depends on it in one round afterwards.  Groups are 2^k * 4 elements inside a
+// warp's 128, or whole multiples of 128.  TAPS: room for the convolution's taps, 0: none.
+constexpr int kFastTop = 8;
+template <typename T, int NV, int TAPS>
+__global__ void __launch_bounds__(512) block_norm_fast_kernel(BlockNormArgs a) {
+  __shared__ float s_part[16 * NV];
+  pdl_trigger();
+  const int tid = threadIdx.x, nt = blockDim.x, lane = tid & 31, w = tid >> 5, nw = nt >> 5;
+  const int d = a.d, gsz = d / a.groups, out_row = blockIdx.x;
+  float w1[NV][4], w2[NV][4], cw[NV][4][TAPS > 0 ? TAPS : 1];
+#pragma unroll
+  for (int u = 0; u < NV; ++u) {
+    const int i = (tid + u * nt) * 4;
+    VecIO<T, 4>::load(reinterpret_cast<const T*>(a.w1) + i, w1[u]);
+    if (a.w2) VecIO<T, 4>::load(reinterpret_cast<const T*>(a.w2) + i, w2[u]);
+    if constexpr (TAPS > 0) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+#pragma unroll
+        for (int q = 0; q < TAPS; ++q)   // q positions back
+          cw[u][e][q] = q < a.taps ? to_f<T>(reinterpret_cast<const T*>(a.conv_w)[(int64_t)(i + e) * a.taps + a.taps - 1 - q]) : 0.0f;
+    }
+  }
+  pdl_wait();
+  int row = out_row;
+  if (a.rows_of) row = a.rows_of[out_row];
+  else if (a.last_of_S > 0) {
+    const int n = a.lens ? a.lens[out_row] : a.last_of_S;
+    row = out_row * a.last_of_S + min(max(n, 1), a.last_of_S) - 1;
+  }
+  float* xr = a.x + (int64_t)row * d;
+  int yp[kFastTop], np[kFastTop];
+#pragma unroll
+  for (int j = 0; j < kFastTop; ++j) {
+    yp[j] = a.y && j < a.top ? a.y_pos[(int64_t)row * a.top + j] : 0;
+    np[j] = a.w2 && j < a.next_top ? a.next_pos[(int64_t)row * a.next_top + j] : 0;
+  }
+  float v[NV][4], past[NV][TAPS > 1 ? TAPS - 1 : 1][4];
+  int pos = 0;
+  T* ring = nullptr;
+  if constexpr (TAPS > 0) {
+    pos = state_len(a.state, out_row, a.T0);
+    ring = reinterpret_cast<T*>(a.conv_ring) + (int64_t)out_row * a.taps * d;
+  }
+#pragma unroll
+  for (int u = 0; u < NV; ++u) {
+    const int i = (tid + u * nt) * 4;
+    VecIO<float, 4>::load(xr + i, v[u]);
+    if constexpr (TAPS > 1) {
+#pragma unroll
+      for (int q = 1; q < TAPS; ++q) {
+        if (q < a.taps && pos >= q) VecIO<T, 4>::load(ring + (int64_t)((pos - q) % a.taps) * d + i, past[u][q - 1]);
+        else past[u][q - 1][0] = past[u][q - 1][1] = past[u][q - 1][2] = past[u][q - 1][3] = 0.0f;
+      }
+    }
+  }
+  if (a.y) {
+    const float inv_top = 1.0f / (float)a.top;
+#pragma unroll
+    for (int u = 0; u < NV; ++u) {
+      const int i = (tid + u * nt) * 4;
+      float g[4] = {1.0f, 1.0f, 1.0f, 1.0f}, sum[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+      if (a.y_gate) VecIO<T, 4>::load(reinterpret_cast<const T*>(a.y_gate) + (int64_t)row * d + i, g);
+#pragma unroll
+      for (int j = 0; j < kFastTop; ++j)
+        if (j < a.top) {
+          float t[4];
+          VecIO<T, 4>::load(reinterpret_cast<const T*>(a.y) + (int64_t)yp[j] * d + i, t);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) sum[e] += t[e];
+        }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[u][e] += sum[e] * inv_top * g[e];
+      if (a.write_x) VecIO<float, 4>::store(xr + i, v[u]);
+    }
+  }
+  float inv[NV];
+#pragma unroll
+  for (int u = 0; u < NV; ++u) {
+    float s = (v[u][0] * v[u][0] + v[u][1] * v[u][1]) + (v[u][2] * v[u][2] + v[u][3] * v[u][3]);
+    if (gsz < 128) {
+      for (int o = gsz >> 3; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    } else {
+      s = warp_sum(s);
+      if (lane == 0) s_part[w + u * nw] = s;
+    }
+    inv[u] = s;
+  }
+  if (gsz >= 128) {
+    __syncthreads();
+    const int per = gsz >> 7;
+#pragma unroll
+    for (int u = 0; u < NV; ++u) {
+      const int first = (w + u * nw) / per * per;
+      float s = 0.0f;
+      for (int q = 0; q < per; ++q) s += s_part[first + q];
+      inv[u] = s;
+    }
+  }
+#pragma unroll
+  for (int u = 0; u < NV; ++u) {
+    const int i = (tid + u * nt) * 4;
+    const float r = 1.0f / sqrtf(inv[u] / (float)gsz + a.eps);
+    float h[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) h[e] = v[u][e] * r * w1[u][e] * a.out_scale;
+    VecIO<T, 4>::store(reinterpret_cast<T*>(a.h1) + (int64_t)out_row * d + i, h);
+    if (a.w2) {
+      float h2[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) h2[e] = v[u][e] * r * w2[u][e];
+      VecIO<T, 4>::store(reinterpret_cast<T*>(a.h2) + (int64_t)out_row * d + i, h2);
+#pragma unroll
+      for (int j = 0; j < kFastTop; ++j)
+        if (j < a.next_top) VecIO<T, 4>::store(reinterpret_cast<T*>(a.h2_sorted) + (int64_t)np[j] * d + i, h2);
+    }
+    if constexpr (TAPS > 0) {
+      float out[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float hr = to_f<T>(from_f<T>(h[e]));   // the value the state keeps
+        float acc = hr;
+#pragma unroll
+        for (int q = TAPS - 1; q >= 1; --q) acc += cw[u][e][q] * past[u][q - 1][e];   // oldest first, as in the other kernels
+        out[e] = acc + cw[u][e][0] * hr;
+      }
+      VecIO<T, 4>::store(ring + (int64_t)(pos % a.taps) * d + i, h);
+      VecIO<T, 4>::store(reinterpret_cast<T*>(a.hc) + (int64_t)out_row * d + i, out);
+    }
+  }
+}
+static bool block_norm_fast_shape(const BlockNormArgs& a) {
+  const int gsz = a.d / a.groups, nv = a.d <= 2048 ? 1 : 2;
+  if (a.d % (128 * nv) != 0 || a.d > 4096 || a.top > kFastTop || a.next_top > kFastTop || (a.conv_ring && a.taps > 4)) return false;
+  return gsz >= 128 ? gsz % 128 == 0 : (gsz >= 4 && (gsz & (gsz - 1)) == 0);
+}
+
 // out[b, s] = h[b, s] + sum_j w[:, j] h[b, s - taps + 1 + j]; positions before the portion come from the ring, none before 0
 template <typename T>
 __global__ void __launch_bounds__(256) short_conv_kernel(T* out, const T* h, const T* wgt, const T* ring, int B, int S, int d, int taps, int T0_arg,
@@ -308,6 +446,18 @@ __global__ void __launch_bounds__(128) pick_linear_kernel(const T* x, const T* W
 int launch_block_norm(int device, int dtype, const BlockNormArgs& a, int out_rows, cudaStream_t s) {
   if (out_rows == 0) return 1;
   TSB_CHECK(a.groups >= 1 && a.d % a.groups == 0, "block_norm: a width of %d is not cut into %d groups", a.d, a.groups);
+  if (block_norm_fast_shape(a)) {
+    const int nv = a.d <= 2048 ? 1 : 2;
+    const dim3 th(a.d / 4 / nv);
+#define TSB_BNF(T)                                                                                                                    \
+  (a.conv_ring ? (nv == 1 ? block_norm_fast_kernel<T, 1, 4> : block_norm_fast_kernel<T, 2, 4>)                                        \
+               : (nv == 1 ? block_norm_fast_kernel<T, 1, 0> : block_norm_fast_kernel<T, 2, 0>))
+    if (dtype == TSB200_F32) TSB_CUDA(launch_k(TSB_BNF(float), dim3(out_rows), th, 0, s, a));
+    else TSB_CUDA(launch_k(TSB_BNF(__nv_bfloat16), dim3(out_rows), th, 0, s, a));
+#undef TSB_BNF
+    count_launch(device);
+    return check_launch("block_norm_fast");
+  }
   const size_t smem = ((size_t)a.d + (a.groups > 8 ? a.groups : 8)) * sizeof(float);
   TSB_CHECK(smem <= 200 * 1024, "block_norm: rows of %d elements are not supported", a.d);
   static bool done[kMaxDevices] = {};

@@ -5,12 +5,12 @@
 //   absorbed   q_lat = [Uk_h^T q_n | q_r] once per query, then all heads attend to the cache rows themselves (one key of
 //              rank + rot elements whose first rank elements are also the value), and Uv_h is applied to the result.  Reads the cache
 //              once for all heads: decoding and short portions.
-//                latent_query_kernel     q_lat (Uk read once per eight rows, its inner dimension split over the warps)
-//                latent_attn_mma_kernel  bf16, split over the key range: 16 (query, head) rows per CTA on mma.sync, cache rows
-//                                        staged once by cp.async as keys AND values; scores meet in shared memory so that each
-//                                        warp can own a slice of the latent in the second product
-//                latent_attn_kernel      any type and size up to a latent of 1024, CUDA cores
-//                latent_value_kernel     merges the splits and applies Uv_h
+//                latent_query_*          q_lat, and the cache rows of the new positions in CTAs of their own
+//                latent_attn_*           the attention, split over the key range
+//                latent_value_*          merges the splits and applies Uv_h
+//              each as an mma.sync kernel (bf16; in the attention 16 (query, head) rows per CTA, cache rows staged once by cp.async as
+//              keys AND values, scores meeting in shared memory so that each warp can own a slice of the latent in the second
+//              product) and on CUDA cores (any type and size up to a latent of 1024)
 //   expanded   keys and values of all heads are materialised from the cache rows by one tensor-core linear, then causal flash
 //              attention per head (latent_prefill_mma_kernel: 128 queries per CTA, mma.sync).  Fewer operations per (query, key)
 //              pair, paid for by the expansion: long portions.
@@ -61,78 +61,155 @@ __device__ __forceinline__ void turn_pair(const T* src, T* dst, int i, int dims,
   dst[i] = from_f<T>(u * cs.x - v * cs.y);
   dst[i + dims / 2] = from_f<T>(v * cs.x + u * cs.y);
 }
-
-constexpr int kLatentAppendThreads = 128;
+// one cache row from a dkv row, by a whole block: latent norm, rotation of the shared key part
 template <typename T>
-__global__ void __launch_bounds__(kLatentAppendThreads) latent_append_kernel(LatentShape a, T* qkv, int row_stride, int dkv_col, const T* norm_w, float eps,
-                                                                             T* cache, int64_t seq_stride, int S, int T0_arg, const int* state, int Tmax,
-                                                                             const float2* tab) {
-  __shared__ float red[32];
-  pdl_trigger();
-  pdl_wait();
-  const int row = blockIdx.x, b = row / S, tid = threadIdx.x;
-  const int pos = state_len(state, b, T0_arg) + row % S;
-  TSB_DEV_CHECK(latent, pos >= 0 && pos < Tmax, 0x601, return)   // append position outside the cache
-  if (pos >= Tmax) return;   // capacity is checked on the host; never write past the cache
-  const int half = a.rot_dims / 2;
-  const float2* cs = tab + (int64_t)pos * half;
-  T* q = qkv + (int64_t)row * row_stride;
-  for (int p = tid; p < a.H * half; p += kLatentAppendThreads) {
-    T* r = q + (int64_t)(p / half) * (a.dim + a.rot) + a.dim;
-    turn_pair<T>(r, r, p % half, a.rot_dims, cs[p % half]);
-  }
-  if (dkv_col < 0) return;
-  const T* x = q + dkv_col;
-  T* out = cache + (int64_t)b * seq_stride + (int64_t)pos * a.row;
+__device__ __forceinline__ void append_row(const LatentShape& a, const T* x, T* out, const T* norm_w, float eps, const float2* cs, float* red) {
+  const int tid = threadIdx.x, nt = blockDim.x, half = a.rot_dims / 2;
   float s = 0.0f;
-  for (int i = tid; i < a.rank; i += kLatentAppendThreads) {
+  for (int i = tid; i < a.rank; i += nt) {
     const float v = to_f<T>(x[i]);
     s += v * v;
   }
+  for (int i = tid; i < half; i += nt) turn_pair<T>(x + a.rank, out + a.rank, i, a.rot_dims, cs[i]);
+  for (int i = a.rot_dims + tid; i < a.rot; i += nt) out[a.rank + i] = x[a.rank + i];
   s = block_sum(s, red);
   const float inv = 1.0f / sqrtf(s / (float)a.rank + eps);
-  for (int i = tid; i < a.rank; i += kLatentAppendThreads) out[i] = from_f<T>(to_f<T>(x[i]) * inv * to_f<T>(norm_w[i]));
-  for (int i = tid; i < half; i += kLatentAppendThreads) turn_pair<T>(x + a.rank, out + a.rank, i, a.rot_dims, cs[i]);
-  for (int i = a.rot_dims + tid; i < a.rot; i += kLatentAppendThreads) out[a.rank + i] = x[a.rank + i];
+  for (int i = tid; i < a.rank; i += nt) out[i] = from_f<T>(to_f<T>(x[i]) * inv * to_f<T>(norm_w[i]));
 }
 
-// q_lat[row, h, :] = [sum_d q[row, h, d] Uk[h * dim + d, :] | rotated part | zeros]
+struct LatentAppend {   // what the append needs beside the rows
+  int dkv_col;          // column of dkv in a q | dkv row; < 0: the layer reads another layer's cache
+  const void* norm_w;
+  float eps;
+  void* cache;
+  int64_t seq_stride;
+  int S, T0;
+  const int* state;
+  int Tmax;
+  const float2* tab;
+};
+
+// rows r0 .. r0 + n - 1 of the batch, one per blockIdx.y
+template <typename T>
+__device__ __forceinline__ void append_rows(const LatentShape& a, const T* q, int q_stride, int r0, int n, const LatentAppend& ap, float* red) {
+  for (int r = blockIdx.y; r < n; r += gridDim.y) {
+    const int row = r0 + r, b = row / ap.S, pos = state_len(ap.state, b, ap.T0) + row % ap.S;
+    TSB_DEV_CHECK(latent, pos >= 0 && pos < ap.Tmax, 0x602, continue)   // append position outside the cache
+    if (pos >= ap.Tmax) continue;
+    append_row<T>(a, q + (int64_t)row * q_stride + ap.dkv_col, reinterpret_cast<T*>(ap.cache) + (int64_t)b * ap.seq_stride + (int64_t)pos * a.row,
+                  (const T*)ap.norm_w, ap.eps, ap.tab + (int64_t)pos * (a.rot_dims / 2), red);
+    __syncthreads();
+  }
+}
+// q_lat[row, h, rank ..] = [rotated part | zeros] for n rows
+template <typename T>
+__device__ __forceinline__ void turn_queries(const LatentShape& a, T* q_lat, const T* q, int q_stride, int h, int r0, int n, const LatentAppend& ap) {
+  const int tail = a.row - a.rank, half = a.rot_dims / 2;
+  for (int i = threadIdx.x; i < n * tail; i += blockDim.x) {
+    const int r = i / tail, e = i % tail, row = r0 + r;
+    const T* x = q + (int64_t)row * q_stride + (int64_t)h * (a.dim + a.rot) + a.dim;
+    float v = 0.0f;
+    if (e < a.rot_dims) {
+      const int pos = min(state_len(ap.state, row / ap.S, ap.T0) + row % ap.S, ap.Tmax - 1);
+      const float2 cs = ap.tab[(int64_t)pos * half + (e < half ? e : e - half)];
+      v = e < half ? to_f<T>(x[e]) * cs.x - to_f<T>(x[e + half]) * cs.y : to_f<T>(x[e]) * cs.x + to_f<T>(x[e - half]) * cs.y;
+    } else if (e < a.rot) {
+      v = to_f<T>(x[e]);
+    }
+    q_lat[((int64_t)row * a.H + h) * a.row + a.rank + e] = from_f<T>(v);
+  }
+}
+
+// expanded form: queries turned in place, cache rows appended.  grid (rows, 2): y = 0 the query, y = 1 the cache row
+constexpr int kLatentAppendThreads = 128;
+template <typename T>
+__global__ void __launch_bounds__(kLatentAppendThreads) latent_append_kernel(LatentShape a, T* qkv, int row_stride, LatentAppend ap) {
+  __shared__ float red[32];
+  pdl_trigger();
+  pdl_wait();
+  const int row = blockIdx.x, b = row / ap.S, tid = threadIdx.x;
+  const int pos = state_len(ap.state, b, ap.T0) + row % ap.S;
+  TSB_DEV_CHECK(latent, pos >= 0 && pos < ap.Tmax, 0x601, return)   // append position outside the cache
+  if (pos >= ap.Tmax) return;   // capacity is checked on the host; never write past the cache
+  const int half = a.rot_dims / 2;
+  const float2* cs = ap.tab + (int64_t)pos * half;
+  T* q = qkv + (int64_t)row * row_stride;
+  if (blockIdx.y == 0) {
+    for (int p = tid; p < a.H * half; p += kLatentAppendThreads) {
+      T* r = q + (int64_t)(p / half) * (a.dim + a.rot) + a.dim;
+      turn_pair<T>(r, r, p % half, a.rot_dims, cs[p % half]);
+    }
+  } else {
+    append_row<T>(a, q + ap.dkv_col, reinterpret_cast<T*>(ap.cache) + (int64_t)b * ap.seq_stride + (int64_t)pos * a.row, (const T*)ap.norm_w, ap.eps, cs, red);
+  }
+}
+
+// absorbed form: q_lat[row, h, :] = [sum_d q[row, h, d] Uk[h * dim + d, :] | rotated part | zeros] for eight rows per CTA; the CTAs with
+// blockIdx.x == H append the rows' cache rows (one row per blockIdx.y)
 constexpr int kLqThreads = 256, kLqCols = 64, kLqRows = 8;
 template <typename T>
-__global__ void __launch_bounds__(kLqThreads) latent_query_kernel(LatentShape a, T* q_lat, const T* q, int q_stride, const T* uk, int rows) {
+__global__ void __launch_bounds__(kLqThreads) latent_query_kernel(LatentShape a, T* q_lat, const T* q, int q_stride, const T* uk, int rows, LatentAppend ap) {
   extern __shared__ float s_q[];              // [8 rows][dim]
   __shared__ float s_red[8][kLqRows][kLqCols];
   pdl_trigger();
-  pdl_wait();
   const int h = blockIdx.x, c0 = blockIdx.y * kLqCols, r0 = blockIdx.z * kLqRows;
   const int n = min(kLqRows, rows - r0);
   const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
-  for (int i = tid; i < kLqRows * a.dim; i += kLqThreads) {
-    const int r = i / a.dim;
-    s_q[i] = r < n ? to_f<T>(q[(int64_t)(r0 + r) * q_stride + (int64_t)h * (a.dim + a.rot) + i % a.dim]) : 0.0f;
+  if (h == a.H) {
+    pdl_wait();
+    append_rows<T>(a, q, q_stride, r0, n, ap, &s_red[0][0][0]);
+    return;
   }
-  if (blockIdx.y == 0) {
-    const int tail = a.row - a.rank;
-    for (int i = tid; i < n * tail; i += kLqThreads) {
-      const int r = i / tail, e = i % tail;
-      const T v = e < a.rot ? q[(int64_t)(r0 + r) * q_stride + (int64_t)h * (a.dim + a.rot) + a.dim + e] : from_f<T>(0.0f);
-      q_lat[((int64_t)(r0 + r) * a.H + h) * a.row + a.rank + e] = v;
+  // this warp's first weights do not depend on the previous kernel
+  const int c = c0 + lane * 2;
+  const bool in0 = c < a.rank, in1 = c + 1 < a.rank;
+  constexpr int PRE = 16;
+  float u0[PRE], u1[PRE];
+#pragma unroll
+  for (int k = 0; k < PRE; ++k) {
+    const int dd = w + 8 * k;
+    const T* u = uk + ((int64_t)h * a.dim + dd) * a.rank + c;
+    u0[k] = u1[k] = 0.0f;
+    if (dd < a.dim && in0) {
+      if (sizeof(T) == 2 && a.rank % 2 == 0) {
+        const float2 t = Pair16<bf16>::get(*reinterpret_cast<const uint32_t*>(u));
+        u0[k] = t.x;
+        u1[k] = t.y;
+      } else {
+        u0[k] = to_f<T>(u[0]);
+        if (in1) u1[k] = to_f<T>(u[1]);
+      }
     }
   }
+  pdl_wait();
+  const T* qh = q + (int64_t)h * (a.dim + a.rot);
+  for (int i = tid; i < kLqRows * a.dim; i += kLqThreads) {
+    const int r = i / a.dim;
+    s_q[i] = r < n ? to_f<T>(qh[(int64_t)(r0 + r) * q_stride + i % a.dim]) : 0.0f;
+  }
+  if (blockIdx.y == 0) turn_queries<T>(a, q_lat, q, q_stride, h, r0, n, ap);
   __syncthreads();
-  const int c = c0 + lane * 2;
   float acc[kLqRows][2];
 #pragma unroll
   for (int r = 0; r < kLqRows; ++r) acc[r][0] = acc[r][1] = 0.0f;
-  const bool in0 = c < a.rank, in1 = c + 1 < a.rank;
-#pragma unroll 8
-  for (int dd = w; dd < a.dim; dd += 8) {
+#pragma unroll
+  for (int k = 0; k < PRE; ++k) {
+    const int dd = w + 8 * k;
+    if (dd < a.dim)
+#pragma unroll
+      for (int r = 0; r < kLqRows; ++r) {
+        acc[r][0] = fmaf(s_q[r * a.dim + dd], u0[k], acc[r][0]);
+        acc[r][1] = fmaf(s_q[r * a.dim + dd], u1[k], acc[r][1]);
+      }
+  }
+#pragma unroll 4
+  for (int dd = w + 8 * PRE; dd < a.dim; dd += 8) {
     const T* u = uk + ((int64_t)h * a.dim + dd) * a.rank + c;
-    const float u0 = in0 ? to_f<T>(u[0]) : 0.0f, u1 = in1 ? to_f<T>(u[1]) : 0.0f;
+    const float t0 = in0 ? to_f<T>(u[0]) : 0.0f, t1 = in1 ? to_f<T>(u[1]) : 0.0f;
 #pragma unroll
     for (int r = 0; r < kLqRows; ++r) {
-      acc[r][0] = fmaf(s_q[r * a.dim + dd], u0, acc[r][0]);
-      acc[r][1] = fmaf(s_q[r * a.dim + dd], u1, acc[r][1]);
+      acc[r][0] = fmaf(s_q[r * a.dim + dd], t0, acc[r][0]);
+      acc[r][1] = fmaf(s_q[r * a.dim + dd], t1, acc[r][1]);
     }
   }
 #pragma unroll
@@ -149,6 +226,77 @@ __global__ void __launch_bounds__(kLqThreads) latent_query_kernel(LatentShape a,
     for (int q8 = 0; q8 < 8; ++q8) v += s_red[q8][r][e];
     q_lat[((int64_t)(r0 + r) * a.H + h) * a.row + c0 + e] = from_f<T>(v);
   }
+}
+
+// The same on the warp-level tensor cores: 16 * MT rows and 64 latent columns per CTA, each warp 16 columns.  Uk's tile is requested
+// before the wait on the previous kernel.
+constexpr int kLqmThreads = 128;
+__host__ __device__ inline int latent_q_pitch(int dim) { return (dim + 15) / 16 * 32 + 16; }
+template <int MT>
+__global__ void __launch_bounds__(kLqmThreads) latent_query_mma_kernel(LatentShape a, bf16* q_lat, const bf16* q, int q_stride, const bf16* uk, int rows,
+                                                                       LatentAppend ap) {
+  extern __shared__ __align__(128) unsigned char smem[];   // Uk tile [dim to 16][64], query rows [16 MT][dim to 16]
+  constexpr int WP = 64 * 2 + 16;
+  __shared__ float red[32];
+  pdl_trigger();
+  const int h = blockIdx.x, c0 = blockIdx.y * 64, r0 = blockIdx.z * 16 * MT, n = min(16 * MT, rows - r0);
+  const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
+  if (h == a.H) {
+    pdl_wait();
+    append_rows<bf16>(a, q, q_stride, r0, n, ap, red);
+    return;
+  }
+  const int kd = (a.dim + 15) / 16 * 16, qp = latent_q_pitch(a.dim);
+  const uint32_t sw = la_smem(smem), sq = sw + kd * WP;
+  for (int i = tid; i < kd * 8; i += kLqmThreads) {
+    const int k = i >> 3, c = c0 + (i & 7) * 8;
+    const bool live = k < a.dim && c < a.rank;
+    la_cp16(sw + k * WP + (i & 7) * 16, uk + ((int64_t)h * a.dim + (live ? k : 0)) * a.rank + (live ? c : 0), live);
+  }
+  pdl_wait();
+  const int qc = kd / 8, dc = a.dim / 8;
+  for (int r = w; r < 16 * MT; r += kLqmThreads / 32)
+    for (int c = lane; c < qc; c += 32) {
+      const bool live = r < n && c < dc;
+      la_cp16(sq + r * qp + c * 16, q + (int64_t)(r0 + (live ? r : 0)) * q_stride + (int64_t)h * (a.dim + a.rot) + (live ? c : 0) * 8, live);
+    }
+  la_commit();
+  if (blockIdx.y == 0) turn_queries<bf16>(a, q_lat, q, q_stride, h, r0, n, ap);
+  la_wait<0>();
+  __syncthreads();
+  float d[MT][2][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) d[m][i][e] = 0.0f;
+  const uint32_t wa = sw + ((lane & 7) + ((lane >> 3) & 1) * 8) * WP + w * 32 + (lane >> 4) * 16;
+  const uint32_t aa = sq + (lane & 15) * qp + (lane >> 4) * 16;
+#pragma unroll 4
+  for (int ks = 0; ks < kd / 16; ++ks) {
+    uint32_t b0, b1, b2, b3;
+    la_ldsm_x4_trans(wa + ks * 16 * WP, b0, b1, b2, b3);
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      uint32_t a0, a1, a2, a3;
+      la_ldsm_x4(aa + m * 16 * qp + ks * 32, a0, a1, a2, a3);
+      mma_16816<bf16>(d[m][0], a0, a1, a2, a3, b0, b1);
+      mma_16816<bf16>(d[m][1], a0, a1, a2, a3, b2, b3);
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int c = c0 + w * 16 + i * 8 + 2 * t4;
+      if (c >= a.rank) continue;   // the latent is a multiple of eight
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int r = m * 16 + g8 + e * 8;
+        if (r < n) *reinterpret_cast<uint32_t*>(q_lat + ((int64_t)(r0 + r) * a.H + h) * a.row + c) = Pair16<bf16>::put(d[m][i][2 * e], d[m][i][2 * e + 1]);
+      }
+    }
 }
 
 // ---- absorbed form on CUDA cores: one CTA per (query, head) row and split -------------------------------------------------------
@@ -208,26 +356,26 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(LatentShape a, float* 
 }
 
 // ---- absorbed form on the warp-level tensor cores -------------------------------------------------------------------------------
-constexpr int kLmThreads = 256, kLmKeys = 64;
+constexpr int kLmThreads = 512, kLmKeys = 64;
 struct LatentMmaLayout {   // shared memory of latent_attn_mma_kernel
   int pitch;               // bytes of a staged row: an odd number of 16-byte units, so that ldmatrix rows fall into different banks
-  int stages;
-  size_t stage_bytes, q_off, s_off, p_off, st_off, total;
+  uint32_t stage_bytes, q_off, s_off, p_off, st_off, total;
 };
 __host__ __device__ inline LatentMmaLayout latent_mma_layout(int row, int stages) {
   LatentMmaLayout L;
   L.pitch = row * 2 + 16;
-  L.stages = stages;
-  L.stage_bytes = (size_t)kLmKeys * L.pitch;
+  L.stage_bytes = (uint32_t)kLmKeys * L.pitch;
   L.q_off = L.stage_bytes * stages;
-  L.s_off = L.q_off + (size_t)16 * L.pitch;
-  L.p_off = L.s_off + 16 * (kLmKeys + 4) * 4;
+  L.s_off = L.q_off + 16u * L.pitch;
+  L.p_off = L.s_off + 2 * 16 * (kLmKeys + 4) * 4;
   L.st_off = L.p_off + 16 * (kLmKeys + 8) * 2;
-  L.total = L.st_off + 48 * 4;
+  L.total = L.st_off + 16 * 4;
   return L;
 }
 
-template <int NBW>   // latent blocks of 8 columns a warp owns in the second product (even)
+// Sixteen warps.  Scores: warp w takes keys (w % 8) * 8 .. + 7 and one half of the inner dimension.  Softmax: warp w takes row w.
+// Second product: warp w owns NBW * 8 latent columns.
+template <int NBW>   // even
 __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape a, float* part, const bf16* q_lat, const bf16* cache, int64_t seq_stride,
                                                                      int S, int T0_arg, const int* state, int Tmax, int splits, int stages) {
   extern __shared__ __align__(128) unsigned char smem[];
@@ -246,36 +394,33 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
   const bf16* base = cache + (int64_t)b * seq_stride;
   const int cpr = a.row / 8;                   // 16-byte chunks per row
   const uint32_t sbase = la_smem(smem);
-  float* sS = reinterpret_cast<float*>(smem + L.s_off);
+  float* sS = reinterpret_cast<float*>(smem + L.s_off);   // [2 halves][16][SP]
   bf16* sP = reinterpret_cast<bf16*>(smem + L.p_off);
-  float* s_m = reinterpret_cast<float*>(smem + L.st_off);
-  float *s_l = s_m + 16, *s_c = s_m + 32;
-  constexpr int SP = kLmKeys + 4, PP = kLmKeys + 8;
+  float* s_c = reinterpret_cast<float*>(smem + L.st_off);
+  constexpr int SP = kLmKeys + 4, PP = kLmKeys + 8, NW = kLmThreads / 32;
 
   auto issue = [&](int tile) {
     if (tile < n_tiles) {
-      const uint32_t dst = sbase + (uint32_t)((tile % stages) * L.stage_bytes);
+      const uint32_t dst = sbase + (uint32_t)(tile % stages) * L.stage_bytes;
       const int t0 = t_beg + tile * kLmKeys;
-      for (int v = tid; v < kLmKeys * cpr; v += kLmThreads) {
-        const int tt = v / cpr, c = v % cpr;
+#pragma unroll
+      for (int q = 0; q < kLmKeys / NW; ++q) {
+        const int tt = w + q * NW;
         const int t = min(t0 + tt, t_end - 1);   // the tail re-reads the last key of the range; its scores are masked
-        la_cp16(dst + tt * L.pitch + c * 16, base + (int64_t)t * a.row + c * 8);
+        const bf16* src = base + (int64_t)t * a.row;
+        for (int c = lane; c < cpr; c += 32) la_cp16(dst + tt * L.pitch + c * 16, src + c * 8);
       }
     }
     la_commit();
   };
   issue(0);
   {
-    const bf16* src = q_lat + ((int64_t)b * R + r0) * a.row;
-    for (int v = tid; v < 16 * cpr; v += kLmThreads) {
-      const int rr = v / cpr, c = v % cpr;
+    const bool live = r0 + w < R;
+    const bf16* src = q_lat + ((int64_t)b * R + r0 + (live ? w : 0)) * a.row;
+    for (int c = lane; c < cpr; c += 32) {
       uint4 x = make_uint4(0, 0, 0, 0);
-      if (r0 + rr < R) x = *reinterpret_cast<const uint4*>(src + (int64_t)rr * a.row + c * 8);
-      *reinterpret_cast<uint4*>(smem + L.q_off + rr * L.pitch + c * 16) = x;
-    }
-    if (tid < 16) {
-      s_m[tid] = -INFINITY;
-      s_l[tid] = 0.0f;
+      if (live) x = *reinterpret_cast<const uint4*>(src + c * 8);
+      *reinterpret_cast<uint4*>(smem + L.q_off + w * L.pitch + c * 16) = x;
     }
   }
   float o[NBW][4];
@@ -284,10 +429,11 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[i][e] = 0.0f;
   const int col0 = w * NBW * 8;                // first latent column of this warp
-  const int ksteps = a.row / 16;
-  // softmax: thread -> row tid / 16, four keys from (tid % 16) * 4
-  const int sr = tid >> 4, sc0 = (tid & 15) * 4;
-  const int row_lim = r0 + sr < R ? T0 + (r0 + sr) / a.H + 1 : 0;   // keys [0, row_lim) are visible
+  const int ksteps = a.row / 16, kh = (ksteps + 1) / 2;
+  const int kb8 = w & 7, khalf = w >> 3;
+  const int ks_beg = khalf * kh, ks_end = khalf ? ksteps : kh;
+  const int row_lim = r0 + w < R ? T0 + (r0 + w) / a.H + 1 : 0;   // softmax row w: keys [0, row_lim) are visible
+  float m_run = -INFINITY, l_run = 0.0f;       // state of row w, the same in every lane
 
   for (int tile = 0; tile < n_tiles; ++tile) {
     if (stages > 1) {
@@ -298,14 +444,14 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
       la_wait<0>();
     }
     __syncthreads();
-    const uint32_t kb = sbase + (uint32_t)((tile % stages) * L.stage_bytes);
-    {   // scores of keys w * 8 .. + 7
+    const uint32_t kb = sbase + (uint32_t)(tile % stages) * L.stage_bytes;
+    {
       float c0[4] = {0.0f, 0.0f, 0.0f, 0.0f}, c1[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-      const uint32_t qa = sbase + (uint32_t)L.q_off + (lane & 15) * L.pitch + (lane >> 4) * 16;
-      const uint32_t ka = kb + (w * 8 + (lane & 7)) * L.pitch + (lane >> 3) * 16;
-      int ks = 0;
-#pragma unroll 2
-      for (; ks + 1 < ksteps; ks += 2) {
+      const uint32_t qa = sbase + L.q_off + (lane & 15) * L.pitch + (lane >> 4) * 16;
+      const uint32_t ka = kb + (kb8 * 8 + (lane & 7)) * L.pitch + (lane >> 3) * 16;
+      int ks = ks_beg;
+#pragma unroll 4
+      for (; ks + 1 < ks_end; ks += 2) {
         uint32_t a0, a1, a2, a3, b0, b1, b2, b3;
         la_ldsm_x4(ka + ks * 32, b0, b1, b2, b3);
         la_ldsm_x4(qa + ks * 32, a0, a1, a2, a3);
@@ -313,48 +459,33 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
         la_ldsm_x4(qa + ks * 32 + 32, a0, a1, a2, a3);
         mma_16816<bf16>(c1, a0, a1, a2, a3, b2, b3);
       }
-      if (ks < ksteps) {
+      if (ks < ks_end) {
         uint32_t a0, a1, a2, a3, b0, b1;
-        la_ldsm_x2(kb + (w * 8 + (lane & 7)) * L.pitch + ((lane >> 3) & 1) * 16 + ks * 32, b0, b1);
+        la_ldsm_x2(kb + (kb8 * 8 + (lane & 7)) * L.pitch + ((lane >> 3) & 1) * 16 + ks * 32, b0, b1);
         la_ldsm_x4(qa + ks * 32, a0, a1, a2, a3);
         mma_16816<bf16>(c0, a0, a1, a2, a3, b0, b1);
       }
-      float* d = sS + w * 8 + 2 * t4;
+      float* d = sS + khalf * 16 * SP + kb8 * 8 + 2 * t4;
       *reinterpret_cast<float2*>(d + g8 * SP) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
       *reinterpret_cast<float2*>(d + (g8 + 8) * SP) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
     }
     __syncthreads();
     {
-      const int t0 = t_beg + tile * kLmKeys + sc0;
-      const float4 z4 = *reinterpret_cast<const float4*>(sS + sr * SP + sc0);
-      float z[4] = {z4.x, z4.y, z4.z, z4.w};
-      float mx = -INFINITY;
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        z[e] = (t0 + e < t_end && t0 + e < row_lim) ? z[e] * a.scale : -INFINITY;
-        mx = fmaxf(mx, z[e]);
-      }
-#pragma unroll
-      for (int q = 8; q > 0; q >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, q));
-      const float m_old = s_m[sr], m_new = fmaxf(m_old, mx);
-      float p[4], sum = 0.0f;
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        p[e] = m_new == -INFINITY ? 0.0f : __expf(z[e] - m_new);   // a row may see none of these keys
-        sum += p[e];
-      }
-#pragma unroll
-      for (int q = 8; q > 0; q >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, q);
-      *reinterpret_cast<uint2*>(sP + sr * PP + sc0) = make_uint2(Pair16<bf16>::put(p[0], p[1]), Pair16<bf16>::put(p[2], p[3]));
-      if ((tid & 15) == 0) {
-        const float corr = m_new == -INFINITY ? 1.0f : __expf(m_old - m_new);
-        s_c[sr] = corr;
-        s_m[sr] = m_new;
-        s_l[sr] = s_l[sr] * corr + sum;
-      }
+      const int t0 = t_beg + tile * kLmKeys + 2 * lane;
+      const float2 zA = *reinterpret_cast<const float2*>(sS + w * SP + 2 * lane), zB = *reinterpret_cast<const float2*>(sS + (16 + w) * SP + 2 * lane);
+      const int lim = min(t_end, row_lim);
+      const float z0 = t0 < lim ? (zA.x + zB.x) * a.scale : -INFINITY, z1 = t0 + 1 < lim ? (zA.y + zB.y) * a.scale : -INFINITY;
+      const float m_new = fmaxf(m_run, warp_max(fmaxf(z0, z1)));
+      const bool none = m_new == -INFINITY;      // a row may see none of these keys
+      const float p0 = none ? 0.0f : __expf(z0 - m_new), p1 = none ? 0.0f : __expf(z1 - m_new);
+      const float corr = none ? 1.0f : __expf(m_run - m_new);
+      *reinterpret_cast<uint32_t*>(sP + w * PP + 2 * lane) = Pair16<bf16>::put(p0, p1);
+      l_run = l_run * corr + warp_sum(p0 + p1);
+      m_run = m_new;
+      if (lane == 0) s_c[w] = corr;
     }
     __syncthreads();
-    {
+    if (col0 < a.rank) {
       const float cA = s_c[g8], cB = s_c[g8 + 8];
 #pragma unroll
       for (int i = 0; i < NBW; ++i) {
@@ -369,7 +500,7 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
 #pragma unroll
         for (int i = 0; i < NBW; i += 2) {
           const int col = col0 + i * 8;
-          if (col < a.row) {   // the row is a multiple of 16 elements: both blocks of the pair are inside
+          if (col < a.rank) {   // the row is a multiple of 16 elements: both blocks of the pair are inside it
             uint32_t b0, b1, b2, b3;
             la_ldsm_x4_trans(va + ks * 16 * L.pitch + col * 2, b0, b1, b2, b3);
             mma_16816<bf16>(o[i], a0, a1, a2, a3, b0, b1);
@@ -383,68 +514,172 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
   la_wait<0>();
   const int rec = a.rank + 2;
   float* pb = part + (((int64_t)b * R + r0) * splits + split) * rec;
-  if (n_tiles == 0) __syncthreads();   // the initial states of an empty range
 #pragma unroll
   for (int i = 0; i < NBW; ++i) {
-    const int col = col0 + i * 8 + 2 * t4;
+    const int c = col0 + i * 8 + 2 * t4;
+    if (c >= a.rank) continue;   // the latent is a multiple of eight
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int rr = g8 + (e >> 1) * 8, c = col + (e & 1);
-      if (r0 + rr < R && c < a.rank) pb[(int64_t)rr * splits * rec + 2 + c] = o[i][e];
+    for (int e = 0; e < 2; ++e) {
+      const int rr = g8 + e * 8;
+      if (r0 + rr < R) *reinterpret_cast<float2*>(pb + (int64_t)rr * splits * rec + 2 + c) = make_float2(o[i][2 * e], o[i][2 * e + 1]);
     }
   }
-  if (tid < 16 && r0 + tid < R) {
-    pb[(int64_t)tid * splits * rec] = s_m[tid];
-    pb[(int64_t)tid * splits * rec + 1] = s_l[tid];
+  if (lane == 0 && r0 + w < R) {
+    pb[(int64_t)w * splits * rec] = m_run;
+    pb[(int64_t)w * splits * rec + 1] = l_run;
   }
 }
 
-// merges the splits of a (query, head) row and applies Uv_h: 32 value elements per CTA
-constexpr int kLvThreads = 256, kLvCols = 32;
-template <typename T>
-__global__ void __launch_bounds__(kLvThreads) latent_value_kernel(LatentShape a, T* out, const float* part, const T* uv, int splits) {
-  extern __shared__ float s_o[];
+// merges the splits of up to eight rows of one head and applies Uv_h: 32 value elements per CTA, four per warp
+constexpr int kLvThreads = 256, kLvCols = 32, kMaxSplits = 64;
+template <typename T, int kLvRows>
+__global__ void __launch_bounds__(kLvThreads) latent_value_kernel(LatentShape a, T* out, const float* part, const T* uv, int splits, int rows) {
+  extern __shared__ float s_o[];   // [8][rank]
+  __shared__ float s_w[kLvRows][kMaxSplits];
   pdl_trigger();
   pdl_wait();
-  const int64_t rr = blockIdx.x;
-  const int h = (int)(rr % a.H), v0 = blockIdx.y * kLvCols;
+  const int h = blockIdx.x, v0 = blockIdx.y * kLvCols, r0 = blockIdx.z * kLvRows;
+  const int n = min(kLvRows, rows - r0);
   const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, rec = a.rank + 2;
-  const float* p = part + rr * splits * rec;
-  float mx = -INFINITY, l = 0.0f;
-  for (int i = 0; i < splits; ++i) mx = fmaxf(mx, p[(int64_t)i * rec]);
-  for (int i = 0; i < splits; ++i) {
-    const float m = p[(int64_t)i * rec];
-    l += m == -INFINITY ? 0.0f : p[(int64_t)i * rec + 1] * expf(m - mx);
-  }
-  const float inv = l > 0.0f ? 1.0f / l : 0.0f;
-  for (int e = tid; e < a.rank; e += kLvThreads) {
-    float v = 0.0f;
-    for (int i = 0; i < splits; ++i) {
-      const float m = p[(int64_t)i * rec];
-      v += m == -INFINITY ? 0.0f : p[(int64_t)i * rec + 2 + e] * expf(m - mx);
-    }
-    s_o[e] = v * inv;
+  if (w < n) {   // weight of every split of row w
+    const float* p = part + ((int64_t)(r0 + w) * a.H + h) * splits * rec;
+    const float m0 = lane < splits ? p[(int64_t)lane * rec] : -INFINITY, m1 = lane + 32 < splits ? p[(int64_t)(lane + 32) * rec] : -INFINITY;
+    const float l0 = lane < splits ? p[(int64_t)lane * rec + 1] : 0.0f, l1 = lane + 32 < splits ? p[(int64_t)(lane + 32) * rec + 1] : 0.0f;
+    const float mx = warp_max(fmaxf(m0, m1));
+    const float e0 = m0 == -INFINITY ? 0.0f : expf(m0 - mx), e1 = m1 == -INFINITY ? 0.0f : expf(m1 - mx);
+    const float l = warp_sum(l0 * e0 + l1 * e1), inv = l > 0.0f ? 1.0f / l : 0.0f;
+    s_w[w][lane] = e0 * inv;
+    s_w[w][lane + 32] = e1 * inv;
   }
   __syncthreads();
-  for (int q = w; q < kLvCols && v0 + q < a.vdim; q += 8) {
-    const T* u = uv + ((int64_t)h * a.vdim + v0 + q) * a.rank;
-    float acc = 0.0f;
-    if constexpr (sizeof(T) == 2) {
-      if (a.rank % 2 == 0) {
-#pragma unroll 4
-        for (int e = lane * 2; e < a.rank; e += 64) {
-          const float2 t = Pair16<bf16>::get(*reinterpret_cast<const uint32_t*>(u + e));
-          acc = fmaf(t.x, s_o[e], acc);
-          acc = fmaf(t.y, s_o[e + 1], acc);
-        }
-      } else {
-        for (int e = lane; e < a.rank; e += 32) acc = fmaf(to_f<T>(u[e]), s_o[e], acc);
-      }
-    } else {
-      for (int e = lane; e < a.rank; e += 32) acc = fmaf(to_f<T>(u[e]), s_o[e], acc);
+  for (int i = tid; i < n * a.rank; i += kLvThreads) {
+    const int r = kLvRows == 1 ? 0 : i / a.rank, e = i - r * a.rank;
+    const float* p = part + ((int64_t)(r0 + r) * a.H + h) * splits * rec + 2 + e;
+    float v = 0.0f;
+#pragma unroll 8
+    for (int q = 0; q < splits; ++q) {
+      v = fmaf(s_w[r][q], p[(int64_t)q * rec], v);   // an empty split left zeros and has weight 0
     }
-    acc = warp_sum(acc);
-    if (lane == 0) out[rr * a.vdim + v0 + q] = from_f<T>(acc);
+    s_o[i] = v;
+  }
+  __syncthreads();
+  float acc[4][kLvRows];
+#pragma unroll
+  for (int q = 0; q < 4; ++q)
+#pragma unroll
+    for (int r = 0; r < kLvRows; ++r) acc[q][r] = 0.0f;
+  const T* u = uv + ((int64_t)h * a.vdim + v0 + w * 4) * a.rank;
+  const int nq = min(4, a.vdim - v0 - w * 4);   // <= 0: this warp's columns do not exist
+  bool pairs = false;
+  if constexpr (sizeof(T) == 2) pairs = a.rank % 2 == 0;
+  if (pairs) {
+    if constexpr (sizeof(T) == 2) {
+#pragma unroll 2
+      for (int e = lane * 2; e < a.rank; e += 64) {
+        float2 t[4];
+#pragma unroll
+        for (int q = 0; q < 4; ++q) t[q] = q < nq ? Pair16<bf16>::get(*reinterpret_cast<const uint32_t*>(u + (int64_t)q * a.rank + e)) : make_float2(0.0f, 0.0f);
+#pragma unroll
+        for (int r = 0; r < kLvRows; ++r)
+          if (r < n) {
+            const float2 o = *reinterpret_cast<const float2*>(s_o + r * a.rank + e);
+#pragma unroll
+            for (int q = 0; q < 4; ++q) acc[q][r] = fmaf(t[q].y, o.y, fmaf(t[q].x, o.x, acc[q][r]));
+          }
+      }
+    }
+  } else {
+    for (int e = lane; e < a.rank; e += 32) {
+      float t[4];
+#pragma unroll
+      for (int q = 0; q < 4; ++q) t[q] = q < nq ? to_f<T>(u[(int64_t)q * a.rank + e]) : 0.0f;
+#pragma unroll
+      for (int r = 0; r < kLvRows; ++r)
+        if (r < n) {
+          const float o = s_o[r * a.rank + e];
+#pragma unroll
+          for (int q = 0; q < 4; ++q) acc[q][r] = fmaf(t[q], o, acc[q][r]);
+        }
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < kLvRows; ++r)
+    if (r < n) {
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const float v = warp_sum(acc[q][r]);
+        if (lane == 0 && q < nq) out[((int64_t)(r0 + r) * a.H + h) * a.vdim + v0 + w * 4 + q] = from_f<T>(v);
+      }
+    }
+}
+
+// The same on the warp-level tensor cores: 16 rows of one head and 32 value elements per CTA.  Uv's tile is requested before the wait on
+// the previous kernel; warp w takes value block w % 4 and every second step of the inner dimension.
+__host__ __device__ inline int latent_v_pitch(int rank) { return (rank + 15) / 16 * 32 + 16; }
+__global__ void __launch_bounds__(kLvThreads) latent_value_mma_kernel(LatentShape a, bf16* out, const float* part, const bf16* uv, int splits, int rows) {
+  extern __shared__ __align__(128) unsigned char smem[];   // Uv tile [32][rank to 16], merged rows [16][rank to 16]
+  __shared__ float s_w[16][kMaxSplits];
+  __shared__ float4 s_half[4][32];
+  pdl_trigger();
+  const int h = blockIdx.x, v0 = blockIdx.y * kLvCols, r0 = blockIdx.z * 16;
+  const int n = min(16, rows - r0);
+  const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, g8 = lane >> 2, t4 = lane & 3, rec = a.rank + 2;
+  const int pitch = latent_v_pitch(a.rank), kr = (a.rank + 15) / 16 * 16, chunks = kr / 8, live_chunks = a.rank / 8;
+  const uint32_t su = la_smem(smem), so = su + 32 * pitch;
+  for (int q = w; q < 32; q += 8)
+    for (int c = lane; c < chunks; c += 32) {
+      const bool live = v0 + q < a.vdim && c < live_chunks;
+      la_cp16(su + q * pitch + c * 16, uv + ((int64_t)h * a.vdim + (live ? v0 + q : 0)) * a.rank + (live ? c : 0) * 8, live);
+    }
+  la_commit();
+  pdl_wait();
+  for (int r = w; r < n; r += 8) {   // weight of every split of row r
+    const float* p = part + ((int64_t)(r0 + r) * a.H + h) * splits * rec;
+    const float m0 = lane < splits ? p[(int64_t)lane * rec] : -INFINITY, m1 = lane + 32 < splits ? p[(int64_t)(lane + 32) * rec] : -INFINITY;
+    const float l0 = lane < splits ? p[(int64_t)lane * rec + 1] : 0.0f, l1 = lane + 32 < splits ? p[(int64_t)(lane + 32) * rec + 1] : 0.0f;
+    const float mx = warp_max(fmaxf(m0, m1));
+    const float e0 = m0 == -INFINITY ? 0.0f : expf(m0 - mx), e1 = m1 == -INFINITY ? 0.0f : expf(m1 - mx);
+    const float l = warp_sum(l0 * e0 + l1 * e1), inv = l > 0.0f ? 1.0f / l : 0.0f;
+    s_w[r][lane] = e0 * inv;
+    s_w[r][lane + 32] = e1 * inv;
+  }
+  __syncthreads();
+  const int half = kr / 2;   // pairs per row
+  for (int i = tid; i < 16 * half; i += kLvThreads) {
+    const int r = i / half, e = (i - r * half) * 2;
+    float x = 0.0f, y = 0.0f;
+    if (r < n && e < a.rank) {
+      const float* p = part + ((int64_t)(r0 + r) * a.H + h) * splits * rec + 2 + e;
+#pragma unroll 8
+      for (int q = 0; q < splits; ++q) {
+        const float2 t = *reinterpret_cast<const float2*>(p + (int64_t)q * rec);
+        x = fmaf(s_w[r][q], t.x, x);
+        y = fmaf(s_w[r][q], t.y, y);
+      }
+    }
+    *reinterpret_cast<uint32_t*>(smem + 32 * pitch + r * pitch + e * 2) = Pair16<bf16>::put(x, y);
+  }
+  la_wait<0>();
+  __syncthreads();
+  float d0[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+  const int nb = w & 3, kh = w >> 2;
+  const uint32_t aa = so + (lane & 15) * pitch + (lane >> 4) * 16, ba = su + (nb * 8 + (lane & 7)) * pitch + ((lane >> 3) & 1) * 16;
+#pragma unroll 4
+  for (int ks = kh; ks < kr / 16; ks += 2) {
+    uint32_t a0, a1, a2, a3, b0, b1;
+    la_ldsm_x4(aa + ks * 32, a0, a1, a2, a3);
+    la_ldsm_x2(ba + ks * 32, b0, b1);
+    mma_16816<bf16>(d0, a0, a1, a2, a3, b0, b1);
+  }
+  if (kh == 1) s_half[nb][lane] = make_float4(d0[0], d0[1], d0[2], d0[3]);
+  __syncthreads();
+  if (kh == 0) {
+    const float4 t = s_half[nb][lane];
+    const int c = v0 + nb * 8 + 2 * t4;
+    if (c < a.vdim) {   // the value size is even: the pair is inside
+      if (g8 < n) *reinterpret_cast<uint32_t*>(out + ((int64_t)(r0 + g8) * a.H + h) * a.vdim + c) = Pair16<bf16>::put(d0[0] + t.x, d0[1] + t.y);
+      if (g8 + 8 < n) *reinterpret_cast<uint32_t*>(out + ((int64_t)(r0 + g8 + 8) * a.H + h) * a.vdim + c) = Pair16<bf16>::put(d0[2] + t.z, d0[3] + t.w);
+    }
   }
 }
 
@@ -606,19 +841,6 @@ int launch_angle_table(int device, DeviceState* st, float2* tab, int Tmax, int d
   return check_launch("angle_table");
 }
 
-int launch_latent_append(int device, int dtype, const LatentShape& a, void* qkv, int row_stride, int dkv_col, const void* norm_w, float eps, void* cache,
-                         int64_t seq_stride, int B, int S, int T0, const int* state, int Tmax, const float2* tab, cudaStream_t s) {
-  TSB_CHECK(state || T0 + S <= Tmax, "latent_append: cache capacity exceeded (%d + %d > %d)", T0, S, Tmax);
-  if (dtype == TSB200_F32)
-    TSB_CUDA(launch_k(latent_append_kernel<float>, dim3(B * S), dim3(kLatentAppendThreads), 0, s, a, (float*)qkv, row_stride, dkv_col, (const float*)norm_w,
-                      eps, (float*)cache, seq_stride, S, T0, state, Tmax, tab));
-  else
-    TSB_CUDA(launch_k(latent_append_kernel<bf16>, dim3(B * S), dim3(kLatentAppendThreads), 0, s, a, (bf16*)qkv, row_stride, dkv_col, (const bf16*)norm_w, eps,
-                      (bf16*)cache, seq_stride, S, T0, state, Tmax, tab));
-  count_launch(device);
-  return check_launch("latent_append");
-}
-
 constexpr size_t kLatentSmemMax = 226 * 1024;
 static bool latent_mma_shape(int dtype, const LatentShape& a) {
   return dtype == TSB200_BF16 && a.rank % 8 == 0 && a.rank <= 1024 && latent_mma_layout(a.row, 1).total <= kLatentSmemMax;
@@ -666,57 +888,86 @@ static int latent_simple(int device, const LatentArgs& a, cudaStream_t s) {
   return 1;
 }
 
-template <typename T>
-static int latent_absorbed(int device, int dtype, const LatentArgs& a, cudaStream_t s) {
+static LatentAppend latent_append_args(const LatentArgs& a) {
+  return LatentAppend{a.dkv_col, a.norm_w, a.eps, a.cache, a.seq_stride, a.S, a.T0, a.state, a.Tmax, a.tab};
+}
+
+// bf16 shapes whose pieces are multiples of 16 bytes: every kernel of the absorbed form on the tensor cores
+static bool latent_mma_pieces(const LatentArgs& a) {
+  const LatentShape& sh = a.shape;
+  return latent_mma_shape(TSB200_BF16, sh) && sh.dim % 8 == 0 && (sh.dim + sh.rot) % 8 == 0 && a.q_stride % 8 == 0 && sh.vdim % 2 == 0;
+}
+static int latent_absorbed_mma(int device, DeviceState* st, const LatentArgs& a, cudaStream_t s) {
   const LatentShape& sh = a.shape;
   const int rows = a.B * a.S;
-  TSB_CHECK((int64_t)rows * sh.H * a.splits * (sh.rank + 2) <= a.part_elems, "latent attention: scratch too small for %d rows in %d splits", rows, a.splits);
+  static bool done[kMaxDevices] = {};
+  if (!done[device]) {
+    const auto dyn = cudaFuncAttributeMaxDynamicSharedMemorySize;
+    TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<2>, dyn, (int)kLatentSmemMax));
+    TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<4>, dyn, (int)kLatentSmemMax));
+    TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<8>, dyn, (int)kLatentSmemMax));
+    TSB_CUDA(cudaFuncSetAttribute(latent_query_mma_kernel<1>, dyn, (int)kLatentSmemMax));
+    TSB_CUDA(cudaFuncSetAttribute(latent_query_mma_kernel<4>, dyn, (int)kLatentSmemMax));
+    TSB_CUDA(cudaFuncSetAttribute(latent_value_mma_kernel, dyn, 48 * latent_v_pitch(1024)));
+    done[device] = true;
+  }
+  const LatentAppend ap = latent_append_args(a);
+  const int kd = (sh.dim + 15) / 16 * 16, mt = rows > 16 ? 4 : 1;
+  const size_t sq = (size_t)kd * (64 * 2 + 16) + (size_t)16 * mt * latent_q_pitch(sh.dim);
+  TSB_CHECK(sq <= kLatentSmemMax, "latent attention: unrotated head size %d is not supported", sh.dim);
+  TSB_CUDA(launch_k(mt == 4 ? latent_query_mma_kernel<4> : latent_query_mma_kernel<1>,
+                    dim3(sh.H + (a.dkv_col >= 0 ? 1 : 0), (sh.rank + 63) / 64, (rows + 16 * mt - 1) / (16 * mt)), dim3(kLqmThreads), sq, s, sh, (bf16*)a.q_lat,
+                    (const bf16*)a.q, a.q_stride, (const bf16*)a.uk, rows, ap));
+  const int stages = latent_mma_layout(sh.row, 2).total <= kLatentSmemMax ? 2 : 1;
+  auto k = sh.rank <= 256 ? latent_attn_mma_kernel<2> : (sh.rank <= 512 ? latent_attn_mma_kernel<4> : latent_attn_mma_kernel<8>);
+  TSB_CUDA(launch_k(k, dim3(a.splits, (a.S * sh.H + 15) / 16, a.B), dim3(kLmThreads), (size_t)latent_mma_layout(sh.row, stages).total, s, sh, a.part,
+                    (const bf16*)a.q_lat, (const bf16*)a.cache, a.seq_stride, a.S, a.T0, a.state, a.Tmax, a.splits, stages));
+  TSB_CUDA(launch_k(latent_value_mma_kernel, dim3(sh.H, (sh.vdim + kLvCols - 1) / kLvCols, (rows + 15) / 16), dim3(kLvThreads),
+                    (size_t)48 * latent_v_pitch(sh.rank), s, sh, (bf16*)a.out, (const float*)a.part, (const bf16*)a.uv, a.splits, rows));
+  count_launch(device, 3);
+  return check_launch("latent attention (tensor cores)");
+}
+
+// any type and size, CUDA cores
+template <typename T>
+static int latent_absorbed(int device, DeviceState* st, const LatentArgs& a, cudaStream_t s) {
+  const LatentShape& sh = a.shape;
+  const int rows = a.B * a.S;
   const size_t sq = (size_t)kLqRows * sh.dim * sizeof(float);
   TSB_CHECK(sq <= 24 * 1024, "latent attention: unrotated head size %d is not supported (at most 768)", sh.dim);
-  TSB_CUDA(launch_k(latent_query_kernel<T>, dim3(sh.H, (sh.rank + kLqCols - 1) / kLqCols, (rows + kLqRows - 1) / kLqRows), dim3(kLqThreads), sq, s, sh,
-                    (T*)a.q_lat, (const T*)a.q, a.q_stride, (const T*)a.uk, rows));
-  count_launch(device);
-  bool done_mma = false;
-  if constexpr (sizeof(T) == 2) {
-    if (latent_mma_shape(dtype, sh)) {
-      const int stages = latent_mma_layout(sh.row, 2).total <= kLatentSmemMax ? 2 : 1;
-      const size_t smem = latent_mma_layout(sh.row, stages).total;
-      const dim3 grid(a.splits, (a.S * sh.H + 15) / 16, a.B);
-      static bool done[kMaxDevices] = {};
-      if (!done[device]) {
-        TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLatentSmemMax));
-        TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLatentSmemMax));
-        TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLatentSmemMax));
-        TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLatentSmemMax));
-        done[device] = true;
-      }
-      auto k = sh.rank <= 128 ? latent_attn_mma_kernel<2>
-                              : (sh.rank <= 256 ? latent_attn_mma_kernel<4> : (sh.rank <= 512 ? latent_attn_mma_kernel<8> : latent_attn_mma_kernel<16>));
-      TSB_CUDA(launch_k(k, grid, dim3(kLmThreads), smem, s, sh, a.part, (const bf16*)a.q_lat, (const bf16*)a.cache, a.seq_stride, a.S, a.T0, a.state, a.Tmax,
-                        a.splits, stages));
-      done_mma = true;
-    }
-  }
-  if (!done_mma) TSB_TRY(latent_simple<T>(device, a, s));
-  count_launch(device);
-  TSB_CUDA(launch_k(latent_value_kernel<T>, dim3(rows * sh.H, (sh.vdim + kLvCols - 1) / kLvCols), dim3(kLvThreads), (size_t)sh.rank * 4, s, sh, (T*)a.out,
-                    (const float*)a.part, (const T*)a.uv, a.splits));
-  count_launch(device);
+  const LatentAppend ap = latent_append_args(a);
+  TSB_CUDA(launch_k(latent_query_kernel<T>, dim3(sh.H + (a.dkv_col >= 0 ? 1 : 0), (sh.rank + kLqCols - 1) / kLqCols, (rows + kLqRows - 1) / kLqRows),
+                    dim3(kLqThreads), sq, s, sh, (T*)a.q_lat, (const T*)a.q, a.q_stride, (const T*)a.uk, rows, ap));
+  TSB_TRY(latent_simple<T>(device, a, s));
+  const int vt = (sh.vdim + kLvCols - 1) / kLvCols;   // few rows: one per CTA, so that the merges run side by side; many: eight share a read of Uv
+  const int rb = (int64_t)sh.H * vt * rows >= 16 * (int64_t)st->sm_count ? 8 : 1;
+  auto k = rb == 8 ? latent_value_kernel<T, 8> : latent_value_kernel<T, 1>;
+  TSB_CUDA(launch_k(k, dim3(sh.H, vt, (rows + rb - 1) / rb), dim3(kLvThreads), (size_t)rb * sh.rank * 4, s, sh, (T*)a.out, (const float*)a.part, (const T*)a.uv,
+                    a.splits, rows));
+  count_launch(device, 3);
   return check_launch("latent attention");
 }
 
 int launch_latent_attention(int device, DeviceState* st, int dtype, const LatentArgs& a, cudaStream_t s) {
   if (a.B == 0 || a.S == 0) return 1;
   const LatentShape& sh = a.shape;
+  TSB_CHECK(a.state || a.T0 + a.S <= a.Tmax, "latent attention: cache capacity exceeded (%d + %d > %d)", a.T0, a.S, a.Tmax);
   if (!a.state && latent_expanded(dtype, sh, a.q_stride, a.S)) {
     const int T = a.T0 + a.S, kvw = sh.H * (sh.dim + sh.vdim);
+    latent_append_kernel<bf16><<<dim3(a.B * a.S, a.dkv_col >= 0 ? 2 : 1), kLatentAppendThreads, 0, s>>>(sh, (bf16*)a.q, a.q_stride, latent_append_args(a));
+    count_launch(device);
+    TSB_TRY(check_launch("latent_append"));
     TSB_CHECK((int64_t)a.B * T * kvw <= a.kv_elems, "latent attention: scratch too small for %d expanded keys", a.B * T);
-    for (int b = 0; b < a.B; ++b) {
-      Epilogue ep{};
-      ep.y = (bf16*)a.kv + (int64_t)b * T * kvw;
-      ep.act = TSB200_ACT_NONE;
-      TSB_TRY(launch_linear(device, st, dtype, (const bf16*)a.cache + (int64_t)b * a.seq_stride, a.ukv_packed, T, sh.row, kvw, ep, a.lin_ws, a.lin_ws_bytes, s, true));
+    const void* rows = a.cache;
+    if (a.B > 1) {   // the sequences' cache rows side by side: one product for the whole batch
+      TSB_CHECK((int64_t)a.B * T * sh.row <= a.compact_elems, "latent attention: scratch too small for %d cache rows", a.B * T);
+      TSB_CUDA(cudaMemcpy2DAsync(a.compact, (size_t)T * sh.row * 2, a.cache, (size_t)a.seq_stride * 2, (size_t)T * sh.row * 2, a.B, cudaMemcpyDeviceToDevice, s));
+      rows = a.compact;
     }
+    Epilogue ep{};
+    ep.y = a.kv;
+    ep.act = TSB200_ACT_NONE;
+    TSB_TRY(launch_linear(device, st, dtype, rows, a.ukv_packed, a.B * T, sh.row, kvw, ep, a.lin_ws, a.lin_ws_bytes, s, true));
     const int qk = (sh.dim + sh.rot + 15) / 16 * 16, vn = latent_vn(sh.vdim);
     const size_t smem = latent_prefill_smem(qk, vn);
     const dim3 grid((a.S + kLpRows - 1) / kLpRows, sh.H, a.B);
@@ -733,8 +984,10 @@ int launch_latent_attention(int device, DeviceState* st, int dtype, const Latent
     count_launch(device);
     return check_launch("latent_prefill_mma");
   }
-  if (dtype == TSB200_F32) return latent_absorbed<float>(device, dtype, a, s);
-  return latent_absorbed<bf16>(device, dtype, a, s);
+  TSB_CHECK(a.splits >= 1 && a.splits <= kMaxSplits, "latent attention: %d splits", a.splits);
+  TSB_CHECK((int64_t)a.B * a.S * sh.H * a.splits * (sh.rank + 2) <= a.part_elems, "latent attention: scratch too small for %d rows in %d splits", a.B * a.S, a.splits);
+  if (dtype == TSB200_F32) return latent_absorbed<float>(device, st, a, s);
+  return latent_mma_pieces(a) ? latent_absorbed_mma(device, st, a, s) : latent_absorbed<bf16>(device, st, a, s);
 }
 
 }  // namespace tsb

@@ -521,7 +521,7 @@ class GPT:
         N.call("TSB200_GptGetStepTimes", self._h, ms.ctypes.data_as(C.c_void_p), n, C.byref(got))
         return ms[:got.value]
 
-    KERNEL_CLASSES = ("embed", "norm", "linear", "rope_append", "attention", "sampling", "commit", "allreduce", "decode_stack")
+    KERNEL_CLASSES = ("embed", "norm", "linear", "rope_append", "attention", "sampling", "commit", "allreduce", "decode_stack", "experts")
 
     def ProfileDecode(self, n_steps, opts: DecodingOptions):
         """{class: (ms_total, launch_groups)} over n_steps un-captured decode steps (CUDA events per launch group)."""
@@ -531,6 +531,17 @@ class GPT:
         c = self._opts(opts)
         N.call("TSB200_GptProfileDecode", self._h, n_steps, C.byref(c), ms.ctypes.data_as(C.c_void_p),
                groups.ctypes.data_as(C.c_void_p), n)
+        return {k: (float(ms[i]), int(groups[i])) for i, k in enumerate(self.KERNEL_CLASSES)}
+
+    def ProfilePrefill(self, tokens, opts: DecodingOptions):
+        """{class: (ms_total, launches)} of one prefill on an empty cache (call Reset first)."""
+        ids = np.ascontiguousarray(np.asarray(tokens, dtype=np.int32))
+        n = len(self.KERNEL_CLASSES)
+        ms, groups = np.zeros(n, dtype=np.float32), np.zeros(n, dtype=np.int64)
+        c = self._opts(opts)
+        N.call("TSB200_GptProfilePrefill", self._h, ids.ctypes.data_as(C.c_void_p), ids.shape[0], ids.shape[1], C.byref(c), ms.ctypes.data_as(C.c_void_p),
+               groups.ctypes.data_as(C.c_void_p), n)
+        self._B = ids.shape[0]
         return {k: (float(ms[i]), int(groups[i])) for i, k in enumerate(self.KERNEL_CLASSES)}
 
     # ---- inspection --------------------------------------------------------------------------------

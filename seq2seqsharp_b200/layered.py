@@ -62,7 +62,10 @@ class LayeredConfig:
     logit_scale: float = 1.0
     dtype: str = "bfloat16"     # "bfloat16" | "float32"
     name: str = ""
+    # what a GPTConfig would say here: no attention over an encoder, no position table (positions are the mixers' business)
     cross_attn = False
+    pe = 0
+    ape_decode_pos0 = False
 
     @property
     def L(self):

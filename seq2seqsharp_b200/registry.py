@@ -48,8 +48,8 @@ def load_model(path: str, dtype: str = "bfloat16", device_id: int = 0, max_batch
         if missing:
             raise ValueError("%s: %d tensors are missing, the first is %s" % (tensors.path, len(missing), missing[0]))
         gpt = LayeredGPT(cfg, device_id=device_id, max_batch=max_batch, max_tokens=max_tokens)
-        for engine, n in names.items():
-            gpt.SetWeight(engine, tensors.get(n))
+        for engine in cfg.weight_shapes():
+            gpt.SetWeight(engine, tensors.get(names[engine]))
         return gpt
     from .model_file import load_gpt
     return load_gpt(path, device_id=device_id, max_batch=max_batch, max_tokens=max_tokens, dtype="float32" if dtype == "float32" else None)[0]
