@@ -318,6 +318,50 @@ __global__ void __launch_bounds__(256) short_conv_kernel(T* out, const T* h, con
     out[q] = from_f<T>(acc);
   }
 }
+// up to four taps, widths that are multiples of four: four channels and a strip of positions per thread, the window in registers
+constexpr int kConvStrip = 16;
+template <typename T>
+__global__ void __launch_bounds__(128) short_conv_strip_kernel(T* out, const T* h, const T* wgt, const T* ring, int S, int d, int taps, int T0_arg,
+                                                               const int* state) {
+  const int i = (blockIdx.x * 128 + threadIdx.x) * 4, s0 = blockIdx.y * kConvStrip, b = blockIdx.z;
+  if (i >= d) return;
+  const int T0 = state_len(state, b, T0_arg);
+  float cw[4][4];   // [positions back][channel]
+#pragma unroll
+  for (int q = 0; q < 4; ++q)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) cw[q][e] = q < taps ? to_f<T>(wgt[(int64_t)(i + e) * taps + taps - 1 - q]) : 0.0f;
+  const T* hb = h + (int64_t)b * S * d + i;
+  T* ob = out + (int64_t)b * S * d + i;
+  float past[3][4];
+#pragma unroll
+  for (int q = 1; q < 4; ++q) {
+    const int s = s0 - q, p = T0 + s;
+    past[q - 1][0] = past[q - 1][1] = past[q - 1][2] = past[q - 1][3] = 0.0f;
+    if (q < taps && p >= 0) {
+      if (s >= 0) VecIO<T, 4>::load(hb + (int64_t)s * d, past[q - 1]);
+      else VecIO<T, 4>::load(ring + ((int64_t)b * taps + p % taps) * d + i, past[q - 1]);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < kConvStrip; ++k) {
+    const int s = s0 + k;
+    if (s >= S) break;
+    float x[4], y[4];
+    VecIO<T, 4>::load(hb + (int64_t)s * d, x);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float acc = x[e];
+#pragma unroll
+      for (int q = 3; q >= 1; --q) acc += cw[q][e] * past[q - 1][e];   // oldest first, as in the other kernels
+      y[e] = acc + cw[0][e] * x[e];
+      past[2][e] = past[1][e];
+      past[1][e] = past[0][e];
+      past[0][e] = x[e];
+    }
+    VecIO<T, 4>::store(ob + (int64_t)s * d, y);
+  }
+}
 template <typename T>
 __global__ void __launch_bounds__(256) short_conv_state_kernel(T* ring, const T* h, int S, int d, int taps, int T0_arg, const int* state, const int* lens) {
   const int b = blockIdx.y;
@@ -482,12 +526,16 @@ int launch_short_conv(int device, DeviceState* st, int dtype, void* out, const v
   int64_t g = ((int64_t)B * S * d + 255) / 256;
   if (g > (int64_t)st->sm_count * 32) g = (int64_t)st->sm_count * 32;
   const dim3 g2((unsigned)((taps * d + 255) / 256), B);
+  const bool strip = taps <= 4 && d % 4 == 0 && B <= 65535 && (S + kConvStrip - 1) / kConvStrip <= 65535;
+  const dim3 gs((d / 4 + 127) / 128, (S + kConvStrip - 1) / kConvStrip, B);
   if (dtype == TSB200_F32) {
-    short_conv_kernel<float><<<(int)g, 256, 0, s>>>((float*)out, (const float*)h, (const float*)w, (const float*)ring, B, S, d, taps, T0, state);
+    if (strip) short_conv_strip_kernel<float><<<gs, 128, 0, s>>>((float*)out, (const float*)h, (const float*)w, (const float*)ring, S, d, taps, T0, state);
+    else short_conv_kernel<float><<<(int)g, 256, 0, s>>>((float*)out, (const float*)h, (const float*)w, (const float*)ring, B, S, d, taps, T0, state);
     short_conv_state_kernel<float><<<g2, 256, 0, s>>>((float*)ring, (const float*)h, S, d, taps, T0, state, lens);
   } else {
     typedef __nv_bfloat16 H;
-    short_conv_kernel<H><<<(int)g, 256, 0, s>>>((H*)out, (const H*)h, (const H*)w, (const H*)ring, B, S, d, taps, T0, state);
+    if (strip) short_conv_strip_kernel<H><<<gs, 128, 0, s>>>((H*)out, (const H*)h, (const H*)w, (const H*)ring, S, d, taps, T0, state);
+    else short_conv_kernel<H><<<(int)g, 256, 0, s>>>((H*)out, (const H*)h, (const H*)w, (const H*)ring, B, S, d, taps, T0, state);
     short_conv_state_kernel<H><<<g2, 256, 0, s>>>((H*)ring, (const H*)h, S, d, taps, T0, state, lens);
   }
   count_launch(device, 2);

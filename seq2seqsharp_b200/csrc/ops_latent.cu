@@ -89,10 +89,10 @@ struct LatentAppend {   // what the append needs beside the rows
   const float2* tab;
 };
 
-// rows r0 .. r0 + n - 1 of the batch, one per blockIdx.y
+// rows r0 .. r0 + n - 1 of the batch, one per CTA of the columns blockIdx.x >= H
 template <typename T>
 __device__ __forceinline__ void append_rows(const LatentShape& a, const T* q, int q_stride, int r0, int n, const LatentAppend& ap, float* red) {
-  for (int r = blockIdx.y; r < n; r += gridDim.y) {
+  for (int r = (blockIdx.x - a.H) * gridDim.y + blockIdx.y; r < n; r += (gridDim.x - a.H) * gridDim.y) {
     const int row = r0 + r, b = row / ap.S, pos = state_len(ap.state, b, ap.T0) + row % ap.S;
     TSB_DEV_CHECK(latent, pos >= 0 && pos < ap.Tmax, 0x602, continue)   // append position outside the cache
     if (pos >= ap.Tmax) continue;
@@ -101,11 +101,11 @@ __device__ __forceinline__ void append_rows(const LatentShape& a, const T* q, in
     __syncthreads();
   }
 }
-// q_lat[row, h, rank ..] = [rotated part | zeros] for n rows
+// q_lat[row, h, rank ..] = [rotated part | zeros] for n rows, shared out over blockIdx.y
 template <typename T>
 __device__ __forceinline__ void turn_queries(const LatentShape& a, T* q_lat, const T* q, int q_stride, int h, int r0, int n, const LatentAppend& ap) {
   const int tail = a.row - a.rank, half = a.rot_dims / 2;
-  for (int i = threadIdx.x; i < n * tail; i += blockDim.x) {
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < n * tail; i += gridDim.y * blockDim.x) {
     const int r = i / tail, e = i % tail, row = r0 + r;
     const T* x = q + (int64_t)row * q_stride + (int64_t)h * (a.dim + a.rot) + a.dim;
     float v = 0.0f;
@@ -145,7 +145,7 @@ __global__ void __launch_bounds__(kLatentAppendThreads) latent_append_kernel(Lat
 }
 
 // absorbed form: q_lat[row, h, :] = [sum_d q[row, h, d] Uk[h * dim + d, :] | rotated part | zeros] for eight rows per CTA; the CTAs with
-// blockIdx.x == H append the rows' cache rows (one row per blockIdx.y)
+// blockIdx.x >= H append the rows' cache rows
 constexpr int kLqThreads = 256, kLqCols = 64, kLqRows = 8;
 template <typename T>
 __global__ void __launch_bounds__(kLqThreads) latent_query_kernel(LatentShape a, T* q_lat, const T* q, int q_stride, const T* uk, int rows, LatentAppend ap) {
@@ -155,7 +155,7 @@ __global__ void __launch_bounds__(kLqThreads) latent_query_kernel(LatentShape a,
   const int h = blockIdx.x, c0 = blockIdx.y * kLqCols, r0 = blockIdx.z * kLqRows;
   const int n = min(kLqRows, rows - r0);
   const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
-  if (h == a.H) {
+  if (h >= a.H) {
     pdl_wait();
     append_rows<T>(a, q, q_stride, r0, n, ap, &s_red[0][0][0]);
     return;
@@ -187,7 +187,7 @@ __global__ void __launch_bounds__(kLqThreads) latent_query_kernel(LatentShape a,
     const int r = i / a.dim;
     s_q[i] = r < n ? to_f<T>(qh[(int64_t)(r0 + r) * q_stride + i % a.dim]) : 0.0f;
   }
-  if (blockIdx.y == 0) turn_queries<T>(a, q_lat, q, q_stride, h, r0, n, ap);
+  turn_queries<T>(a, q_lat, q, q_stride, h, r0, n, ap);
   __syncthreads();
   float acc[kLqRows][2];
 #pragma unroll
@@ -241,7 +241,7 @@ __global__ void __launch_bounds__(kLqmThreads) latent_query_mma_kernel(LatentSha
   pdl_trigger();
   const int h = blockIdx.x, c0 = blockIdx.y * 64, r0 = blockIdx.z * 16 * MT, n = min(16 * MT, rows - r0);
   const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
-  if (h == a.H) {
+  if (h >= a.H) {
     pdl_wait();
     append_rows<bf16>(a, q, q_stride, r0, n, ap, red);
     return;
@@ -261,7 +261,7 @@ __global__ void __launch_bounds__(kLqmThreads) latent_query_mma_kernel(LatentSha
       la_cp16(sq + r * qp + c * 16, q + (int64_t)(r0 + (live ? r : 0)) * q_stride + (int64_t)h * (a.dim + a.rot) + (live ? c : 0) * 8, live);
     }
   la_commit();
-  if (blockIdx.y == 0) turn_queries<bf16>(a, q_lat, q, q_stride, h, r0, n, ap);
+  turn_queries<bf16>(a, q_lat, q, q_stride, h, r0, n, ap);
   la_wait<0>();
   __syncthreads();
   float d[MT][2][4];
@@ -356,26 +356,27 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(LatentShape a, float* 
 }
 
 // ---- absorbed form on the warp-level tensor cores -------------------------------------------------------------------------------
-constexpr int kLmThreads = 512, kLmKeys = 64;
+constexpr int kLmThreads = 512, kLmKeys = 32, kLmMaxStages = 5;
 struct LatentMmaLayout {   // shared memory of latent_attn_mma_kernel
   int pitch;               // bytes of a staged row: an odd number of 16-byte units, so that ldmatrix rows fall into different banks
-  uint32_t stage_bytes, q_off, s_off, p_off, st_off, total;
+  uint32_t stage_bytes, s_off, p_off, c_off, total;
 };
 __host__ __device__ inline LatentMmaLayout latent_mma_layout(int row, int stages) {
   LatentMmaLayout L;
   L.pitch = row * 2 + 16;
   L.stage_bytes = (uint32_t)kLmKeys * L.pitch;
-  L.q_off = L.stage_bytes * stages;
-  L.s_off = L.q_off + 16u * L.pitch;
-  L.p_off = L.s_off + 2 * 16 * (kLmKeys + 4) * 4;
-  L.st_off = L.p_off + 16 * (kLmKeys + 8) * 2;
-  L.total = L.st_off + 16 * 4;
+  L.s_off = L.stage_bytes * stages;
+  L.p_off = L.s_off + 4 * 16 * (kLmKeys + 4) * 4;
+  L.c_off = L.p_off + 16 * (kLmKeys + 8) * 2;
+  L.total = L.c_off + 16 * 4;
   return L;
 }
 
-// Sixteen warps.  Scores: warp w takes keys (w % 8) * 8 .. + 7 and one half of the inner dimension.  Softmax: warp w takes row w.
-// Second product: warp w owns NBW * 8 latent columns.
-template <int NBW>   // even
+// 16 (query, head) rows, sixteen warps, tiles of 32 keys in a ring of 3..5 stages.  Scores: warp w takes keys (w % 4) * 8 .. + 7 and a
+// quarter of the inner dimension, its query fragments in registers (KQ steps at most).  Softmax: warp w takes row w, one key per lane.
+// Second product: warp w owns NBW * 8 latent columns.  The scores of tile t and the second product of tile t - 1 share an interval between
+// two barriers, so a tile costs two of them.
+template <int NBW, int KQ>   // NBW even
 __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape a, float* part, const bf16* q_lat, const bf16* cache, int64_t seq_stride,
                                                                      int S, int T0_arg, const int* state, int Tmax, int splits, int stages) {
   extern __shared__ __align__(128) unsigned char smem[];
@@ -394,9 +395,9 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
   const bf16* base = cache + (int64_t)b * seq_stride;
   const int cpr = a.row / 8;                   // 16-byte chunks per row
   const uint32_t sbase = la_smem(smem);
-  float* sS = reinterpret_cast<float*>(smem + L.s_off);   // [2 halves][16][SP]
+  float* sS = reinterpret_cast<float*>(smem + L.s_off);   // [4 quarters][16][SP]
   bf16* sP = reinterpret_cast<bf16*>(smem + L.p_off);
-  float* s_c = reinterpret_cast<float*>(smem + L.st_off);
+  float* s_c = reinterpret_cast<float*>(smem + L.c_off);
   constexpr int SP = kLmKeys + 4, PP = kLmKeys + 8, NW = kLmThreads / 32;
 
   auto issue = [&](int tile) {
@@ -413,14 +414,21 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
     }
     la_commit();
   };
-  issue(0);
+  const int ahead = stages - 2;                // tiles in flight beside the one being scored and the one before it
+  for (int i = 0; i < ahead; ++i) issue(i);
+  const int ksteps = a.row / 16, kq4 = (ksteps + 3) / 4;
+  const int kblk = w & 3, ks_beg = (w >> 2) * kq4, ks_n = max(0, min(ksteps - ks_beg, kq4));
+  uint32_t qf[KQ][4];
   {
-    const bool live = r0 + w < R;
-    const bf16* src = q_lat + ((int64_t)b * R + r0 + (live ? w : 0)) * a.row;
-    for (int c = lane; c < cpr; c += 32) {
-      uint4 x = make_uint4(0, 0, 0, 0);
-      if (live) x = *reinterpret_cast<const uint4*>(src + c * 8);
-      *reinterpret_cast<uint4*>(smem + L.q_off + w * L.pitch + c * 16) = x;
+    const bool la = r0 + g8 < R, lb = r0 + g8 + 8 < R;
+    const bf16* qa = q_lat + ((int64_t)b * R + r0 + (la ? g8 : 0)) * a.row + ks_beg * 16 + 2 * t4;
+    const bf16* qb = q_lat + ((int64_t)b * R + r0 + (lb ? g8 + 8 : 0)) * a.row + ks_beg * 16 + 2 * t4;
+#pragma unroll
+    for (int k = 0; k < KQ; ++k) {
+      qf[k][0] = k < ks_n && la ? *reinterpret_cast<const uint32_t*>(qa + k * 16) : 0u;
+      qf[k][1] = k < ks_n && lb ? *reinterpret_cast<const uint32_t*>(qb + k * 16) : 0u;
+      qf[k][2] = k < ks_n && la ? *reinterpret_cast<const uint32_t*>(qa + k * 16 + 8) : 0u;
+      qf[k][3] = k < ks_n && lb ? *reinterpret_cast<const uint32_t*>(qb + k * 16 + 8) : 0u;
     }
   }
   float o[NBW][4];
@@ -429,70 +437,39 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[i][e] = 0.0f;
   const int col0 = w * NBW * 8;                // first latent column of this warp
-  const int ksteps = a.row / 16, kh = (ksteps + 1) / 2;
-  const int kb8 = w & 7, khalf = w >> 3;
-  const int ks_beg = khalf * kh, ks_end = khalf ? ksteps : kh;
-  const int row_lim = r0 + w < R ? T0 + (r0 + w) / a.H + 1 : 0;   // softmax row w: keys [0, row_lim) are visible
+  const int row_lim = min(t_end, r0 + w < R ? T0 + (r0 + w) / a.H + 1 : 0);   // softmax row w: keys below are visible to it
   float m_run = -INFINITY, l_run = 0.0f;       // state of row w, the same in every lane
 
-  for (int tile = 0; tile < n_tiles; ++tile) {
-    if (stages > 1) {
-      issue(tile + 1);
-      la_wait<1>();
-    } else {
-      if (tile > 0) issue(tile);
-      la_wait<0>();
-    }
+  for (int tile = 0; tile <= n_tiles; ++tile) {
+    issue(tile + ahead);                       // over the stage of tile - 2, which the previous interval was the last to read
+    if (ahead == 3) la_wait<3>();
+    else if (ahead == 2) la_wait<2>();
+    else la_wait<1>();
     __syncthreads();
-    const uint32_t kb = sbase + (uint32_t)(tile % stages) * L.stage_bytes;
-    {
+    if (tile < n_tiles) {
+      const uint32_t ka = sbase + (uint32_t)(tile % stages) * L.stage_bytes + (kblk * 8 + (lane & 7)) * L.pitch + (lane >> 3) * 16 + ks_beg * 32;
       float c0[4] = {0.0f, 0.0f, 0.0f, 0.0f}, c1[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-      const uint32_t qa = sbase + L.q_off + (lane & 15) * L.pitch + (lane >> 4) * 16;
-      const uint32_t ka = kb + (kb8 * 8 + (lane & 7)) * L.pitch + (lane >> 3) * 16;
-      int ks = ks_beg;
-#pragma unroll 4
-      for (; ks + 1 < ks_end; ks += 2) {
-        uint32_t a0, a1, a2, a3, b0, b1, b2, b3;
-        la_ldsm_x4(ka + ks * 32, b0, b1, b2, b3);
-        la_ldsm_x4(qa + ks * 32, a0, a1, a2, a3);
-        mma_16816<bf16>(c0, a0, a1, a2, a3, b0, b1);
-        la_ldsm_x4(qa + ks * 32 + 32, a0, a1, a2, a3);
-        mma_16816<bf16>(c1, a0, a1, a2, a3, b2, b3);
+#pragma unroll
+      for (int k = 0; k < KQ; k += 2) {
+        if (k < ks_n) {                        // an odd end also reads the next 32 bytes of shared memory and does not use them
+          uint32_t b0, b1, b2, b3;
+          la_ldsm_x4(ka + k * 32, b0, b1, b2, b3);
+          mma_16816<bf16>(c0, qf[k][0], qf[k][1], qf[k][2], qf[k][3], b0, b1);
+          if (k + 1 < KQ && k + 1 < ks_n) mma_16816<bf16>(c1, qf[k + 1 < KQ ? k + 1 : k][0], qf[k + 1 < KQ ? k + 1 : k][1], qf[k + 1 < KQ ? k + 1 : k][2], qf[k + 1 < KQ ? k + 1 : k][3], b2, b3);
+        }
       }
-      if (ks < ks_end) {
-        uint32_t a0, a1, a2, a3, b0, b1;
-        la_ldsm_x2(kb + (kb8 * 8 + (lane & 7)) * L.pitch + ((lane >> 3) & 1) * 16 + ks * 32, b0, b1);
-        la_ldsm_x4(qa + ks * 32, a0, a1, a2, a3);
-        mma_16816<bf16>(c0, a0, a1, a2, a3, b0, b1);
-      }
-      float* d = sS + khalf * 16 * SP + kb8 * 8 + 2 * t4;
+      float* d = sS + (w >> 2) * 16 * SP + kblk * 8 + 2 * t4;
       *reinterpret_cast<float2*>(d + g8 * SP) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
       *reinterpret_cast<float2*>(d + (g8 + 8) * SP) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
     }
-    __syncthreads();
-    {
-      const int t0 = t_beg + tile * kLmKeys + 2 * lane;
-      const float2 zA = *reinterpret_cast<const float2*>(sS + w * SP + 2 * lane), zB = *reinterpret_cast<const float2*>(sS + (16 + w) * SP + 2 * lane);
-      const int lim = min(t_end, row_lim);
-      const float z0 = t0 < lim ? (zA.x + zB.x) * a.scale : -INFINITY, z1 = t0 + 1 < lim ? (zA.y + zB.y) * a.scale : -INFINITY;
-      const float m_new = fmaxf(m_run, warp_max(fmaxf(z0, z1)));
-      const bool none = m_new == -INFINITY;      // a row may see none of these keys
-      const float p0 = none ? 0.0f : __expf(z0 - m_new), p1 = none ? 0.0f : __expf(z1 - m_new);
-      const float corr = none ? 1.0f : __expf(m_run - m_new);
-      *reinterpret_cast<uint32_t*>(sP + w * PP + 2 * lane) = Pair16<bf16>::put(p0, p1);
-      l_run = l_run * corr + warp_sum(p0 + p1);
-      m_run = m_new;
-      if (lane == 0) s_c[w] = corr;
-    }
-    __syncthreads();
-    if (col0 < a.rank) {
+    if (tile > 0 && col0 < a.rank) {
       const float cA = s_c[g8], cB = s_c[g8 + 8];
 #pragma unroll
       for (int i = 0; i < NBW; ++i) {
         o[i][0] *= cA; o[i][1] *= cA; o[i][2] *= cB; o[i][3] *= cB;
       }
       const uint32_t pa = la_smem(sP) + (lane & 15) * (PP * 2) + (lane >> 4) * 16;
-      const uint32_t va = kb + ((lane & 7) + ((lane >> 3) & 1) * 8) * L.pitch + (lane >> 4) * 16;
+      const uint32_t va = sbase + (uint32_t)((tile - 1) % stages) * L.stage_bytes + ((lane & 7) + ((lane >> 3) & 1) * 8) * L.pitch + (lane >> 4) * 16;
 #pragma unroll
       for (int ks = 0; ks < kLmKeys / 16; ++ks) {
         uint32_t a0, a1, a2, a3;
@@ -509,7 +486,19 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
         }
       }
     }
-    __syncthreads();   // the stage is overwritten by the copy issued in the next iteration
+    __syncthreads();
+    if (tile < n_tiles) {
+      const int t = t_beg + tile * kLmKeys + lane;
+      const float* z4 = sS + w * SP + lane;
+      const float z = t < row_lim ? ((z4[0] + z4[16 * SP]) + (z4[32 * SP] + z4[48 * SP])) * a.scale : -INFINITY;
+      const float m_new = fmaxf(m_run, warp_max(z));
+      const bool none = m_new == -INFINITY;      // the row has seen no key yet
+      const float p = none ? 0.0f : __expf(z - m_new), corr = none ? 1.0f : __expf(m_run - m_new);
+      sP[w * PP + lane] = from_f<bf16>(p);
+      l_run = l_run * corr + warp_sum(p);
+      m_run = m_new;
+      if (lane == 0) s_c[w] = corr;
+    }
   }
   la_wait<0>();
   const int rec = a.rank + 2;
@@ -613,16 +602,17 @@ __global__ void __launch_bounds__(kLvThreads) latent_value_kernel(LatentShape a,
     }
 }
 
-// The same on the warp-level tensor cores: 16 rows of one head and 32 value elements per CTA.  Uv's tile is requested before the wait on
+// The same on the warp-level tensor cores: up to 16 rows of one head and 32 value elements per CTA.  Uv's tile is requested before the wait on
 // the previous kernel; warp w takes value block w % 4 and every second step of the inner dimension.
 __host__ __device__ inline int latent_v_pitch(int rank) { return (rank + 15) / 16 * 32 + 16; }
-__global__ void __launch_bounds__(kLvThreads) latent_value_mma_kernel(LatentShape a, bf16* out, const float* part, const bf16* uv, int splits, int rows) {
+__global__ void __launch_bounds__(kLvThreads) latent_value_mma_kernel(LatentShape a, bf16* out, const float* part, const bf16* uv, int splits, int rows,
+                                                                      int rows_per_cta) {
   extern __shared__ __align__(128) unsigned char smem[];   // Uv tile [32][rank to 16], merged rows [16][rank to 16]
   __shared__ float s_w[16][kMaxSplits];
   __shared__ float4 s_half[4][32];
   pdl_trigger();
-  const int h = blockIdx.x, v0 = blockIdx.y * kLvCols, r0 = blockIdx.z * 16;
-  const int n = min(16, rows - r0);
+  const int h = blockIdx.x, v0 = blockIdx.y * kLvCols, r0 = blockIdx.z * rows_per_cta;
+  const int n = min(rows_per_cta, rows - r0);
   const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, g8 = lane >> 2, t4 = lane & 3, rec = a.rank + 2;
   const int pitch = latent_v_pitch(a.rank), kr = (a.rank + 15) / 16 * 16, chunks = kr / 8, live_chunks = a.rank / 8;
   const uint32_t su = la_smem(smem), so = su + 32 * pitch;
@@ -645,19 +635,41 @@ __global__ void __launch_bounds__(kLvThreads) latent_value_mma_kernel(LatentShap
   }
   __syncthreads();
   const int half = kr / 2;   // pairs per row
-  for (int i = tid; i < 16 * half; i += kLvThreads) {
-    const int r = i / half, e = (i - r * half) * 2;
-    float x = 0.0f, y = 0.0f;
-    if (r < n && e < a.rank) {
-      const float* p = part + ((int64_t)(r0 + r) * a.H + h) * splits * rec + 2 + e;
-#pragma unroll 8
-      for (int q = 0; q < splits; ++q) {
-        const float2 t = *reinterpret_cast<const float2*>(p + (int64_t)q * rec);
-        x = fmaf(s_w[r][q], t.x, x);
-        y = fmaf(s_w[r][q], t.y, y);
+  if (n <= 2) {
+    for (int i = tid; i < 16 * half; i += kLvThreads) {
+      const int r = i / half, e = (i - r * half) * 2;
+      float x = 0.0f, y = 0.0f;
+      if (r < n && e < a.rank) {
+        const float* p = part + ((int64_t)(r0 + r) * a.H + h) * splits * rec + 2 + e;
+#pragma unroll 16
+        for (int q = 0; q < splits; ++q) {
+          const float2 t = *reinterpret_cast<const float2*>(p + (int64_t)q * rec);
+          x = fmaf(s_w[r][q], t.x, x);
+          y = fmaf(s_w[r][q], t.y, y);
+        }
       }
+      *reinterpret_cast<uint32_t*>(smem + 32 * pitch + r * pitch + e * 2) = Pair16<bf16>::put(x, y);
     }
-    *reinterpret_cast<uint32_t*>(smem + 32 * pitch + r * pitch + e * 2) = Pair16<bf16>::put(x, y);
+  } else {
+    for (int i = tid; i < 4 * half; i += kLvThreads) {   // four rows of a pair of columns at a time
+      const int rg = i / half * 4, e = (i % half) * 2;
+      float x[4] = {0.0f, 0.0f, 0.0f, 0.0f}, y[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+      if (rg < n && e < a.rank) {
+        const float* p = part + ((int64_t)(r0 + rg) * a.H + h) * splits * rec + 2 + e;
+        const int64_t row_step = (int64_t)a.H * splits * rec;
+#pragma unroll 4
+        for (int q = 0; q < splits; ++q)
+#pragma unroll
+          for (int r = 0; r < 4; ++r)
+            if (rg + r < n) {
+              const float2 t = *reinterpret_cast<const float2*>(p + r * row_step + (int64_t)q * rec);
+              x[r] = fmaf(s_w[rg + r][q], t.x, x[r]);
+              y[r] = fmaf(s_w[rg + r][q], t.y, y[r]);
+            }
+      }
+#pragma unroll
+      for (int r = 0; r < 4; ++r) *reinterpret_cast<uint32_t*>(smem + 32 * pitch + (rg + r) * pitch + e * 2) = Pair16<bf16>::put(x[r], y[r]);
+    }
   }
   la_wait<0>();
   __syncthreads();
@@ -843,14 +855,14 @@ int launch_angle_table(int device, DeviceState* st, float2* tab, int Tmax, int d
 
 constexpr size_t kLatentSmemMax = 226 * 1024;
 static bool latent_mma_shape(int dtype, const LatentShape& a) {
-  return dtype == TSB200_BF16 && a.rank % 8 == 0 && a.rank <= 1024 && latent_mma_layout(a.row, 1).total <= kLatentSmemMax;
+  return dtype == TSB200_BF16 && a.rank % 8 == 0 && a.rank <= 1024 && a.row <= 17 * 64 && latent_mma_layout(a.row, 3).total <= kLatentSmemMax;
 }
 
-// splits of the key range: about one CTA per SM, at least 64 keys each
+// splits of the key range: about one CTA per SM, at least 128 keys each
 int latent_pick_splits(DeviceState* st, const LatentShape& a, int B, int S, int T) {
   const int64_t base = (int64_t)B * (((int64_t)S * a.H + 15) / 16);
   int64_t n = (st->sm_count + base / 2) / base;
-  const int by_len = (T + 63) / 64;
+  const int by_len = (T + 127) / 128;
   if (n > by_len) n = by_len;
   if (n > 64) n = 64;
   return n < 1 ? 1 : (int)n;
@@ -892,6 +904,13 @@ static LatentAppend latent_append_args(const LatentArgs& a) {
   return LatentAppend{a.dkv_col, a.norm_w, a.eps, a.cache, a.seq_stride, a.S, a.T0, a.state, a.Tmax, a.tab};
 }
 
+// CTA columns for the append beside the heads': one row per CTA
+static int latent_append_columns(const LatentArgs& a, int rows_per_z, int grid_y) {
+  if (a.dkv_col < 0) return 0;
+  const int rows = a.B * a.S < rows_per_z ? a.B * a.S : rows_per_z;
+  return (rows + grid_y - 1) / grid_y;
+}
+
 // bf16 shapes whose pieces are multiples of 16 bytes: every kernel of the absorbed form on the tensor cores
 static bool latent_mma_pieces(const LatentArgs& a) {
   const LatentShape& sh = a.shape;
@@ -903,9 +922,11 @@ static int latent_absorbed_mma(int device, DeviceState* st, const LatentArgs& a,
   static bool done[kMaxDevices] = {};
   if (!done[device]) {
     const auto dyn = cudaFuncAttributeMaxDynamicSharedMemorySize;
-    TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<2>, dyn, (int)kLatentSmemMax));
-    TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<4>, dyn, (int)kLatentSmemMax));
-    TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<8>, dyn, (int)kLatentSmemMax));
+    TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<2, 5>, dyn, (int)kLatentSmemMax));
+    TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<2, 17>, dyn, (int)kLatentSmemMax));
+    TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<4, 9>, dyn, (int)kLatentSmemMax));
+    TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<4, 17>, dyn, (int)kLatentSmemMax));
+    TSB_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<8, 17>, dyn, (int)kLatentSmemMax));
     TSB_CUDA(cudaFuncSetAttribute(latent_query_mma_kernel<1>, dyn, (int)kLatentSmemMax));
     TSB_CUDA(cudaFuncSetAttribute(latent_query_mma_kernel<4>, dyn, (int)kLatentSmemMax));
     TSB_CUDA(cudaFuncSetAttribute(latent_value_mma_kernel, dyn, 48 * latent_v_pitch(1024)));
@@ -916,14 +937,21 @@ static int latent_absorbed_mma(int device, DeviceState* st, const LatentArgs& a,
   const size_t sq = (size_t)kd * (64 * 2 + 16) + (size_t)16 * mt * latent_q_pitch(sh.dim);
   TSB_CHECK(sq <= kLatentSmemMax, "latent attention: unrotated head size %d is not supported", sh.dim);
   TSB_CUDA(launch_k(mt == 4 ? latent_query_mma_kernel<4> : latent_query_mma_kernel<1>,
-                    dim3(sh.H + (a.dkv_col >= 0 ? 1 : 0), (sh.rank + 63) / 64, (rows + 16 * mt - 1) / (16 * mt)), dim3(kLqmThreads), sq, s, sh, (bf16*)a.q_lat,
+                    dim3(sh.H + latent_append_columns(a, 16 * mt, (sh.rank + 63) / 64), (sh.rank + 63) / 64, (rows + 16 * mt - 1) / (16 * mt)), dim3(kLqmThreads), sq, s, sh, (bf16*)a.q_lat,
                     (const bf16*)a.q, a.q_stride, (const bf16*)a.uk, rows, ap));
-  const int stages = latent_mma_layout(sh.row, 2).total <= kLatentSmemMax ? 2 : 1;
-  auto k = sh.rank <= 256 ? latent_attn_mma_kernel<2> : (sh.rank <= 512 ? latent_attn_mma_kernel<4> : latent_attn_mma_kernel<8>);
+  int stages = kLmMaxStages;
+  while (stages > 3 && latent_mma_layout(sh.row, stages).total > kLatentSmemMax) --stages;
+  const int kq = (sh.row / 16 + 3) / 4;
+  auto k = sh.rank <= 256 ? (kq <= 5 ? latent_attn_mma_kernel<2, 5> : latent_attn_mma_kernel<2, 17>)
+                          : (sh.rank <= 512 ? (kq <= 9 ? latent_attn_mma_kernel<4, 9> : latent_attn_mma_kernel<4, 17>) : latent_attn_mma_kernel<8, 17>);
   TSB_CUDA(launch_k(k, dim3(a.splits, (a.S * sh.H + 15) / 16, a.B), dim3(kLmThreads), (size_t)latent_mma_layout(sh.row, stages).total, s, sh, a.part,
                     (const bf16*)a.q_lat, (const bf16*)a.cache, a.seq_stride, a.S, a.T0, a.state, a.Tmax, a.splits, stages));
-  TSB_CUDA(launch_k(latent_value_mma_kernel, dim3(sh.H, (sh.vdim + kLvCols - 1) / kLvCols, (rows + 15) / 16), dim3(kLvThreads),
-                    (size_t)48 * latent_v_pitch(sh.rank), s, sh, (bf16*)a.out, (const float*)a.part, (const bf16*)a.uv, a.splits, rows));
+  // few rows: one per CTA, so that the merges run side by side
+  const int vt = (sh.vdim + kLvCols - 1) / kLvCols;
+  int rt = (int)(((int64_t)sh.H * vt * rows + 4 * st->sm_count - 1) / (4 * st->sm_count));
+  rt = rt < 1 ? 1 : (rt > 16 ? 16 : rt);
+  TSB_CUDA(launch_k(latent_value_mma_kernel, dim3(sh.H, vt, (rows + rt - 1) / rt), dim3(kLvThreads), (size_t)48 * latent_v_pitch(sh.rank), s, sh, (bf16*)a.out,
+                    (const float*)a.part, (const bf16*)a.uv, a.splits, rows, rt));
   count_launch(device, 3);
   return check_launch("latent attention (tensor cores)");
 }
@@ -936,7 +964,7 @@ static int latent_absorbed(int device, DeviceState* st, const LatentArgs& a, cud
   const size_t sq = (size_t)kLqRows * sh.dim * sizeof(float);
   TSB_CHECK(sq <= 24 * 1024, "latent attention: unrotated head size %d is not supported (at most 768)", sh.dim);
   const LatentAppend ap = latent_append_args(a);
-  TSB_CUDA(launch_k(latent_query_kernel<T>, dim3(sh.H + (a.dkv_col >= 0 ? 1 : 0), (sh.rank + kLqCols - 1) / kLqCols, (rows + kLqRows - 1) / kLqRows),
+  TSB_CUDA(launch_k(latent_query_kernel<T>, dim3(sh.H + latent_append_columns(a, kLqRows, (sh.rank + kLqCols - 1) / kLqCols), (sh.rank + kLqCols - 1) / kLqCols, (rows + kLqRows - 1) / kLqRows),
                     dim3(kLqThreads), sq, s, sh, (T*)a.q_lat, (const T*)a.q, a.q_stride, (const T*)a.uk, rows, ap));
   TSB_TRY(latent_simple<T>(device, a, s));
   const int vt = (sh.vdim + kLvCols - 1) / kLvCols;   // few rows: one per CTA, so that the merges run side by side; many: eight share a read of Uv

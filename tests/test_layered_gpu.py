@@ -124,6 +124,27 @@ def test_long_prompt_in_large_and_small_portions(cuda, dtype):
     g.close()
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("rank,rot", [(24, 8), (256, 16), (256, 96), (264, 8), (512, 64), (512, 96), (648, 32), (1024, 16), (1000, 88)])
+def test_latent_sizes(cuda, rank, rot, dtype):
+    """Every register and staging variant of the absorbed form."""
+    cfg = M.config([M.layer(5, 16, rot, 24, rank, scale=0.2), M.layer(3, 24, rot, 40, rank, kv_from=0, scale=0.2)], 64, 50, groups=2, taps=3)
+    w = M.weights(cfg, 18)
+    ids = M.tokens(cfg, 150)
+    want = M.oracle(cfg, w).forward(ids)
+    g = engine(cfg, w, dtype)
+    tol = M.TOL[dtype]
+    assert M.rel(score(g, ids, cuts=[13, 5, 2, 40, 64, 3]), want) < tol
+    g.Reset()
+    rows = [g.SlotLogits(0, ids[:120], [119])[0]]
+    for t in ids[120:]:
+        g.StepHost([t], GREEDY)
+        rows.append(g.Logits(want_probs=False)[0][0])
+    assert M.rel(rows, want[119:]) < tol
+    g.CheckGuards()
+    g.close()
+
+
 # ---- keys far away, at tile borders, the first tokens ----------------------------------------------------------------------------
 def _needle(scale=6.0, n=200, at=0):
     """A model whose attention is nearly one-hot: the marker token's key stands out for every query."""
