@@ -303,7 +303,7 @@ static int ensure_layered(Gpt* g, int B, int S, int T) {
     na = std::max(na, rows * L.sh.H * L.sh.vdim);
     if (!latent_expanded(dt, L.sh, L.Nq + L.Nkv, S)) {
       nlat = std::max(nlat, rows * L.sh.H * L.sh.row);
-      npart = std::max(npart, rows * L.sh.H * latent_pick_splits(g->st, L.sh, B, S, T) * (L.sh.rank + 2));
+      npart = std::max(npart, rows * L.sh.H * latent_pick_splits(g->st, L.sh, B, S, T) * latent_rec(L.sh.rank));
     } else {
       nkv = std::max(nkv, (int64_t)B * T * L.sh.H * (L.sh.dim + L.sh.vdim));
       if (B > 1) ncomp = std::max(ncomp, (int64_t)B * T * L.sh.row);

@@ -324,6 +324,9 @@ struct LatentShape {
   int row;                       // elements of a cache row: [latent | rotated key part | zeros]
   float scale;
 };
+// what a split of the key range leaves per (query, head) row: [max, sum of weights, -, - | accumulator], in 16-byte units
+constexpr int kRecHead = 4;
+__host__ __device__ inline int latent_rec(int rank) { return kRecHead + (rank + 3) / 4 * 4; }
 inline int latent_row_elems(int rank, int rot) { return (rank + rot + 15) / 16 * 16; }
 // full-precision cos / sin table [Tmax, dims / 2] of base^(-2 i / dims) * position
 int launch_angle_table(int device, DeviceState* st, float2* tab, int Tmax, int dims, double base, cudaStream_t s);
@@ -343,7 +346,7 @@ struct LatentArgs {
   const void *uk, *uv;           // [H * dim, rank], [H * vdim, rank] row-major in the model type
   const void* ukv_packed;        // packed [row, H * (dim + vdim)]: latent -> keys | values (zero rows beyond the latent)
   void* q_lat;                   // scratch [B * S, H, row]
-  float* part;                   // scratch [B * S * H][splits][rank + 2]
+  float* part;                   // scratch [B * S * H][splits][latent_rec(rank)]
   int64_t part_elems;
   void* kv;                      // scratch [B][T0 + S][H * (dim + vdim)], expanded form only
   int64_t kv_elems;

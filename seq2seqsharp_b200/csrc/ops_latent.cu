@@ -346,11 +346,11 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(LatentShape a, float* 
   __syncthreads();
   float mx = -INFINITY;
   for (int q = 0; q < 8; ++q) mx = fmaxf(mx, st[q * rec]);
-  float* out = part + (rr * splits + split) * rec;
-  for (int e = tid; e < a.rank + 1; e += 256) {
+  float* out = part + (rr * splits + split) * latent_rec(a.rank);
+  for (int e = tid; e < a.rank + 1; e += 256) {   // e = 0: the sum of the weights
     float v = 0.0f;
     for (int q = 0; q < 8; ++q) v += (st[q * rec] == -INFINITY) ? 0.0f : st[q * rec + 1 + e] * expf(st[q * rec] - mx);
-    out[1 + e] = v;
+    out[e == 0 ? 1 : kRecHead + e - 1] = v;
   }
   if (tid == 0) out[0] = mx;
 }
@@ -400,22 +400,33 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
   float* s_c = reinterpret_cast<float*>(smem + L.c_off);
   constexpr int SP = kLmKeys + 4, PP = kLmKeys + 8, NW = kLmThreads / 32;
 
-  auto issue = [&](int tile) {
-    if (tile < n_tiles) {
-      const uint32_t dst = sbase + (uint32_t)(tile % stages) * L.stage_bytes;
-      const int t0 = t_beg + tile * kLmKeys;
+  // this thread's share of a tile: chunks lane, lane + 32, ... of the rows w and w + 16
+  constexpr int NCH = (KQ * 8 + 31) / 32;
+  const bf16* src = base + (int64_t)(t_beg + w) * a.row + lane * 8;
+  const uint32_t dst0 = sbase + w * L.pitch + lane * 16;
+  uint32_t dst_off = 0;
+  const int row16 = NW * a.row;
+  int to_issue = 0;                            // tile the next call requests
+  auto issue = [&]() {
+    if (to_issue < n_tiles) {
+      const int t = t_beg + to_issue * kLmKeys + w;
+      const bool whole = t - w + kLmKeys <= t_end;
 #pragma unroll
       for (int q = 0; q < kLmKeys / NW; ++q) {
-        const int tt = w + q * NW;
-        const int t = min(t0 + tt, t_end - 1);   // the tail re-reads the last key of the range; its scores are masked
-        const bf16* src = base + (int64_t)t * a.row;
-        for (int c = lane; c < cpr; c += 32) la_cp16(dst + tt * L.pitch + c * 16, src + c * 8);
+        // keys beyond the range re-read its last one; their scores are masked
+        const bf16* sr = whole || t + q * NW < t_end ? src + q * row16 : base + (int64_t)(t_end - 1) * a.row + lane * 8;
+#pragma unroll
+        for (int c = 0; c < NCH; ++c)
+          if (lane + c * 32 < cpr) la_cp16(dst0 + dst_off + q * NW * L.pitch + c * 512, sr + c * 256);
       }
+      src += kLmKeys * a.row;
+      ++to_issue;
+      dst_off = dst_off + L.stage_bytes == L.s_off ? 0 : dst_off + L.stage_bytes;
     }
     la_commit();
   };
   const int ahead = stages - 2;                // tiles in flight beside the one being scored and the one before it
-  for (int i = 0; i < ahead; ++i) issue(i);
+  for (int i = 0; i < ahead; ++i) issue();
   const int ksteps = a.row / 16, kq4 = (ksteps + 3) / 4;
   const int kblk = w & 3, ks_beg = (w >> 2) * kq4, ks_n = max(0, min(ksteps - ks_beg, kq4));
   uint32_t qf[KQ][4];
@@ -431,32 +442,48 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
       qf[k][3] = k < ks_n && lb ? *reinterpret_cast<const uint32_t*>(qb + k * 16 + 8) : 0u;
     }
   }
+  const uint32_t ka0 = sbase + (kblk * 8 + (lane & 7)) * L.pitch + (lane >> 3) * 16 + ks_beg * 32;
+  const uint32_t ka2 = sbase + (kblk * 8 + (lane & 7)) * L.pitch + ((lane >> 3) & 1) * 16 + ks_beg * 32;
   float o[NBW][4];
 #pragma unroll
   for (int i = 0; i < NBW; ++i)
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[i][e] = 0.0f;
   const int col0 = w * NBW * 8;                // first latent column of this warp
+  const uint32_t pa = la_smem(sP) + (lane & 15) * (PP * 2) + (lane >> 4) * 16;
+  const uint32_t va0 = sbase + ((lane & 7) + ((lane >> 3) & 1) * 8) * L.pitch + (lane >> 4) * 16 + col0 * 2;
   const int row_lim = min(t_end, r0 + w < R ? T0 + (r0 + w) / a.H + 1 : 0);   // softmax row w: keys below are visible to it
   float m_run = -INFINITY, l_run = 0.0f;       // state of row w, the same in every lane
 
+  const bool whole_q = ks_n == KQ, whole_o = col0 + NBW * 8 <= a.rank;
+  uint32_t k_off = 0, v_off = 0;               // stages of this tile's keys and of the previous tile's values
   for (int tile = 0; tile <= n_tiles; ++tile) {
-    issue(tile + ahead);                       // over the stage of tile - 2, which the previous interval was the last to read
+    issue();                                   // over the stage of tile - 2, which the previous interval was the last to read
     if (ahead == 3) la_wait<3>();
     else if (ahead == 2) la_wait<2>();
     else la_wait<1>();
     __syncthreads();
     if (tile < n_tiles) {
-      const uint32_t ka = sbase + (uint32_t)(tile % stages) * L.stage_bytes + (kblk * 8 + (lane & 7)) * L.pitch + (lane >> 3) * 16 + ks_beg * 32;
+      const uint32_t ka = ka0 + k_off;
       float c0[4] = {0.0f, 0.0f, 0.0f, 0.0f}, c1[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+      if (whole_q) {
 #pragma unroll
-      for (int k = 0; k < KQ; k += 2) {
-        if (k < ks_n) {                        // an odd end also reads the next 32 bytes of shared memory and does not use them
+        for (int k = 0; k < KQ; k += 2) {
           uint32_t b0, b1, b2, b3;
-          la_ldsm_x4(ka + k * 32, b0, b1, b2, b3);
+          if (k + 1 < KQ) la_ldsm_x4(ka + k * 32, b0, b1, b2, b3);
+          else la_ldsm_x2(ka2 + k_off + k * 32, b0, b1);
           mma_16816<bf16>(c0, qf[k][0], qf[k][1], qf[k][2], qf[k][3], b0, b1);
-          if (k + 1 < KQ && k + 1 < ks_n) mma_16816<bf16>(c1, qf[k + 1 < KQ ? k + 1 : k][0], qf[k + 1 < KQ ? k + 1 : k][1], qf[k + 1 < KQ ? k + 1 : k][2], qf[k + 1 < KQ ? k + 1 : k][3], b2, b3);
+          if (k + 1 < KQ) mma_16816<bf16>(c1, qf[k + 1 < KQ ? k + 1 : k][0], qf[k + 1 < KQ ? k + 1 : k][1], qf[k + 1 < KQ ? k + 1 : k][2], qf[k + 1 < KQ ? k + 1 : k][3], b2, b3);
         }
+      } else {
+#pragma unroll
+        for (int k = 0; k < KQ; k += 2)
+          if (k < ks_n) {                      // an odd end also reads the next 32 bytes of shared memory and does not use them
+            uint32_t b0, b1, b2, b3;
+            la_ldsm_x4(ka + k * 32, b0, b1, b2, b3);
+            mma_16816<bf16>(c0, qf[k][0], qf[k][1], qf[k][2], qf[k][3], b0, b1);
+            if (k + 1 < KQ && k + 1 < ks_n) mma_16816<bf16>(c1, qf[k + 1 < KQ ? k + 1 : k][0], qf[k + 1 < KQ ? k + 1 : k][1], qf[k + 1 < KQ ? k + 1 : k][2], qf[k + 1 < KQ ? k + 1 : k][3], b2, b3);
+          }
       }
       float* d = sS + (w >> 2) * 16 * SP + kblk * 8 + 2 * t4;
       *reinterpret_cast<float2*>(d + g8 * SP) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
@@ -468,18 +495,16 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
       for (int i = 0; i < NBW; ++i) {
         o[i][0] *= cA; o[i][1] *= cA; o[i][2] *= cB; o[i][3] *= cB;
       }
-      const uint32_t pa = la_smem(sP) + (lane & 15) * (PP * 2) + (lane >> 4) * 16;
-      const uint32_t va = sbase + (uint32_t)((tile - 1) % stages) * L.stage_bytes + ((lane & 7) + ((lane >> 3) & 1) * 8) * L.pitch + (lane >> 4) * 16;
+      const uint32_t va = va0 + v_off;
 #pragma unroll
       for (int ks = 0; ks < kLmKeys / 16; ++ks) {
         uint32_t a0, a1, a2, a3;
         la_ldsm_x4(pa + ks * 32, a0, a1, a2, a3);
 #pragma unroll
         for (int i = 0; i < NBW; i += 2) {
-          const int col = col0 + i * 8;
-          if (col < a.rank) {   // the row is a multiple of 16 elements: both blocks of the pair are inside it
+          if (whole_o || col0 + i * 8 < a.rank) {   // the row is a multiple of 16 elements: both blocks of the pair are inside it
             uint32_t b0, b1, b2, b3;
-            la_ldsm_x4_trans(va + ks * 16 * L.pitch + col * 2, b0, b1, b2, b3);
+            la_ldsm_x4_trans(va + ks * 16 * L.pitch + i * 16, b0, b1, b2, b3);
             mma_16816<bf16>(o[i], a0, a1, a2, a3, b0, b1);
             mma_16816<bf16>(o[i + 1], a0, a1, a2, a3, b2, b3);
           }
@@ -499,9 +524,11 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
       m_run = m_new;
       if (lane == 0) s_c[w] = corr;
     }
+    v_off = k_off;
+    k_off = k_off + L.stage_bytes == L.s_off ? 0 : k_off + L.stage_bytes;
   }
   la_wait<0>();
-  const int rec = a.rank + 2;
+  const int rec = latent_rec(a.rank);
   float* pb = part + (((int64_t)b * R + r0) * splits + split) * rec;
 #pragma unroll
   for (int i = 0; i < NBW; ++i) {
@@ -510,7 +537,7 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int rr = g8 + e * 8;
-      if (r0 + rr < R) *reinterpret_cast<float2*>(pb + (int64_t)rr * splits * rec + 2 + c) = make_float2(o[i][2 * e], o[i][2 * e + 1]);
+      if (r0 + rr < R) *reinterpret_cast<float2*>(pb + (int64_t)rr * splits * rec + kRecHead + c) = make_float2(o[i][2 * e], o[i][2 * e + 1]);
     }
   }
   if (lane == 0 && r0 + w < R) {
@@ -529,7 +556,7 @@ __global__ void __launch_bounds__(kLvThreads) latent_value_kernel(LatentShape a,
   pdl_wait();
   const int h = blockIdx.x, v0 = blockIdx.y * kLvCols, r0 = blockIdx.z * kLvRows;
   const int n = min(kLvRows, rows - r0);
-  const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, rec = a.rank + 2;
+  const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, rec = latent_rec(a.rank);
   if (w < n) {   // weight of every split of row w
     const float* p = part + ((int64_t)(r0 + w) * a.H + h) * splits * rec;
     const float m0 = lane < splits ? p[(int64_t)lane * rec] : -INFINITY, m1 = lane + 32 < splits ? p[(int64_t)(lane + 32) * rec] : -INFINITY;
@@ -543,7 +570,7 @@ __global__ void __launch_bounds__(kLvThreads) latent_value_kernel(LatentShape a,
   __syncthreads();
   for (int i = tid; i < n * a.rank; i += kLvThreads) {
     const int r = kLvRows == 1 ? 0 : i / a.rank, e = i - r * a.rank;
-    const float* p = part + ((int64_t)(r0 + r) * a.H + h) * splits * rec + 2 + e;
+    const float* p = part + ((int64_t)(r0 + r) * a.H + h) * splits * rec + kRecHead + e;
     float v = 0.0f;
 #pragma unroll 8
     for (int q = 0; q < splits; ++q) {
@@ -613,7 +640,7 @@ __global__ void __launch_bounds__(kLvThreads) latent_value_mma_kernel(LatentShap
   pdl_trigger();
   const int h = blockIdx.x, v0 = blockIdx.y * kLvCols, r0 = blockIdx.z * rows_per_cta;
   const int n = min(rows_per_cta, rows - r0);
-  const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, g8 = lane >> 2, t4 = lane & 3, rec = a.rank + 2;
+  const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, g8 = lane >> 2, t4 = lane & 3, rec = latent_rec(a.rank);
   const int pitch = latent_v_pitch(a.rank), kr = (a.rank + 15) / 16 * 16, chunks = kr / 8, live_chunks = a.rank / 8;
   const uint32_t su = la_smem(smem), so = su + 32 * pitch;
   for (int q = w; q < 32; q += 8)
@@ -635,40 +662,45 @@ __global__ void __launch_bounds__(kLvThreads) latent_value_mma_kernel(LatentShap
   }
   __syncthreads();
   const int half = kr / 2;   // pairs per row
-  if (n <= 2) {
-    for (int i = tid; i < 16 * half; i += kLvThreads) {
-      const int r = i / half, e = (i - r * half) * 2;
-      float x = 0.0f, y = 0.0f;
-      if (r < n && e < a.rank) {
-        const float* p = part + ((int64_t)(r0 + r) * a.H + h) * splits * rec + 2 + e;
-#pragma unroll 16
-        for (int q = 0; q < splits; ++q) {
-          const float2 t = *reinterpret_cast<const float2*>(p + (int64_t)q * rec);
-          x = fmaf(s_w[r][q], t.x, x);
-          y = fmaf(s_w[r][q], t.y, y);
+  for (int i = tid; i < (16 - n) * half; i += kLvThreads) *reinterpret_cast<uint32_t*>(smem + (32 + n + i / half) * pitch + (i % half) * 4) = 0u;
+  const int64_t split_step = rec / 4, row_step = (int64_t)a.H * splits * split_step;
+  const int groups = n <= 2 ? n : (n + 3) / 4;   // four columns of one row (few rows) or of four rows at a time
+  const int quads = kr / 4;
+  for (int idx = tid; idx < groups * quads; idx += kLvThreads) {
+    const int g = idx / quads, e = idx - g * quads;
+    const bool live = e * 4 < a.rank;
+    if (n <= 2) {
+      const float4* p = reinterpret_cast<const float4*>(part + ((int64_t)(r0 + g) * a.H + h) * splits * rec + kRecHead) + e;
+      float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      if (live) {
+#pragma unroll 8
+        for (int q = 0; q < splits; ++q, p += split_step) {
+          const float4 t = *p;
+          const float f = s_w[g][q];
+          x.x = fmaf(f, t.x, x.x); x.y = fmaf(f, t.y, x.y); x.z = fmaf(f, t.z, x.z); x.w = fmaf(f, t.w, x.w);
         }
       }
-      *reinterpret_cast<uint32_t*>(smem + 32 * pitch + r * pitch + e * 2) = Pair16<bf16>::put(x, y);
-    }
-  } else {
-    for (int i = tid; i < 4 * half; i += kLvThreads) {   // four rows of a pair of columns at a time
-      const int rg = i / half * 4, e = (i % half) * 2;
-      float x[4] = {0.0f, 0.0f, 0.0f, 0.0f}, y[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-      if (rg < n && e < a.rank) {
-        const float* p = part + ((int64_t)(r0 + rg) * a.H + h) * splits * rec + 2 + e;
-        const int64_t row_step = (int64_t)a.H * splits * rec;
-#pragma unroll 4
-        for (int q = 0; q < splits; ++q)
+      *reinterpret_cast<uint2*>(smem + (32 + g) * pitch + e * 8) = make_uint2(Pair16<bf16>::put(x.x, x.y), Pair16<bf16>::put(x.z, x.w));
+    } else {
+      const int rg = g * 4;
+      const float4* p = reinterpret_cast<const float4*>(part + ((int64_t)(r0 + rg) * a.H + h) * splits * rec + kRecHead) + e;
+      float4 x[4];
+#pragma unroll
+      for (int r = 0; r < 4; ++r) x[r] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      if (live) {
+#pragma unroll 2
+        for (int q = 0; q < splits; ++q, p += split_step)
 #pragma unroll
           for (int r = 0; r < 4; ++r)
             if (rg + r < n) {
-              const float2 t = *reinterpret_cast<const float2*>(p + r * row_step + (int64_t)q * rec);
-              x[r] = fmaf(s_w[rg + r][q], t.x, x[r]);
-              y[r] = fmaf(s_w[rg + r][q], t.y, y[r]);
+              const float4 t = p[r * row_step];
+              const float f = s_w[rg + r][q];
+              x[r].x = fmaf(f, t.x, x[r].x); x[r].y = fmaf(f, t.y, x[r].y); x[r].z = fmaf(f, t.z, x[r].z); x[r].w = fmaf(f, t.w, x[r].w);
             }
       }
 #pragma unroll
-      for (int r = 0; r < 4; ++r) *reinterpret_cast<uint32_t*>(smem + 32 * pitch + (rg + r) * pitch + e * 2) = Pair16<bf16>::put(x[r], y[r]);
+      for (int r = 0; r < 4; ++r)
+        if (rg + r < n) *reinterpret_cast<uint2*>(smem + (32 + rg + r) * pitch + e * 8) = make_uint2(Pair16<bf16>::put(x[r].x, x[r].y), Pair16<bf16>::put(x[r].z, x[r].w));
     }
   }
   la_wait<0>();
@@ -1013,7 +1045,7 @@ int launch_latent_attention(int device, DeviceState* st, int dtype, const Latent
     return check_launch("latent_prefill_mma");
   }
   TSB_CHECK(a.splits >= 1 && a.splits <= kMaxSplits, "latent attention: %d splits", a.splits);
-  TSB_CHECK((int64_t)a.B * a.S * sh.H * a.splits * (sh.rank + 2) <= a.part_elems, "latent attention: scratch too small for %d rows in %d splits", a.B * a.S, a.splits);
+  TSB_CHECK((int64_t)a.B * a.S * sh.H * a.splits * latent_rec(sh.rank) <= a.part_elems, "latent attention: scratch too small for %d rows in %d splits", a.B * a.S, a.splits);
   if (dtype == TSB200_F32) return latent_absorbed<float>(device, st, a, s);
   return latent_mma_pieces(a) ? latent_absorbed_mma(device, st, a, s) : latent_absorbed<bf16>(device, st, a, s);
 }
