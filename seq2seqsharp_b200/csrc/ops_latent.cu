@@ -35,6 +35,12 @@ __device__ __forceinline__ void la_ldsm_x2(uint32_t addr, uint32_t& r0, uint32_t
 __device__ __forceinline__ void la_ldsm_x4_trans(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
 }
+// not volatile: the products may be scheduled around the fragment loads that follow them
+__device__ __forceinline__ void la_mma(float* d, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
 // 16 bytes to shared memory; with live == false the destination is zero-filled and the source is not read
 __device__ __forceinline__ void la_cp16(uint32_t dst, const void* src, bool live = true) {
   const int n = live ? 16 : 0;
@@ -281,8 +287,8 @@ __global__ void __launch_bounds__(kLqmThreads) latent_query_mma_kernel(LatentSha
     for (int m = 0; m < MT; ++m) {
       uint32_t a0, a1, a2, a3;
       la_ldsm_x4(aa + m * 16 * qp + ks * 32, a0, a1, a2, a3);
-      mma_16816<bf16>(d[m][0], a0, a1, a2, a3, b0, b1);
-      mma_16816<bf16>(d[m][1], a0, a1, a2, a3, b2, b3);
+      la_mma(d[m][0], a0, a1, a2, a3, b0, b1);
+      la_mma(d[m][1], a0, a1, a2, a3, b2, b3);
     }
   }
 #pragma unroll
@@ -467,22 +473,22 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
       const uint32_t ka = ka0 + k_off;
       float c0[4] = {0.0f, 0.0f, 0.0f, 0.0f}, c1[4] = {0.0f, 0.0f, 0.0f, 0.0f};
       if (whole_q) {
+        uint32_t kf[KQ + 1][2];
 #pragma unroll
         for (int k = 0; k < KQ; k += 2) {
-          uint32_t b0, b1, b2, b3;
-          if (k + 1 < KQ) la_ldsm_x4(ka + k * 32, b0, b1, b2, b3);
-          else la_ldsm_x2(ka2 + k_off + k * 32, b0, b1);
-          mma_16816<bf16>(c0, qf[k][0], qf[k][1], qf[k][2], qf[k][3], b0, b1);
-          if (k + 1 < KQ) mma_16816<bf16>(c1, qf[k + 1 < KQ ? k + 1 : k][0], qf[k + 1 < KQ ? k + 1 : k][1], qf[k + 1 < KQ ? k + 1 : k][2], qf[k + 1 < KQ ? k + 1 : k][3], b2, b3);
+          if (k + 1 < KQ) la_ldsm_x4(ka + k * 32, kf[k][0], kf[k][1], kf[k + 1][0], kf[k + 1][1]);
+          else la_ldsm_x2(ka2 + k_off + k * 32, kf[k][0], kf[k][1]);
         }
+#pragma unroll
+        for (int k = 0; k < KQ; ++k) la_mma(k & 1 ? c1 : c0, qf[k][0], qf[k][1], qf[k][2], qf[k][3], kf[k][0], kf[k][1]);
       } else {
 #pragma unroll
         for (int k = 0; k < KQ; k += 2)
           if (k < ks_n) {                      // an odd end also reads the next 32 bytes of shared memory and does not use them
             uint32_t b0, b1, b2, b3;
             la_ldsm_x4(ka + k * 32, b0, b1, b2, b3);
-            mma_16816<bf16>(c0, qf[k][0], qf[k][1], qf[k][2], qf[k][3], b0, b1);
-            if (k + 1 < KQ && k + 1 < ks_n) mma_16816<bf16>(c1, qf[k + 1 < KQ ? k + 1 : k][0], qf[k + 1 < KQ ? k + 1 : k][1], qf[k + 1 < KQ ? k + 1 : k][2], qf[k + 1 < KQ ? k + 1 : k][3], b2, b3);
+            la_mma(c0, qf[k][0], qf[k][1], qf[k][2], qf[k][3], b0, b1);
+            if (k + 1 < KQ && k + 1 < ks_n) la_mma(c1, qf[k + 1 < KQ ? k + 1 : k][0], qf[k + 1 < KQ ? k + 1 : k][1], qf[k + 1 < KQ ? k + 1 : k][2], qf[k + 1 < KQ ? k + 1 : k][3], b2, b3);
           }
       }
       float* d = sS + (w >> 2) * 16 * SP + kblk * 8 + 2 * t4;
@@ -505,8 +511,8 @@ __global__ void __launch_bounds__(kLmThreads) latent_attn_mma_kernel(LatentShape
           if (whole_o || col0 + i * 8 < a.rank) {   // the row is a multiple of 16 elements: both blocks of the pair are inside it
             uint32_t b0, b1, b2, b3;
             la_ldsm_x4_trans(va + ks * 16 * L.pitch + i * 16, b0, b1, b2, b3);
-            mma_16816<bf16>(o[i], a0, a1, a2, a3, b0, b1);
-            mma_16816<bf16>(o[i + 1], a0, a1, a2, a3, b2, b3);
+            la_mma(o[i], a0, a1, a2, a3, b0, b1);
+            la_mma(o[i + 1], a0, a1, a2, a3, b2, b3);
           }
         }
       }
@@ -713,7 +719,7 @@ __global__ void __launch_bounds__(kLvThreads) latent_value_mma_kernel(LatentShap
     uint32_t a0, a1, a2, a3, b0, b1;
     la_ldsm_x4(aa + ks * 32, a0, a1, a2, a3);
     la_ldsm_x2(ba + ks * 32, b0, b1);
-    mma_16816<bf16>(d0, a0, a1, a2, a3, b0, b1);
+    la_mma(d0, a0, a1, a2, a3, b0, b1);
   }
   if (kh == 1) s_half[nb][lane] = make_float4(d0[0], d0[1], d0[2], d0[3]);
   __syncthreads();
@@ -803,11 +809,11 @@ __global__ void __launch_bounds__(kLpThreads, VN <= 16 ? 2 : 1) latent_prefill_m
         uint32_t a0, a1, a2, a3, b0, b1, b2, b3;
         la_ldsm_x4(qa + ks * 32, a0, a1, a2, a3);
         la_ldsm_x4(ka + ks * 32, b0, b1, b2, b3);
-        mma_16816<bf16>(sc[0], a0, a1, a2, a3, b0, b1);
-        mma_16816<bf16>(sc[1], a0, a1, a2, a3, b2, b3);
+        la_mma(sc[0], a0, a1, a2, a3, b0, b1);
+        la_mma(sc[1], a0, a1, a2, a3, b2, b3);
         la_ldsm_x4(ka + 16 * qpitch + ks * 32, b0, b1, b2, b3);
-        mma_16816<bf16>(sc[2], a0, a1, a2, a3, b0, b1);
-        mma_16816<bf16>(sc[3], a0, a1, a2, a3, b2, b3);
+        la_mma(sc[2], a0, a1, a2, a3, b0, b1);
+        la_mma(sc[3], a0, a1, a2, a3, b2, b3);
       }
       float mxA = -INFINITY, mxB = -INFINITY;
 #pragma unroll
@@ -853,8 +859,8 @@ __global__ void __launch_bounds__(kLpThreads, VN <= 16 ? 2 : 1) latent_prefill_m
         for (int i = 0; i < VN; i += 2) {
           uint32_t b0, b1, b2, b3;
           la_ldsm_x4_trans(va + i * 16, b0, b1, b2, b3);
-          mma_16816<bf16>(o[i], p0, p1, p2, p3, b0, b1);
-          mma_16816<bf16>(o[i + 1], p0, p1, p2, p3, b2, b3);
+          la_mma(o[i], p0, p1, p2, p3, b0, b1);
+          la_mma(o[i + 1], p0, p1, p2, p3, b2, b3);
         }
       }
     }
@@ -980,8 +986,8 @@ static int latent_absorbed_mma(int device, DeviceState* st, const LatentArgs& a,
                     (const bf16*)a.q_lat, (const bf16*)a.cache, a.seq_stride, a.S, a.T0, a.state, a.Tmax, a.splits, stages));
   // few rows: one per CTA, so that the merges run side by side
   const int vt = (sh.vdim + kLvCols - 1) / kLvCols;
-  int rt = (int)(((int64_t)sh.H * vt * rows + 4 * st->sm_count - 1) / (4 * st->sm_count));
-  rt = rt < 1 ? 1 : (rt > 16 ? 16 : rt);
+  int rt = 1;
+  while (rt < 16 && (int64_t)sh.H * vt * ((rows + rt - 1) / rt) > 4 * (int64_t)st->sm_count) ++rt;   // four CTAs fit on an SM: one wave
   TSB_CUDA(launch_k(latent_value_mma_kernel, dim3(sh.H, vt, (rows + rt - 1) / rt), dim3(kLvThreads), (size_t)48 * latent_v_pitch(sh.rank), s, sh, (bf16*)a.out,
                     (const float*)a.part, (const bf16*)a.uv, a.splits, rows, rt));
   count_launch(device, 3);
