@@ -896,10 +896,10 @@ static bool latent_mma_shape(int dtype, const LatentShape& a) {
   return dtype == TSB200_BF16 && a.rank % 8 == 0 && a.rank <= 1024 && a.row <= 17 * 64 && latent_mma_layout(a.row, 3).total <= kLatentSmemMax;
 }
 
-// splits of the key range: about one CTA per SM, at least 128 keys each
+// splits of the key range: about one CTA per SM (two with short cache rows, which fit twice), at least 128 keys each
 int latent_pick_splits(DeviceState* st, const LatentShape& a, int B, int S, int T) {
   const int64_t base = (int64_t)B * (((int64_t)S * a.H + 15) / 16);
-  int64_t n = (st->sm_count + base / 2) / base;
+  int64_t n = ((a.row <= 320 ? 2 : 1) * (int64_t)st->sm_count + base / 2) / base;
   const int by_len = (T + 127) / 128;
   if (n > by_len) n = by_len;
   if (n > 64) n = 64;
