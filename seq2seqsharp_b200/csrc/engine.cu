@@ -902,7 +902,7 @@ static int ensure_stack(Gpt* g, int B) {
 // With use_state the cache length is read from g->state[0] by the kernels (graph replay), else from T0.
 static int enqueue_forward(Gpt* g, int B, int S, int T0, bool use_state, int splits) {
   if (g->ly) {
-    if (!use_state) TSB_TRY(ensure_layered(g, B, S, T0 + S));
+    if (!use_state) TSB_TRY(ensure_layered(g, B, S, T0 + S, false));
     return enqueue_layered(g, B, S, T0, use_state, use_state ? splits : T0 + S);
   }
   NvtxRange nvtx_(S == 1 ? "tsb200.forward.step" : "tsb200.forward.prompt");
@@ -1175,7 +1175,7 @@ static int ensure_graph(Gpt* g, const TSB200DecodingOptions* opt, int n_steps) {
   GraphKey key;
   if (g->ly) {
     if (Tp > c.max_tokens) Tp = c.max_tokens;
-    TSB_TRY(ensure_layered(g, B, 1, Tp));
+    TSB_TRY(ensure_layered(g, B, 1, Tp, true));
   }
   key.B = B; key.strategy = opt->strategy; key.splits = g->ly ? Tp : attn_pick_splits(g->st, c.dtype, B, c.H, c.Hkv, c.hd, Tp);
   key.n_blocked = opt->n_blocked; key.blocked_hash = hash_blocked(opt->blocked, opt->n_blocked);
@@ -2580,7 +2580,7 @@ int TSB200_GptProfileDecode(void* h, int n_steps, const TSB200DecodingOptions* o
   TSB_TRY(set_state(g, 0));
   int Tp = 256;
   while (Tp < g->T + n_steps) Tp <<= 1;
-  if (g->ly) TSB_TRY(ensure_layered(g, g->B, 1, Tp));
+  if (g->ly) TSB_TRY(ensure_layered(g, g->B, 1, Tp, true));
   const int splits = g->ly ? Tp : attn_pick_splits(g->st, c.dtype, g->B, c.H, c.Hkv, c.hd, Tp);
   TSB_TRY(ensure_stack(g, g->B));
   g->prof = true;

@@ -28,7 +28,7 @@ struct LayeredLayer {
   int* table = nullptr;
   void* cache = nullptr;          // [max_batch][max_tokens][row]; null: kv_from's
   void* ring = nullptr;           // [max_batch][taps][d]
-  RouteLayer route{};             // host copy of the routing scratch
+  RouteLayer routes[2]{};         // host copies of the routing scratch (prompts, captured decode step)
   int route_index = -1;
 };
 
@@ -39,9 +39,9 @@ struct Layered {
   int n_route = 0, max_experts = 0;
   // scratch, grown on demand (ensure_layered)
   struct Buf { void* p = nullptr; int64_t bytes = 0; };
-  Buf hcat, gate1, gate2, qkv, attn, hs, hidden, y, q_lat, part, kv, compact, ints, routes, ws;
-  int64_t route_rows = 0;
-  int route_block = 0;
+  Buf hcat, gate1, gate2, qkv, attn, hs, hidden, y, q_lat, part, kv, compact, ws;
+  // routing scratch, one set for prompts and one for the decode step: a prompt between two steps leaves the captured step valid
+  struct Routing { Buf ints, layers; int64_t rows = 0; int block = 0; } routing[2];
 };
 
 template <typename TD, typename TS>
@@ -282,8 +282,8 @@ static int grow(Gpt* g, Layered::Buf& b, int64_t bytes, bool zero = false) {
   return 1;
 }
 
-// Scratch of a forward pass over B sequences of S new positions on up to T cached ones (T: after the pass).
-static int ensure_layered(Gpt* g, int B, int S, int T) {
+// Scratch of a forward pass over B sequences of S new positions on up to T cached ones (T: after the pass); step: for the decode step.
+static int ensure_layered(Gpt* g, int B, int S, int T, bool step) {
   Layered* ly = g->ly;
   const int64_t rows = (int64_t)B * S, d = ly->c.d, es = g->es;
   const int dt = g->c.dtype;
@@ -349,17 +349,18 @@ static int ensure_layered(Gpt* g, int B, int S, int T) {
   TSB_TRY(grow(g, ly->kv, nkv * es));
   TSB_TRY(grow(g, ly->compact, ncomp * es));
   TSB_TRY(grow(g, ly->ws, ws, true));
-  if (ly->n_route > 0 && (ly->route_rows != rows || ly->route_block != br)) {
-    // routing scratch of every expert layer, laid out for this many rows; the captured step holds pointers into it
-    TSB_TRY(grow(g, ly->ints, nints * 4 + 64));
-    TSB_TRY(grow(g, ly->routes, (int64_t)ly->n_route * sizeof(RouteLayer)));
-    if (g->gexec) { cudaGraphExecDestroy(g->gexec); g->gexec = nullptr; }
+  Layered::Routing& rt = ly->routing[step ? 1 : 0];
+  if (ly->n_route > 0 && (rt.rows != rows || rt.block != br)) {
+    // routing scratch of every expert layer, laid out for this many rows; the captured step holds pointers into its set
+    TSB_TRY(grow(g, rt.ints, nints * 4 + 64));
+    TSB_TRY(grow(g, rt.layers, (int64_t)ly->n_route * sizeof(RouteLayer)));
+    if (step && g->gexec) { cudaGraphExecDestroy(g->gexec); g->gexec = nullptr; }
     std::vector<RouteLayer> host((size_t)ly->n_route);
-    int* at = (int*)ly->ints.p;
+    int* at = (int*)rt.ints.p;
     for (auto& L : ly->L) {
       if (L.d.experts <= 0) continue;
       const int64_t p = rows * L.d.top;
-      RouteLayer& r = L.route;
+      RouteLayer& r = L.routes[step ? 1 : 0];
       r.table = L.table;
       r.top = L.d.top;
       r.experts = L.d.experts;
@@ -373,10 +374,10 @@ static int ensure_layered(Gpt* g, int B, int S, int T) {
       at += (p + 3) / 4 * 4;
       host[(size_t)L.route_index] = r;
     }
-    TSB_CUDA(cudaMemcpyAsync(ly->routes.p, host.data(), host.size() * sizeof(RouteLayer), cudaMemcpyHostToDevice, g->s));
+    TSB_CUDA(cudaMemcpyAsync(rt.layers.p, host.data(), host.size() * sizeof(RouteLayer), cudaMemcpyHostToDevice, g->s));
     TSB_CUDA(cudaStreamSynchronize(g->s));   // `host` is pageable
-    ly->route_rows = rows;
-    ly->route_block = br;
+    rt.rows = rows;
+    rt.block = br;
   }
   return 1;
 }
@@ -394,6 +395,8 @@ static int enqueue_layered(Gpt* g, int B, int S, int T0, bool use_state, int T_p
   TSB_CHECK(ly->missing.empty(), "layered engine: %d weights have not been given, the first is '%s'", (int)ly->missing.size(), ly->missing.begin()->c_str());
   const int* ids = (S == 1 && use_state) ? g->ids_cur : g->ids_in;
   const bool pdl = g->pdl;
+  const Layered::Routing& rt = ly->routing[use_state ? 1 : 0];
+  auto route_of = [&](const LayeredLayer& L) -> const RouteLayer& { return L.routes[use_state ? 1 : 0]; };
   void *ws = ly->ws.p;
   const int64_t wsb = ly->ws.bytes;
   g->lin_syms_used = true;
@@ -406,7 +409,7 @@ static int enqueue_layered(Gpt* g, int B, int S, int T0, bool use_state, int T_p
       TSB_CUDA(launch_k(embed_kernel<__nv_bfloat16>, dim3(gsz), dim3(256), 0, g->s, g->x, (const __nv_bfloat16*)g->E, (const __nv_bfloat16*)nullptr, ids, rows, S, d, g->c.V, ly->c.embed_scale, 0, 0, T0, dT));
     count_launch(dev);
     TSB_TRY(check_launch("embed"));
-    TSB_TRY(launch_table_route(dev, (const RouteLayer*)ly->routes.p, ly->n_route, ly->max_experts, ids, rows, g->c.V, ly->route_block, g->s));
+    TSB_TRY(launch_table_route(dev, (const RouteLayer*)rt.layers.p, ly->n_route, ly->max_experts, ids, rows, g->c.V, rt.block, g->s));
     prof_end(g, KC_EMBED);
   }
   char* h1 = (char*)ly->hcat.p;
@@ -415,7 +418,7 @@ static int enqueue_layered(Gpt* g, int B, int S, int T0, bool use_state, int T_p
   auto pending = [&](BlockNormArgs& a) {
     if (!prev) return;
     a.y = ly->y.p;
-    a.y_pos = prev->route.pos;
+    a.y_pos = route_of(*prev).pos;
     a.top = prev->d.top;
     a.y_gate = ly->gate2.p;
   };
@@ -427,7 +430,7 @@ static int enqueue_layered(Gpt* g, int B, int S, int T0, bool use_state, int T_p
     a.x = g->x; a.d = d; a.groups = ly->c.norm_groups; a.eps = ly->c.eps;
     a.w1 = L.norm1; a.h1 = h1; a.out_scale = 1.0f;
     if (ff) {
-      a.w2 = L.norm2; a.h2 = h2; a.h2_sorted = ly->hs.p; a.next_pos = L.route.pos; a.next_top = L.d.top;
+      a.w2 = L.norm2; a.h2 = h2; a.h2_sorted = ly->hs.p; a.next_pos = route_of(L).pos; a.next_top = L.d.top;
     }
     pending(a);
     a.write_x = 1;
@@ -473,14 +476,14 @@ static int enqueue_layered(Gpt* g, int B, int S, int T0, bool use_state, int T_p
     if (ff) {
       const int picks = rows * L.d.top;
       RowGroups gr{};
-      gr.table = L.route.blocks; gr.n_blocks = L.route.n_blocks;
-      gr.max_blocks = layered_max_blocks(picks, L.d.experts, ly->route_block);
+      gr.table = route_of(L).blocks; gr.n_blocks = route_of(L).n_blocks;
+      gr.max_blocks = layered_max_blocks(picks, L.d.experts, rt.block);
       auto grouped = [&](const void* x, const void* W, int64_t matrix_bytes, int K, int N, const Epilogue& e) -> int {
         gr.matrix_bytes = matrix_bytes;
         int r = 2;
-        if (ly->route_block <= 16) r = launch_gemm_stream_grouped(dev, g->st, dt, x, W, picks, ly->route_block, K, N, e, gr, pdl, ws, wsb, g->s);
+        if (rt.block <= 16) r = launch_gemm_stream_grouped(dev, g->st, dt, x, W, picks, rt.block, K, N, e, gr, pdl, ws, wsb, g->s);
         if (r == 2) r = launch_gemm_tc_grouped(dev, g->st, dt, x, W, picks, K, N, e, gr, g->s);
-        if (r == 2) r = launch_pick_linear(dev, dt, x, W, L.route.matrix_of, matrix_bytes, picks, K, N, e, g->s);
+        if (r == 2) r = launch_pick_linear(dev, dt, x, W, route_of(L).matrix_of, matrix_bytes, picks, K, N, e, g->s);
         return r;
       };
       Epilogue eu = make_ep(nullptr, nullptr, ly->hidden.p, nullptr, TSB200_ACT_CLAMP_GLU, 1);
