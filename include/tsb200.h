@@ -336,31 +336,55 @@ TSB200_API int TSB200_GptCreate(const TSB200GptConfig* cfg, void** gpt);
  * handle is an ordinary engine: prefill, decode, slots, snapshots, beams and sampling work as for TSB200_GptCreate.  (The reference
  * has no counterpart: its GPTDecoder repeats one layer, Networks/GPTDecoder.cs:104-133.)  dtype TSB200_F32 or TSB200_BF16; the
  * residual stream, norms, scores, softmax and angles are fp32 in both.  One GPU.
- *   x = embed[id] * embed_scale
+ *   x = embed[id] * embed_scale;   logits = norm(x) head^T * logit_scale, head: a matrix of its own or (tied_head) the embedding
+ * block TSB200_BLOCK_GATED (latent attention, experts by token id):
  *   x <- x + gate1 * attention(h1 + conv(h1)) + gate2 * experts(h2),   h1 / h2: RMS norm in norm_groups equal parts, weights norm1 /
  *        norm2; gate = sigmoid(h G + b); conv: causal, per channel, conv_taps taps (the newest is the position itself)
- *   logits = norm(x) embed^T * logit_scale
- * Weights (TSB200_GptSetWeight; matrices [out, in] row-major, F32 or BF16, tables I32): embed [V, d], final_norm [1, d] and per layer i
- *   layer.<i>.{norm1, norm2 [1, d], conv1 [d, taps], gate1.w, gate2.w [d, d], gate1.b, gate2.b [1, d]}
+ * block TSB200_BLOCK_SANDWICH (grouped attention, matrix memory, dense feed-forward; norm_groups 1, conv_taps 1):
+ *   x <- x + scale1 * norm1b(mixer(norm1(x))),   x <- x + scale2 * norm2b(ff(norm2(x))),   ff(h) = down(silu(gate h) * up h)
+ * Mixers:
+ *   TSB200_MIXER_LATENT   attention over one cached latent and rotated key part per position, shared by all heads
+ *   TSB200_MIXER_GROUPED  attention with kv_heads key/value heads, query head h reads key/value head h / (heads / kv_heads):
+ *        score = scale q . k + bias[bucket(i - j)][h] for j <= i and (window == 0 or i - j < window or j < keep_first);
+ *        bucket(n) = n below bias_rows / 2, then logarithmic up to bias_max; the softmax's denominator also holds exp(sink[h]);
+ *        head outputs times sigmoid(gate h).  Every part is optional (flags, bias_rows, window).
+ *   TSB200_MIXER_MEMORY   matrix memory with exponential gates (mLSTM): per head a state [dim, vdim], gate logits softly capped at gate_cap
+ * Weights (TSB200_GptSetWeight; matrices [out, in] row-major, F32 or BF16, tables I32): embed [V, d], final_norm [1, d], head [V, d] and per layer
+ *   layer.<i>.{norm1, norm2 [1, d], conv1 [d, taps], gate1.w, gate2.w [d, d], gate1.b, gate2.b [1, d]}              (gated blocks)
+ *   layer.<i>.{norm1, norm1b, scale1, norm2, norm2b, scale2 [1, d]}                                              (sandwich blocks)
  *   layer.<i>.attn.{q [H (dim + rot), d], dkv [rank + rot, d], dkv_norm [1, rank], uk [H dim, rank], uv [H vdim, rank], o [d, H vdim]}
- *   layer.<i>.experts.{table [V, top] I32, <e>.gate, <e>.up [ff, d], <e>.down [d, ff]}
- * Layers with kv_from >= 0 have no dkv / dkv_norm; layers without experts have no norm2 / gate2 / experts. */
+ *   layer.<i>.attn.{q [H dim, d], k [G dim, d], v [G vdim, d], q.b, k.b, v.b, q_norm, k_norm [1, dim], bias [bias_rows, H], sink [1, H],
+ *                   gate [H, d], o [d, H vdim]}                                                                  (grouped attention)
+ *   layer.<i>.mem.{q, k [H dim, d], v, gate [H vdim, d], i, f [H, d], i.b, f.b [1, H], norm [1, H vdim], o [d, H vdim]}
+ *   layer.<i>.experts.{table [V, top] I32, <e>.gate, <e>.up [ff, d], <e>.down [d, ff]},   layer.<i>.ff.{gate, up [ff, d], down [d, ff]}
+ * Layers with kv_from >= 0 have no weights of keys and values; layers without a feed-forward have no second norm, gate or scale. */
+enum { TSB200_MIXER_LATENT = 0, TSB200_MIXER_GROUPED = 1, TSB200_MIXER_MEMORY = 2 };
+enum { TSB200_BLOCK_GATED = 0, TSB200_BLOCK_SANDWICH = 1 };
+enum { TSB200_ATTN_QK_NORM = 1, TSB200_ATTN_QKV_BIAS = 2, TSB200_ATTN_SINK = 4, TSB200_ATTN_HEAD_GATE = 8 };   /* LayerDesc.flags */
 typedef struct TSB200LayerDesc {
-  int32_t mixer;              /* 0: latent attention */
-  int32_t heads, dim, rot_dim, vdim, kv_rank;   /* per head: unrotated and rotated query/key size, value size; size of the latent */
+  int32_t mixer;              /* TSB200_MIXER_* */
+  int32_t heads, dim, rot_dim, vdim, kv_rank;   /* per head: (unrotated) and rotated query/key size, value size; size of the latent */
   int32_t rot_dims;           /* leading dimensions of the rotated part that turn (pairs i, i + rot_dims / 2) */
-  int32_t kv_from;            /* -1: own latent and cache; else the layer whose cached latents and rotated keys are attended to */
+  int32_t kv_from;            /* -1: own cache; else the layer whose cached keys and values are attended to */
   float scale;                /* of the scores */
   double rot_base;
-  int32_t experts, top;       /* experts 0: no feed-forward; else `top` experts per token id by table, each with weight 1 / top */
-  int32_t ff;
+  int32_t experts, top;       /* experts > 0: `top` experts per token id by table, each with weight 1 / top */
+  int32_t ff;                 /* size of an expert, or (experts 0, ff > 0) of the dense feed-forward; both 0: none */
   float glu_limit, glu_slope, glu_shift;   /* expert: a = min(gate, limit), u = clamp(up, limit), a sigmoid(slope a) (u + shift) */
+  int32_t kv_heads;           /* grouped attention from here on */
+  int32_t window, keep_first; /* window 0: every earlier position is seen */
+  int32_t bias_rows, bias_max;
+  int32_t flags;              /* TSB200_ATTN_* */
+  float gate_cap;             /* matrix memory */
+  int32_t reserved;
 } TSB200LayerDesc;
 typedef struct TSB200LayeredConfig {
   int32_t L, d, V, dtype;
   int32_t norm_groups, conv_taps;
   float eps, embed_scale, logit_scale;
   int32_t max_batch, max_tokens, device;
+  int32_t block;              /* TSB200_BLOCK_* */
+  int32_t tied_head;
 } TSB200LayeredConfig;
 TSB200_API int TSB200_GptCreateLayered(const TSB200LayeredConfig* cfg, const TSB200LayerDesc* layers, void** gpt);
 TSB200_API int TSB200_GptDestroy(void* gpt);

@@ -15,6 +15,9 @@ LIB_PATH = os.environ.get("TSB200_LIB") or os.path.join(_HERE, "libtsb200.so")
 HEADER_PATH = os.path.join(_HERE, "..", "include", "tsb200.h")
 
 F32, F16, F64, I32, U8, BF16 = 0, 1, 2, 3, 4, 5
+MIXER_LATENT, MIXER_GROUPED, MIXER_MEMORY = 0, 1, 2
+BLOCK_GATED, BLOCK_SANDWICH = 0, 1
+ATTN_QK_NORM, ATTN_QKV_BIAS, ATTN_SINK, ATTN_HEAD_GATE = 1, 2, 4, 8
 ACT_NONE, ACT_RELU, ACT_SILU, ACT_LEAKYRELU, ACT_GLU_NOACT, ACT_SWIGLU, ACT_GELU = -1, 0, 1, 2, 3, 4, 5
 
 
@@ -43,13 +46,15 @@ class GptConfig(C.Structure):
 class LayerDescC(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "rot_dim", "vdim", "kv_rank", "rot_dims", "kv_from")] + \
                [("scale", C.c_float), ("rot_base", C.c_double)] + [(n, C.c_int32) for n in ("experts", "top", "ff")] + \
-               [(n, C.c_float) for n in ("glu_limit", "glu_slope", "glu_shift")]
+               [(n, C.c_float) for n in ("glu_limit", "glu_slope", "glu_shift")] + \
+               [(n, C.c_int32) for n in ("kv_heads", "window", "keep_first", "bias_rows", "bias_max", "flags")] + \
+               [("gate_cap", C.c_float), ("reserved", C.c_int32)]
 
 
 class LayeredConfigC(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("L", "d", "V", "dtype", "norm_groups", "conv_taps")] + \
                [(n, C.c_float) for n in ("eps", "embed_scale", "logit_scale")] + \
-               [(n, C.c_int32) for n in ("max_batch", "max_tokens", "device")]
+               [(n, C.c_int32) for n in ("max_batch", "max_tokens", "device", "block", "tied_head")]
 
 
 class DecodingOptionsC(C.Structure):

@@ -294,7 +294,7 @@ struct Gpt {
   int own_B = 0;                     // batch the owner kernel serves for the current program (0: not in use)
 };
 
-enum KernelClass { KC_EMBED = 0, KC_NORM = 1, KC_LINEAR = 2, KC_ROPE_APPEND = 3, KC_ATTENTION = 4, KC_SAMPLE = 5, KC_COMMIT = 6, KC_ALLREDUCE = 7, KC_STACK = 8, KC_EXPERTS = 9, KC_COUNT = 10 };
+enum KernelClass { KC_EMBED = 0, KC_NORM = 1, KC_LINEAR = 2, KC_ROPE_APPEND = 3, KC_ATTENTION = 4, KC_SAMPLE = 5, KC_COMMIT = 6, KC_ALLREDUCE = 7, KC_STACK = 8, KC_EXPERTS = 9, KC_MEMORY = 10, KC_COUNT = 11 };
 
 // Profiling pass (TSB200_GptProfileDecode): CUDA events around RUNS of consecutive launches of one class.  Inside a run no
 // event is recorded between the launches, so they chain exactly as they do in the captured step (an event between two
@@ -666,7 +666,12 @@ static std::vector<CachePart> cache_parts(Gpt* g) {
   if (g->ly) {
     for (auto& L : g->ly->L) {
       if (L.cache) v.push_back({&L.cache, 1, (size_t)L.sh.row * g->es, 0});
-      v.push_back({&L.ring, 1, 0, (size_t)g->ly->c.conv_taps * g->ly->c.d * g->es});
+      if (L.cK) {
+        v.push_back({&L.cK, L.gs.G, (size_t)L.gs.dk * g->es, 0});
+        v.push_back({&L.cV, L.gs.G, (size_t)L.gs.dv * g->es, 0});
+      }
+      if (L.mem) v.push_back({&L.mem, 1, 0, (size_t)memory_state_floats(L.ms) * sizeof(float)});
+      if (L.ring) v.push_back({&L.ring, 1, 0, (size_t)g->ly->c.conv_taps * g->ly->c.d * g->es});
     }
     return v;
   }
@@ -1068,6 +1073,8 @@ static int check_err_flag(Gpt* g, const int* pre = nullptr) {
     if (!c) c = chk_take_moe();
     if (!c) c = chk_take_blocks();
     if (!c) c = chk_take_latent();
+    if (!c) c = chk_take_grouped();
+    if (!c) c = chk_take_memory();
     if (!c) c = chk_take_sampling();
     TSB_CHECK(c == 0, "checked build: device-side check 0x%x failed (an index or a capacity was out of range; the access was skipped)", c);
   }
@@ -1391,11 +1398,35 @@ int TSB200_GptCreateLayered(const TSB200LayeredConfig* cfg, const TSB200LayerDes
   TSB_CHECK(c.L > 0 && c.d > 0 && c.V > 0, "gpt_create_layered: bad dimensions");
   TSB_CHECK(c.dtype == TSB200_F32 || c.dtype == TSB200_BF16, "gpt_create_layered: dtype must be F32 or BF16");
   TSB_CHECK(c.norm_groups > 0 && c.d % c.norm_groups == 0, "gpt_create_layered: a width of %d is not cut into %d norm groups", c.d, c.norm_groups);
+  TSB_CHECK(c.block == TSB200_BLOCK_GATED || c.block == TSB200_BLOCK_SANDWICH, "gpt_create_layered: unknown kind of block %d", c.block);
+  TSB_CHECK(c.block == TSB200_BLOCK_GATED || (c.norm_groups == 1 && c.conv_taps == 1 && c.logit_scale == 1.0f),
+            "gpt_create_layered: sandwich blocks have one norm group, no convolution and unscaled logits");
   TSB_CHECK(c.conv_taps >= 1 && c.conv_taps <= 64, "gpt_create_layered: %d convolution taps are not supported", c.conv_taps);
   TSB_CHECK(c.max_batch > 0 && c.max_batch <= 1024 && c.max_tokens > 0, "gpt_create_layered: bad cache capacity");
   for (int i = 0; i < c.L; ++i) {
     const TSB200LayerDesc& l = layers[i];
-    TSB_CHECK(l.mixer == 0, "gpt_create_layered: layer %d has an unknown mixer %d", i, l.mixer);
+    const bool sandwich = c.block == TSB200_BLOCK_SANDWICH;
+    TSB_CHECK(sandwich ? (l.mixer == TSB200_MIXER_GROUPED || l.mixer == TSB200_MIXER_MEMORY) : l.mixer == TSB200_MIXER_LATENT,
+              "gpt_create_layered: layer %d has an unknown mixer %d for this kind of block", i, l.mixer);
+    if (sandwich) {
+      TSB_CHECK(l.heads > 0 && l.dim > 0 && l.vdim > 0 && l.ff >= 0 && l.experts == 0, "gpt_create_layered: layer %d has bad sizes", i);
+      if (l.mixer == TSB200_MIXER_MEMORY) {
+        TSB_CHECK(l.gate_cap > 0.0f && l.kv_from < 0, "gpt_create_layered: layer %d: a matrix memory has a positive gate cap and no cache to share", i);
+        continue;
+      }
+      TSB_CHECK(l.kv_heads > 0 && l.heads % l.kv_heads == 0, "gpt_create_layered: layer %d: %d heads do not share %d key/value heads", i, l.heads, l.kv_heads);
+      TSB_CHECK(l.window >= 0 && l.keep_first >= 0, "gpt_create_layered: layer %d has a bad window", i);
+      TSB_CHECK(l.bias_rows >= 0 && (l.bias_rows == 0 || l.bias_max > l.bias_rows / 2), "gpt_create_layered: layer %d has a bad distance bias (%d rows up to %d)", i,
+                l.bias_rows, l.bias_max);
+      if (l.kv_from >= 0) {
+        TSB_CHECK(l.kv_from < i && layers[l.kv_from].kv_from < 0 && layers[l.kv_from].mixer == TSB200_MIXER_GROUPED,
+                  "gpt_create_layered: layer %d reads the cache of layer %d, which is not an earlier layer with its own", i, l.kv_from);
+        const TSB200LayerDesc& o = layers[l.kv_from];
+        TSB_CHECK(o.kv_heads == l.kv_heads && o.dim == l.dim && o.vdim == l.vdim,
+                  "gpt_create_layered: layer %d and layer %d, whose cache it reads, differ in the key/value heads", i, l.kv_from);
+      }
+      continue;
+    }
     TSB_CHECK(l.heads > 0 && l.dim > 0 && l.rot_dim > 0 && l.vdim > 0 && l.kv_rank > 0 && l.kv_rank <= 1024 && l.dim <= 768,
               "gpt_create_layered: layer %d has unsupported attention sizes (latent up to 1024, unrotated head size up to 768)", i);
     TSB_CHECK(l.rot_dims > 0 && l.rot_dims <= l.rot_dim && l.rot_dims % 2 == 0 && l.rot_base > 0.0, "gpt_create_layered: layer %d has a bad rotation", i);
@@ -1437,6 +1468,56 @@ int TSB200_GptCreateLayered(const TSB200LayeredConfig* cfg, const TSB200LayerDes
   for (int i = 0; i < c.L; ++i) {
     LayeredLayer& L = ly->L[i];
     L.d = layers[i];
+    if (c.block == TSB200_BLOCK_SANDWICH) {
+      const LayerDescView v{L.d};
+      const bool grouped = L.d.mixer == TSB200_MIXER_GROUPED, own = grouped && L.d.kv_from < 0;
+      int cols = v.q();
+      if (own || !grouped) {
+        L.k_col = cols;
+        L.v_col = L.k_col + v.k();
+        cols = L.v_col + v.v();
+      }
+      if (!grouped || (L.d.flags & TSB200_ATTN_HEAD_GATE)) {
+        L.g_col = cols;
+        cols += grouped ? L.d.heads : v.o();
+      }
+      L.Nq = cols;
+      L.ct_gates = (cols + NT - 1) / NT;
+      G_ALLOC(L.norm1, d * es); G_ALLOC(L.norm1b, d * es); G_ALLOC(L.scale1, d * es);
+      G_ALLOC(L.fused, packed_bytes(dt, (int)d, grouped ? cols : L.ct_gates * NT + 2 * L.d.heads));
+      G_ALLOC(L.wo, packed_bytes(dt, v.o(), (int)d));
+      if (grouped) {
+        L.gs = GroupedShape{L.d.heads, L.d.kv_heads, L.d.dim, L.d.vdim, grouped_row_elems(L.d.dim), grouped_row_elems(L.d.vdim), L.d.scale, L.d.window, L.d.keep_first,
+                            L.d.bias_rows > 0 ? std::min(L.d.bias_max, c.max_tokens - 1) + 1 : 0, c.eps};
+        if (L.d.flags & TSB200_ATTN_QKV_BIAS) G_ALLOC(L.qkv_b, (int64_t)cols * es);   // zeros for the gates
+        if (L.d.flags & TSB200_ATTN_QK_NORM) {
+          G_ALLOC(L.q_norm, (int64_t)L.d.dim * es);
+          if (own) G_ALLOC(L.k_norm, (int64_t)L.d.dim * es);
+        }
+        if (L.d.flags & TSB200_ATTN_SINK) G_ALLOC(L.sink, (int64_t)L.d.heads * 4);
+        if (L.gs.n_bias > 0) {
+          G_ALLOC(L.bias, (int64_t)L.gs.n_bias * L.d.heads * 4); G_ALLOC(L.bucket, (int64_t)L.gs.n_bias * 4);
+          std::vector<int> bucket((size_t)L.gs.n_bias);
+          for (int n = 0; n < L.gs.n_bias; ++n) bucket[(size_t)n] = distance_bucket(n, L.d.bias_rows, L.d.bias_max);
+          if (cudaMemcpyAsync(L.bucket, bucket.data(), bucket.size() * 4, cudaMemcpyHostToDevice, g->s) != cudaSuccess || cudaStreamSynchronize(g->s) != cudaSuccess) {
+            set_last_error("gpt_create_layered: upload of the distance table failed");
+            return fail();
+          }
+        }
+        if (own) {
+          G_ALLOC(L.cK, MB * L.gs.G * c.max_tokens * L.gs.dk * es); G_ALLOC(L.cV, MB * L.gs.G * c.max_tokens * L.gs.dv * es);
+        }
+      } else {
+        L.ms = MemoryShape{L.d.heads, L.d.dim, L.d.vdim, L.d.gate_cap, c.eps};
+        G_ALLOC(L.gates_b, 2LL * L.d.heads * es); G_ALLOC(L.mem_norm, (int64_t)v.o() * es);
+        G_ALLOC(L.mem, MB * memory_state_floats(L.ms) * 4);
+      }
+      if (L.d.ff > 0) {
+        G_ALLOC(L.norm2, d * es); G_ALLOC(L.norm2b, d * es); G_ALLOC(L.scale2, d * es);
+        G_ALLOC(L.up, packed_bytes(dt, (int)d, 2 * L.d.ff)); G_ALLOC(L.down, packed_bytes(dt, L.d.ff, (int)d));
+      }
+      continue;
+    }
     L.sh = LatentShape{L.d.heads, L.d.dim, L.d.rot_dim, L.d.vdim, L.d.kv_rank, L.d.rot_dims, latent_row_elems(L.d.kv_rank, L.d.rot_dim), L.d.scale};
     L.Nq = L.sh.H * (L.sh.dim + L.sh.rot);
     L.Nkv = L.d.kv_from < 0 ? L.sh.rank + L.sh.rot : 0;

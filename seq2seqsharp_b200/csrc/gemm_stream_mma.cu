@@ -36,6 +36,7 @@ constexpr int kGsMaxSections = 4;
 struct GsSection {
   int ct_end;   // first column tile after the section
   int N;
+  int x_block;  // stacked row block it reads
   Epilogue ep;
 };
 
@@ -87,7 +88,7 @@ __device__ __forceinline__ void gs_consumers_sync() { asm volatile("bar.sync 1, 
 // rows are read from the fp32 residual stream, normed by the consumer warps (LayerNorm / RMSNorm, the arithmetic of
 // norm_kernel) and kept in shared memory as fp16 for the whole kernel - the norm launch in front of the linear disappears and
 // a stage is the weight tile alone.
-// MODE kGsSections: column tile ct belongs to section i (the first with ct < ct_end), which reads activation rows i * M ..;
+// MODE kGsSections: column tile ct belongs to section i (the first with ct < ct_end), which reads activation rows x_block * M ..;
 // MODE kGsGrouped: "column tiles" run over (row block, column tile of its matrix) pairs; how many there are is read from the device.
 template <typename H, int NB, int KQ = 0, int MODE = kGsPlain>  // row blocks of 8: M <= 8 * NB
 __global__ void __launch_bounds__(kStreamThreads, 1) gemm_stream_mma_kernel(const __grid_constant__ CUtensorMap mapX, GsArgs a) {
@@ -142,7 +143,7 @@ __global__ void __launch_bounds__(kStreamThreads, 1) gemm_stream_mma_kernel(cons
     if constexpr (MODE == kGsSections) {
       int i = 0;
       while (i < a.n_sec - 1 && vct >= a.sec[i].ct_end) ++i;
-      return i * a.M;
+      return a.sec[i].x_block * a.M;
     }
     return 0;
   };
@@ -518,7 +519,7 @@ __global__ void __launch_bounds__(kGcThreads, 3) gemm_chunk_mma_kernel(const __g
   int si = 0;
   if constexpr (MODE == kGsSections)
     while (si < a.n_sec - 1 && ct >= a.sec[si].ct_end) ++si;
-  const int xrow = si * M;
+  const int xrow = MODE == kGsSections ? a.sec[si].x_block * M : 0;
   const int k2_total = (KB + 1) / 2;
   const int k2_beg = ks * a.k2_per, k2_end = min(k2_total, k2_beg + a.k2_per);
   const int n_st = max(k2_end - k2_beg, 0);
@@ -944,6 +945,8 @@ int launch_gemm_stream_sections(int device, DeviceState* st, int dtype, const vo
   if (dtype != TSB200_BF16 || M < 1 || M > 64 || n_sec < 1 || n_sec > kGsMaxSections || K % 8 != 0 || ((uintptr_t)x % 16) != 0 ||
       ((uintptr_t)Wp % 16) != 0)
     return 2;
+  int x_blocks = 1;
+  for (int i = 0; i < n_sec; ++i) x_blocks = sec[i].x_block + 1 > x_blocks ? sec[i].x_block + 1 : x_blocks;
   if (M > 16) {   // the column-chunk kernel; every section starts on a column tile, so its boxes are whole tiles but for the last section's
     GcArgs c{};
     c.Wp = reinterpret_cast<const unsigned char*>(Wp);
@@ -955,12 +958,13 @@ int launch_gemm_stream_sections(int device, DeviceState* st, int dtype, const vo
       c.sec[i].ct_end = c.CT;
       c.sec[i].N = sec[i].N;
       c.sec[i].ep = sec[i].ep;
+      c.sec[i].x_block = sec[i].x_block;
     }
     const int last = (sec[n_sec - 1].N + 255) / 256, boxes = (c.CT - last) * 4 + (sec[n_sec - 1].N + 63) / 64;
     if (gc_plan(&c, st, boxes, ws, ws_bytes) != 1) return 2;
     const int nb = M <= 32 ? 4 : 8;
     CUtensorMap map;
-    const int r = gc_map_x(&map, dtype, x, n_sec * M, K, nb);
+    const int r = gc_map_x(&map, dtype, x, x_blocks * M, K, nb);
     if (r != 1) return r;
     return nb == 4 ? gc_launch<__nv_bfloat16, 4, kGsSections>(device, map, c, boxes * c.ksplit, pdl, s)
                    : gc_launch<__nv_bfloat16, 8, kGsSections>(device, map, c, boxes * c.ksplit, pdl, s);
@@ -976,6 +980,7 @@ int launch_gemm_stream_sections(int device, DeviceState* st, int dtype, const vo
     a.sec[i].ct_end = a.CT;
     a.sec[i].N = sec[i].N;
     a.sec[i].ep = sec[i].ep;
+    a.sec[i].x_block = sec[i].x_block;
   }
   const long long U = (long long)a.KB * a.CT;
   long long g = st->sm_count;
@@ -987,7 +992,7 @@ int launch_gemm_stream_sections(int device, DeviceState* st, int dtype, const vo
   a.counters = reinterpret_cast<unsigned int*>(ws);
   a.partials = reinterpret_cast<float*>(reinterpret_cast<char*>(ws) + kWsCounterBytes);
   CUtensorMap mapX;
-  const int r = gs_map_x(&mapX, dtype, x, n_sec * M, K, NB);
+  const int r = gs_map_x(&mapX, dtype, x, x_blocks * M, K, NB);
   if (r != 1) return r;
   const size_t smem = gs_ring(&a);
   return NB == 1 ? gs_launch<__nv_bfloat16, 1, 0, kGsSections>(device, mapX, a, (int)g, smem, pdl, s)

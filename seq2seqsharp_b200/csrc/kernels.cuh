@@ -136,6 +136,8 @@ int chk_take_moe();
 int chk_take_sampling();
 int chk_take_blocks();
 int chk_take_latent();
+int chk_take_grouped();
+int chk_take_memory();
 
 constexpr int kStackMaxRanks = 8;
 constexpr int kStackXchSites = 4;     // exchange buffers: {out-projection, FFN down} x layer parity
@@ -232,11 +234,12 @@ int launch_gemm_tc_grouped(int device, DeviceState* st, int dtype, const void* x
 int launch_gemm_stream_grouped(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int rows, int block_rows, int K, int N,
                                const Epilogue& ep, const RowGroups& groups, bool pdl, void* ws, int64_t ws_bytes, cudaStream_t s);
 int64_t gemm_stream_grouped_workspace_bytes(int block_rows, int N, int max_blocks, int sm_count);
-// Several linears of equal K in one launch: section i multiplies rows [i * M, (i + 1) * M) of x (stacked [sections * M, K])
+// Several linears of equal K in one launch: a section multiplies rows [x_block * M, (x_block + 1) * M) of x (stacked [blocks * M, K])
 // with columns of its own in Wp (each section starts on a column tile).  At most 64 rows.
 struct LinearSection {
   int N;
   Epilogue ep;
+  int x_block;             // which of the stacked row blocks of x the section reads
 };
 int launch_gemm_stream_sections(int device, DeviceState* st, int dtype, const void* x, const void* Wp, int M, int K, const LinearSection* sec,
                                 int n_sec, bool pdl, void* ws, int64_t ws_bytes, cudaStream_t s);
@@ -305,6 +308,23 @@ struct BlockNormArgs {
 int launch_block_norm(int device, int dtype, const BlockNormArgs& a, int out_rows, cudaStream_t s);
 int launch_short_conv(int device, DeviceState* st, int dtype, void* out, const void* h, const void* w, void* ring, int B, int S, int d, int taps,
                       int T0, const int* state, const int* lens, cudaStream_t s);
+// Sandwich norms: the sublayer's output joins the residual through a norm of its own, and the sum is normed for what comes next.
+//   x += scale * (rms(y) * post_w);  h = rms(x) * next_w
+struct SandwichNormArgs {
+  float* x;               // [rows, d] residual stream
+  int d;
+  float eps;
+  const void* y;          // [rows, d] sublayer output in the model type, null: nothing pending
+  const void* post_w;
+  const void* scale;      // per element, may be null (1)
+  int write_x;            // store the sum back into x
+  const void* next_w;
+  void* h;                // [out rows, d]
+  const int* rows_of;     // which row of x (and y) an output row is, as in BlockNormArgs
+  int last_of_S;
+  const int* lens;
+};
+int launch_sandwich_norm(int device, int dtype, const SandwichNormArgs& a, int out_rows, cudaStream_t s);
 struct RouteLayer {       // one expert layer of table_route_kernel
   const int* table;       // [vocab, top]
   int top, experts;
@@ -359,6 +379,68 @@ struct LatentArgs {
 int latent_pick_splits(DeviceState* st, const LatentShape& a, int B, int S, int T);
 bool latent_expanded(int dtype, const LatentShape& a, int q_stride, int S);
 int launch_latent_attention(int device, DeviceState* st, int dtype, const LatentArgs& a, cudaStream_t s);
+// ---- grouped-query attention with a window, a distance bias, a sink and gated heads (ops_grouped.cu) ------------------------
+struct GroupedShape {
+  int H, G, dim, vdim;           // query heads, key/value heads, query-key size, value size
+  int dk, dv;                    // elements of a cache row of keys / values: dim and vdim rounded up to 8, the rest zero
+  float scale;                   // of the scores (not of the bias)
+  int window;                    // position i sees j if i - j < window (0: every earlier position) ...
+  int keep_first;                // ... or j < keep_first
+  int n_bias;                    // entries of a head's distance bias (the last one serves all larger distances); 0: no bias
+  float eps;                     // of the query and key norm
+};
+inline int grouped_row_elems(int n) { return (n + 7) / 8 * 8; }
+struct GroupedArgs {
+  GroupedShape shape;
+  const void* qkv;               // projected rows: q at column 0, k and v at k_col and v_col, head gates at g_col
+  int q_stride;
+  int k_col, v_col;              // < 0: the layer reads another layer's cache
+  int g_col;                     // < 0: heads are not gated
+  const void *q_norm, *k_norm;   // per-head RMS norm weights [dim], null: none
+  const float* bias;             // [H][n_bias]
+  const float* sink;             // [H] logits of a key without value, null: none
+  void *cK, *cV;                 // [sequences][G][Tmax][dk], [..][dv]
+  int B, S, T0, Tmax;
+  const int* state;
+  int splits;                    // of the key range (decode)
+  void* qn;                      // scratch [B * S][H][dk]: normed queries
+  float* part;                   // scratch of grouped_part_elems() values, decode with several splits
+  int64_t part_elems;
+  unsigned int* counters;        // [B * G * 64], zero, self-resetting
+  void* out;                     // [B * S, H * vdim]
+};
+constexpr int kGroupedMaxSplits = 64;
+int grouped_pick_splits(DeviceState* st, int dtype, const GroupedShape& a, int B, int T);
+int64_t grouped_part_elems(const GroupedShape& a, int B, int splits);
+int launch_grouped_attention(int device, DeviceState* st, int dtype, const GroupedArgs& a, cudaStream_t s);
+// Expanded distance bias [H][n] from a table [rows, H] whose row bucket[i] serves distance i
+int launch_expand_bias(int device, int src_dtype, float* out, const void* table, const int* bucket, int n, int H, cudaStream_t s);
+// ---- matrix memory with exponential gates (ops_memory.cu) ------------------------------------------------------------------
+struct MemoryShape {
+  int H, dim, vdim;
+  float cap;                     // soft cap of the gates' logits
+  float eps;                     // of the norm of a head's output
+};
+__host__ __device__ inline int64_t memory_state_floats(const MemoryShape& a) { return ((int64_t)a.H * ((int64_t)a.dim * a.vdim + a.dim + 1) + 3) / 4 * 4; }
+struct MemoryArgs {
+  MemoryShape shape;
+  const void* x;                 // projected rows q | k | v | output gate (H dim, H dim, H vdim, H vdim)
+  int stride;
+  const float* gates;            // [B * S, 2 H] logits of the input and forget gates
+  const void* norm_w;            // [H * vdim]
+  float* state;                  // [sequences][memory_state_floats]: H matrices [dim, vdim], H vectors [dim], H running maxima
+  int B, S, T0;
+  const int* step_state;         // device step state, null: T0
+  const int* lens;               // prompts of different lengths padded to S, null: all S
+  // a sequence whose current id is 0 stands still when stop_fin is set and the step state is per sequence: its memory keeps
+  const int* ids;
+  int stop_fin;
+  void* scratch;                 // memory_scratch_bytes(), prompts
+  int64_t scratch_bytes;
+  void* out;                     // [B * S, H * vdim]
+};
+int64_t memory_scratch_bytes(int dtype, const MemoryShape& a, int B, int S);
+int launch_matrix_memory(int device, DeviceState* st, int dtype, const MemoryArgs& a, cudaStream_t s);
 int init_tc_attrs(int device);
 int tc_take_error();
 int64_t linear_workspace_bytes(int M, int K, int N);

@@ -2,6 +2,7 @@
 //   block_norm_kernel    pending expert outputs -> residual, RMS norm in groups with one or two weights from one pass over the
 //                        row, the second result optionally also in the row order of a grouped product, and for one new
 //                        position per sequence the short causal convolution with its state;
+//   sandwich_norm_kernel the sublayer output's own norm and scale -> residual, norm of the sum for the next sublayer, one pass;
 //   short_conv_kernel    the same convolution for many new positions; short_conv_state_kernel then leaves the sequence's last
 //                        inputs in its ring (a kernel of its own: the ring is read by the first positions of a portion);
 //   table_route_kernel   experts chosen by token id: for every layer the picks of all rows sorted by expert, cut into blocks of
@@ -298,6 +299,101 @@ static bool block_norm_fast_shape(const BlockNormArgs& a) {
   return gsz >= 128 ? gsz % 128 == 0 : (gsz >= 4 && (gsz & (gsz - 1)) == 0);
 }
 
+// Both norms of a sandwich block in one pass: the row of x and of the sublayer output y in registers (thread t holds elements
+// (t + u * threads) * V .. + V - 1), weights requested before the wait on the previous kernel.
+__device__ __forceinline__ float sandwich_sum(float v, float* red) {   // block-wide sum, one barrier; red: 32 floats of its own per call
+  const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  v = warp_sum(v);
+  if (lane == 0) red[w] = v;
+  __syncthreads();
+  return warp_sum(lane < nw ? red[lane] : 0.0f);
+}
+template <typename T, int V, int NV>
+__global__ void __launch_bounds__(512) sandwich_norm_kernel(SandwichNormArgs a) {
+  __shared__ float s_red[2][32];
+  pdl_trigger();
+  const int tid = threadIdx.x, nt = blockDim.x, d = a.d, out_row = blockIdx.x;
+  constexpr bool kEarly = NV <= 2;   // room to hold the weights across the wait
+  float pw[kEarly ? NV : 1][V], nw[kEarly ? NV : 1][V];
+  auto post_weight = [&](int i, float* o) {
+    VecIO<T, V>::load(reinterpret_cast<const T*>(a.post_w) + i, o);
+    if (a.scale) {
+      float sc[V];
+      VecIO<T, V>::load(reinterpret_cast<const T*>(a.scale) + i, sc);
+#pragma unroll
+      for (int e = 0; e < V; ++e) o[e] *= sc[e];
+    }
+  };
+  if constexpr (kEarly) {
+#pragma unroll
+    for (int u = 0; u < NV; ++u) {
+      const int i = (tid + u * nt) * V;
+      if (i < d) {
+        if (a.y) post_weight(i, pw[u]);
+        VecIO<T, V>::load(reinterpret_cast<const T*>(a.next_w) + i, nw[u]);
+      }
+    }
+  }
+  pdl_wait();
+  int row = out_row;
+  if (a.rows_of) row = a.rows_of[out_row];
+  else if (a.last_of_S > 0) {
+    const int n = a.lens ? a.lens[out_row] : a.last_of_S;
+    row = out_row * a.last_of_S + min(max(n, 1), a.last_of_S) - 1;
+  }
+  float* xr = a.x + (int64_t)row * d;
+  float x[NV][V];
+#pragma unroll
+  for (int u = 0; u < NV; ++u) {
+    const int i = (tid + u * nt) * V;
+#pragma unroll
+    for (int e = 0; e < V; ++e) x[u][e] = 0.0f;
+    if (i < d) VecIO<float, V>::load(xr + i, x[u]);
+  }
+  if (a.y) {
+    const T* yr = reinterpret_cast<const T*>(a.y) + (int64_t)row * d;
+    float y[NV][V], s = 0.0f;
+#pragma unroll
+    for (int u = 0; u < NV; ++u) {
+      const int i = (tid + u * nt) * V;
+#pragma unroll
+      for (int e = 0; e < V; ++e) y[u][e] = 0.0f;
+      if (i < d) VecIO<T, V>::load(yr + i, y[u]);
+#pragma unroll
+      for (int e = 0; e < V; ++e) s += y[u][e] * y[u][e];
+    }
+    const float r = 1.0f / sqrtf(sandwich_sum(s, s_red[0]) / (float)d + a.eps);
+#pragma unroll
+    for (int u = 0; u < NV; ++u) {
+      const int i = (tid + u * nt) * V;
+      if (i < d) {
+        float w[V];
+        if constexpr (!kEarly) post_weight(i, w);
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[u][e] += y[u][e] * r * (kEarly ? pw[kEarly ? u : 0][e] : w[e]);
+        if (a.write_x) VecIO<float, V>::store(xr + i, x[u]);
+      }
+    }
+  }
+  float s = 0.0f;
+#pragma unroll
+  for (int u = 0; u < NV; ++u)
+#pragma unroll
+    for (int e = 0; e < V; ++e) s += x[u][e] * x[u][e];
+  const float r = 1.0f / sqrtf(sandwich_sum(s, s_red[1]) / (float)d + a.eps);
+#pragma unroll
+  for (int u = 0; u < NV; ++u) {
+    const int i = (tid + u * nt) * V;
+    if (i < d) {
+      float w[V], h[V];
+      if constexpr (!kEarly) VecIO<T, V>::load(reinterpret_cast<const T*>(a.next_w) + i, w);
+#pragma unroll
+      for (int e = 0; e < V; ++e) h[e] = x[u][e] * r * (kEarly ? nw[kEarly ? u : 0][e] : w[e]);
+      VecIO<T, V>::store(reinterpret_cast<T*>(a.h) + (int64_t)out_row * d + i, h);
+    }
+  }
+}
+
 // out[b, s] = h[b, s] + sum_j w[:, j] h[b, s - taps + 1 + j]; positions before the portion come from the ring, none before 0
 template <typename T>
 __global__ void __launch_bounds__(256) short_conv_kernel(T* out, const T* h, const T* wgt, const T* ring, int B, int S, int d, int taps, int T0_arg,
@@ -519,6 +615,28 @@ int launch_block_norm(int device, int dtype, const BlockNormArgs& a, int out_row
     TSB_CUDA(launch_k(v4 ? block_norm_kernel<__nv_bfloat16, 4> : block_norm_kernel<__nv_bfloat16, 1>, dim3(out_rows), dim3(kBlockNormThreads), smem, s, a));
   count_launch(device);
   return check_launch("block_norm");
+}
+
+template <typename T, int V>
+static cudaError_t sandwich_go(const SandwichNormArgs& a, int out_rows, cudaStream_t s) {
+  const int units = (a.d + V - 1) / V;
+  int nt = units >= 512 ? 512 : (units + 31) / 32 * 32;
+  const int nv = (units + nt - 1) / nt;
+  const dim3 g(out_rows), b(nt);
+  if (nv <= 1) return launch_k(sandwich_norm_kernel<T, V, 1>, g, b, 0, s, a);
+  if (nv <= 2) return launch_k(sandwich_norm_kernel<T, V, 2>, g, b, 0, s, a);
+  if (nv <= 4) return launch_k(sandwich_norm_kernel<T, V, 4>, g, b, 0, s, a);
+  return launch_k(sandwich_norm_kernel<T, V, 8>, g, b, 0, s, a);
+}
+
+int launch_sandwich_norm(int device, int dtype, const SandwichNormArgs& a, int out_rows, cudaStream_t s) {
+  if (out_rows == 0) return 1;
+  const bool v4 = a.d % 4 == 0;
+  TSB_CHECK(a.d > 0 && a.d <= (v4 ? 16384 : 4096), "sandwich_norm: rows of %d elements are not supported", a.d);
+  if (dtype == TSB200_F32) TSB_CUDA((v4 ? sandwich_go<float, 4>(a, out_rows, s) : sandwich_go<float, 1>(a, out_rows, s)));
+  else TSB_CUDA((v4 ? sandwich_go<__nv_bfloat16, 4>(a, out_rows, s) : sandwich_go<__nv_bfloat16, 1>(a, out_rows, s)));
+  count_launch(device);
+  return check_launch("sandwich_norm");
 }
 
 int launch_short_conv(int device, DeviceState* st, int dtype, void* out, const void* h, const void* w, void* ring, int B, int S, int d, int taps,

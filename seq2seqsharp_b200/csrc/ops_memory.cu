@@ -1,0 +1,640 @@
+// Matrix memory with exponential gates (the mLSTM recurrence): per head a matrix S [dim, vdim], a vector n [dim] and a running maximum m
+// that keeps the exponentials in range.  With log gates i = cap tanh(z_i / cap) and f = logsigmoid(cap tanh(z_f / cap)):
+//
+//   m' = max(f + m, i);   S' = e^(f + m - m') S + e^(i - m') k v^T;   n' likewise with k;   (all zero before the first token)
+//   o  = S'^T q / (max(|n' . q|, e^(-m')) + 1e-6),  q scaled by dim^(-1/2)
+//   out = o / rms(o) * w * sigmoid(g)
+//
+// State of a sequence and layer: fp32, S [H][dim][vdim], n [H][dim], m [H].  Position 0 starts from zero, so a slot that is used again
+// needs no clearing.
+//
+//   memory_step_kernel   token by token, a cluster of CTAs per (sequence, head) with the value columns shared out; the sum of squares of
+//                        the norm crosses the cluster through distributed shared memory.  Decoding, short portions, fp32 models.
+//   prompts (bf16), in chunks of 128 tokens, with F the running sum of f inside a chunk:
+//   memory_gates_kernel  log gates, F and the running maximum of every token (a scan with (max, +))
+//   memory_state_kernel  a tile of S per CTA, chunk by chunk in registers: S <- e^(F_C + m_0 - m_C) S + sum_s e^(F_C - F_s + i_s - m_C) k_s v_s^T
+//                        on the warp-level tensor cores; leaves the state before every chunk in scratch
+//   memory_out_kernel    64 tokens per CTA: inside the chunk (q_t . k_s) e^(F_t - F_s + i_s - m_t), before it e^(F_t + m_0 - m_t) S^T q,
+//                        denominator, norm and output gate
+// The chunk kernels keep fp32 quality on bf16 products: weighted values, scores and states enter as a sum of two bf16 numbers.
+#include <algorithm>
+
+#include "kernels.cuh"
+#include "warp_tiles.cuh"
+
+namespace tsb {
+
+TSB_CHECKED_WORD(memory)
+#ifndef TSB200_CHECKED
+int chk_take_memory() { return 0; }
+#endif
+
+__device__ __forceinline__ float log_sigmoid(float z) { return z >= 0.0f ? -log1pf(expf(-z)) : z - log1pf(expf(z)); }
+__device__ __forceinline__ float soft_cap(float z, float cap) { return cap * tanhf(z / cap); }
+
+__device__ __forceinline__ void cluster_sync() {
+  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+  asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+__device__ __forceinline__ float cluster_read(const float* p, unsigned rank) {
+  uint32_t a;
+  float v;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(a) : "r"(la_smem(p)), "r"(rank));
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(a) : "memory");
+  return v;
+}
+
+// ---- token by token ----------------------------------------------------------------------------------------------------------------
+constexpr int kMsThreads = 256, kMsBatch = 8;
+
+template <int V> struct MsVec;
+template <> struct MsVec<1> {
+  static __device__ __forceinline__ void load(const float* p, float* f) { f[0] = *p; }
+  static __device__ __forceinline__ void store(float* p, const float* f) { *p = f[0]; }
+};
+template <> struct MsVec<4> {
+  static __device__ __forceinline__ void load(const float* p, float* f) {
+    const float4 t = *reinterpret_cast<const float4*>(p);
+    f[0] = t.x; f[1] = t.y; f[2] = t.z; f[3] = t.w;
+  }
+  static __device__ __forceinline__ void store(float* p, const float* f) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+};
+
+// grid (cluster size, heads, sequences); the CTA of rank r has value columns [r * cw, min(vdim, (r + 1) * cw)), cw a multiple of V.
+// Dynamic shared memory: q, k, n [dim each], v [cw], partial outputs [row groups][cw], 32 for sums.
+template <typename T, int V>
+__global__ void __launch_bounds__(kMsThreads) memory_step_kernel(MemoryArgs a, int cw) {
+  extern __shared__ __align__(16) float s_mem[];
+  __shared__ float s_sq[2];
+  const MemoryShape& sh = a.shape;
+  pdl_trigger();
+  pdl_wait();
+  const int tid = threadIdx.x, rank = blockIdx.x, ranks = gridDim.x, h = blockIdx.y, b = blockIdx.z;
+  const int dim = sh.dim, c0 = rank * cw, nc = min(cw, sh.vdim - c0);   // every rank has columns
+  const int tpr = cw / V, groups = kMsThreads / tpr;                    // threads per matrix row, rows at a time
+  float *s_q = s_mem, *s_k = s_q + dim, *s_n = s_k + dim, *s_v = s_n + dim, *s_o = s_v + cw, *s_red = s_o + groups * cw;
+  const int T0 = state_len(a.step_state, b, a.T0);
+  const int n_tok = a.lens ? min(max(a.lens[b], 1), a.S) : a.S;
+  const bool still = a.stop_fin && a.step_state && a.step_state[kStateRagged] != 0 && a.ids[b] == 0;
+  float* st = a.state + (int64_t)b * memory_state_floats(sh);
+  float* S = st + (int64_t)h * dim * sh.vdim;
+  float* gn = st + (int64_t)sh.H * dim * sh.vdim + (int64_t)h * dim;
+  float* gm = st + (int64_t)sh.H * dim * sh.vdim + (int64_t)sh.H * dim + h;
+  float m = T0 > 0 ? *gm : 0.0f;
+  for (int i = tid; i < dim; i += kMsThreads) s_n[i] = T0 > 0 ? gn[i] : 0.0f;
+  const float qs = 1.0f / sqrtf((float)dim);
+  const int grp = tid / tpr, col = (tid % tpr) * V;
+  const bool mine = grp < groups && col < nc;   // nc is a multiple of V
+  const int64_t qk = (int64_t)sh.H * dim, vg = (int64_t)sh.H * sh.vdim;
+
+  for (int t = 0; t < n_tok; ++t) {
+    const int64_t row = (int64_t)b * a.S + t;
+    const T* x = reinterpret_cast<const T*>(a.x) + row * a.stride;
+    const float gi = soft_cap(a.gates[row * 2 * sh.H + h], sh.cap);
+    const float gf = log_sigmoid(soft_cap(a.gates[row * 2 * sh.H + sh.H + h], sh.cap));
+    const float mn = fmaxf(gf + m, gi), keep = expf(gf + m - mn), add = expf(gi - mn);
+    m = mn;
+    __syncthreads();   // the previous token's vectors have been read
+    for (int i = tid; i < dim; i += kMsThreads) {
+      s_q[i] = to_f<T>(x[(int64_t)h * dim + i]) * qs;
+      s_k[i] = to_f<T>(x[qk + (int64_t)h * dim + i]);
+    }
+    for (int i = tid; i < nc; i += kMsThreads) s_v[i] = to_f<T>(x[2 * qk + (int64_t)h * sh.vdim + c0 + i]);
+    __syncthreads();
+    float dot = 0.0f;
+    for (int i = tid; i < dim; i += kMsThreads) {
+      const float nn = keep * s_n[i] + add * s_k[i];
+      s_n[i] = nn;
+      dot = fmaf(nn, s_q[i], dot);
+    }
+    if (mine) {
+      float acc[V], v[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        acc[e] = 0.0f;
+        v[e] = s_v[col + e] * add;
+      }
+      float* base = S + c0 + col;
+      const bool zero = T0 + t == 0;
+      for (int r0 = grp; r0 < dim; r0 += groups * kMsBatch) {
+        float s[kMsBatch][V];
+#pragma unroll
+        for (int q = 0; q < kMsBatch; ++q) {
+          const int r = r0 + q * groups;
+#pragma unroll
+          for (int e = 0; e < V; ++e) s[q][e] = 0.0f;
+          if (r < dim && !zero) MsVec<V>::load(base + (int64_t)r * sh.vdim, s[q]);
+        }
+#pragma unroll
+        for (int q = 0; q < kMsBatch; ++q) {
+          const int r = r0 + q * groups;
+          if (r >= dim) break;
+          const float kk = s_k[r], qq = s_q[r];
+#pragma unroll
+          for (int e = 0; e < V; ++e) {
+            s[q][e] = fmaf(v[e], kk, keep * s[q][e]);
+            acc[e] = fmaf(s[q][e], qq, acc[e]);
+          }
+          if (!still) MsVec<V>::store(base + (int64_t)r * sh.vdim, s[q]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < V; ++e) s_o[grp * cw + col + e] = acc[e];
+    }
+    dot = block_sum(dot, s_red);   // its barriers also publish s_o
+    const float inv_den = 1.0f / (fmaxf(fabsf(dot), expf(-m)) + 1e-6f);
+    float sq = 0.0f;
+    for (int c = tid; c < nc; c += kMsThreads) {
+      float o = 0.0f;
+      for (int q = 0; q < groups; ++q) o += s_o[q * cw + c];
+      o *= inv_den;
+      sq = fmaf(o, o, sq);
+      s_v[c] = o;
+    }
+    sq = block_sum(sq, s_red);
+    if (ranks > 1) {
+      if (tid == 0) s_sq[t & 1] = sq;
+      cluster_sync();
+      sq = 0.0f;
+      for (int q = 0; q < ranks; ++q) sq += cluster_read(&s_sq[t & 1], q);
+    }
+    const float r = 1.0f / sqrtf(sq / (float)sh.vdim + sh.eps);
+    for (int c = tid; c < nc; c += kMsThreads) {
+      const int64_t e = (int64_t)h * sh.vdim + c0 + c;
+      const float g = to_f<T>(x[2 * qk + vg + e]);
+      reinterpret_cast<T*>(a.out)[row * vg + e] = from_f<T>(s_v[c] * r * to_f<T>(reinterpret_cast<const T*>(a.norm_w)[e]) / (1.0f + expf(-g)));
+    }
+  }
+  // every rank has read n and m: the first cluster barrier lies behind
+  if (rank == 0 && !still) {
+    for (int i = tid; i < dim; i += kMsThreads) gn[i] = s_n[i];
+    if (tid == 0) *gm = m;
+  }
+  if (ranks > 1) cluster_sync();   // no CTA leaves while another reads its sum
+}
+
+// ---- chunks ------------------------------------------------------------------------------------------------------------------------
+constexpr int kMcTokens = 128;      // tokens per chunk
+constexpr int kMcTile = 64;         // state tile, value slice, rows of an output CTA
+constexpr int kMcPitch = kMcTile * 2 + 16;
+constexpr int kMgThreads = 1024;
+
+struct MemoryChunks {               // scratch of the chunk kernels
+  float *F, *I, *M;                 // [B * H][chunks * 128]: sum of f inside the chunk, i, running maximum
+  float* m0;                        // [B * H] running maximum before the portion
+  float* n0;                        // [B * H][chunks][dim] state vector before every chunk
+  bf16 *hi, *lo;                    // [B * H][chunks][dim][vdim] state before every chunk, as a sum of two numbers
+  int chunks;
+};
+__device__ __forceinline__ float2 split_bf16(float v) {
+  const float h = to_f<bf16>(from_f<bf16>(v));
+  return make_float2(h, v - h);
+}
+
+__global__ void __launch_bounds__(kMgThreads) memory_gates_kernel(MemoryArgs a, MemoryChunks ck) {
+  __shared__ float s_a[32], s_b[32];
+  const MemoryShape& sh = a.shape;
+  const int bh = blockIdx.x, b = bh / sh.H, h = bh % sh.H, tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
+  const int T0 = state_len(a.step_state, b, a.T0);
+  const int n_tok = a.lens ? min(max(a.lens[b], 1), a.S) : a.S, padded = ck.chunks * kMcTokens;
+  float* gm = a.state + (int64_t)b * memory_state_floats(sh) + (int64_t)sh.H * sh.dim * sh.vdim + (int64_t)sh.H * sh.dim + h;
+  float carry = T0 > 0 ? *gm : 0.0f;
+  __syncthreads();
+  if (tid == 0) ck.m0[bh] = carry;
+  for (int t0 = 0; t0 < padded; t0 += kMgThreads) {
+    const int t = t0 + tid;
+    float gi = -INFINITY, gf = 0.0f;   // tokens beyond the end change nothing
+    if (t < n_tok) {
+      const int64_t row = (int64_t)b * a.S + t;
+      gi = soft_cap(a.gates[row * 2 * sh.H + h], sh.cap);
+      gf = log_sigmoid(soft_cap(a.gates[row * 2 * sh.H + sh.H + h], sh.cap));
+    }
+    // (A, B) of a range of tokens: m after it = max(A + m before it, B)
+    float A = gf, B = gi;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float pa = __shfl_up_sync(0xffffffffu, A, o), pb = __shfl_up_sync(0xffffffffu, B, o);
+      if (lane >= o) {
+        B = fmaxf(pb + A, B);
+        A += pa;
+      }
+    }
+    __syncthreads();
+    if (lane == 31) {
+      s_a[w] = A;
+      s_b[w] = B;
+    }
+    __syncthreads();
+    float F = A, m = carry;
+    for (int q = w & ~3; q < w; ++q) F += s_a[q];          // four warps to a chunk
+    for (int q = 0; q < w; ++q) m = fmaxf(s_a[q] + m, s_b[q]);
+    m = fmaxf(A + m, B);
+    for (int q = 0; q < 32; ++q) carry = fmaxf(s_a[q] + carry, s_b[q]);
+    if (t < padded) {
+      const int64_t at = (int64_t)bh * padded + t;
+      ck.F[at] = F;
+      ck.I[at] = gi;
+      ck.M[at] = m;
+    }
+  }
+  if (tid == 0) *gm = carry;
+}
+
+// grid (value tiles, key tiles, B * H), 4 warps of 16 matrix rows
+__global__ void __launch_bounds__(128) memory_state_kernel(MemoryArgs a, MemoryChunks ck) {
+  extern __shared__ __align__(128) unsigned char smem[];   // k [128], weighted v hi [128], lo [128]: rows of kMcPitch bytes
+  __shared__ float s_w[kMcTokens];
+  const MemoryShape& sh = a.shape;
+  const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
+  const int v0 = blockIdx.x * kMcTile, d0 = blockIdx.y * kMcTile, bh = blockIdx.z, b = bh / sh.H, h = bh % sh.H;
+  const int nv = min(kMcTile, sh.vdim - v0), nd = min(kMcTile, sh.dim - d0);
+  const int T0 = state_len(a.step_state, b, a.T0), padded = ck.chunks * kMcTokens;
+  float* st = a.state + (int64_t)b * memory_state_floats(sh);
+  float* S = st + (int64_t)h * sh.dim * sh.vdim;
+  float* gn = st + (int64_t)sh.H * sh.dim * sh.vdim + (int64_t)h * sh.dim;
+  const uint32_t sk = la_smem(smem), sv = sk + kMcTokens * kMcPitch, sl = sv + kMcTokens * kMcPitch;
+  const int64_t qk = (int64_t)sh.H * sh.dim;
+  const bf16* x0 = reinterpret_cast<const bf16*>(a.x) + (int64_t)b * a.S * a.stride;
+  float s[8][4], nvec = 0.0f;
+#pragma unroll
+  for (int nb = 0; nb < 8; ++nb)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = w * 16 + g8 + (e >> 1) * 8, c = nb * 8 + 2 * t4 + (e & 1);
+      s[nb][e] = T0 > 0 && r < nd && c < nv ? S[(int64_t)(d0 + r) * sh.vdim + v0 + c] : 0.0f;
+    }
+  const bool vec = blockIdx.x == 0 && tid < nd;   // one element of n per thread of the first value tile
+  if (vec && T0 > 0) nvec = gn[d0 + tid];
+  float m0 = ck.m0[bh];
+  for (int c = 0; c < ck.chunks; ++c) {
+    const float* F = ck.F + (int64_t)bh * padded + c * kMcTokens;
+    const float* I = ck.I + (int64_t)bh * padded + c * kMcTokens;
+    const float FC = F[kMcTokens - 1], mC = ck.M[(int64_t)bh * padded + c * kMcTokens + kMcTokens - 1];
+    const float keep = expf(FC + m0 - mC);
+    __syncthreads();
+    for (int v = tid; v < kMcTokens * 8; v += 128) {   // keys: 8 units of 16 bytes per row
+      const int r = v >> 3, u = v & 7, t = c * kMcTokens + r;
+      const bool live = t < a.S && u * 8 < nd;
+      la_cp16(sk + r * kMcPitch + u * 16, live ? x0 + (int64_t)t * a.stride + qk + (int64_t)h * sh.dim + d0 + u * 8 : x0, live);
+    }
+    la_commit();
+    s_w[tid] = expf(FC - F[tid] + I[tid] - mC);
+    // the state before the chunk
+    const int64_t plane = ((int64_t)bh * ck.chunks + c) * sh.dim * sh.vdim;
+#pragma unroll
+    for (int nb = 0; nb < 8; ++nb)
+#pragma unroll
+      for (int q = 0; q < 2; ++q) {
+        const int r = w * 16 + g8 + q * 8, cc = nb * 8 + 2 * t4;
+        if (r < nd && cc < nv) {
+          const float2 p0 = split_bf16(s[nb][2 * q]), p1 = split_bf16(s[nb][2 * q + 1]);
+          const int64_t at = plane + (int64_t)(d0 + r) * sh.vdim + v0 + cc;
+          *reinterpret_cast<uint32_t*>(ck.hi + at) = Pair16<bf16>::put(p0.x, p1.x);
+          *reinterpret_cast<uint32_t*>(ck.lo + at) = Pair16<bf16>::put(p0.y, p1.y);
+        }
+      }
+    if (vec) ck.n0[((int64_t)bh * ck.chunks + c) * sh.dim + d0 + tid] = nvec;
+    __syncthreads();
+    for (int v = tid; v < kMcTokens * 8; v += 128) {   // values times their weight
+      const int r = v >> 3, u = v & 7, t = c * kMcTokens + r;
+      uint4 in = make_uint4(0u, 0u, 0u, 0u), hi, lo;
+      if (t < a.S && u * 8 < nv) in = *reinterpret_cast<const uint4*>(x0 + (int64_t)t * a.stride + 2 * qk + (int64_t)h * sh.vdim + v0 + u * 8);
+      const float wt = s_w[r];
+      const uint32_t* pi = &in.x;
+      uint32_t *ph = &hi.x, *pl = &lo.x;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 f = Pair16<bf16>::get(pi[e]);
+        const float2 p0 = split_bf16(f.x * wt), p1 = split_bf16(f.y * wt);
+        ph[e] = Pair16<bf16>::put(p0.x, p1.x);
+        pl[e] = Pair16<bf16>::put(p0.y, p1.y);
+      }
+      *reinterpret_cast<uint4*>(smem + kMcTokens * kMcPitch + r * kMcPitch + u * 16) = hi;
+      *reinterpret_cast<uint4*>(smem + 2 * kMcTokens * kMcPitch + r * kMcPitch + u * 16) = lo;
+    }
+    la_wait<0>();
+    __syncthreads();
+#pragma unroll
+    for (int nb = 0; nb < 8; ++nb)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[nb][e] *= keep;
+    // S += K^T V: rows of the product are key elements (fragments of K transposed), the sum runs over tokens
+    const uint32_t ka = sk + ((lane & 7) + ((lane >> 4) & 1) * 8) * kMcPitch + (w * 16 + ((lane >> 3) & 1) * 8) * 2;
+    const uint32_t va = sv + ((lane & 7) + ((lane >> 3) & 1) * 8) * kMcPitch + (lane >> 4) * 16;
+#pragma unroll
+    for (int ks = 0; ks < kMcTokens / 16; ++ks) {
+      uint32_t a0, a1, a2, a3;
+      la_ldsm_x4_trans(ka + ks * 16 * kMcPitch, a0, a1, a2, a3);
+#pragma unroll
+      for (int np = 0; np < 4; ++np) {
+        uint32_t b0, b1, b2, b3;
+        la_ldsm_x4_trans(va + ks * 16 * kMcPitch + np * 32, b0, b1, b2, b3);
+        la_mma(s[2 * np], a0, a1, a2, a3, b0, b1);
+        la_mma(s[2 * np + 1], a0, a1, a2, a3, b2, b3);
+        la_ldsm_x4_trans(va + (sl - sv) + ks * 16 * kMcPitch + np * 32, b0, b1, b2, b3);
+        la_mma(s[2 * np], a0, a1, a2, a3, b0, b1);
+        la_mma(s[2 * np + 1], a0, a1, a2, a3, b2, b3);
+      }
+    }
+    if (vec) {
+      float d = 0.0f;
+#pragma unroll 8
+      for (int r = 0; r < kMcTokens; ++r) d = fmaf(s_w[r], to_f<bf16>(*reinterpret_cast<const bf16*>(smem + r * kMcPitch + tid * 2)), d);
+      nvec = keep * nvec + d;
+    }
+    m0 = mC;
+  }
+#pragma unroll
+  for (int nb = 0; nb < 8; ++nb)
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      const int r = w * 16 + g8 + q * 8, c = nb * 8 + 2 * t4;
+      if (r < nd && c < nv) *reinterpret_cast<float2*>(S + (int64_t)(d0 + r) * sh.vdim + v0 + c) = make_float2(s[nb][2 * q], s[nb][2 * q + 1]);
+    }
+  if (vec) gn[d0 + tid] = nvec;
+}
+
+// grid (tiles of 64 tokens, heads, sequences), 4 warps of 16 tokens.  Shared memory: q [64] rows; then k [64] rows, or a value slice [128]
+// and the two planes of a state slice [dim].  Rows of q and k hold dim elements rounded up to 16 (zero beyond) and 16 bytes.
+__global__ void __launch_bounds__(128) memory_out_kernel(MemoryArgs a, MemoryChunks ck) {
+  extern __shared__ __align__(128) unsigned char smem[];
+  __shared__ float s_F[kMcTokens], s_I[kMcTokens], s_nq[kMcTile];
+  const MemoryShape& sh = a.shape;
+  const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
+  const int t0 = blockIdx.x * kMcTile, h = blockIdx.y, b = blockIdx.z, bh = b * sh.H + h;
+  const int c = t0 / kMcTokens, cb = c * kMcTokens, padded = ck.chunks * kMcTokens;
+  const int n_keys = t0 - cb + kMcTile;                       // 64 or 128, the tile's own tokens last
+  const int dp = (sh.dim + 15) / 16 * 16, pitch = dp * 2 + 16, du = dp / 8;
+  const uint32_t sq = la_smem(smem), sk = sq + kMcTile * pitch;
+  const uint32_t sv = sk, sh_hi = sv + kMcTokens * kMcPitch, sh_lo = sh_hi + dp * kMcPitch;
+  const int64_t qk = (int64_t)sh.H * sh.dim, vg = (int64_t)sh.H * sh.vdim;
+  const bf16* x0 = reinterpret_cast<const bf16*>(a.x) + (int64_t)b * a.S * a.stride;
+  auto rows = [&](uint32_t dst, int first, int64_t col) {     // 64 rows of q or k
+    for (int v = tid; v < kMcTile * du; v += 128) {
+      const int r = v / du, u = v % du, t = first + r;
+      const bool live = t < a.S && u * 8 < sh.dim;
+      la_cp16(dst + r * pitch + u * 16, live ? x0 + (int64_t)t * a.stride + col + (int64_t)h * sh.dim + u * 8 : x0, live);
+    }
+    la_commit();
+  };
+  rows(sq, t0, 0);
+  rows(sk, cb, qk);
+  s_F[tid] = ck.F[(int64_t)bh * padded + cb + tid];
+  s_I[tid] = ck.I[(int64_t)bh * padded + cb + tid];
+  const float m0 = c > 0 ? ck.M[(int64_t)bh * padded + cb - 1] : ck.m0[bh];
+  const int rA = w * 16 + g8, off = t0 - cb;
+  float mt[2], ft[2], inter[2];
+  const float qs = 1.0f / sqrtf((float)sh.dim);
+  la_wait<0>();
+  __syncthreads();
+#pragma unroll
+  for (int q = 0; q < 2; ++q) {
+    mt[q] = ck.M[(int64_t)bh * padded + t0 + rA + q * 8];
+    ft[q] = s_F[off + rA + q * 8];
+    inter[q] = expf(ft[q] + m0 - mt[q]) * qs;
+  }
+  {   // n . q of every row: two threads per row
+    const float* n0 = ck.n0 + ((int64_t)bh * ck.chunks + c) * sh.dim;
+    const bf16* qr = reinterpret_cast<const bf16*>(smem + (tid >> 1) * pitch);
+    float d = 0.0f;
+    for (int i = (tid & 1); i < sh.dim; i += 2) d = fmaf(n0[i], to_f<bf16>(qr[i]), d);
+    d += __shfl_xor_sync(0xffffffffu, d, 1);
+    if ((tid & 1) == 0) s_nq[tid >> 1] = d;
+  }
+  // weights of the chunk's keys up to each row, as operands of the second product
+  uint32_t ph[8][4], pl[8][4];
+  float rs[2] = {0.0f, 0.0f};
+  const uint32_t qa = sq + (w * 16 + (lane & 15)) * pitch + (lane >> 4) * 16;
+#pragma unroll
+  for (int kt = 0; kt < 2; ++kt) {
+    if (kt * kMcTile < n_keys) {
+      if (kt > 0) {
+        __syncthreads();
+        rows(sk, cb + kMcTile, qk);
+        la_wait<0>();
+        __syncthreads();
+      }
+      float sc[8][4];
+#pragma unroll
+      for (int nb = 0; nb < 8; ++nb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sc[nb][e] = 0.0f;
+      const uint32_t ka = sk + ((lane & 7) + (lane >> 4) * 8) * pitch + ((lane >> 3) & 1) * 16;
+      for (int ks = 0; ks < dp / 16; ++ks) {
+        uint32_t a0, a1, a2, a3;
+        la_ldsm_x4(qa + ks * 32, a0, a1, a2, a3);
+#pragma unroll
+        for (int np = 0; np < 4; ++np) {   // two blocks of 8 keys
+          uint32_t b0, b1, b2, b3;
+          la_ldsm_x4(ka + np * 16 * pitch + ks * 32, b0, b1, b2, b3);
+          la_mma(sc[2 * np], a0, a1, a2, a3, b0, b1);
+          la_mma(sc[2 * np + 1], a0, a1, a2, a3, b2, b3);
+        }
+      }
+#pragma unroll
+      for (int nb = 0; nb < 8; ++nb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int q = e >> 1, key = kt * kMcTile + nb * 8 + 2 * t4 + (e & 1);
+          const float p = key <= off + rA + q * 8 ? sc[nb][e] * qs * expf(ft[q] - s_F[key] + s_I[key] - mt[q]) : 0.0f;
+          sc[nb][e] = p;
+          rs[q] += p;
+        }
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float* p = &sc[2 * kk + (e >> 1)][2 * (e & 1)];
+          const float2 p0 = split_bf16(p[0]), p1 = split_bf16(p[1]);
+          ph[kt * 4 + kk][e] = Pair16<bf16>::put(p0.x, p1.x);
+          pl[kt * 4 + kk][e] = Pair16<bf16>::put(p0.y, p1.y);
+        }
+    } else {
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) ph[kt * 4 + kk][e] = pl[kt * 4 + kk][e] = 0u;
+    }
+  }
+  __syncthreads();
+  float inv_den[2], sq_sum[2] = {0.0f, 0.0f};
+#pragma unroll
+  for (int q = 0; q < 2; ++q) {
+    rs[q] += __shfl_xor_sync(0xffffffffu, rs[q], 1);
+    rs[q] += __shfl_xor_sync(0xffffffffu, rs[q], 2);
+    inv_den[q] = 1.0f / (fmaxf(fabsf(rs[q] + inter[q] * s_nq[rA + q * 8]), expf(-mt[q])) + 1e-6f);
+  }
+  bf16* out = reinterpret_cast<bf16*>(a.out) + ((int64_t)b * a.S + t0) * vg + (int64_t)h * sh.vdim;
+  const int64_t plane = ((int64_t)bh * ck.chunks + c) * sh.dim * sh.vdim;
+  for (int v0 = 0; v0 < sh.vdim; v0 += kMcTile) {
+    const int nv = min(kMcTile, sh.vdim - v0);
+    if (v0 > 0) __syncthreads();
+    for (int v = tid; v < n_keys * 8; v += 128) {
+      const int r = v >> 3, u = v & 7, t = cb + r;
+      const bool live = t < a.S && u * 8 < nv;
+      la_cp16(sv + r * kMcPitch + u * 16, live ? x0 + (int64_t)t * a.stride + 2 * qk + (int64_t)h * sh.vdim + v0 + u * 8 : x0, live);
+    }
+    for (int v = tid; v < dp * 8; v += 128) {
+      const int r = v >> 3, u = v & 7;
+      const bool live = r < sh.dim && u * 8 < nv;
+      const int64_t at = live ? plane + (int64_t)r * sh.vdim + v0 + u * 8 : 0;
+      la_cp16(sh_hi + r * kMcPitch + u * 16, ck.hi + at, live);
+      la_cp16(sh_lo + r * kMcPitch + u * 16, ck.lo + at, live);
+    }
+    la_commit();
+    la_wait<0>();
+    __syncthreads();
+    float o[8][4];
+#pragma unroll
+    for (int nb = 0; nb < 8; ++nb)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[nb][e] = 0.0f;
+    const uint32_t vrow = ((lane & 7) + ((lane >> 3) & 1) * 8) * kMcPitch + (lane >> 4) * 16;
+    for (int ks = 0; ks < dp / 16; ++ks) {
+      uint32_t a0, a1, a2, a3;
+      la_ldsm_x4(qa + ks * 32, a0, a1, a2, a3);
+#pragma unroll
+      for (int np = 0; np < 4; ++np) {
+        uint32_t b0, b1, b2, b3;
+        la_ldsm_x4_trans(sh_hi + vrow + ks * 16 * kMcPitch + np * 32, b0, b1, b2, b3);
+        la_mma(o[2 * np], a0, a1, a2, a3, b0, b1);
+        la_mma(o[2 * np + 1], a0, a1, a2, a3, b2, b3);
+        la_ldsm_x4_trans(sh_lo + vrow + ks * 16 * kMcPitch + np * 32, b0, b1, b2, b3);
+        la_mma(o[2 * np], a0, a1, a2, a3, b0, b1);
+        la_mma(o[2 * np + 1], a0, a1, a2, a3, b2, b3);
+      }
+    }
+#pragma unroll
+    for (int nb = 0; nb < 8; ++nb)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[nb][e] *= inter[e >> 1];
+#pragma unroll
+    for (int kk = 0; kk < 8; ++kk) {
+      if (kk * 16 >= n_keys) break;
+#pragma unroll
+      for (int np = 0; np < 4; ++np) {
+        uint32_t b0, b1, b2, b3;
+        la_ldsm_x4_trans(sv + vrow + kk * 16 * kMcPitch + np * 32, b0, b1, b2, b3);
+        la_mma(o[2 * np], ph[kk][0], ph[kk][1], ph[kk][2], ph[kk][3], b0, b1);
+        la_mma(o[2 * np + 1], ph[kk][0], ph[kk][1], ph[kk][2], ph[kk][3], b2, b3);
+        la_mma(o[2 * np], pl[kk][0], pl[kk][1], pl[kk][2], pl[kk][3], b0, b1);
+        la_mma(o[2 * np + 1], pl[kk][0], pl[kk][1], pl[kk][2], pl[kk][3], b2, b3);
+      }
+    }
+#pragma unroll
+    for (int nb = 0; nb < 8; ++nb)
+#pragma unroll
+      for (int q = 0; q < 2; ++q) {
+        const float u0 = o[nb][2 * q] * inv_den[q], u1 = o[nb][2 * q + 1] * inv_den[q];
+        sq_sum[q] += u0 * u0 + u1 * u1;   // columns beyond the slice are zero
+        const int r = rA + q * 8, cc = nb * 8 + 2 * t4;
+        if (t0 + r < a.S && cc < nv) *reinterpret_cast<uint32_t*>(out + (int64_t)r * vg + v0 + cc) = Pair16<bf16>::put(u0, u1);
+      }
+  }
+  // norm and output gate on the values this thread has just written
+#pragma unroll
+  for (int q = 0; q < 2; ++q) {
+    sq_sum[q] += __shfl_xor_sync(0xffffffffu, sq_sum[q], 1);
+    sq_sum[q] += __shfl_xor_sync(0xffffffffu, sq_sum[q], 2);
+    const int r = rA + q * 8;
+    if (t0 + r >= a.S) continue;
+    const float f = 1.0f / sqrtf(sq_sum[q] / (float)sh.vdim + sh.eps);
+    const bf16* gr = x0 + (int64_t)(t0 + r) * a.stride + 2 * qk + vg + (int64_t)h * sh.vdim;
+    const bf16* wr = reinterpret_cast<const bf16*>(a.norm_w) + (int64_t)h * sh.vdim;
+#pragma unroll 4
+    for (int cc = 2 * t4; cc < sh.vdim; cc += 8) {
+      uint32_t* op = reinterpret_cast<uint32_t*>(out + (int64_t)r * vg + cc);
+      const float2 o = Pair16<bf16>::get(*op), g = Pair16<bf16>::get(*reinterpret_cast<const uint32_t*>(gr + cc)), wt = Pair16<bf16>::get(*reinterpret_cast<const uint32_t*>(wr + cc));
+      *op = Pair16<bf16>::put(o.x * f * wt.x / (1.0f + __expf(-g.x)), o.y * f * wt.y / (1.0f + __expf(-g.y)));
+    }
+  }
+}
+
+// ---- host side -------------------------------------------------------------------------------------------------------------------
+constexpr int kMemoryChunkMin = 32;   // shorter portions go token by token
+static bool memory_chunked(int dtype, const MemoryShape& a, int S) {
+  return dtype == TSB200_BF16 && S >= kMemoryChunkMin && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.dim <= 256;
+}
+static int64_t align16(int64_t n) { return (n + 255) / 256 * 256; }
+static int64_t memory_layout(const MemoryShape& a, int B, int S, char* base, MemoryChunks* ck) {
+  const int64_t bh = (int64_t)B * a.H, chunks = (S + kMcTokens - 1) / kMcTokens, tok = align16(bh * chunks * kMcTokens * 4), m0 = align16(bh * 4);
+  const int64_t n0 = align16(bh * chunks * a.dim * 4), st = align16(bh * chunks * a.dim * a.vdim * 2);
+  if (ck) {
+    ck->chunks = (int)chunks;
+    ck->F = (float*)base;
+    ck->I = (float*)(base + tok);
+    ck->M = (float*)(base + 2 * tok);
+    ck->m0 = (float*)(base + 3 * tok);
+    ck->n0 = (float*)(base + 3 * tok + m0);
+    ck->hi = (bf16*)(base + 3 * tok + m0 + n0);
+    ck->lo = (bf16*)(base + 3 * tok + m0 + n0 + st);
+  }
+  return 3 * tok + m0 + n0 + 2 * st;
+}
+int64_t memory_scratch_bytes(int dtype, const MemoryShape& a, int B, int S) { return memory_chunked(dtype, a, S) ? memory_layout(a, B, S, nullptr, nullptr) : 0; }
+
+template <typename T, int V>
+static int memory_step_go(int device, const MemoryArgs& a, int ranks, int cw, size_t smem, cudaStream_t s) {
+  static bool done[kMaxDevices] = {};
+  if (!done[device]) {
+    TSB_CUDA(cudaFuncSetAttribute(memory_step_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+    done[device] = true;
+  }
+  cudaLaunchConfig_t cfg{};
+  cfg.gridDim = dim3(ranks, a.shape.H, a.B);
+  cfg.blockDim = dim3(kMsThreads);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = s;
+  cudaLaunchAttribute at[2];
+  at[0].id = cudaLaunchAttributeClusterDimension;
+  at[0].val.clusterDim.x = (unsigned)ranks;
+  at[0].val.clusterDim.y = at[0].val.clusterDim.z = 1;
+  at[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  at[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = at;
+  cfg.numAttrs = pdl_enabled() ? 2 : 1;
+  TSB_CUDA(cudaLaunchKernelEx(&cfg, memory_step_kernel<T, V>, a, cw));
+  count_launch(device);
+  return check_launch("memory_step");
+}
+
+int launch_matrix_memory(int device, DeviceState* st, int dtype, const MemoryArgs& a, cudaStream_t s) {
+  if (a.B == 0 || a.S == 0) return 1;
+  const MemoryShape& sh = a.shape;
+  TSB_CHECK(a.B <= 65535 && sh.H <= 65535, "matrix memory: %d heads of %d sequences are not supported", sh.H, a.B);
+  if (!a.step_state && memory_chunked(dtype, sh, a.S) && a.stride % 8 == 0 && ((uintptr_t)a.x % 16) == 0 && ((uintptr_t)a.state % 16) == 0) {
+    MemoryChunks ck;
+    TSB_CHECK(memory_layout(sh, a.B, a.S, (char*)a.scratch, &ck) <= a.scratch_bytes, "matrix memory: scratch too small for %d tokens", a.B * a.S);
+    const int dp = (sh.dim + 15) / 16 * 16;
+    const size_t s1 = 3 * (size_t)kMcTokens * kMcPitch;
+    const size_t q = (size_t)kMcTile * (dp * 2 + 16), s2 = q + std::max<size_t>(q, (size_t)(kMcTokens + 2 * dp) * kMcPitch);
+    static bool done[kMaxDevices] = {};
+    if (!done[device]) {
+      TSB_CUDA(cudaFuncSetAttribute(memory_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024));
+      TSB_CUDA(cudaFuncSetAttribute(memory_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+      done[device] = true;
+    }
+    TSB_CHECK((int64_t)a.B * sh.H <= 65535, "matrix memory: %d heads of %d sequences are not supported", sh.H, a.B);
+    memory_gates_kernel<<<a.B * sh.H, kMgThreads, 0, s>>>(a, ck);
+    memory_state_kernel<<<dim3((sh.vdim + kMcTile - 1) / kMcTile, (sh.dim + kMcTile - 1) / kMcTile, a.B * sh.H), 128, s1, s>>>(a, ck);
+    memory_out_kernel<<<dim3((a.S + kMcTile - 1) / kMcTile, sh.H, a.B), 128, s2, s>>>(a, ck);
+    count_launch(device, 3);
+    return check_launch("matrix_memory");
+  }
+  // columns of a CTA: enough CTAs for the machine, at least 16 columns, clusters of up to 8
+  const bool v4 = sh.vdim % 4 == 0 && ((uintptr_t)a.state % 16) == 0;
+  const int V = v4 ? 4 : 1;
+  int ranks = 1;
+  while (ranks < 8 && (int64_t)a.B * sh.H * ranks < 2 * st->sm_count && sh.vdim / (2 * ranks) >= 16) ranks *= 2;
+  auto cols = [&](int r) { return ((sh.vdim + r - 1) / r + V - 1) / V * V; };
+  while (cols(ranks) / V > kMsThreads && ranks < 8) ranks *= 2;
+  while (ranks > 1 && (int64_t)(ranks - 1) * cols(ranks) >= sh.vdim) ranks /= 2;   // every rank has columns
+  const int cw = cols(ranks);
+  TSB_CHECK(cw / V <= kMsThreads, "matrix memory: values of %d elements are not supported", sh.vdim);
+  const size_t smem = ((size_t)3 * sh.dim + cw + (size_t)(kMsThreads / (cw / V)) * cw + 32) * sizeof(float);
+  TSB_CHECK(smem <= 160 * 1024, "matrix memory: keys of %d elements are not supported", sh.dim);
+  if (dtype == TSB200_F32) return v4 ? memory_step_go<float, 4>(device, a, ranks, cw, smem, s) : memory_step_go<float, 1>(device, a, ranks, cw, smem, s);
+  return v4 ? memory_step_go<bf16, 4>(device, a, ranks, cw, smem, s) : memory_step_go<bf16, 1>(device, a, ranks, cw, smem, s);
+}
+
+}  // namespace tsb

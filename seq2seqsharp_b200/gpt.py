@@ -521,7 +521,7 @@ class GPT:
         N.call("TSB200_GptGetStepTimes", self._h, ms.ctypes.data_as(C.c_void_p), n, C.byref(got))
         return ms[:got.value]
 
-    KERNEL_CLASSES = ("embed", "norm", "linear", "rope_append", "attention", "sampling", "commit", "allreduce", "decode_stack", "experts")
+    KERNEL_CLASSES = ("embed", "norm", "linear", "rope_append", "attention", "sampling", "commit", "allreduce", "decode_stack", "experts", "memory")
 
     def ProfileDecode(self, n_steps, opts: DecodingOptions):
         """{class: (ms_total, launch_groups)} over n_steps un-captured decode steps (CUDA events per launch group)."""

@@ -6,7 +6,7 @@ snapshots, KV pool, beam search, sampling and the slot scheduler work on it unch
 """
 import ctypes as C
 from dataclasses import dataclass, field
-from typing import Dict, List, Optional
+from typing import Dict, List, Optional, Union
 
 import numpy as np
 
@@ -45,9 +45,45 @@ class TableExperts:
 
 
 @dataclass
+class GroupedAttention:
+    """Attention with kv_heads key/value heads (query head h reads key/value head h // (heads // kv_heads)) over cached keys and values.
+    score = scale q . k + bias[bucket(i - j)]; position i sees j <= i with i - j < window or j < keep_first."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float             # of the scores (not of the bias)
+    window: int = 0          # 0: every earlier position
+    keep_first: int = 0
+    bias_rows: int = 0       # rows of the distance bias table, 0: none; half of them for single distances, half logarithmic up to bias_max
+    bias_max: int = 0
+    qk_norm: bool = False    # per-head RMS norm of queries and keys
+    qkv_bias: bool = False
+    sink: bool = False       # a logit per head that joins the softmax's denominator
+    head_gate: bool = False  # head outputs times sigmoid(gate h)
+    kv_from: int = -1        # attend to another layer's cache instead of an own one
+
+
+@dataclass
+class MatrixMemory:
+    """Matrix memory with exponential gates (mLSTM): per head a state [dim, vdim] of fixed size instead of a cache."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float          # soft cap of the gates' logits
+
+
+@dataclass
+class DenseGated:
+    """down(silu(gate h) * up h)."""
+    ff: int
+
+
+@dataclass
 class BlockLayer:
-    mixer: LatentAttention
-    experts: Optional[TableExperts] = None
+    mixer: Union[LatentAttention, GroupedAttention, MatrixMemory]
+    experts: Optional[TableExperts] = None     # feed-forward of gated blocks
+    dense: Optional[DenseGated] = None         # feed-forward of sandwich blocks
 
 
 @dataclass
@@ -55,11 +91,13 @@ class LayeredConfig:
     d: int
     V: int
     layers: List[BlockLayer] = field(default_factory=list)
+    block: str = "gated"        # "gated": latent attention and experts, parallel and gated; "sandwich": norms around every sublayer
     norm_groups: int = 1
     conv_taps: int = 1
     eps: float = 1e-6
     embed_scale: float = 1.0
     logit_scale: float = 1.0
+    tied_head: bool = True      # logits from the embedding table; False: a "head" matrix
     dtype: str = "bfloat16"     # "bfloat16" | "float32"
     name: str = ""
     # what a GPTConfig would say here: no attention over an encoder, no position table (positions are the mixers' business)
@@ -73,35 +111,70 @@ class LayeredConfig:
 
     def weight_shapes(self) -> Dict[str, tuple]:
         """Engine weight names -> shapes ([out, in] for matrices)."""
-        d, V = self.d, self.V
-        s = {"embed": (V, d), "final_norm": (1, d)}
+        s = {"embed": (self.V, self.d), "final_norm": (1, self.d)}
+        if not self.tied_head:
+            s["head"] = (self.V, self.d)
         for i, layer in enumerate(self.layers):
-            p, m, x = "layer.%d." % i, layer.mixer, layer.experts
-            s[p + "norm1"], s[p + "conv1"], s[p + "gate1.w"], s[p + "gate1.b"] = (1, d), (d, self.conv_taps), (d, d), (1, d)
-            s[p + "attn.q"] = (m.heads * (m.dim + m.rot_dim), d)
-            if m.kv_from < 0:
-                s[p + "attn.dkv"], s[p + "attn.dkv_norm"] = (m.kv_rank + m.rot_dim, d), (1, m.kv_rank)
-            s[p + "attn.uk"], s[p + "attn.uv"] = (m.heads * m.dim, m.kv_rank), (m.heads * m.vdim, m.kv_rank)
-            s[p + "attn.o"] = (d, m.heads * m.vdim)
-            if x is not None:
-                s[p + "norm2"], s[p + "gate2.w"], s[p + "gate2.b"] = (1, d), (d, d), (1, d)
-                s[p + "experts.table"] = (V, x.top)
-                for e in range(x.experts):
-                    q = p + "experts.%d." % e
-                    s[q + "gate"], s[q + "up"], s[q + "down"] = (x.ff, d), (x.ff, d), (d, x.ff)
+            p = "layer.%d." % i
+            s.update({p + n: v for n, v in (self._sandwich_shapes(layer) if self.block == "sandwich" else self._gated_shapes(layer)).items()})
+        return s
+
+    def _gated_shapes(self, layer) -> Dict[str, tuple]:
+        d, m, x = self.d, layer.mixer, layer.experts
+        s = {"norm1": (1, d), "conv1": (d, self.conv_taps), "gate1.w": (d, d), "gate1.b": (1, d), "attn.q": (m.heads * (m.dim + m.rot_dim), d)}
+        if m.kv_from < 0:
+            s["attn.dkv"], s["attn.dkv_norm"] = (m.kv_rank + m.rot_dim, d), (1, m.kv_rank)
+        s["attn.uk"], s["attn.uv"] = (m.heads * m.dim, m.kv_rank), (m.heads * m.vdim, m.kv_rank)
+        s["attn.o"] = (d, m.heads * m.vdim)
+        if x is not None:
+            s["norm2"], s["gate2.w"], s["gate2.b"] = (1, d), (d, d), (1, d)
+            s["experts.table"] = (self.V, x.top)
+            for e in range(x.experts):
+                q = "experts.%d." % e
+                s[q + "gate"], s[q + "up"], s[q + "down"] = (x.ff, d), (x.ff, d), (d, x.ff)
+        return s
+
+    def _sandwich_shapes(self, layer) -> Dict[str, tuple]:
+        d, m = self.d, layer.mixer
+        s = {"norm1": (1, d), "norm1b": (1, d), "scale1": (1, d)}
+        if isinstance(m, GroupedAttention):
+            own = m.kv_from < 0
+            rows = {"q": m.heads * m.dim, **({"k": m.kv_heads * m.dim, "v": m.kv_heads * m.vdim} if own else {})}
+            for n, r in rows.items():
+                s["attn." + n] = (r, d)
+                if m.qkv_bias:
+                    s["attn.%s.b" % n] = (1, r)
+                if m.qk_norm and n != "v":
+                    s["attn.%s_norm" % n] = (1, m.dim)
+            if m.bias_rows:
+                s["attn.bias"] = (m.bias_rows, m.heads)
+            if m.sink:
+                s["attn.sink"] = (1, m.heads)
+            if m.head_gate:
+                s["attn.gate"] = (m.heads, d)
+            s["attn.o"] = (d, m.heads * m.vdim)
+        else:
+            for n, r in (("q", m.heads * m.dim), ("k", m.heads * m.dim), ("v", m.heads * m.vdim), ("gate", m.heads * m.vdim), ("i", m.heads), ("f", m.heads)):
+                s["mem." + n] = (r, d)
+            s["mem.i.b"], s["mem.f.b"], s["mem.norm"] = (1, m.heads), (1, m.heads), (1, m.heads * m.vdim)
+            s["mem.o"] = (d, m.heads * m.vdim)
+        if layer.dense is not None:
+            ff = layer.dense.ff
+            s["norm2"], s["norm2b"], s["scale2"] = (1, d), (1, d), (1, d)
+            s["ff.gate"], s["ff.up"], s["ff.down"] = (ff, d), (ff, d), (d, ff)
         return s
 
     def active_matmul_params(self) -> int:
         """Multiply-adds of the matrices per token (experts: the ones a token uses; keys and values once per position)."""
-        n = self.d * self.V
-        for layer in self.layers:
-            m, x = layer.mixer, layer.experts
-            n += self.d * self.d * (2 if x is not None else 1) + self.d * m.heads * (m.dim + m.rot_dim) + m.heads * m.vdim * self.d
-            n += m.heads * (m.dim + m.vdim) * m.kv_rank
-            if m.kv_from < 0:
-                n += self.d * (m.kv_rank + m.rot_dim)
-            if x is not None:
-                n += 3 * self.d * x.ff * x.top
+        n = 0
+        for name, (r, c) in self.weight_shapes().items():
+            layer = self.layers[int(name.split(".")[1])] if name.startswith("layer.") else None
+            if name == "embed":
+                n += r * c if self.tied_head else 0
+            elif ".experts." in name:
+                n += 0 if name.endswith("table") else r * c * layer.experts.top // layer.experts.experts
+            elif r > 1 and not name.endswith(("conv1", "attn.bias")):
+                n += r * c
         return n
 
 
@@ -118,14 +191,25 @@ class LayeredGPT(GPT):
         c.norm_groups, c.conv_taps = cfg.norm_groups, cfg.conv_taps
         c.eps, c.embed_scale, c.logit_scale = cfg.eps, cfg.embed_scale, cfg.logit_scale
         c.max_batch, c.max_tokens, c.device = max_batch, max_tokens, device_id
+        c.block, c.tied_head = {"gated": N.BLOCK_GATED, "sandwich": N.BLOCK_SANDWICH}[cfg.block], int(cfg.tied_head)
         descs = (N.LayerDescC * cfg.L)()
         for t, layer in zip(descs, cfg.layers):
             m, x = layer.mixer, layer.experts
-            t.mixer, t.heads, t.dim, t.rot_dim, t.vdim, t.kv_rank = 0, m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank
-            t.rot_dims, t.kv_from, t.scale, t.rot_base = m.rot_dims, m.kv_from, m.scale, m.rot_base
+            t.heads, t.dim, t.vdim, t.kv_from = m.heads, m.dim, m.vdim, -1
+            if isinstance(m, LatentAttention):
+                t.mixer, t.rot_dim, t.kv_rank = N.MIXER_LATENT, m.rot_dim, m.kv_rank
+                t.rot_dims, t.kv_from, t.scale, t.rot_base = m.rot_dims, m.kv_from, m.scale, m.rot_base
+            elif isinstance(m, GroupedAttention):
+                t.mixer, t.kv_heads, t.scale, t.kv_from = N.MIXER_GROUPED, m.kv_heads, m.scale, m.kv_from
+                t.window, t.keep_first, t.bias_rows, t.bias_max = m.window, m.keep_first, m.bias_rows, m.bias_max
+                t.flags = (N.ATTN_QK_NORM * m.qk_norm) | (N.ATTN_QKV_BIAS * m.qkv_bias) | (N.ATTN_SINK * m.sink) | (N.ATTN_HEAD_GATE * m.head_gate)
+            else:
+                t.mixer, t.gate_cap = N.MIXER_MEMORY, m.gate_cap
             if x is not None:
                 t.experts, t.top, t.ff = x.experts, x.top, x.ff
                 t.glu_limit, t.glu_slope, t.glu_shift = x.limit, x.slope, x.shift
+            elif layer.dense is not None:
+                t.ff = layer.dense.ff
         self._h = C.c_void_p()
         N.call("TSB200_GptCreateLayered", C.byref(c), descs, C.byref(self._h))
 
@@ -144,7 +228,7 @@ class LayeredGPT(GPT):
 
 
 def synthetic_layered_weights(cfg: LayeredConfig, seed: int, std: float = 0.02, bias_std: float = 0.0):
-    """Seeded weights by engine name (float32 values that bfloat16 holds exactly): matrices N(0, std), norm gains 1, biases N(0, bias_std)."""
+    """Seeded weights by engine name (float32 values that bfloat16 holds exactly): matrices N(0, std), norm gains and scales 1, biases N(0, bias_std)."""
     from .safetensors_file import to_bfloat16, to_float32
     rng = np.random.default_rng(seed)
     out = {}
@@ -153,7 +237,7 @@ def synthetic_layered_weights(cfg: LayeredConfig, seed: int, std: float = 0.02, 
             x = cfg.layers[int(name.split(".")[1])].experts
             out[name] = np.stack([rng.permutation(x.experts)[:x.top] for _ in range(shape[0])]).astype(np.int32)
             continue
-        if name == "final_norm" or name.endswith(("norm1", "norm2", "dkv_norm")):
+        if "norm" in name or ".scale" in name:
             w = np.ones(shape, dtype=np.float32)
         elif name.endswith(".b"):
             w = synth(name, shape, seed, bias_std) if bias_std > 0 else np.zeros(shape, dtype=np.float32)

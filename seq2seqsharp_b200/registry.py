@@ -6,23 +6,28 @@ reference's protobuf model file (model_file.py).  `load_model` is what the comma
 import json
 import os
 from dataclasses import dataclass
-from typing import Callable, Dict
+from typing import Callable, Dict, Mapping
 
-from . import pepilix
+from . import gunuvik, pepilix
 from .layered import LayeredConfig, LayeredGPT
 from .safetensors_file import SafetensorsFile
 
 
 @dataclass
 class Architecture:
-    config: Callable[[dict, str], LayeredConfig]     # (config.json, dtype) -> configuration
-    tensor_name: Callable[[str], str]                # tensor name in the file -> engine name
+    config: Callable[[dict, str, Mapping], LayeredConfig]     # (config.json, dtype, tensor shapes of the file) -> configuration
+    tensor_name: Callable[[str, LayeredConfig], str]          # tensor name in the file -> engine name
     dtypes: tuple = ("bfloat16", "float32")
 
 
 ARCHITECTURES: Dict[str, Architecture] = {
-    pepilix.ARCHITECTURE: Architecture(pepilix.config_from_json, pepilix.engine_name),
+    pepilix.ARCHITECTURE: Architecture(lambda j, dtype, shapes: pepilix.config_from_json(j, dtype), lambda n, cfg: pepilix.engine_name(n)),
+    gunuvik.ARCHITECTURE: Architecture(gunuvik.config_from_json, gunuvik.engine_name),
 }
+
+
+def weights_file(path: str) -> SafetensorsFile:
+    return SafetensorsFile(os.path.join(path, "model.safetensors"))
 
 
 def read_config(path: str, dtype: str = "bfloat16"):
@@ -35,15 +40,16 @@ def read_config(path: str, dtype: str = "bfloat16"):
     arch = ARCHITECTURES[name]
     if dtype not in arch.dtypes:
         raise ValueError("%s models are not served in %s" % (name, dtype))
-    return arch, arch.config(j, dtype)
+    tensors = weights_file(path)
+    return arch, arch.config(j, dtype, {n: tensors.shape(n) for n in tensors.names()})
 
 
 def load_model(path: str, dtype: str = "bfloat16", device_id: int = 0, max_batch: int = 1, max_tokens: int = 512):
     """An engine with the model's weights, ready to run."""
     if os.path.isdir(path):
         arch, cfg = read_config(path, dtype)
-        tensors = SafetensorsFile(os.path.join(path, "model.safetensors"))
-        names = {arch.tensor_name(n): n for n in tensors.names()}
+        tensors = weights_file(path)
+        names = {arch.tensor_name(n, cfg): n for n in tensors.names()}
         missing = sorted(set(cfg.weight_shapes()) - set(names))
         if missing:
             raise ValueError("%s: %d tensors are missing, the first is %s" % (tensors.path, len(missing), missing[0]))

@@ -71,6 +71,6 @@ def test_config_struct_layout_matches_header():
     # field order/size of the ctypes mirrors = the C structs (all 4-byte fields, no padding until the pointers)
     assert C.sizeof(N.GptConfig) == 24 * 4
     assert C.sizeof(N.Tensor) == 8 + 4 + 4 + 32 + 32
-    assert C.sizeof(N.LayeredConfigC) == 12 * 4
-    assert C.sizeof(N.LayerDescC) == 9 * 4 + 4 + 8 + 6 * 4 and N.LayerDescC.rot_base.offset == 40   # the double is 8-byte aligned
+    assert C.sizeof(N.LayeredConfigC) == 14 * 4
+    assert C.sizeof(N.LayerDescC) == 9 * 4 + 4 + 8 + 14 * 4 and N.LayerDescC.rot_base.offset == 40   # the double is 8-byte aligned
     assert N.DecodingOptionsC.blocked.offset == 16 and N.DecodingOptionsC.seed.offset == 32

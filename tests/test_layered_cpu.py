@@ -243,6 +243,7 @@ def _create(cfg_edit=None, layer_edit=None, n=2):
     c = N.LayeredConfigC()
     c.L, c.d, c.V, c.dtype, c.norm_groups, c.conv_taps, c.max_batch, c.max_tokens = n, 32, 50, N.F32, 2, 2, 1, 16
     c.eps = c.embed_scale = c.logit_scale = 1.0
+    c.tied_head = 1
     ls = (N.LayerDescC * n)()
     for t in ls:
         t.heads, t.dim, t.rot_dim, t.rot_dims, t.vdim, t.kv_rank, t.kv_from, t.scale, t.rot_base = 2, 8, 4, 4, 8, 16, -1, 1.0, 100.0
