@@ -15,7 +15,7 @@ Workloads (synthetic seeded weights and prompts of the named shapes; no dataset 
     c4_b4   the same 1B-class model, B=4, 16384-token prompts, greedy (long-context KV-cache stress)
     c1      tiny fp32 model, B=1, prompt 32, greedy
 
-`--design pepilix` measures prefill and decode of a layered design at a few sizes beside the closest uniform model instead (one GPU).
+`--design pepilix` or `--design gunuvik` measures prefill and decode of a layered design at a few sizes beside the closest uniform model instead (one GPU).
 
 With N > 1 the 7B-class workloads (c5_*) run ONE model tensor-parallel over the N GPUs (strong scaling: `value` is the
 tokens/s of the one sharded model); the other workloads run N batch-sharded replicas (weak scaling).  `--parallelism`
@@ -642,37 +642,60 @@ def run_b200(args):
 
 
 # ---- layered designs beside the closest uniform model ---------------------------------------------------------------------------
-# sizes that resemble the layers of real models; every entry: layers, width, heads, unrotated / rotated / value head size, latent,
-# experts, experts per token, expert width.  The closest existing model of equal size: GPTDecoder with grouped-query attention, RoPE,
-# RMSNorm and a dense gated feed-forward as wide as the experts a token uses, fp16.
+# sizes that resemble the layers of real models.  The closest existing model of equal size: GPTDecoder with grouped-query attention, RoPE,
+# RMSNorm and a dense gated feed-forward, fp16.
+# pepilix: layers, width, heads, unrotated / rotated / value head size, latent, experts, experts per token, expert width (the uniform model's
+# feed-forward is as wide as the experts a token uses).
+# gunuvik: layers, width, heads, key/value heads, head size, feed-forward; window, kept first tokens, distance bias rows and range; heads, key
+# and value size of the memories.  Every fourth layer is a memory, the layer after it reads an earlier layer's cache.
 DESIGN_SIZES = {
-    "1k": dict(L=12, d=1024, H=16, dim=64, rot=32, vdim=64, rank=256, E=16, top=2, ff=1024),
-    "2k": dict(L=12, d=2048, H=16, dim=128, rot=64, vdim=128, rank=512, E=32, top=4, ff=1408),
-    "4k": dict(L=6, d=4096, H=32, dim=128, rot=64, vdim=128, rank=512, E=16, top=2, ff=4096),
+    "pepilix": {
+        "1k": dict(L=12, d=1024, H=16, dim=64, rot=32, vdim=64, rank=256, E=16, top=2, ff=1024),
+        "2k": dict(L=12, d=2048, H=16, dim=128, rot=64, vdim=128, rank=512, E=32, top=4, ff=1408),
+        "4k": dict(L=6, d=4096, H=32, dim=128, rot=64, vdim=128, rank=512, E=16, top=2, ff=4096),
+    },
+    "gunuvik": {
+        "1k": dict(L=12, d=1024, H=16, G=4, hd=64, ff=2816, window=1024, keep=4, rows=32, far=128, mH=4, mdim=128, mvdim=256),
+        "2k": dict(L=12, d=2048, H=16, G=4, hd=128, ff=5632, window=1024, keep=4, rows=32, far=128, mH=8, mdim=128, mvdim=256),
+        "4k": dict(L=8, d=4096, H=32, G=8, hd=128, ff=11008, window=2048, keep=4, rows=32, far=128, mH=8, mdim=256, mvdim=512),
+    },
 }
 DESIGN_V = 32000
 
 
-def design_models(z, local, max_batch, max_tokens):
+def design_models(design, z, local, max_batch, max_tokens):
     """(layered model, closest uniform model), random weights."""
     from seq2seqsharp_b200.gpt import (ActivateFuncEnums as A, GPT, GPTConfig, MultiHeadAttentionTypeEnums as MA, NormEnums as Nm,
                                        PositionEmbeddingEnums as PE)
-    from seq2seqsharp_b200.layered import BlockLayer, LatentAttention, LayeredConfig, LayeredGPT, TableExperts
-    from seq2seqsharp_b200.pepilix import EXPERT_SHIFT, EXPERT_SLOPE
-    ex = TableExperts(experts=z["E"], top=z["top"], ff=z["ff"], limit=7.0, slope=EXPERT_SLOPE, shift=EXPERT_SHIFT)
-    at = dict(heads=z["H"], dim=z["dim"], rot_dim=z["rot"], vdim=z["vdim"], kv_rank=z["rank"], rot_base=1e6, scale=(z["dim"] + z["rot"]) ** -0.5)
-    lay = LayeredConfig(d=z["d"], V=DESIGN_V, norm_groups=8, conv_taps=4, embed_scale=z["d"] ** 0.5,
-                        layers=[BlockLayer(LatentAttention(**at), ex) for _ in range(z["L"])])
-    uni = GPTConfig(L=z["L"], d=z["d"], H=z["H"], Hkv=max(1, z["H"] // 4), hd=z["vdim"], F=z["top"] * z["ff"], V=DESIGN_V, norm=Nm.RMSNorm, act=A.SwiGLU_SiLU,
-                    pe=PE.RoPE, attn=MA.GQA, dtype="float16")
+    from seq2seqsharp_b200.layered import BlockLayer, DenseGated, GroupedAttention, LatentAttention, LayeredConfig, LayeredGPT, MatrixMemory, TableExperts
+    if design == "pepilix":
+        from seq2seqsharp_b200.pepilix import EXPERT_SHIFT, EXPERT_SLOPE
+        ex = TableExperts(experts=z["E"], top=z["top"], ff=z["ff"], limit=7.0, slope=EXPERT_SLOPE, shift=EXPERT_SHIFT)
+        at = dict(heads=z["H"], dim=z["dim"], rot_dim=z["rot"], vdim=z["vdim"], kv_rank=z["rank"], rot_base=1e6, scale=(z["dim"] + z["rot"]) ** -0.5)
+        lay = LayeredConfig(d=z["d"], V=DESIGN_V, norm_groups=8, conv_taps=4, embed_scale=z["d"] ** 0.5,
+                            layers=[BlockLayer(LatentAttention(**at), ex) for _ in range(z["L"])])
+        G, hd, F = max(1, z["H"] // 4), z["vdim"], z["top"] * z["ff"]
+    else:
+        G, hd, F = z["G"], z["hd"], z["ff"]
+        at = dict(heads=z["H"], kv_heads=G, dim=hd, vdim=hd, scale=hd ** -0.5, window=z["window"], keep_first=z["keep"], bias_rows=z["rows"], bias_max=z["far"],
+                  qk_norm=True, qkv_bias=True, sink=True, head_gate=True)
+        lay = LayeredConfig(d=z["d"], V=DESIGN_V, block="sandwich", embed_scale=z["d"] ** 0.5, tied_head=False,
+                            layers=[BlockLayer(MatrixMemory(z["mH"], z["mdim"], z["mvdim"], 15.0) if i % 4 == 2 else GroupedAttention(**at, kv_from=i - 2 if i % 4 == 3 else -1),
+                                               dense=DenseGated(F)) for i in range(z["L"])])
+    uni = GPTConfig(L=z["L"], d=z["d"], H=z["H"], Hkv=G, hd=hd, F=F, V=DESIGN_V, norm=Nm.RMSNorm, act=A.SwiGLU_SiLU, pe=PE.RoPE, attn=MA.GQA, dtype="float16")
     return (lambda: LayeredGPT(lay, device_id=local, max_batch=max_batch, max_tokens=max_tokens),
             lambda: GPT(uni, device_id=local, max_batch=max_batch, max_tokens=max_tokens), lay, uni)
 
 
-def design_costs(z, which, B, S, T):
+def design_costs(design, z, which, B, S, T):
     """Algorithmic (bytes of a decode step at context T with B sequences, flops of a prefill of B x S) per kernel class."""
     L, d, H, V = z["L"], z["d"], z["H"], DESIGN_V
-    if which == "layered":
+    if which == "uniform":
+        hd, kv, F = (z["vdim"], max(1, H // 4), z["top"] * z["ff"]) if design == "pepilix" else (z["hd"], z["G"], z["ff"])
+        proj = d * (H + 2 * kv) * hd + H * hd * d + 3 * d * F
+        by = {"linear": 2.0 * (L * proj + d * V), "attention": 2.0 * L * B * T * 2 * kv * hd}
+        fl = {"linear": 2.0 * B * S * L * proj + 2.0 * B * d * V, "attention": L * 4.0 * B * H * hd * S * S / 2.0}
+    elif design == "pepilix":
         proj = 2 * d * d + d * (H * (z["dim"] + z["rot"]) + z["rank"] + z["rot"]) + H * z["vdim"] * d
         lat = H * (z["dim"] + z["vdim"]) * z["rank"]
         seen = z["E"] * (1.0 - (1.0 - z["top"] / z["E"]) ** B)       # experts that B tokens use, on average
@@ -681,10 +704,16 @@ def design_costs(z, which, B, S, T):
         fl = {"linear": 2.0 * B * S * L * proj + 2.0 * B * d * V, "experts": 2.0 * B * S * L * 3 * d * z["ff"] * z["top"],
               "attention": L * (2.0 * B * S * lat + 2.0 * B * H * (z["dim"] + z["rot"] + z["vdim"]) * S * S / 2.0)}
     else:
-        hd, kv = z["vdim"], max(1, H // 4)
-        proj = d * (H + 2 * kv) * hd + H * hd * d + 3 * d * z["top"] * z["ff"]
-        by = {"linear": 2.0 * (L * proj + d * V), "attention": 2.0 * L * B * T * 2 * kv * hd}
-        fl = {"linear": 2.0 * B * S * L * proj + 2.0 * B * d * V, "attention": L * 4.0 * B * H * hd * S * S / 2.0}
+        hd, G, span = z["hd"], z["G"], z["window"] + z["keep"]
+        n_mem = sum(i % 4 == 2 for i in range(L))
+        n_att, n_own = L - n_mem, sum(i % 4 < 2 for i in range(L))
+        mqk, mv = z["mH"] * z["mdim"], z["mH"] * z["mvdim"]
+        proj = n_att * (d * H * hd + d * H + H * hd * d) + n_own * 2 * d * G * hd + n_mem * (d * (2 * mqk + 2 * mv + 2 * z["mH"]) + mv * d) + L * 3 * d * z["ff"]
+        pairs = sum(min(i + 1, span) for i in range(S))              # (query, key) pairs of a prompt
+        by = {"linear": 2.0 * (proj + d * V), "attention": 2.0 * n_att * B * min(T, span) * 2 * G * hd,
+              "memory": 2.0 * 4.0 * n_mem * B * z["mH"] * z["mdim"] * (z["mvdim"] + 1)}
+        fl = {"linear": 2.0 * B * S * proj + 2.0 * B * d * V, "attention": n_att * 4.0 * B * H * hd * pairs,
+              "memory": n_mem * 4.0 * B * S * z["mH"] * z["mdim"] * z["mvdim"]}
     return by, fl
 
 
@@ -705,13 +734,13 @@ def run_design(args):
     sampler = ClockSampler(local)
     sampler.start()
     for name in args.design_sizes.split(","):
-        z = DESIGN_SIZES[name]
+        z = DESIGN_SIZES[args.design][name]
         res = {}
         for which in ("layered", "uniform"):
             r = {}
             for B, S in ((1, 1024), (8, 1024), (64, 512)):
                 max_tokens = S + W + K + 24
-                lay, uni, _, _ = design_models(z, local, B, max_tokens)
+                lay, uni, _, _ = design_models(args.design, z, local, B, max_tokens)
                 g = (lay if which == "layered" else uni)()
                 g.FillSynthetic(SEED, 0.02, 0.0)
                 opts = make_options("greedy", 1.0, max_tokens, SEED, 0)
@@ -722,14 +751,14 @@ def run_design(args):
                 ms, _ = g.LastTiming()
                 T = S + W + K // 2
                 prof = g.ProfileDecode(8, opts)
-                by, _ = design_costs(z, which, B, S, T)
+                by, _ = design_costs(args.design, z, which, B, S, T)
                 r["decode_B%d_T%d" % (B, T)] = {
                     "tokens_per_s": B * K / (ms / 1e3), "ms_per_step": ms / K, "launches_per_step": sum(v[1] for v in prof.values()) // 8,
                     "classes": {k: {"ms": v[0] / 8, **({"gbs": by[k] / 1e6 / (v[0] / 8), "frac_of_hbm_peak": by[k] / 1e6 / (v[0] / 8) / hbm} if k in by else {})}
                                 for k, v in prof.items() if v[1]}}
                 g.close()
             for B, S in ((1, 2048), (4, 2048)):
-                lay, uni, _, _ = design_models(z, local, B, S + 8)
+                lay, uni, _, _ = design_models(args.design, z, local, B, S + 8)
                 g = (lay if which == "layered" else uni)()
                 g.FillSynthetic(SEED, 0.02, 0.0)
                 opts = make_options("greedy", 1.0, S + 8, SEED, 0)
@@ -742,7 +771,7 @@ def run_design(args):
                 ms = statistics.median(times[W:])
                 g.Reset()
                 prof = g.ProfilePrefill(ids, opts)
-                _, fl = design_costs(z, which, B, S, 0)
+                _, fl = design_costs(args.design, z, which, B, S, 0)
                 r["prefill_B%d_S%d" % (B, S)] = {
                     "tokens_per_s": B * S / (ms / 1e3), "ms": ms, "tflops": sum(fl.values()) / 1e9 / ms, "frac_of_tensor_peak": sum(fl.values()) / 1e9 / ms / burst,
                     "classes": {k: {"ms": v[0], **({"tflops": fl[k] / 1e9 / v[0], "frac_of_tensor_peak": fl[k] / 1e9 / v[0] / burst} if k in fl else {})}
@@ -762,7 +791,7 @@ def main():
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--workload", default="c5_b1", choices=sorted(WORKLOADS))
-    ap.add_argument("--design", default="", choices=["", "pepilix"],
+    ap.add_argument("--design", default="", choices=["", *sorted(DESIGN_SIZES)],
                     help="instead of a workload: prefill and decode throughput of a layered design at a few sizes beside the closest uniform model")
     ap.add_argument("--design-sizes", default="1k,2k,4k")
     ap.add_argument("--no-cpu-baseline", action="store_true")
