@@ -83,11 +83,12 @@ __global__ void __launch_bounds__(256) head_prep_kernel(GroupedArgs a) {
   const GroupedShape& sh = a.shape;
   const int lane = threadIdx.x & 31;
   const int units = sh.H + (a.k_col >= 0 ? 2 * sh.G : 0);
-  const int64_t n_all = (int64_t)a.B * a.S * units;
-  for (int64_t w = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5); w < n_all; w += (int64_t)gridDim.x * 8) {
-    const int u = (int)(w % units);
-    const int64_t row = w / units;
-    const int b = (int)(row / a.S), pos = state_len(a.state, b, a.T0) + (int)(row % a.S);
+  const unsigned n_all = (unsigned)(a.B * a.S) * (unsigned)units;
+  for (unsigned w = blockIdx.x * 8 + (threadIdx.x >> 5); w < n_all; w += gridDim.x * 8) {
+    const unsigned r = w / (unsigned)units;
+    const int u = (int)(w - r * (unsigned)units);
+    const int64_t row = r;
+    const int b = (int)(r / (unsigned)a.S), pos = state_len(a.state, b, a.T0) + (int)(r % (unsigned)a.S);
     TSB_DEV_CHECK(grouped, pos >= 0 && pos < a.Tmax, 0x601, (void)0)   // append position outside the cache (row skipped)
     const T* src = reinterpret_cast<const T*>(a.qkv) + row * a.q_stride;
     const T* wt = nullptr;
@@ -109,6 +110,31 @@ __global__ void __launch_bounds__(256) head_prep_kernel(GroupedArgs a) {
         src += a.v_col + (int64_t)g * sh.vdim;
         dst = reinterpret_cast<T*>(a.cV) + (((int64_t)b * sh.G + g) * a.Tmax + pos) * sh.dv;
       }
+    }
+    if (n <= 32 * V) {   // the row in registers
+      float v[V], g[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        v[e] = 0.0f;
+        g[e] = 1.0f;
+      }
+      const int i = lane * V;
+      if (i < n) {
+        HeadVec<T, V>::load(src + i, v);
+        if (wt) HeadVec<T, V>::load(wt + i, g);
+      }
+      if (wt) {
+        float s = 0.0f;
+#pragma unroll
+        for (int e = 0; e < V; ++e) s += v[e] * v[e];
+        const float inv = 1.0f / sqrtf(warp_sum(s) / (float)n + sh.eps);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = v[e] * inv * g[e];
+      }
+      if (i < n) HeadVec<T, V>::store(dst + i, v);
+      if (u < sh.H)
+        for (int e = n + lane; e < sh.dk; e += 32) dst[e] = from_f<T>(0.0f);
+      continue;
     }
     float inv = 1.0f;
     if (wt) {
@@ -255,10 +281,12 @@ __global__ void __launch_bounds__(kGaThreads) grouped_prefill_kernel(GroupedArgs
   for (int i = 0; i < kGaStages - 1; ++i) issue(i);
   ga_zero_pads<D>(smem, kGaStages, sh.dk, sh.dv);
 
-  // this lane's two rows, (query, head) pairs
+  // this lane's two rows, (query, head) pairs; scores, maxima and bias in powers of two
   int pos[2], head[2];
   bool live[2];
   const float* bias[2];
+  float far_bias[2];   // of every distance from n_bias - 1 on
+  const float bias_unit = bias_in_smem ? 1.0f : kLog2e, scale = sh.scale * kLog2e;
   float* s_bias = reinterpret_cast<float*>(smem + kGaStages * GaTile<D>::stage);
   uint32_t qa[KS][4];
 #pragma unroll
@@ -268,6 +296,7 @@ __global__ void __launch_bounds__(kGaThreads) grouped_prefill_kernel(GroupedArgs
     pos[r] = T0 + q0 + (live[r] ? qi : 0);
     head[r] = kvh * group + (live[r] ? gh : gh0);
     bias[r] = bias_in_smem ? s_bias + (live[r] ? rr % hp : 0) * sh.n_bias : a.bias + (int64_t)head[r] * sh.n_bias;
+    far_bias[r] = sh.n_bias > 0 ? a.bias[(int64_t)head[r] * sh.n_bias + sh.n_bias - 1] * kLog2e : 0.0f;
     const bf16* qp = reinterpret_cast<const bf16*>(a.qn) + (((int64_t)b * a.S + pos[r] - T0) * sh.H + head[r]) * sh.dk + 2 * t4;
 #pragma unroll
     for (int ks = 0; ks < KS; ++ks) {
@@ -276,14 +305,14 @@ __global__ void __launch_bounds__(kGaThreads) grouped_prefill_kernel(GroupedArgs
     }
   }
   if (bias_in_smem)
-    for (int i = threadIdx.x; i < min(hp, group - gh0) * sh.n_bias; i += kGaThreads) s_bias[i] = a.bias[(int64_t)(kvh * group + gh0) * sh.n_bias + i];
+    for (int i = threadIdx.x; i < min(hp, group - gh0) * sh.n_bias; i += kGaThreads) s_bias[i] = a.bias[(int64_t)(kvh * group + gh0) * sh.n_bias + i] * kLog2e;
   // this warp's range of query positions
   const int wq0 = (w * 16) / hp, wq1 = min((w * 16 + 15) / hp, n_q - 1);
   const int wp0 = T0 + q0 + wq0, wp1 = T0 + q0 + wq1;
   float m[2], l[2], o[NBO][4];
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
-    m[r] = a.sink ? a.sink[head[r]] : -INFINITY;
+    m[r] = a.sink ? a.sink[head[r]] * kLog2e : -INFINITY;
     l[r] = a.sink && t4 == 0 ? 1.0f : 0.0f;   // the quad's parts are added at the end
   }
 #pragma unroll
@@ -297,16 +326,16 @@ __global__ void __launch_bounds__(kGaThreads) grouped_prefill_kernel(GroupedArgs
     __syncthreads();
     const uint32_t kb = s0 + (uint32_t)(tile % kGaStages) * GaTile<D>::stage, vb = kb + GaTile<D>::plane;
 #pragma unroll 1
-    for (int sl = 0; sl < kGaKeys / 16; ++sl) {
-      const int u0 = tile * kGaKeys + sl * 16;
+    for (int sl = 0; sl < kGaKeys / 32; ++sl) {
+      const int u0 = tile * kGaKeys + sl * 32;
       if (u0 >= keys.n || wq0 >= n_q) break;
-      const int ja = keys.at(u0), jb = keys.at(min(u0 + 15, keys.n - 1));
+      const int ja = keys.at(u0), jb = keys.at(min(u0 + 31, keys.n - 1));
       if (ja > wp1) break;   // later keys are later positions: nothing more for this warp
       if (sh.window > 0 && ja >= sh.keep_first && jb <= wp0 - sh.window) continue;
-      const int tw = sl * 16;
-      float sc[2][4];
+      const int tw = sl * 32;
+      float sc[4][4];
 #pragma unroll
-      for (int nb = 0; nb < 2; ++nb) {
+      for (int nb = 0; nb < 4; ++nb) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) sc[nb][e] = 0.0f;
         const uint32_t ka = kb + (tw + nb * 8 + (lane & 7)) * PITCH + (lane >> 3) * 16;
@@ -318,55 +347,69 @@ __global__ void __launch_bounds__(kGaThreads) grouped_prefill_kernel(GroupedArgs
           la_mma(sc[nb], qa[2 * kp + 1][0], qa[2 * kp + 1][1], qa[2 * kp + 1][2], qa[2 * kp + 1][3], b2, b3);
         }
       }
-      // row r: elements 2r, 2r + 1 of both blocks; keys nb * 8 + 2 * t4 + e
-      float mx[2] = {-INFINITY, -INFINITY};
+      // row r: elements 2r, 2r + 1 of every block; keys nb * 8 + 2 * t4 + e
+      const bool all_seen = u0 + 31 < keys.n && jb <= wp0 && (sh.window <= 0 || wp1 - ja < sh.window || jb < sh.keep_first);
+      if (all_seen && wp0 - jb >= sh.n_bias - 1) {   // (most slices) nothing to mask, one bias for all distances
 #pragma unroll
-      for (int nb = 0; nb < 2; ++nb)
+        for (int nb = 0; nb < 4; ++nb)
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int u = u0 + nb * 8 + 2 * t4 + e, j = keys.at(u);
+          for (int e = 0; e < 4; ++e) sc[nb][e] = fmaf(sc[nb][e], scale, far_bias[e >> 1]);
+      } else {
 #pragma unroll
-          for (int r = 0; r < 2; ++r) {
-            const bool vis = live[r] && u < keys.n && key_visible(sh, pos[r], j);
-            float z = sc[nb][2 * r + e] * sh.scale;
-            if (sh.n_bias > 0) z += bias[r][min(max(pos[r] - j, 0), sh.n_bias - 1)];
-            sc[nb][2 * r + e] = vis ? z : -INFINITY;
-            mx[r] = fmaxf(mx[r], sc[nb][2 * r + e]);
-          }
-        }
-      float corr[2];
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
-        mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
-        const float mn = fmaxf(m[r], mx[r]);
-        const bool none = mn == -INFINITY;   // the row has seen nothing yet: keep its state (no exp(-inf - -inf))
-        corr[r] = none ? 1.0f : __expf(m[r] - mn);
-        float s = 0.0f;
-#pragma unroll
-        for (int nb = 0; nb < 2; ++nb)
+        for (int nb = 0; nb < 4; ++nb)
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
-            sc[nb][2 * r + e] = none ? 0.0f : __expf(sc[nb][2 * r + e] - mn);
+            const int u = u0 + nb * 8 + 2 * t4 + e, j = keys.at(u);
+#pragma unroll
+            for (int r = 0; r < 2; ++r) {
+              const bool vis = live[r] && u < keys.n && key_visible(sh, pos[r], j);
+              float z = sc[nb][2 * r + e] * scale;
+              if (sh.n_bias > 0) z += bias[r][min(max(pos[r] - j, 0), sh.n_bias - 1)] * bias_unit;
+              sc[nb][2 * r + e] = vis ? z : -INFINITY;
+            }
+          }
+      }
+      float corr[2];
+      bool moved = false;
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        float mx = -INFINITY;
+#pragma unroll
+        for (int nb = 0; nb < 4; ++nb) mx = fmaxf(mx, fmaxf(sc[nb][2 * r], sc[nb][2 * r + 1]));
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+        const float mn = fmaxf(m[r], mx), base = mn == -INFINITY ? 0.0f : mn;   // a row that has seen nothing yet: all weights 0
+        corr[r] = exp2_fast(m[r] - base);
+        moved = moved || mn != m[r];
+        float s = 0.0f;
+#pragma unroll
+        for (int nb = 0; nb < 4; ++nb)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            sc[nb][2 * r + e] = exp2_fast(sc[nb][2 * r + e] - base);
             s += sc[nb][2 * r + e];
           }
         l[r] = l[r] * corr[r] + s;
         m[r] = mn;
       }
-      const uint32_t pa0 = Pair16<bf16>::put(sc[0][0], sc[0][1]), pa1 = Pair16<bf16>::put(sc[0][2], sc[0][3]);
-      const uint32_t pa2 = Pair16<bf16>::put(sc[1][0], sc[1][1]), pa3 = Pair16<bf16>::put(sc[1][2], sc[1][3]);
-      const uint32_t va = vb + (tw + (lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + (lane >> 4) * 16;
+      if (__any_sync(0xffffffffu, moved)) {
 #pragma unroll
-      for (int np = 0; np < NBO / 2; ++np) {
-        uint32_t b0, b1, b2, b3;
-        la_ldsm_x4_trans(va + np * 32, b0, b1, b2, b3);
+        for (int nb = 0; nb < NBO; ++nb)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          o[2 * np][e] *= corr[e >> 1];
-          o[2 * np + 1][e] *= corr[e >> 1];
+          for (int e = 0; e < 4; ++e) o[nb][e] *= corr[e >> 1];
+      }
+#pragma unroll
+      for (int hh = 0; hh < 2; ++hh) {
+        const uint32_t pa0 = Pair16<bf16>::put(sc[2 * hh][0], sc[2 * hh][1]), pa1 = Pair16<bf16>::put(sc[2 * hh][2], sc[2 * hh][3]);
+        const uint32_t pa2 = Pair16<bf16>::put(sc[2 * hh + 1][0], sc[2 * hh + 1][1]), pa3 = Pair16<bf16>::put(sc[2 * hh + 1][2], sc[2 * hh + 1][3]);
+        const uint32_t va = vb + (tw + hh * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + (lane >> 4) * 16;
+#pragma unroll
+        for (int np = 0; np < NBO / 2; ++np) {
+          uint32_t b0, b1, b2, b3;
+          la_ldsm_x4_trans(va + np * 32, b0, b1, b2, b3);
+          la_mma(o[2 * np], pa0, pa1, pa2, pa3, b0, b1);
+          la_mma(o[2 * np + 1], pa0, pa1, pa2, pa3, b2, b3);
         }
-        la_mma(o[2 * np], pa0, pa1, pa2, pa3, b0, b1);
-        la_mma(o[2 * np + 1], pa0, pa1, pa2, pa3, b2, b3);
       }
     }
     __syncthreads();   // the stage is overwritten by the copy issued in the next iteration
@@ -436,29 +479,45 @@ __global__ void __launch_bounds__(kGaThreads) grouped_decode_kernel(GroupedArgs 
   unsigned char* s_q = smem + kGaStages * GaTile<D>::stage;
   bf16* s_new = reinterpret_cast<bf16*>(s_q + ROWS * PITCH);   // [2][D]
   const bf16* row = reinterpret_cast<const bf16*>(a.qkv) + (int64_t)b * a.q_stride;
-  for (int r = w; r < ROWS + (fresh ? 2 : 0); r += kGaThreads / 32) {
-    const bool is_q = r < ROWS, is_k = r == ROWS;
-    const int n = is_q || is_k ? sh.dim : sh.vdim, n_pad = is_q ? D : (is_k ? sh.dk : sh.dv);
-    const bf16* src = is_q ? row + (int64_t)(h0 + min(r, nh - 1)) * sh.dim : (is_k ? row + a.k_col + kvh * sh.dim : row + a.v_col + kvh * sh.vdim);
-    const bf16* wt = reinterpret_cast<const bf16*>(is_q ? a.q_norm : (is_k ? a.k_norm : nullptr));
-    bf16* dst = is_q ? reinterpret_cast<bf16*>(s_q + r * PITCH) : s_new + (is_k ? 0 : D);
-    float v[D / 32], g[D / 32], s = 0.0f;
+  for (int i = tid; i < (ROWS - nh) * (PITCH / 16); i += kGaThreads)   // rows without a head
+    reinterpret_cast<uint4*>(s_q + (nh + i / (PITCH / 16)) * PITCH)[i % (PITCH / 16)] = make_uint4(0u, 0u, 0u, 0u);
+  const int n_items = nh + (fresh ? 2 : 0);   // query heads, the key row, the value row
+  for (int i0 = w; i0 < n_items; i0 += 2 * (kGaThreads / 32)) {
+    float v[2][D / 32], g[2][D / 32];
 #pragma unroll
-    for (int i = 0; i < D / 32; ++i) {
-      const int e = lane + i * 32;
-      v[i] = e < n ? to_f<bf16>(src[e]) : 0.0f;
-      g[i] = wt && e < n ? to_f<bf16>(wt[e]) : 1.0f;
-      s += v[i] * v[i];
+    for (int q = 0; q < 2; ++q) {   // two rows requested at a time
+      const int it = i0 + q * (kGaThreads / 32);
+      const bool is_v = it == nh + 1, is_k = it == nh;
+      const int n = it >= n_items ? 0 : (is_v ? sh.vdim : sh.dim);
+      const bf16* src = row + (is_v ? a.v_col + kvh * sh.vdim : (is_k ? a.k_col + kvh * sh.dim : (h0 + min(it, nh - 1)) * sh.dim));
+      const bf16* wt = reinterpret_cast<const bf16*>(is_v ? nullptr : (is_k ? a.k_norm : a.q_norm));
+#pragma unroll
+      for (int i = 0; i < D / 32; ++i) {
+        const int e = lane + i * 32;
+        v[q][i] = e < n ? to_f<bf16>(src[e]) : 0.0f;
+        g[q][i] = wt && e < n ? to_f<bf16>(wt[e]) : 1.0f;
+      }
     }
-    const float inv = wt ? 1.0f / sqrtf(warp_sum(s) / (float)n + sh.eps) : 1.0f;
-    bf16* cache = is_q || chunk != 0 ? nullptr : (is_k ? Kb + (int64_t)p * sh.dk : Vb + (int64_t)p * sh.dv);
 #pragma unroll
-    for (int i = 0; i < D / 32; ++i) {
-      const int e = lane + i * 32;
-      if (e >= n_pad) continue;
-      const bf16 t = from_f<bf16>(is_q && r >= nh ? 0.0f : v[i] * inv * g[i]);
-      dst[e] = t;
-      if (cache && e < n) cache[e] = t;
+    for (int q = 0; q < 2; ++q) {
+      const int it = i0 + q * (kGaThreads / 32);
+      if (it >= n_items) break;
+      const bool is_v = it == nh + 1, is_k = it == nh;
+      const int n = is_v ? sh.vdim : sh.dim, n_pad = is_v ? sh.dv : (is_k ? sh.dk : D);
+      float s = 0.0f;
+#pragma unroll
+      for (int i = 0; i < D / 32; ++i) s += v[q][i] * v[q][i];
+      const float inv = !is_v && (is_k ? a.k_norm : a.q_norm) ? 1.0f / sqrtf(warp_sum(s) / (float)n + sh.eps) : 1.0f;
+      bf16* dst = is_v ? s_new + D : (is_k ? s_new : reinterpret_cast<bf16*>(s_q + it * PITCH));
+      bf16* cache = chunk != 0 || it < nh ? nullptr : (is_k ? Kb + (int64_t)p * sh.dk : Vb + (int64_t)p * sh.dv);
+#pragma unroll
+      for (int i = 0; i < D / 32; ++i) {
+        const int e = lane + i * 32;
+        if (e >= n_pad) continue;
+        const bf16 t = from_f<bf16>(v[q][i] * inv * g[q][i]);
+        dst[e] = t;
+        if (cache && e < n) cache[e] = t;
+      }
     }
   }
   __syncthreads();
@@ -474,8 +533,12 @@ __global__ void __launch_bounds__(kGaThreads) grouped_decode_kernel(GroupedArgs 
     }
   }
   const float* bias[RH];
+  float far_bias[RH];   // of every distance from n_bias - 1 on
 #pragma unroll
-  for (int r = 0; r < RH; ++r) bias[r] = a.bias + (int64_t)(h0 + min(g8 + 8 * r, nh - 1)) * sh.n_bias;
+  for (int r = 0; r < RH; ++r) {
+    bias[r] = a.bias + (int64_t)(h0 + min(g8 + 8 * r, nh - 1)) * sh.n_bias;
+    far_bias[r] = sh.n_bias > 0 ? bias[r][sh.n_bias - 1] : 0.0f;
+  }
   float m[RH], l[RH], o[NBO][2 * RH];
 #pragma unroll
   for (int r = 0; r < RH; ++r) {
@@ -501,7 +564,9 @@ __global__ void __launch_bounds__(kGaThreads) grouped_decode_kernel(GroupedArgs 
     const int tw = w * 16, u0 = u_beg + tile * kGaKeys + tw;
     if (u0 < u_end) {
       float bv[RH][2][2];
-      if (sh.n_bias > 0) {
+#pragma unroll
+      for (int r = 0; r < RH; ++r) bv[r][0][0] = bv[r][0][1] = bv[r][1][0] = bv[r][1][1] = far_bias[r];
+      if (p - keys.at(min(u0 + 15, u_end - 1)) < sh.n_bias - 1) {
 #pragma unroll
         for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
@@ -533,8 +598,7 @@ __global__ void __launch_bounds__(kGaThreads) grouped_decode_kernel(GroupedArgs 
         for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
-            float z = sc[nb][2 * r + e] * sh.scale;
-            if (sh.n_bias > 0) z += bv[r][nb][e];
+            float z = fmaf(sc[nb][2 * r + e], sh.scale, bv[r][nb][e]);
             z = u0 + nb * 8 + 2 * t4 + e < u_end ? z : -INFINITY;
             sc[nb][2 * r + e] = z;
             mx = fmaxf(mx, z);
@@ -701,7 +765,7 @@ int grouped_pick_splits(DeviceState* st, int dtype, const GroupedShape& a, int B
   const int group = a.H / a.G, hp = grouped_decode_heads(a);
   const int64_t base = (int64_t)B * a.G * ((group + hp - 1) / hp);
   const int n = a.window > 0 ? std::min(T, a.window + a.keep_first) : T;
-  int s = (int)((2LL * st->sm_count + base - 1) / base);
+  int s = (int)(2LL * st->sm_count / base);   // one wave of two CTAs per SM
   s = std::min(s, (n + 127) / 128);
   return std::max(1, std::min(s, kGroupedMaxSplits));
 }
@@ -768,6 +832,7 @@ int launch_grouped_attention(int device, DeviceState* st, int dtype, const Group
   // queries normed into the scratch, keys and values appended
   {
     const int64_t units = (int64_t)a.B * a.S * (sh.H + (a.k_col >= 0 ? 2 * sh.G : 0));
+    TSB_CHECK(units < (1LL << 31), "grouped attention: portions of %d tokens are not supported", a.B * a.S);
     const int g = (int)std::min<int64_t>((units + 7) / 8, (int64_t)st->sm_count * 16);
     const bool v4 = sh.dim % 4 == 0 && sh.vdim % 4 == 0 && a.q_stride % 4 == 0 && a.k_col % 4 == 0 && a.v_col % 4 == 0 && ((uintptr_t)a.qkv % 16) == 0;
     const bool v4s = v4 || (a.k_col < 0 && sh.dim % 4 == 0 && a.q_stride % 4 == 0 && ((uintptr_t)a.qkv % 16) == 0);

@@ -177,6 +177,7 @@ __global__ void __launch_bounds__(kMsThreads) memory_step_kernel(MemoryArgs a, i
 constexpr int kMcTokens = 128;      // tokens per chunk
 constexpr int kMcTile = 64;         // state tile, value slice, rows of an output CTA
 constexpr int kMcPitch = kMcTile * 2 + 16;
+constexpr int kMcMaxDim = 256;
 constexpr int kMgThreads = 1024;
 
 struct MemoryChunks {               // scratch of the chunk kernels
@@ -240,9 +241,16 @@ __global__ void __launch_bounds__(kMgThreads) memory_gates_kernel(MemoryArgs a, 
   if (tid == 0) *gm = carry;
 }
 
-// grid (value tiles, key tiles, B * H), 4 warps of 16 matrix rows
+// grid (value tiles, key tiles, B * H), 4 warps of 16 matrix rows; keys, values and gate sums of a chunk are copied one chunk ahead
+struct McStage {                    // shared memory of memory_state_kernel
+  unsigned char k[2][kMcTokens * kMcPitch];
+  unsigned char v[2][kMcTokens * kMcPitch];   // becomes the upper part of the weighted values
+  unsigned char lo[kMcTokens * kMcPitch];
+  float F[2][kMcTokens], I[2][kMcTokens];
+};
 __global__ void __launch_bounds__(128) memory_state_kernel(MemoryArgs a, MemoryChunks ck) {
-  extern __shared__ __align__(128) unsigned char smem[];   // k [128], weighted v hi [128], lo [128]: rows of kMcPitch bytes
+  extern __shared__ __align__(128) unsigned char smem[];
+  McStage& sm = *reinterpret_cast<McStage*>(smem);
   __shared__ float s_w[kMcTokens];
   const MemoryShape& sh = a.shape;
   const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
@@ -252,9 +260,26 @@ __global__ void __launch_bounds__(128) memory_state_kernel(MemoryArgs a, MemoryC
   float* st = a.state + (int64_t)b * memory_state_floats(sh);
   float* S = st + (int64_t)h * sh.dim * sh.vdim;
   float* gn = st + (int64_t)sh.H * sh.dim * sh.vdim + (int64_t)h * sh.dim;
-  const uint32_t sk = la_smem(smem), sv = sk + kMcTokens * kMcPitch, sl = sv + kMcTokens * kMcPitch;
   const int64_t qk = (int64_t)sh.H * sh.dim;
   const bf16* x0 = reinterpret_cast<const bf16*>(a.x) + (int64_t)b * a.S * a.stride;
+  auto issue = [&](int c) {
+    if (c < ck.chunks) {
+      const uint32_t dk = la_smem(sm.k[c & 1]), dv = la_smem(sm.v[c & 1]);
+      for (int v = tid; v < kMcTokens * 8; v += 128) {   // 8 units of 16 bytes per row
+        const int r = v >> 3, u = v & 7, t = c * kMcTokens + r;
+        const bool lk = t < a.S && u * 8 < nd, lv = t < a.S && u * 8 < nv;
+        const bf16* xr = x0 + (int64_t)min(t, a.S - 1) * a.stride;
+        la_cp16(dk + r * kMcPitch + u * 16, lk ? xr + qk + (int64_t)h * sh.dim + d0 + u * 8 : xr, lk);
+        la_cp16(dv + r * kMcPitch + u * 16, lv ? xr + 2 * qk + (int64_t)h * sh.vdim + v0 + u * 8 : xr, lv);
+      }
+      if (tid < 64) {
+        const int64_t at = (int64_t)bh * padded + c * kMcTokens + (tid & 31) * 4;
+        la_cp16(la_smem(tid < 32 ? &sm.F[c & 1][tid * 4] : &sm.I[c & 1][(tid & 31) * 4]), (tid < 32 ? ck.F : ck.I) + at);
+      }
+    }
+    la_commit();
+  };
+  issue(0);
   float s[8][4], nvec = 0.0f;
 #pragma unroll
   for (int nb = 0; nb < 8; ++nb)
@@ -265,20 +290,11 @@ __global__ void __launch_bounds__(128) memory_state_kernel(MemoryArgs a, MemoryC
     }
   const bool vec = blockIdx.x == 0 && tid < nd;   // one element of n per thread of the first value tile
   if (vec && T0 > 0) nvec = gn[d0 + tid];
-  float m0 = ck.m0[bh];
+  float m0 = ck.m0[bh], m_next = ck.M[(int64_t)bh * padded + kMcTokens - 1];
   for (int c = 0; c < ck.chunks; ++c) {
-    const float* F = ck.F + (int64_t)bh * padded + c * kMcTokens;
-    const float* I = ck.I + (int64_t)bh * padded + c * kMcTokens;
-    const float FC = F[kMcTokens - 1], mC = ck.M[(int64_t)bh * padded + c * kMcTokens + kMcTokens - 1];
-    const float keep = expf(FC + m0 - mC);
-    __syncthreads();
-    for (int v = tid; v < kMcTokens * 8; v += 128) {   // keys: 8 units of 16 bytes per row
-      const int r = v >> 3, u = v & 7, t = c * kMcTokens + r;
-      const bool live = t < a.S && u * 8 < nd;
-      la_cp16(sk + r * kMcPitch + u * 16, live ? x0 + (int64_t)t * a.stride + qk + (int64_t)h * sh.dim + d0 + u * 8 : x0, live);
-    }
-    la_commit();
-    s_w[tid] = expf(FC - F[tid] + I[tid] - mC);
+    issue(c + 1);
+    const float mC = m_next;
+    if (c + 1 < ck.chunks) m_next = ck.M[(int64_t)bh * padded + (c + 1) * kMcTokens + kMcTokens - 1];
     // the state before the chunk
     const int64_t plane = ((int64_t)bh * ck.chunks + c) * sh.dim * sh.vdim;
 #pragma unroll
@@ -294,11 +310,16 @@ __global__ void __launch_bounds__(128) memory_state_kernel(MemoryArgs a, MemoryC
         }
       }
     if (vec) ck.n0[((int64_t)bh * ck.chunks + c) * sh.dim + d0 + tid] = nvec;
+    la_wait<1>();
     __syncthreads();
-    for (int v = tid; v < kMcTokens * 8; v += 128) {   // values times their weight
-      const int r = v >> 3, u = v & 7, t = c * kMcTokens + r;
-      uint4 in = make_uint4(0u, 0u, 0u, 0u), hi, lo;
-      if (t < a.S && u * 8 < nv) in = *reinterpret_cast<const uint4*>(x0 + (int64_t)t * a.stride + 2 * qk + (int64_t)h * sh.vdim + v0 + u * 8);
+    const float *F = sm.F[c & 1], FC = F[kMcTokens - 1];
+    const float keep = expf(FC + m0 - mC);
+    s_w[tid] = expf(FC - F[tid] + sm.I[c & 1][tid] - mC);
+    __syncthreads();
+    for (int v = tid; v < kMcTokens * 8; v += 128) {   // values times their weight, in two parts
+      const int r = v >> 3, at = r * kMcPitch + (v & 7) * 16;
+      const uint4 in = *reinterpret_cast<const uint4*>(sm.v[c & 1] + at);
+      uint4 hi, lo;
       const float wt = s_w[r];
       const uint32_t* pi = &in.x;
       uint32_t *ph = &hi.x, *pl = &lo.x;
@@ -309,18 +330,18 @@ __global__ void __launch_bounds__(128) memory_state_kernel(MemoryArgs a, MemoryC
         ph[e] = Pair16<bf16>::put(p0.x, p1.x);
         pl[e] = Pair16<bf16>::put(p0.y, p1.y);
       }
-      *reinterpret_cast<uint4*>(smem + kMcTokens * kMcPitch + r * kMcPitch + u * 16) = hi;
-      *reinterpret_cast<uint4*>(smem + 2 * kMcTokens * kMcPitch + r * kMcPitch + u * 16) = lo;
+      *reinterpret_cast<uint4*>(sm.v[c & 1] + at) = hi;
+      *reinterpret_cast<uint4*>(sm.lo + at) = lo;
     }
-    la_wait<0>();
     __syncthreads();
 #pragma unroll
     for (int nb = 0; nb < 8; ++nb)
 #pragma unroll
       for (int e = 0; e < 4; ++e) s[nb][e] *= keep;
     // S += K^T V: rows of the product are key elements (fragments of K transposed), the sum runs over tokens
-    const uint32_t ka = sk + ((lane & 7) + ((lane >> 4) & 1) * 8) * kMcPitch + (w * 16 + ((lane >> 3) & 1) * 8) * 2;
-    const uint32_t va = sv + ((lane & 7) + ((lane >> 3) & 1) * 8) * kMcPitch + (lane >> 4) * 16;
+    const uint32_t ka = la_smem(sm.k[c & 1]) + ((lane & 7) + ((lane >> 4) & 1) * 8) * kMcPitch + (w * 16 + ((lane >> 3) & 1) * 8) * 2;
+    const uint32_t vrow = ((lane & 7) + ((lane >> 3) & 1) * 8) * kMcPitch + (lane >> 4) * 16;
+    const uint32_t va = la_smem(sm.v[c & 1]) + vrow, vl = la_smem(sm.lo) + vrow;
 #pragma unroll
     for (int ks = 0; ks < kMcTokens / 16; ++ks) {
       uint32_t a0, a1, a2, a3;
@@ -331,7 +352,7 @@ __global__ void __launch_bounds__(128) memory_state_kernel(MemoryArgs a, MemoryC
         la_ldsm_x4_trans(va + ks * 16 * kMcPitch + np * 32, b0, b1, b2, b3);
         la_mma(s[2 * np], a0, a1, a2, a3, b0, b1);
         la_mma(s[2 * np + 1], a0, a1, a2, a3, b2, b3);
-        la_ldsm_x4_trans(va + (sl - sv) + ks * 16 * kMcPitch + np * 32, b0, b1, b2, b3);
+        la_ldsm_x4_trans(vl + ks * 16 * kMcPitch + np * 32, b0, b1, b2, b3);
         la_mma(s[2 * np], a0, a1, a2, a3, b0, b1);
         la_mma(s[2 * np + 1], a0, a1, a2, a3, b2, b3);
       }
@@ -339,11 +360,13 @@ __global__ void __launch_bounds__(128) memory_state_kernel(MemoryArgs a, MemoryC
     if (vec) {
       float d = 0.0f;
 #pragma unroll 8
-      for (int r = 0; r < kMcTokens; ++r) d = fmaf(s_w[r], to_f<bf16>(*reinterpret_cast<const bf16*>(smem + r * kMcPitch + tid * 2)), d);
+      for (int r = 0; r < kMcTokens; ++r) d = fmaf(s_w[r], to_f<bf16>(*reinterpret_cast<const bf16*>(sm.k[c & 1] + r * kMcPitch + tid * 2)), d);
       nvec = keep * nvec + d;
     }
     m0 = mC;
+    __syncthreads();   // the next copy overwrites this chunk's stage
   }
+  la_wait<0>();
 #pragma unroll
   for (int nb = 0; nb < 8; ++nb)
 #pragma unroll
@@ -354,18 +377,21 @@ __global__ void __launch_bounds__(128) memory_state_kernel(MemoryArgs a, MemoryC
   if (vec) gn[d0 + tid] = nvec;
 }
 
-// grid (tiles of 64 tokens, heads, sequences), 4 warps of 16 tokens.  Shared memory: q [64] rows; then k [64] rows, or a value slice [128]
-// and the two planes of a state slice [dim].  Rows of q and k hold dim elements rounded up to 16 (zero beyond) and 16 bytes.
+// grid (tiles of 64 tokens, heads, sequences), 4 warps of 16 tokens.  Shared memory: q [64] rows; gated outputs [64] rows of vdim and 16
+// bytes; then k [64] rows, or a value slice [128] and the two planes of a state slice [dim].  Rows of q and k hold dim elements rounded up to
+// 16 (zero beyond) and 16 bytes.
 __global__ void __launch_bounds__(128) memory_out_kernel(MemoryArgs a, MemoryChunks ck) {
   extern __shared__ __align__(128) unsigned char smem[];
-  __shared__ float s_F[kMcTokens], s_I[kMcTokens], s_nq[kMcTile];
+  __shared__ float s_F[kMcTokens], s_I[kMcTokens], s_nq[kMcTile], s_n[kMcMaxDim];
   const MemoryShape& sh = a.shape;
   const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
   const int t0 = blockIdx.x * kMcTile, h = blockIdx.y, b = blockIdx.z, bh = b * sh.H + h;
   const int c = t0 / kMcTokens, cb = c * kMcTokens, padded = ck.chunks * kMcTokens;
   const int n_keys = t0 - cb + kMcTile;                       // 64 or 128, the tile's own tokens last
   const int dp = (sh.dim + 15) / 16 * 16, pitch = dp * 2 + 16, du = dp / 8;
-  const uint32_t sq = la_smem(smem), sk = sq + kMcTile * pitch;
+  const int opitch = sh.vdim * 2 + 16;
+  unsigned char* s_out = smem + kMcTile * pitch;
+  const uint32_t sq = la_smem(smem), sk = la_smem(s_out) + kMcTile * opitch;
   const uint32_t sv = sk, sh_hi = sv + kMcTokens * kMcPitch, sh_lo = sh_hi + dp * kMcPitch;
   const int64_t qk = (int64_t)sh.H * sh.dim, vg = (int64_t)sh.H * sh.vdim;
   const bf16* x0 = reinterpret_cast<const bf16*>(a.x) + (int64_t)b * a.S * a.stride;
@@ -381,6 +407,7 @@ __global__ void __launch_bounds__(128) memory_out_kernel(MemoryArgs a, MemoryChu
   rows(sk, cb, qk);
   s_F[tid] = ck.F[(int64_t)bh * padded + cb + tid];
   s_I[tid] = ck.I[(int64_t)bh * padded + cb + tid];
+  for (int i = tid; i < sh.dim; i += 128) s_n[i] = ck.n0[((int64_t)bh * ck.chunks + c) * sh.dim + i];
   const float m0 = c > 0 ? ck.M[(int64_t)bh * padded + cb - 1] : ck.m0[bh];
   const int rA = w * 16 + g8, off = t0 - cb;
   float mt[2], ft[2], inter[2];
@@ -394,10 +421,10 @@ __global__ void __launch_bounds__(128) memory_out_kernel(MemoryArgs a, MemoryChu
     inter[q] = expf(ft[q] + m0 - mt[q]) * qs;
   }
   {   // n . q of every row: two threads per row
-    const float* n0 = ck.n0 + ((int64_t)bh * ck.chunks + c) * sh.dim;
     const bf16* qr = reinterpret_cast<const bf16*>(smem + (tid >> 1) * pitch);
     float d = 0.0f;
-    for (int i = (tid & 1); i < sh.dim; i += 2) d = fmaf(n0[i], to_f<bf16>(qr[i]), d);
+#pragma unroll 4
+    for (int i = (tid & 1); i < sh.dim; i += 2) d = fmaf(s_n[i], to_f<bf16>(qr[i]), d);
     d += __shfl_xor_sync(0xffffffffu, d, 1);
     if ((tid & 1) == 0) s_nq[tid >> 1] = d;
   }
@@ -464,7 +491,6 @@ __global__ void __launch_bounds__(128) memory_out_kernel(MemoryArgs a, MemoryChu
     rs[q] += __shfl_xor_sync(0xffffffffu, rs[q], 2);
     inv_den[q] = 1.0f / (fmaxf(fabsf(rs[q] + inter[q] * s_nq[rA + q * 8]), expf(-mt[q])) + 1e-6f);
   }
-  bf16* out = reinterpret_cast<bf16*>(a.out) + ((int64_t)b * a.S + t0) * vg + (int64_t)h * sh.vdim;
   const int64_t plane = ((int64_t)bh * ck.chunks + c) * sh.dim * sh.vdim;
   for (int v0 = 0; v0 < sh.vdim; v0 += kMcTile) {
     const int nv = min(kMcTile, sh.vdim - v0);
@@ -482,6 +508,16 @@ __global__ void __launch_bounds__(128) memory_out_kernel(MemoryArgs a, MemoryChu
       la_cp16(sh_lo + r * kMcPitch + u * 16, ck.lo + at, live);
     }
     la_commit();
+    uint32_t gate[8][2], nw[8];   // output gates and norm weights of this thread's values, requested while the slice travels
+#pragma unroll
+    for (int nb = 0; nb < 8; ++nb) {
+      const int cc = v0 + nb * 8 + 2 * t4;
+      nw[nb] = cc < sh.vdim ? *reinterpret_cast<const uint32_t*>(reinterpret_cast<const bf16*>(a.norm_w) + (int64_t)h * sh.vdim + cc) : 0u;
+#pragma unroll
+      for (int q = 0; q < 2; ++q)
+        gate[nb][q] = cc < sh.vdim && t0 + rA + q * 8 < a.S
+                          ? *reinterpret_cast<const uint32_t*>(x0 + (int64_t)(t0 + rA + q * 8) * a.stride + 2 * qk + vg + (int64_t)h * sh.vdim + cc) : 0u;
+    }
     la_wait<0>();
     __syncthreads();
     float o[8][4];
@@ -527,33 +563,49 @@ __global__ void __launch_bounds__(128) memory_out_kernel(MemoryArgs a, MemoryChu
       for (int q = 0; q < 2; ++q) {
         const float u0 = o[nb][2 * q] * inv_den[q], u1 = o[nb][2 * q + 1] * inv_den[q];
         sq_sum[q] += u0 * u0 + u1 * u1;   // columns beyond the slice are zero
-        const int r = rA + q * 8, cc = nb * 8 + 2 * t4;
-        if (t0 + r < a.S && cc < nv) *reinterpret_cast<uint32_t*>(out + (int64_t)r * vg + v0 + cc) = Pair16<bf16>::put(u0, u1);
+        const int cc = nb * 8 + 2 * t4;
+        const float2 g = Pair16<bf16>::get(gate[nb][q]), wt = Pair16<bf16>::get(nw[nb]);
+        if (cc < nv)
+          *reinterpret_cast<uint32_t*>(s_out + (rA + q * 8) * opitch + (v0 + cc) * 2) = Pair16<bf16>::put(u0 * wt.x / (1.0f + __expf(-g.x)), u1 * wt.y / (1.0f + __expf(-g.y)));
       }
   }
-  // norm and output gate on the values this thread has just written
+  // the norm's factor of every row; rows leave in 16-byte units
+  float f[2];
 #pragma unroll
   for (int q = 0; q < 2; ++q) {
     sq_sum[q] += __shfl_xor_sync(0xffffffffu, sq_sum[q], 1);
     sq_sum[q] += __shfl_xor_sync(0xffffffffu, sq_sum[q], 2);
-    const int r = rA + q * 8;
-    if (t0 + r >= a.S) continue;
-    const float f = 1.0f / sqrtf(sq_sum[q] / (float)sh.vdim + sh.eps);
-    const bf16* gr = x0 + (int64_t)(t0 + r) * a.stride + 2 * qk + vg + (int64_t)h * sh.vdim;
-    const bf16* wr = reinterpret_cast<const bf16*>(a.norm_w) + (int64_t)h * sh.vdim;
-#pragma unroll 4
-    for (int cc = 2 * t4; cc < sh.vdim; cc += 8) {
-      uint32_t* op = reinterpret_cast<uint32_t*>(out + (int64_t)r * vg + cc);
-      const float2 o = Pair16<bf16>::get(*op), g = Pair16<bf16>::get(*reinterpret_cast<const uint32_t*>(gr + cc)), wt = Pair16<bf16>::get(*reinterpret_cast<const uint32_t*>(wr + cc));
-      *op = Pair16<bf16>::put(o.x * f * wt.x / (1.0f + __expf(-g.x)), o.y * f * wt.y / (1.0f + __expf(-g.y)));
+    f[q] = 1.0f / sqrtf(sq_sum[q] / (float)sh.vdim + sh.eps);
+  }
+  __syncwarp();
+  bf16* out = reinterpret_cast<bf16*>(a.out) + ((int64_t)b * a.S + t0) * vg + (int64_t)h * sh.vdim;
+#pragma unroll
+  for (int r = 0; r < 16; ++r) {
+    const float fr = __shfl_sync(0xffffffffu, f[r >> 3], (r & 7) * 4);
+    if (t0 + w * 16 + r >= a.S) break;
+    for (int u = lane; u < sh.vdim / 8; u += 32) {
+      uint4 v = *reinterpret_cast<const uint4*>(s_out + (w * 16 + r) * opitch + u * 16);
+      uint32_t* pv = &v.x;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 x = Pair16<bf16>::get(pv[e]);
+        pv[e] = Pair16<bf16>::put(x.x * fr, x.y * fr);
+      }
+      *reinterpret_cast<uint4*>(out + (int64_t)(w * 16 + r) * vg + u * 8) = v;
     }
   }
 }
 
 // ---- host side -------------------------------------------------------------------------------------------------------------------
 constexpr int kMemoryChunkMin = 32;   // shorter portions go token by token
+constexpr size_t kMemorySmem = 220 * 1024;
+static size_t memory_out_smem(const MemoryShape& a) {
+  const int dp = (a.dim + 15) / 16 * 16;
+  const size_t q = (size_t)kMcTile * (dp * 2 + 16);
+  return q + (size_t)kMcTile * (a.vdim * 2 + 16) + std::max<size_t>(q, (size_t)(kMcTokens + 2 * dp) * kMcPitch);
+}
 static bool memory_chunked(int dtype, const MemoryShape& a, int S) {
-  return dtype == TSB200_BF16 && S >= kMemoryChunkMin && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.dim <= 256;
+  return dtype == TSB200_BF16 && S >= kMemoryChunkMin && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.dim <= kMcMaxDim && memory_out_smem(a) <= kMemorySmem;
 }
 static int64_t align16(int64_t n) { return (n + 255) / 256 * 256; }
 static int64_t memory_layout(const MemoryShape& a, int B, int S, char* base, MemoryChunks* ck) {
@@ -605,13 +657,11 @@ int launch_matrix_memory(int device, DeviceState* st, int dtype, const MemoryArg
   if (!a.step_state && memory_chunked(dtype, sh, a.S) && a.stride % 8 == 0 && ((uintptr_t)a.x % 16) == 0 && ((uintptr_t)a.state % 16) == 0) {
     MemoryChunks ck;
     TSB_CHECK(memory_layout(sh, a.B, a.S, (char*)a.scratch, &ck) <= a.scratch_bytes, "matrix memory: scratch too small for %d tokens", a.B * a.S);
-    const int dp = (sh.dim + 15) / 16 * 16;
-    const size_t s1 = 3 * (size_t)kMcTokens * kMcPitch;
-    const size_t q = (size_t)kMcTile * (dp * 2 + 16), s2 = q + std::max<size_t>(q, (size_t)(kMcTokens + 2 * dp) * kMcPitch);
+    const size_t s1 = sizeof(McStage), s2 = memory_out_smem(sh);
     static bool done[kMaxDevices] = {};
     if (!done[device]) {
-      TSB_CUDA(cudaFuncSetAttribute(memory_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024));
-      TSB_CUDA(cudaFuncSetAttribute(memory_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+      TSB_CUDA(cudaFuncSetAttribute(memory_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(McStage)));
+      TSB_CUDA(cudaFuncSetAttribute(memory_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMemorySmem));
       done[device] = true;
     }
     TSB_CHECK((int64_t)a.B * sh.H <= 65535, "matrix memory: %d heads of %d sequences are not supported", sh.H, a.B);
