@@ -223,11 +223,34 @@ __global__ void __launch_bounds__(kGsimThreads) grouped_simple_kernel(GroupedArg
 // ---- bf16 tensor-core kernels -------------------------------------------------------------------------------------------------------
 // Staged rows are D elements (dim and vdim rounded up to one of a few sizes, zero beyond) plus 16 bytes, so that the eight rows of an
 // ldmatrix fall into different banks.
-constexpr int kGaThreads = 128, kGaKeys = 64, kGaStages = 3;
+constexpr int kGaThreads = 128, kGaKeys = 64, kGaStages = 2;   // two stages: more CTAs per SM hide more than a third stage would
+
 template <int D> struct GaTile {
   static constexpr int pitch = D * 2 + 16;
   static constexpr uint32_t plane = (uint32_t)kGaKeys * pitch;   // keys, or values, of a stage
   static constexpr uint32_t stage = 2 * plane;
+};
+// The 16-byte units of a stage's rows that a thread copies, walked without divisions.
+struct UnitWalk {
+  int r0, c0, dr, dc, cols;
+  __device__ __forceinline__ explicit UnitWalk(int n) : cols(n) {
+    r0 = threadIdx.x / n;
+    c0 = threadIdx.x % n;
+    dr = kGaThreads / n;
+    dc = kGaThreads % n;
+  }
+  template <typename F>
+  __device__ __forceinline__ void each(F f) const {
+    for (int r = r0, c = c0; r < kGaKeys;) {
+      f(r, c);
+      r += dr;
+      c += dc;
+      if (c >= cols) {
+        c -= cols;
+        ++r;
+      }
+    }
+  }
 };
 // zeros into the columns that no copy writes
 template <int D>
@@ -244,7 +267,7 @@ __device__ __forceinline__ void ga_zero_pads(unsigned char* smem, int stages, in
 
 // grid (tiles of qt query positions, key/value heads x chunks of hp query heads, sequences)
 template <int D>
-__global__ void __launch_bounds__(kGaThreads) grouped_prefill_kernel(GroupedArgs a, int hp, int qt, int bias_in_smem) {
+__global__ void __launch_bounds__(kGaThreads, D <= 64 ? 4 : D <= 128 ? 3 : 1) grouped_prefill_kernel(GroupedArgs a, int hp, int qt, int bias_in_smem) {
   constexpr int PITCH = GaTile<D>::pitch, KS = D / 16, NBO = D / 8;
   extern __shared__ __align__(128) unsigned char smem[];
   const GroupedShape& sh = a.shape;
@@ -262,19 +285,19 @@ __global__ void __launch_bounds__(kGaThreads) grouped_prefill_kernel(GroupedArgs
   const bf16* Kb = reinterpret_cast<const bf16*>(a.cK) + ((int64_t)b * sh.G + kvh) * a.Tmax * sh.dk;
   const bf16* Vb = reinterpret_cast<const bf16*>(a.cV) + ((int64_t)b * sh.G + kvh) * a.Tmax * sh.dv;
   const uint32_t s0 = la_smem(smem);
-  const int kc = sh.dk / 8, vc = sh.dv / 8;
+  const UnitWalk walk_k(sh.dk / 8), walk_v(sh.dv / 8);
 
   auto issue = [&](int tile) {
     if (tile < n_tiles) {
       const uint32_t st = s0 + (uint32_t)(tile % kGaStages) * GaTile<D>::stage;
-      for (int v = threadIdx.x; v < kGaKeys * kc; v += kGaThreads) {
-        const int r = v / kc, c = v % kc, u = tile * kGaKeys + r;
+      walk_k.each([&](int r, int c) {
+        const int u = tile * kGaKeys + r;
         la_cp16(st + r * PITCH + c * 16, Kb + (int64_t)keys.at(min(u, keys.n - 1)) * sh.dk + c * 8, u < keys.n);
-      }
-      for (int v = threadIdx.x; v < kGaKeys * vc; v += kGaThreads) {
-        const int r = v / vc, c = v % vc, u = tile * kGaKeys + r;
+      });
+      walk_v.each([&](int r, int c) {
+        const int u = tile * kGaKeys + r;
         la_cp16(st + GaTile<D>::plane + r * PITCH + c * 16, Vb + (int64_t)keys.at(min(u, keys.n - 1)) * sh.dv + c * 8, u < keys.n);
-      }
+      });
     }
     la_commit();
   };
@@ -335,17 +358,19 @@ __global__ void __launch_bounds__(kGaThreads) grouped_prefill_kernel(GroupedArgs
       const int tw = sl * 32;
       float sc[4][4];
 #pragma unroll
-      for (int nb = 0; nb < 4; ++nb) {
+      for (int nb = 0; nb < 4; ++nb)
 #pragma unroll
         for (int e = 0; e < 4; ++e) sc[nb][e] = 0.0f;
-        const uint32_t ka = kb + (tw + nb * 8 + (lane & 7)) * PITCH + (lane >> 3) * 16;
+      const uint32_t ka = kb + (tw + (lane & 7)) * PITCH + (lane >> 3) * 16;
 #pragma unroll
-        for (int kp = 0; kp < KS / 2; ++kp) {
-          uint32_t b0, b1, b2, b3;
-          la_ldsm_x4(ka + kp * 64, b0, b1, b2, b3);
-          la_mma(sc[nb], qa[2 * kp][0], qa[2 * kp][1], qa[2 * kp][2], qa[2 * kp][3], b0, b1);
-          la_mma(sc[nb], qa[2 * kp + 1][0], qa[2 * kp + 1][1], qa[2 * kp + 1][2], qa[2 * kp + 1][3], b2, b3);
-        }
+      for (int kp = 0; kp < KS / 2; ++kp) {   // four independent sums side by side
+        uint32_t kf[4][4];
+#pragma unroll
+        for (int nb = 0; nb < 4; ++nb) la_ldsm_x4(ka + nb * 8 * PITCH + kp * 64, kf[nb][0], kf[nb][1], kf[nb][2], kf[nb][3]);
+#pragma unroll
+        for (int nb = 0; nb < 4; ++nb) la_mma(sc[nb], qa[2 * kp][0], qa[2 * kp][1], qa[2 * kp][2], qa[2 * kp][3], kf[nb][0], kf[nb][1]);
+#pragma unroll
+        for (int nb = 0; nb < 4; ++nb) la_mma(sc[nb], qa[2 * kp + 1][0], qa[2 * kp + 1][1], qa[2 * kp + 1][2], qa[2 * kp + 1][3], kf[nb][2], kf[nb][3]);
       }
       // row r: elements 2r, 2r + 1 of every block; keys nb * 8 + 2 * t4 + e
       const bool all_seen = u0 + 31 < keys.n && jb <= wp0 && (sh.window <= 0 || wp1 - ja < sh.window || jb < sh.keep_first);
@@ -435,7 +460,7 @@ __global__ void __launch_bounds__(kGaThreads) grouped_prefill_kernel(GroupedArgs
 // splits in `part`, where the CTA that finishes last merges them.
 template <int D, int RH>
 __global__ void __launch_bounds__(kGaThreads) grouped_decode_kernel(GroupedArgs a, int hp) {
-  constexpr int PITCH = GaTile<D>::pitch, KS = D / 16, NBO = D / 8, ROWS = 8 * RH, REC = D + 4;
+  constexpr int PITCH = GaTile<D>::pitch, KS = D / 16, NBO = D / 8, ROWS = 8 * RH, REC = D + 4, NS = kGaStages;
   extern __shared__ __align__(128) unsigned char smem[];   // stages, queries [ROWS] rows, the new key and value row
   __shared__ int s_last;
   const GroupedShape& sh = a.shape;
@@ -457,26 +482,27 @@ __global__ void __launch_bounds__(kGaThreads) grouped_decode_kernel(GroupedArgs 
   bf16* Vb = reinterpret_cast<bf16*>(a.cV) + ((int64_t)b * sh.G + kvh) * a.Tmax * sh.dv;
   const uint32_t s0 = la_smem(smem);
   const int kc = sh.dk / 8, vc = sh.dv / 8;
+  const UnitWalk walk_k(kc), walk_v(vc);
 
   auto issue = [&](int tile) {
     if (tile < n_tiles) {
-      const uint32_t st = s0 + (uint32_t)(tile % kGaStages) * GaTile<D>::stage;
-      for (int v = tid; v < kGaKeys * kc; v += kGaThreads) {
-        const int r = v / kc, c = v % kc, u = u_beg + tile * kGaKeys + r, j = keys.at(min(u, u_end - 1));
+      const uint32_t st = s0 + (uint32_t)(tile % NS) * GaTile<D>::stage;
+      walk_k.each([&](int r, int c) {
+        const int u = u_beg + tile * kGaKeys + r, j = keys.at(min(u, u_end - 1));
         la_cp16(st + r * PITCH + c * 16, Kb + (int64_t)j * sh.dk + c * 8, u < u_end && !(fresh && j == p));
-      }
-      for (int v = tid; v < kGaKeys * vc; v += kGaThreads) {
-        const int r = v / vc, c = v % vc, u = u_beg + tile * kGaKeys + r, j = keys.at(min(u, u_end - 1));
+      });
+      walk_v.each([&](int r, int c) {
+        const int u = u_beg + tile * kGaKeys + r, j = keys.at(min(u, u_end - 1));
         la_cp16(st + GaTile<D>::plane + r * PITCH + c * 16, Vb + (int64_t)j * sh.dv + c * 8, u < u_end && !(fresh && j == p));
-      }
+      });
     }
     la_commit();
   };
-  for (int i = 0; i < kGaStages - 1; ++i) issue(i);
-  ga_zero_pads<D>(smem, kGaStages, sh.dk, sh.dv);
+  for (int i = 0; i < NS - 1; ++i) issue(i);
+  ga_zero_pads<D>(smem, NS, sh.dk, sh.dv);
 
   // while the first rows travel: queries normed into shared memory, the new key and value row into shared memory and the cache
-  unsigned char* s_q = smem + kGaStages * GaTile<D>::stage;
+  unsigned char* s_q = smem + NS * GaTile<D>::stage;
   bf16* s_new = reinterpret_cast<bf16*>(s_q + ROWS * PITCH);   // [2][D]
   const bf16* row = reinterpret_cast<const bf16*>(a.qkv) + (int64_t)b * a.q_stride;
   for (int i = tid; i < (ROWS - nh) * (PITCH / 16); i += kGaThreads)   // rows without a head
@@ -551,12 +577,12 @@ __global__ void __launch_bounds__(kGaThreads) grouped_decode_kernel(GroupedArgs 
     for (int e = 0; e < 2 * RH; ++e) o[nb][e] = 0.0f;
 
   for (int tile = 0; tile < n_tiles; ++tile) {
-    issue(tile + kGaStages - 1);
-    la_wait<kGaStages - 1>();
+    issue(tile + NS - 1);
+    la_wait<NS - 1>();
     __syncthreads();
-    const uint32_t kb = s0 + (uint32_t)(tile % kGaStages) * GaTile<D>::stage, vb = kb + GaTile<D>::plane;
+    const uint32_t kb = s0 + (uint32_t)(tile % NS) * GaTile<D>::stage, vb = kb + GaTile<D>::plane;
     if (fresh && tile == n_tiles - 1) {   // the new row takes its place
-      unsigned char* st = smem + (tile % kGaStages) * GaTile<D>::stage + ((u_end - 1 - u_beg) % kGaKeys) * PITCH;
+      unsigned char* st = smem + (tile % NS) * GaTile<D>::stage + ((u_end - 1 - u_beg) % kGaKeys) * PITCH;
       if (tid < kc) reinterpret_cast<uint4*>(st)[tid] = reinterpret_cast<const uint4*>(s_new)[tid];
       else if (tid >= 64 && tid < 64 + vc) reinterpret_cast<uint4*>(st + GaTile<D>::plane)[tid - 64] = reinterpret_cast<const uint4*>(s_new + D)[tid - 64];
       __syncthreads();
@@ -576,20 +602,27 @@ __global__ void __launch_bounds__(kGaThreads) grouped_decode_kernel(GroupedArgs 
             for (int r = 0; r < RH; ++r) bv[r][nb][e] = bias[r][n];
           }
       }
-      float sc[2][4];
+      float sc[2][4], sd[2][4];   // even and odd steps: four independent sums
 #pragma unroll
-      for (int nb = 0; nb < 2; ++nb) {
+      for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) sc[nb][e] = 0.0f;
-        const uint32_t ka = kb + (tw + nb * 8 + (lane & 7)) * PITCH + (lane >> 3) * 16;
+        for (int e = 0; e < 4; ++e) sc[nb][e] = sd[nb][e] = 0.0f;
+      const uint32_t ka = kb + (tw + (lane & 7)) * PITCH + (lane >> 3) * 16;
 #pragma unroll
-        for (int kp = 0; kp < KS / 2; ++kp) {
-          uint32_t b0, b1, b2, b3;
-          la_ldsm_x4(ka + kp * 64, b0, b1, b2, b3);
-          la_mma(sc[nb], qa[2 * kp][0], qa[2 * kp][1], qa[2 * kp][2], qa[2 * kp][3], b0, b1);
-          la_mma(sc[nb], qa[2 * kp + 1][0], qa[2 * kp + 1][1], qa[2 * kp + 1][2], qa[2 * kp + 1][3], b2, b3);
+      for (int kp = 0; kp < KS / 2; ++kp) {
+        uint32_t kf[2][4];
+#pragma unroll
+        for (int nb = 0; nb < 2; ++nb) la_ldsm_x4(ka + nb * 8 * PITCH + kp * 64, kf[nb][0], kf[nb][1], kf[nb][2], kf[nb][3]);
+#pragma unroll
+        for (int nb = 0; nb < 2; ++nb) {
+          la_mma(sc[nb], qa[2 * kp][0], qa[2 * kp][1], qa[2 * kp][2], qa[2 * kp][3], kf[nb][0], kf[nb][1]);
+          la_mma(sd[nb], qa[2 * kp + 1][0], qa[2 * kp + 1][1], qa[2 * kp + 1][2], qa[2 * kp + 1][3], kf[nb][2], kf[nb][3]);
         }
       }
+#pragma unroll
+      for (int nb = 0; nb < 2; ++nb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sc[nb][e] += sd[nb][e];
       float corr[RH];
 #pragma unroll
       for (int r = 0; r < RH; ++r) {
@@ -761,13 +794,23 @@ static int grouped_decode_heads(const GroupedShape& a) {   // query heads of a C
   return group < 16 ? group : 16;
 }
 int grouped_pick_splits(DeviceState* st, int dtype, const GroupedShape& a, int B, int T) {
-  if (!grouped_tile(dtype, a)) return 1;
+  const int D = grouped_tile(dtype, a);
+  if (!D) return 1;
   const int group = a.H / a.G, hp = grouped_decode_heads(a);
   const int64_t base = (int64_t)B * a.G * ((group + hp - 1) / hp);
   const int n = a.window > 0 ? std::min(T, a.window + a.keep_first) : T;
-  int s = (int)(2LL * st->sm_count / base);   // one wave of two CTAs per SM
-  s = std::min(s, (n + 127) / 128);
-  return std::max(1, std::min(s, kGroupedMaxSplits));
+  // CTAs that run at a time; a split costs its keys, about two tiles for its start and three for its part in the merge (measured)
+  const int64_t slots = (int64_t)st->sm_count * (D <= 64 ? 5 : D <= 96 ? 4 : D <= 128 ? 3 : D <= 192 ? 2 : 1);
+  int best = 1;
+  int64_t best_cost = 0;
+  for (int s = 1; s <= std::min(kGroupedMaxSplits, (n + 127) / 128); ++s) {
+    const int64_t cost = (base * s + slots - 1) / slots * ((n + s - 1) / s + (s > 1 ? 5 : 2) * kGaKeys);
+    if (s == 1 || cost < best_cost) {
+      best = s;
+      best_cost = cost;
+    }
+  }
+  return best;
 }
 int64_t grouped_part_elems(const GroupedShape& a, int B, int splits) {
   if (splits <= 1) return 0;

@@ -187,9 +187,11 @@ struct MemoryChunks {               // scratch of the chunk kernels
   bf16 *hi, *lo;                    // [B * H][chunks][dim][vdim] state before every chunk, as a sum of two numbers
   int chunks;
 };
-__device__ __forceinline__ float2 split_bf16(float v) {
-  const float h = to_f<bf16>(from_f<bf16>(v));
-  return make_float2(h, v - h);
+// a pair of values as the sum of two bf16 pairs
+__device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = Pair16<bf16>::put(a, b);
+  const float2 h = Pair16<bf16>::get(hi);
+  lo = Pair16<bf16>::put(a - h.x, b - h.y);
 }
 
 __global__ void __launch_bounds__(kMgThreads) memory_gates_kernel(MemoryArgs a, MemoryChunks ck) {
@@ -303,10 +305,11 @@ __global__ void __launch_bounds__(128) memory_state_kernel(MemoryArgs a, MemoryC
       for (int q = 0; q < 2; ++q) {
         const int r = w * 16 + g8 + q * 8, cc = nb * 8 + 2 * t4;
         if (r < nd && cc < nv) {
-          const float2 p0 = split_bf16(s[nb][2 * q]), p1 = split_bf16(s[nb][2 * q + 1]);
+          uint32_t hi, lo;
+          split_pair(s[nb][2 * q], s[nb][2 * q + 1], hi, lo);
           const int64_t at = plane + (int64_t)(d0 + r) * sh.vdim + v0 + cc;
-          *reinterpret_cast<uint32_t*>(ck.hi + at) = Pair16<bf16>::put(p0.x, p1.x);
-          *reinterpret_cast<uint32_t*>(ck.lo + at) = Pair16<bf16>::put(p0.y, p1.y);
+          *reinterpret_cast<uint32_t*>(ck.hi + at) = hi;
+          *reinterpret_cast<uint32_t*>(ck.lo + at) = lo;
         }
       }
     if (vec) ck.n0[((int64_t)bh * ck.chunks + c) * sh.dim + d0 + tid] = nvec;
@@ -326,9 +329,7 @@ __global__ void __launch_bounds__(128) memory_state_kernel(MemoryArgs a, MemoryC
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const float2 f = Pair16<bf16>::get(pi[e]);
-        const float2 p0 = split_bf16(f.x * wt), p1 = split_bf16(f.y * wt);
-        ph[e] = Pair16<bf16>::put(p0.x, p1.x);
-        pl[e] = Pair16<bf16>::put(p0.y, p1.y);
+        split_pair(f.x * wt, f.y * wt, ph[e], pl[e]);
       }
       *reinterpret_cast<uint4*>(sm.v[c & 1] + at) = hi;
       *reinterpret_cast<uint4*>(sm.lo + at) = lo;
@@ -347,14 +348,15 @@ __global__ void __launch_bounds__(128) memory_state_kernel(MemoryArgs a, MemoryC
       uint32_t a0, a1, a2, a3;
       la_ldsm_x4_trans(ka + ks * 16 * kMcPitch, a0, a1, a2, a3);
 #pragma unroll
-      for (int np = 0; np < 4; ++np) {
-        uint32_t b0, b1, b2, b3;
-        la_ldsm_x4_trans(va + ks * 16 * kMcPitch + np * 32, b0, b1, b2, b3);
-        la_mma(s[2 * np], a0, a1, a2, a3, b0, b1);
-        la_mma(s[2 * np + 1], a0, a1, a2, a3, b2, b3);
-        la_ldsm_x4_trans(vl + ks * 16 * kMcPitch + np * 32, b0, b1, b2, b3);
-        la_mma(s[2 * np], a0, a1, a2, a3, b0, b1);
-        la_mma(s[2 * np + 1], a0, a1, a2, a3, b2, b3);
+      for (int part = 0; part < 2; ++part) {   // eight independent sums side by side
+        uint32_t b[4][4];
+#pragma unroll
+        for (int np = 0; np < 4; ++np) la_ldsm_x4_trans((part ? vl : va) + ks * 16 * kMcPitch + np * 32, b[np][0], b[np][1], b[np][2], b[np][3]);
+#pragma unroll
+        for (int np = 0; np < 4; ++np) {
+          la_mma(s[2 * np], a0, a1, a2, a3, b[np][0], b[np][1]);
+          la_mma(s[2 * np + 1], a0, a1, a2, a3, b[np][2], b[np][3]);
+        }
       }
     }
     if (vec) {
@@ -382,7 +384,7 @@ __global__ void __launch_bounds__(128) memory_state_kernel(MemoryArgs a, MemoryC
 // 16 (zero beyond) and 16 bytes.
 __global__ void __launch_bounds__(128) memory_out_kernel(MemoryArgs a, MemoryChunks ck) {
   extern __shared__ __align__(128) unsigned char smem[];
-  __shared__ float s_F[kMcTokens], s_I[kMcTokens], s_nq[kMcTile], s_n[kMcMaxDim];
+  __shared__ float s_F[kMcTokens], s_key[kMcTokens], s_nq[kMcTile], s_n[kMcMaxDim];   // s_key: (i - F) in powers of two
   const MemoryShape& sh = a.shape;
   const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
   const int t0 = blockIdx.x * kMcTile, h = blockIdx.y, b = blockIdx.z, bh = b * sh.H + h;
@@ -396,29 +398,31 @@ __global__ void __launch_bounds__(128) memory_out_kernel(MemoryArgs a, MemoryChu
   const int64_t qk = (int64_t)sh.H * sh.dim, vg = (int64_t)sh.H * sh.vdim;
   const bf16* x0 = reinterpret_cast<const bf16*>(a.x) + (int64_t)b * a.S * a.stride;
   auto rows = [&](uint32_t dst, int first, int64_t col) {     // 64 rows of q or k
-    for (int v = tid; v < kMcTile * du; v += 128) {
-      const int r = v / du, u = v % du, t = first + r;
-      const bool live = t < a.S && u * 8 < sh.dim;
-      la_cp16(dst + r * pitch + u * 16, live ? x0 + (int64_t)t * a.stride + col + (int64_t)h * sh.dim + u * 8 : x0, live);
-    }
+    for (int r = w; r < kMcTile; r += 4)
+      for (int u = lane; u < du; u += 32) {
+        const int t = first + r;
+        const bool live = t < a.S && u * 8 < sh.dim;
+        la_cp16(dst + r * pitch + u * 16, live ? x0 + (int64_t)t * a.stride + col + (int64_t)h * sh.dim + u * 8 : x0, live);
+      }
     la_commit();
   };
   rows(sq, t0, 0);
   rows(sk, cb, qk);
   s_F[tid] = ck.F[(int64_t)bh * padded + cb + tid];
-  s_I[tid] = ck.I[(int64_t)bh * padded + cb + tid];
+  s_key[tid] = (ck.I[(int64_t)bh * padded + cb + tid] - s_F[tid]) * kLog2e;
   for (int i = tid; i < sh.dim; i += 128) s_n[i] = ck.n0[((int64_t)bh * ck.chunks + c) * sh.dim + i];
   const float m0 = c > 0 ? ck.M[(int64_t)bh * padded + cb - 1] : ck.m0[bh];
   const int rA = w * 16 + g8, off = t0 - cb;
-  float mt[2], ft[2], inter[2];
+  float mt[2], query[2], inter[2];   // query: (F - m) in powers of two
   const float qs = 1.0f / sqrtf((float)sh.dim);
   la_wait<0>();
   __syncthreads();
 #pragma unroll
   for (int q = 0; q < 2; ++q) {
     mt[q] = ck.M[(int64_t)bh * padded + t0 + rA + q * 8];
-    ft[q] = s_F[off + rA + q * 8];
-    inter[q] = expf(ft[q] + m0 - mt[q]) * qs;
+    const float ft = s_F[off + rA + q * 8];
+    query[q] = (ft - mt[q]) * kLog2e;
+    inter[q] = expf(ft + m0 - mt[q]) * qs;
   }
   {   // n . q of every row: two threads per row
     const bf16* qr = reinterpret_cast<const bf16*>(smem + (tid >> 1) * pitch);
@@ -463,7 +467,7 @@ __global__ void __launch_bounds__(128) memory_out_kernel(MemoryArgs a, MemoryChu
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int q = e >> 1, key = kt * kMcTile + nb * 8 + 2 * t4 + (e & 1);
-          const float p = key <= off + rA + q * 8 ? sc[nb][e] * qs * expf(ft[q] - s_F[key] + s_I[key] - mt[q]) : 0.0f;
+          const float p = key <= off + rA + q * 8 ? sc[nb][e] * qs * exp2_fast(query[q] + s_key[key]) : 0.0f;
           sc[nb][e] = p;
           rs[q] += p;
         }
@@ -472,9 +476,7 @@ __global__ void __launch_bounds__(128) memory_out_kernel(MemoryArgs a, MemoryChu
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const float* p = &sc[2 * kk + (e >> 1)][2 * (e & 1)];
-          const float2 p0 = split_bf16(p[0]), p1 = split_bf16(p[1]);
-          ph[kt * 4 + kk][e] = Pair16<bf16>::put(p0.x, p1.x);
-          pl[kt * 4 + kk][e] = Pair16<bf16>::put(p0.y, p1.y);
+          split_pair(p[0], p[1], ph[kt * 4 + kk][e], pl[kt * 4 + kk][e]);
         }
     } else {
 #pragma unroll
@@ -530,14 +532,15 @@ __global__ void __launch_bounds__(128) memory_out_kernel(MemoryArgs a, MemoryChu
       uint32_t a0, a1, a2, a3;
       la_ldsm_x4(qa + ks * 32, a0, a1, a2, a3);
 #pragma unroll
-      for (int np = 0; np < 4; ++np) {
-        uint32_t b0, b1, b2, b3;
-        la_ldsm_x4_trans(sh_hi + vrow + ks * 16 * kMcPitch + np * 32, b0, b1, b2, b3);
-        la_mma(o[2 * np], a0, a1, a2, a3, b0, b1);
-        la_mma(o[2 * np + 1], a0, a1, a2, a3, b2, b3);
-        la_ldsm_x4_trans(sh_lo + vrow + ks * 16 * kMcPitch + np * 32, b0, b1, b2, b3);
-        la_mma(o[2 * np], a0, a1, a2, a3, b0, b1);
-        la_mma(o[2 * np + 1], a0, a1, a2, a3, b2, b3);
+      for (int part = 0; part < 2; ++part) {
+        uint32_t b[4][4];
+#pragma unroll
+        for (int np = 0; np < 4; ++np) la_ldsm_x4_trans((part ? sh_lo : sh_hi) + vrow + ks * 16 * kMcPitch + np * 32, b[np][0], b[np][1], b[np][2], b[np][3]);
+#pragma unroll
+        for (int np = 0; np < 4; ++np) {
+          la_mma(o[2 * np], a0, a1, a2, a3, b[np][0], b[np][1]);
+          la_mma(o[2 * np + 1], a0, a1, a2, a3, b[np][2], b[np][3]);
+        }
       }
     }
 #pragma unroll
@@ -547,14 +550,18 @@ __global__ void __launch_bounds__(128) memory_out_kernel(MemoryArgs a, MemoryChu
 #pragma unroll
     for (int kk = 0; kk < 8; ++kk) {
       if (kk * 16 >= n_keys) break;
+      uint32_t b[4][4];
+#pragma unroll
+      for (int np = 0; np < 4; ++np) la_ldsm_x4_trans(sv + vrow + kk * 16 * kMcPitch + np * 32, b[np][0], b[np][1], b[np][2], b[np][3]);
 #pragma unroll
       for (int np = 0; np < 4; ++np) {
-        uint32_t b0, b1, b2, b3;
-        la_ldsm_x4_trans(sv + vrow + kk * 16 * kMcPitch + np * 32, b0, b1, b2, b3);
-        la_mma(o[2 * np], ph[kk][0], ph[kk][1], ph[kk][2], ph[kk][3], b0, b1);
-        la_mma(o[2 * np + 1], ph[kk][0], ph[kk][1], ph[kk][2], ph[kk][3], b2, b3);
-        la_mma(o[2 * np], pl[kk][0], pl[kk][1], pl[kk][2], pl[kk][3], b0, b1);
-        la_mma(o[2 * np + 1], pl[kk][0], pl[kk][1], pl[kk][2], pl[kk][3], b2, b3);
+        la_mma(o[2 * np], ph[kk][0], ph[kk][1], ph[kk][2], ph[kk][3], b[np][0], b[np][1]);
+        la_mma(o[2 * np + 1], ph[kk][0], ph[kk][1], ph[kk][2], ph[kk][3], b[np][2], b[np][3]);
+      }
+#pragma unroll
+      for (int np = 0; np < 4; ++np) {
+        la_mma(o[2 * np], pl[kk][0], pl[kk][1], pl[kk][2], pl[kk][3], b[np][0], b[np][1]);
+        la_mma(o[2 * np + 1], pl[kk][0], pl[kk][1], pl[kk][2], pl[kk][3], b[np][2], b[np][3]);
       }
     }
 #pragma unroll
@@ -566,7 +573,7 @@ __global__ void __launch_bounds__(128) memory_out_kernel(MemoryArgs a, MemoryChu
         const int cc = nb * 8 + 2 * t4;
         const float2 g = Pair16<bf16>::get(gate[nb][q]), wt = Pair16<bf16>::get(nw[nb]);
         if (cc < nv)
-          *reinterpret_cast<uint32_t*>(s_out + (rA + q * 8) * opitch + (v0 + cc) * 2) = Pair16<bf16>::put(u0 * wt.x / (1.0f + __expf(-g.x)), u1 * wt.y / (1.0f + __expf(-g.y)));
+          *reinterpret_cast<uint32_t*>(s_out + (rA + q * 8) * opitch + (v0 + cc) * 2) = Pair16<bf16>::put(__fdividef(u0 * wt.x, 1.0f + exp2_fast(-g.x * kLog2e)), __fdividef(u1 * wt.y, 1.0f + exp2_fast(-g.y * kLog2e)));
       }
   }
   // the norm's factor of every row; rows leave in 16-byte units
