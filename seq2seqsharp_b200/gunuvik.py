@@ -7,15 +7,14 @@ attention without rotation (distance bias, sink, gated heads, caches shared betw
 import re
 from typing import Dict, Mapping, Optional
 
-from .layered import BlockLayer, DenseGated, GroupedAttention, LayeredConfig, MatrixMemory
-from .pepilix import _only
+from .layered import BlockLayer, DenseGated, GroupedAttention, LayeredConfig, MatrixMemory, only_keys
 
 ARCHITECTURE = "Gunuvik"
 
 
 def _attention(m: dict, where: str, rel_rows: int) -> GroupedAttention:
-    _only(m, ("bias_max", "dim", "heads", "kv_heads", "mask", "scale", "vdim", "kv_from"), where + " mixer")
-    _only(m["mask"], ("size", "keep_first"), where + " mask")
+    only_keys(m, ("bias_max", "dim", "heads", "kv_heads", "mask", "scale", "vdim", "kv_from"), where + " mixer")
+    only_keys(m["mask"], ("size", "keep_first"), where + " mask")
     src = m.get("kv_from")
     if int(m["mask"]["size"]) < 1:
         raise ValueError("%s: a window of %r positions" % (where, m["mask"]["size"]))
@@ -29,14 +28,14 @@ def config_from_json(j: dict, dtype: str = "bfloat16", shapes: Optional[Mapping[
     Unknown kinds and keys are refused: they would change the model."""
     if j.get("architecture") != ARCHITECTURE:
         raise ValueError("not a %s model: architecture %r" % (ARCHITECTURE, j.get("architecture")))
-    _only(j, ("architecture", "embedding", "layers", "norm", "vocab", "width"), "config.json")
-    _only(j["embedding"], ("scale",), "embedding")
-    _only(j["norm"], ("eps",), "norm")
+    only_keys(j, ("architecture", "embedding", "layers", "norm", "vocab", "width"), "config.json")
+    only_keys(j["embedding"], ("scale",), "embedding")
+    only_keys(j["norm"], ("eps",), "norm")
     cfg = LayeredConfig(d=int(j["width"]), V=int(j["vocab"]), block="sandwich", eps=float(j["norm"]["eps"]), embed_scale=float(j["embedding"]["scale"]),
                         tied_head=False, dtype=dtype, name=ARCHITECTURE)
     for i, layer in enumerate(j["layers"]):
         where = "layer %d" % i
-        _only(layer, ("type", "mixer", "mlp"), where)
+        only_keys(layer, ("type", "mixer", "mlp"), where)
         m = layer["mixer"]
         if layer["type"] == "attention":
             rel = "l%d.mix.rel" % i
@@ -44,13 +43,13 @@ def config_from_json(j: dict, dtype: str = "bfloat16", shapes: Optional[Mapping[
                 raise ValueError("%s: the shape of %s is needed" % (where, rel))
             mixer = _attention(m, where, int(shapes[rel][0]))
         elif layer["type"] == "mlstm":
-            _only(m, ("dim", "gate_cap", "heads", "vdim"), where + " mixer")
+            only_keys(m, ("dim", "gate_cap", "heads", "vdim"), where + " mixer")
             mixer = MatrixMemory(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), gate_cap=float(m["gate_cap"]))
         else:
             raise ValueError("%s: unknown type %r" % (where, layer["type"]))
         dense = None
         if layer.get("mlp") is not None:
-            _only(layer["mlp"], ("kind", "ff"), where + " mlp")
+            only_keys(layer["mlp"], ("kind", "ff"), where + " mlp")
             if layer["mlp"].get("kind", "dense") != "dense":
                 raise ValueError("%s: unknown feed-forward %r" % (where, layer["mlp"]["kind"]))
             dense = DenseGated(int(layer["mlp"]["ff"]))

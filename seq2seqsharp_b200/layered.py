@@ -15,6 +15,13 @@ from .gpt import GPT
 from .synthetic import synth
 
 
+def only_keys(d: dict, known, where: str):
+    """For readers of model configurations: a key that is not known would change the model, so it is refused."""
+    unknown = set(d) - set(known)
+    if unknown:
+        raise ValueError("%s: unknown keys %s" % (where, sorted(unknown)))
+
+
 @dataclass
 class LatentAttention:
     """Attention over one cached vector per position: a normed latent and a rotated key part shared by all heads."""

@@ -6,35 +6,29 @@ RMS norms of the same residual stream, each multiplied by a sigmoid gate of its 
 import re
 from typing import Dict
 
-from .layered import BlockLayer, LatentAttention, LayeredConfig, TableExperts
+from .layered import BlockLayer, LatentAttention, LayeredConfig, TableExperts, only_keys
 
 ARCHITECTURE = "Pepilix"
 # constants of the design's experts: hidden = a sigmoid(1.702 a) (u + 1)
 EXPERT_SLOPE, EXPERT_SHIFT = 1.702, 1.0
 
 
-def _only(d: dict, known, where: str):
-    unknown = set(d) - set(known)
-    if unknown:
-        raise ValueError("%s: unknown keys %s" % (where, sorted(unknown)))
-
-
 def config_from_json(j: dict, dtype: str = "bfloat16") -> LayeredConfig:
     """The parsed config.json as a `LayeredConfig`.  Unknown kinds and keys are refused: they would change the model."""
     if j.get("architecture") != ARCHITECTURE:
         raise ValueError("not a %s model: architecture %r" % (ARCHITECTURE, j.get("architecture")))
-    _only(j, ("architecture", "canon", "embedding", "layers", "logit_scale", "norm", "vocab", "width"), "config.json")
+    only_keys(j, ("architecture", "canon", "embedding", "layers", "logit_scale", "norm", "vocab", "width"), "config.json")
     cfg = LayeredConfig(d=int(j["width"]), V=int(j["vocab"]), norm_groups=int(j["norm"]["groups"]), conv_taps=int(j["canon"]["taps"]),
                         eps=float(j["norm"]["eps"]), embed_scale=float(j["embedding"]["scale"]), logit_scale=float(j["logit_scale"]), dtype=dtype,
                         name=ARCHITECTURE)
     for i, layer in enumerate(j["layers"]):
         where = "layer %d" % i
-        _only(layer, ("type", "mixer", "mlp"), where)
+        only_keys(layer, ("type", "mixer", "mlp"), where)
         if layer["type"] != "latent_attention":
             raise ValueError("%s: unknown type %r" % (where, layer["type"]))
         m = layer["mixer"]
-        _only(m, ("dim", "heads", "kv_rank", "rot", "rot_dim", "scale", "vdim", "kv_from"), where + " mixer")
-        _only(m["rot"], ("base", "dims"), where + " rotation")
+        only_keys(m, ("dim", "heads", "kv_rank", "rot", "rot_dim", "scale", "vdim", "kv_from"), where + " mixer")
+        only_keys(m["rot"], ("base", "dims"), where + " rotation")
         src = m.get("kv_from")
         mixer = LatentAttention(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]), kv_rank=int(m["kv_rank"]),
                                 rot_base=float(m["rot"]["base"]), rot_dims=int(m["rot"]["dims"]), scale=float(m["scale"]),
@@ -42,11 +36,11 @@ def config_from_json(j: dict, dtype: str = "bfloat16") -> LayeredConfig:
         experts = None
         if layer.get("mlp") is not None:
             f = layer["mlp"]
-            _only(f, ("kind", "expert", "router"), where + " mlp")
+            only_keys(f, ("kind", "expert", "router"), where + " mlp")
             if f.get("kind", "moe") != "moe":
                 raise ValueError("%s: unknown feed-forward %r" % (where, f["kind"]))
-            _only(f["expert"], ("ff", "limit"), where + " expert")
-            _only(f["router"], ("experts", "top"), where + " router")
+            only_keys(f["expert"], ("ff", "limit"), where + " expert")
+            only_keys(f["router"], ("experts", "top"), where + " router")
             experts = TableExperts(experts=int(f["router"]["experts"]), top=int(f["router"]["top"]), ff=int(f["expert"]["ff"]),
                                    limit=float(f["expert"]["limit"]), slope=EXPERT_SLOPE, shift=EXPERT_SHIFT)
         cfg.layers.append(BlockLayer(mixer, experts))

@@ -81,11 +81,11 @@ def weights(cfg, seed=1, rows=None):
         else:
             w = rng.normal(0, (2.0 if part in ("mix.g", "mix.i", "mix.f") else 1.0) / np.sqrt(shape[1]), size=shape)
         a = to_float32(to_bfloat16(w.astype(np.float32)))
-        out[n] = a.reshape(-1) if shape[0] == 1 and part not in ("mix.g", "mix.i", "mix.f", "mlp.down") and a.ndim == 2 and is_vector(part) else a
+        out[n] = a.reshape(-1) if is_vector(part) else a
     return out
 
 
-def is_vector(part):
+def is_vector(part):   # stored with one dimension
     return "norm" in part or part in ("ls1", "ls2", "mix.sink") or part.endswith(".b")
 
 
